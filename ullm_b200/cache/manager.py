@@ -19,7 +19,7 @@ What it owns
 
 Groups: executions (schedule entries) with equal CacheNeed share a group; an
 execution that reads another's cache has none of its own.  A group with a
-window gives pages back as soon as every position in them is out of reach of
+window (or stretches of positions) gives pages back as soon as every position in them is out of reach of
 any later token; a finished request gives back everything (full pages of a
 prefix-cached group go to the tree instead and stay findable until evicted).
 """
@@ -88,7 +88,7 @@ def plan_groups_with_aux(needs):
         if need is None:
             where_aux.append(None)
             continue
-        if need.window is not None and need.every > 1:
+        if not need.keeps_all and need.every > 1:
             raise ValueError(f"schedule entry {i}: a cache with one entry per {need.every} tokens keeps all of them")
         for g, info in enumerate(groups):
             if info.need == need:
@@ -118,7 +118,9 @@ def _plan_main(needs):
                 need.num_kv_heads, need.head_dim, need.v_dim):
             raise ValueError(f"schedule entry {i} cannot read the cache of entry {cache_of}: different geometry")
         have = kept[cache_of]
-        window = None if (have.window is None or need.window is None) else max(have.window, need.window)
+        if have.chunk is not None and have.chunk == need.chunk:
+            continue  # (stretches of the same size: the reader sees what the writer sees)
+        window = None if (have.keeps_all or need.keeps_all) else max(have.reach, need.reach)
         kept[cache_of] = CacheNeed(have.num_kv_heads, have.head_dim, window, have.value_dim,
                                    0 if window is None else max(have.keep_first, need.keep_first),
                                    have.values_in_keys, have.every)
@@ -163,7 +165,7 @@ class CacheManager:
         self.needs = list(needs)
         self.groups, self.where, self.where_aux = plan_groups_with_aux(self.needs)
         for g in self.groups:
-            if g.need.every < 1 or (g.need.every > 1 and g.need.window is not None):
+            if g.need.every < 1 or (g.need.every > 1 and not g.need.keeps_all):
                 raise ValueError("a cache with one entry per several tokens keeps all its entries (no window)")
         # a group with one entry per n tokens needs a page per n pages of tokens, and one more per request for
         # the page each is filling
@@ -172,7 +174,7 @@ class CacheManager:
         self.allocators = [PageAllocator(n) for n in self.group_pages]
         self.slots = SlotAllocator(max_requests)
         has_state = any(n[1] is not None for n in self.needs)
-        only_full = len(self.groups) == 1 and self.groups[0].need.window is None
+        only_full = len(self.groups) == 1 and self.groups[0].need.keeps_all
         self.tree = PrefixTree(page_size) if (enable_prefix_cache and only_full and not has_state) else None
         if enable_prefix_cache and self.tree is None:
             why = ("a mixer keeps per-request state" if has_state else
@@ -329,17 +331,16 @@ class CacheManager:
         return held[pos // ps - first] * ps + pos % ps
 
     def commit(self, rc: RequestCache, n_new: int) -> None:
-        """The step wrote n_new tokens.  Pages of windowed groups that no later
+        """The step wrote n_new tokens.  Pages of groups with a window (or stretches) that no later
         token can reach are given back."""
         rc.num_tokens += n_new
         ps = self.page_size
         for g, info in enumerate(self.groups):
-            w = info.need.window
-            if w is None:
+            if info.need.keeps_all:
                 continue
-            # the next token sits at position num_tokens and sees positions >= num_tokens - w + 1, and the first
+            # the next token sits at position num_tokens and sees positions >= first_needed, and the first
             # keep_first positions for ever: the pages that hold those are never given back
-            first_needed = max(0, rc.num_tokens - w + 1) // ps
+            first_needed = info.need.first_needed(rc.num_tokens) // ps
             lo = max(rc.first_live_page[g], -(-info.need.keep_first // ps))
             if first_needed > lo:
                 gone = [p for p in rc.pages[g][lo:first_needed] if p >= 0]

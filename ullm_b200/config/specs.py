@@ -121,6 +121,8 @@ class ModelSpec:
     # "engine": the residual stream has the engine's dtype; "float32": it is kept in 32-bit whatever the engine's
     # dtype (the blocks of such a model take and return a 32-bit stream)
     stream_dtype: str = "engine"
+    # logits <- logit_scale * logits
+    logit_scale: float = 1.0
     # logits <- logit_softcap * tanh(logits / logit_softcap) when set
     logit_softcap: float | None = None
     # a per-layer token input table that blocks read through the step's context (`ctx.token_side`)

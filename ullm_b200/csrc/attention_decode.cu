@@ -91,7 +91,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
   const int group = num_q / num_kv;
   const int kvl = kv_len[b];
   const int pos = kvl - 1;
-  const int lo = (window > 0 && pos >= 0) ? max(0, pos - window + 1) : 0;
+  const int lo = pos >= 0 ? first_seen(pos, window) : 0;
   // The keys a row sees are numbered 0 .. n_keys - 1: first the kept first positions that the window has left
   // behind (0 .. kept - 1), then the window (lo .. pos).  Blocks and warps split this numbering; only the page
   // lookup needs the position itself.
@@ -630,7 +630,7 @@ static int decode_attention_impl(const void* q, long long q_row_stride, const vo
                                  int page_size, int window, float scale, int num_splits, long long num_pages,
                                  int* status, void* stream, const DecFuse& fu) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (batch < 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0 || num_splits <= 0 || window < 0)
+  if (batch < 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0 || num_splits <= 0)
     return ULLM_ERR_BAD_SIZE;
   if (!ullm_decode_attention_supported(head_dim, num_q, num_kv)) return ULLM_ERR_UNSUPPORTED;
   if (num_splits > 1 && scratch == nullptr) return ULLM_ERR_BAD_SIZE;

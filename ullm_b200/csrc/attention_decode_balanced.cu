@@ -113,7 +113,7 @@ decode_attention_balanced_kernel(const __grid_constant__ CUtensorMap map_k, cons
   // ---- prologue (the only block-wide part): every request's visible keys, tiles and their running sum -----
   for (int b = threadIdx.x; b < p.batch; b += blockDim.x) {
     const int pos = p.kv_len[b] - 1;
-    const int lo = (p.window > 0 && pos >= 0) ? max(0, pos - p.window + 1) : 0;
+    const int lo = pos >= 0 ? first_seen(pos, p.window) : 0;
     const int n = pos >= 0 ? pos - lo + 1 : 0;
     s_lo[b] = lo;
     s_end[b] = lo + n;
@@ -496,7 +496,7 @@ extern "C" int ullm_decode_attention_balanced(const void* q, long long q_row_str
                                               int page_size, int window, float scale, long long num_pages, int* status,
                                               void* stream) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (batch < 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0 || window < 0) return ULLM_ERR_BAD_SIZE;
+  if (batch < 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0) return ULLM_ERR_BAD_SIZE;
   if (!ullm_decode_attention_balanced_supported(head_dim, num_q, num_kv, batch, page_size)) return ULLM_ERR_UNSUPPORTED;
   if (((uintptr_t)k_cache | (uintptr_t)v_cache) & 15) return ULLM_ERR_UNSUPPORTED;
   if (part == nullptr || prefix == nullptr || flags == nullptr) return ULLM_ERR_BAD_SIZE;

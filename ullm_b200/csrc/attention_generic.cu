@@ -16,7 +16,8 @@
 //
 // Batch row r reads row req_slots[r] of the block table.  Request r owns query rows cu_q[r] .. cu_q[r+1]-1 and holds kv_len[r] tokens
 // after this step; row j of it sits at position kv_len[r] - q_len[r] + j and
-// sees positions max(0, pos - window + 1) .. pos (window 0 = all), and with
+// sees positions first_seen(pos, window) .. pos (window 0: all; w > 0: the last
+// w; -c: its stretch of c positions, see common.cuh), and with
 // `keep_first` > 0 also the positions below keep_first that the window has
 // left behind (they are visited first, in groups of 32 of their own).
 // Values may have a head size of their own (`v_dim`): the value pages are
@@ -95,7 +96,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, long lon
     }
     return;
   }
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = first_seen(pos, window);
   const T* q_ptr = q + (long long)t * q_row_stride + (long long)h * head_dim;
   float* qv = qs[warp];
   for (int e = lane; e < head_dim; e += 32) qv[e] = to_f32(q_ptr[e]);
@@ -287,7 +288,7 @@ extern "C" int ullm_paged_attention_generic_ex2(int dtype, const void* q, long l
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || page_size <= 0 || max_pages <= 0)
     return ULLM_ERR_BAD_SIZE;
-  if (num_q % num_kv != 0 || head_dim > ATT_MAX_HEAD_DIM || window < 0 || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
+  if (num_q % num_kv != 0 || head_dim > ATT_MAX_HEAD_DIM || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
       keep_first < 0 || softcap < 0.f)
     return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;
@@ -323,7 +324,7 @@ extern "C" int ullm_paged_attention_generic_ex3(int dtype, const void* q, long l
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || page_size <= 0 || max_pages <= 0)
     return ULLM_ERR_BAD_SIZE;
-  if (num_q % num_kv != 0 || head_dim > ATT_MAX_KEY_DIM || window < 0 || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
+  if (num_q % num_kv != 0 || head_dim > ATT_MAX_KEY_DIM || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
       keep_first < 0 || softcap < 0.f || pool < 0)
     return ULLM_ERR_UNSUPPORTED;
   if (values_in_keys && v_dim > head_dim) return ULLM_ERR_BAD_SIZE;
@@ -387,7 +388,7 @@ extern "C" int ullm_paged_attention_generic_ex(int dtype, const void* q, long lo
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || page_size <= 0 || max_pages <= 0)
     return ULLM_ERR_BAD_SIZE;
-  if (num_q % num_kv != 0 || head_dim > ATT_MAX_HEAD_DIM || window < 0 || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
+  if (num_q % num_kv != 0 || head_dim > ATT_MAX_HEAD_DIM || v_dim <= 0 || v_dim > ATT_MAX_HEAD_DIM ||
       keep_first < 0)
     return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;

@@ -8,7 +8,7 @@
 // Rows are (token, query head of the group) pairs: with G query heads per kv
 // head a block covers 128 / G consecutive tokens, so one pass over K and V serves
 // all heads that share them.  Row i of a block: token j0 + i / G, head kh * G +
-// i % G, position start + j0 + i / G; it sees keys max(0, pos - window + 1) ..
+// i % G, position start + j0 + i / G; it sees keys first_seen(pos, window) ..
 // pos.  K and V tiles are gathered from the pages with cp.async into a two-stage
 // ring shared by the block's four warps (16-byte chunks, XOR-swizzled by row);
 // each warp owns 32 rows, so a K or V fragment read from shared memory feeds two
@@ -140,7 +140,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_st
     }
     return;
   }
-  const int key0 = window > 0 ? max(0, p0 - window + 1) : 0;
+  const int key0 = first_seen(p0, window);
   // With kept first positions the block's key tiles are: those of positions 0 .. kept - 1 (what the window of
   // the block's first token has left behind of them), then those from key0 on.
   const int kept = min(keep_first, key0);
@@ -198,12 +198,13 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_st
     for (int h = 0; h < 2; ++h) {
       const int row = wrow + mt * 16 + (lane >> 2) + h * 8;
       pos[mt][h] = row < rows_valid ? p0 + row / G : -1;
-      lo[mt][h] = window > 0 ? pos[mt][h] - window + 1 : 0;
+      lo[mt][h] = first_seen(pos[mt][h], window);
     }
   const int w_last = min(rows_valid, wrow + PRE_ROWS_PER_WARP) - 1;
   const bool warp_live = wrow < rows_valid;
   const int wp_max = warp_live ? p0 + w_last / G : -1;
-  const int wp_lo = (warp_live && window > 0) ? p0 + wrow / G - window + 1 : 0;
+  const int wp_lo = warp_live ? first_seen(p0 + wrow / G, window) : 0;
+  const int wp_lo_last = warp_live ? first_seen(wp_max, window) : 0;  // what the warp's last row sees first
   const int wp_min = p0 + wrow / G;                               // position of the warp's first row
   const bool warp_full = wrow + PRE_ROWS_PER_WARP <= rows_valid;  // no padding rows in this warp
 
@@ -292,7 +293,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_st
               for (int e = 0; e < 4; ++e) sc[mt][t][e] = pre_tanh(sc[mt][t][e]);
         }
       }
-      const bool need_mask = sink || !warp_full || kb + PRE_N - 1 > wp_min || (window > 0 && kb < wp_max - window + 1);
+      const bool need_mask = sink || !warp_full || kb + PRE_N - 1 > wp_min || kb < wp_lo_last;
       float alpha[2][2];
 #pragma unroll
       for (int mt = 0; mt < 2; ++mt) {
@@ -439,8 +440,7 @@ extern "C" int ullm_prefill_attention_ex(const void* q, long long q_row_stride, 
                                          int window, float scale, long long num_pages, int* status, void* stream,
                                          int keep_first, float softcap, float* parts) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (tokens < 0 || num_requests <= 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0 || window < 0 ||
-      keep_first < 0 || softcap < 0.f)
+  if (tokens < 0 || num_requests <= 0 || num_q <= 0 || num_kv <= 0 || page_size <= 0 || max_pages <= 0 || keep_first < 0 || softcap < 0.f)
     return ULLM_ERR_BAD_SIZE;
   if (!ullm_prefill_attention_supported(head_dim, num_q, num_kv)) return ULLM_ERR_UNSUPPORTED;
   if (softcap > 0.f && parts != nullptr) return ULLM_ERR_UNSUPPORTED;

@@ -287,7 +287,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
     }
     return;
   }
-  const int key_lo = p.window > 0 ? max(0, p0 - p.window + 1) : 0;
+  const int key_lo = first_seen(p0, p.window);
   const int k_start = key_lo / TP_KEYS * TP_KEYS;
   // key tiles each query tile walks (tile 1 sees later keys: tiles1 >= tiles0 when it has rows)
   const int tiles0 = (p0 + ntok0 - 1 - k_start) / TP_KEYS + 1;
@@ -484,7 +484,8 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
     const int pf = p0 + i * tpt;                 // position of the tile's first token
     const int pl = pf + ntok_i - 1;              // and of its last
     const int pos = row_ok ? pf + row / G : -1;
-    const int lo = p.window > 0 ? pos - p.window + 1 : 0;
+    const int lo = first_seen(pos, p.window);
+    const int lo_last = first_seen(pl, p.window);  // what the tile's last token sees first
     const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t tmem_s = tmem + i * TP_KEYS + lane_base;
     const uint32_t tmem_o = tmem + 2 * TP_KEYS + i * TP_D + lane_base;
@@ -524,7 +525,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
           for (int k = 0; k < TP_KEYS; ++k) sr[k] = __float_as_uint(tp_tanh(__uint_as_float(sr[k])));
         }
       }
-      const bool need_mask = rows_valid < TP_ROWS || key0 + TP_KEYS - 1 > pf || (p.window > 0 && key0 < pl - p.window + 1);
+      const bool need_mask = rows_valid < TP_ROWS || key0 + TP_KEYS - 1 > pf || key0 < lo_last;
       if (need_mask) {
 #pragma unroll
         for (int k = 0; k < TP_KEYS; ++k) {
@@ -699,7 +700,7 @@ static int tp_launch(const void* q, long long q_row_stride, void* out, const voi
                      int tokens, int num_requests, int num_q, int num_kv, int head_dim, int page_size, int window,
                      float scale, long long num_pages, int* status, void* stream, float softcap, float* parts) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (tokens < 0 || num_requests <= 0 || max_pages <= 0 || window < 0) return ULLM_ERR_BAD_SIZE;
+  if (tokens < 0 || num_requests <= 0 || max_pages <= 0) return ULLM_ERR_BAD_SIZE;
   if (CAP && !(softcap > 0.f)) return ULLM_ERR_BAD_SIZE;
   if (PARTS && (parts == nullptr || ((uintptr_t)parts) % 16)) return ULLM_ERR_BAD_SIZE;
   if (!ullm_prefill_attention_pair_supported(head_dim, num_q, num_kv, page_size)) return ULLM_ERR_UNSUPPORTED;

@@ -250,7 +250,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     }
     return;
   }
-  const int key_lo = p.window > 0 ? max(0, p0 - p.window + 1) : 0;
+  const int key_lo = first_seen(p0, p.window);
   const int k_start = key_lo / TA_KEYS * TA_KEYS;
   const int tiles = (p1 - k_start) / TA_KEYS + 1;
   const int* bt = p.block_table + (long long)p.req_slots[r] * p.max_pages;
@@ -386,7 +386,8 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const int row = tid;
     const bool row_ok = row < rows_valid;
     const int pos = row_ok ? p0 + row / G : -1;
-    const int lo = p.window > 0 ? pos - p.window + 1 : 0;
+    const int lo = first_seen(pos, p.window);
+    const int lo_last = first_seen(p1, p.window);  // what the tile's last token sees first
     const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
@@ -400,7 +401,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       float s[TA_KEYS];
       ta_tmem_ld64(tmem_s + (t & 1) * TA_KEYS + lane_base, s);
-      const bool need_mask = rows_valid < TA_ROWS || key0 + TA_KEYS - 1 > p0 || (p.window > 0 && key0 < p1 - p.window + 1);
+      const bool need_mask = rows_valid < TA_ROWS || key0 + TA_KEYS - 1 > p0 || key0 < lo_last;
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < TA_KEYS; ++i) {
@@ -575,7 +576,7 @@ extern "C" int ullm_prefill_attention_tcgen05(const void* q, long long q_row_str
                                               int num_requests, int num_q, int num_kv, int head_dim, int page_size,
                                               int window, float scale, long long num_pages, int* status, void* stream) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (tokens < 0 || num_requests <= 0 || max_pages <= 0 || window < 0) return ULLM_ERR_BAD_SIZE;
+  if (tokens < 0 || num_requests <= 0 || max_pages <= 0) return ULLM_ERR_BAD_SIZE;
   if (!ullm_prefill_attention_tcgen05_supported(head_dim, num_q, num_kv, page_size)) return ULLM_ERR_UNSUPPORTED;
   if (q_row_stride % 8 || ((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16)
     return ULLM_ERR_UNSUPPORTED;

@@ -16,7 +16,8 @@
 // row size that is a multiple of 32 bytes the eight rows of an ldmatrix fall into distinct banks); value pages
 // of their own have one stage, awaited between the softmax and P V.  A block walks first the pooled entries its
 // rows can see (entry b stands for positions bP .. bP + P - 1 and is seen by a row at position i when
-// bP + P - 1 <= i - window), then the keys from the window's start of its first token to its last token.  All
+// bP + P - 1 <= i - window), then the keys from the first one that its first token
+// sees (the window's start, or the start of its stretch of positions) to its last token.  All
 // stretches share one online softmax.  For steps of few rows the tiles of a block are cut into runs (grid.y)
 // whose unnormalised results a second kernel merges.  The only waits are cp.async groups and block barriers.
 #include "common.cuh"
@@ -174,7 +175,7 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
     }
     return;
   }
-  const int key0 = W > 0 ? max(0, p0 - W + 1) : 0;
+  const int key0 = first_seen(p0, W);
   const int nb = (W > 0 && a.pool > 0 && p1 - W + 1 > 0) ? (p1 - W + 1) / a.pool : 0;  // pooled entries in sight
   const int ptiles = (nb + WIN_N - 1) / WIN_N;
   const int tiles = ptiles + (p1 - key0 + WIN_N) / WIN_N;
@@ -255,7 +256,7 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
     const int row = wrow + (lane >> 2) + h * 8;
     const bool valid = row < rows_valid;
     pos[h] = valid ? p0 + row / G : -1;
-    lo[h] = W > 0 ? pos[h] - W + 1 : 0;
+    lo[h] = first_seen(pos[h], W);
     nblk[h] = (valid && a.pool > 0 && W > 0 && lo[h] > 0) ? lo[h] / a.pool : 0;
     slope[h] = (valid && a.slopes != nullptr) ? a.slopes[kh * G + row % G] * log2e : 0.f;
     slope_pos[h] = -slope[h] * (float)pos[h];
@@ -265,7 +266,8 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
   const int w_last = min(rows_valid, wrow + 16) - 1;
   const int wp_max = warp_live ? p0 + w_last / G : -1;
   const int wp_min = p0 + wrow / G;
-  const int wp_lo = (warp_live && W > 0) ? wp_min - W + 1 : 0;
+  const int wp_lo = warp_live ? first_seen(wp_min, W) : 0;
+  const int wp_lo_last = warp_live ? first_seen(wp_max, W) : 0;  // what the warp's last row sees first
   const bool warp_full = wrow + 16 <= rows_valid;
   const int w_nblk = (warp_live && a.pool > 0 && W > 0 && wp_max - W + 1 > 0) ? (wp_max - W + 1) / a.pool : 0;
   const int c0 = cw * DVW;  // this warp's first value column
@@ -338,7 +340,7 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
         }
       }
       // ---- scale, distance bias, mask: scores in units of log2 from here on ------------------
-      const bool edge = pooled || !warp_full || kb + WIN_N - 1 > wp_min || (W > 0 && kb < wp_max - W + 1);
+      const bool edge = pooled || !warp_full || kb + WIN_N - 1 > wp_min || kb < wp_lo_last;
       if (has_slopes && !pooled) {
         // score * scale - slope (pos - key), as two multiply-adds per score
         const float kf = (float)(kb + (lane & 3) * 2);
@@ -578,7 +580,7 @@ extern "C" int ullm_window_attention(const void* q, long long q_row_stride, void
                                      int p_max_pages, long long p_num_pages, const void* gate, long long gate_stride,
                                      float out_scale, int nsplit, float* parts) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (tokens < 0 || num_requests <= 0 || page_size <= 0 || max_pages <= 0 || window < 0 || pool < 0)
+  if (tokens < 0 || num_requests <= 0 || page_size <= 0 || max_pages <= 0 || pool < 0)
     return ULLM_ERR_BAD_SIZE;
   if (!ullm_window_attention_supported(dk, dv, num_q, num_kv, v_cache == nullptr)) return ULLM_ERR_UNSUPPORTED;
   if (pool > 0 && (window <= 0 || pk == nullptr || p_block_table == nullptr || p_max_pages <= 0 || slopes != nullptr ||

@@ -47,6 +47,15 @@ __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { retu
 template <>
 __device__ __forceinline__ __half from_f32<__half>(float v) { return __float2half_rn(v); }
 
+// The first position that a query at `pos` sees, from the `window` argument that every attention kernel takes:
+// 0: position 0 (all earlier ones are seen);  w > 0: a sliding window, the last w positions;  -c < 0: the stretch of c
+// positions that holds `pos`, stretches being counted from position 0.  It never falls when `pos` grows, which is all
+// that the kernels' tile walks rely on.
+__device__ __forceinline__ int first_seen(int pos, int window) {
+  if (window > 0) return max(0, pos - window + 1);
+  return window < 0 ? pos - pos % (-window) : 0;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -89,6 +98,61 @@ template <typename T>
 __device__ __host__ __forceinline__ bool rows_are_16B(const void* p, long long cols, long long row_stride) {
   return (reinterpret_cast<uintptr_t>(p) % 16 == 0) && ((cols * sizeof(T)) % 16 == 0) &&
          ((row_stride * sizeof(T)) % 16 == 0);
+}
+
+// VEC neighbouring elements from / to p as 32-bit values: one 16-byte access when they are 16 bytes, else one by one.
+template <typename T, int VEC>
+__device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
+  if constexpr (VEC * sizeof(T) == 16) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = to_f32(e[i]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = to_f32(p[i]);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC * sizeof(T) == 16) {
+    uint4 raw;
+    T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) e[i] = from_f32<T>(v[i]);
+    *reinterpret_cast<uint4*>(p) = raw;
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) p[i] = from_f32<T>(v[i]);
+  }
+}
+// VEC 32-bit floats in 16-byte pieces (VEC a multiple of 4, p on a 16-byte border), else one by one.
+template <int VEC>
+__device__ __forceinline__ void load_vec32(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(p + i);
+      v[i] = x.x;
+      v[i + 1] = x.y;
+      v[i + 2] = x.z;
+      v[i + 3] = x.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = p[i];
+  }
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec32(float* p, const float (&v)[VEC]) {
+  if constexpr (VEC % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4)
+      *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) p[i] = v[i];
+  }
 }
 
 // Programmatic dependent launch.  Every kernel of this library starts with

@@ -2,7 +2,11 @@
 //
 //   moe_route     per token: scores from the 32-bit router logits (sigmoid, or softmax over the experts), the
 //                 `top` largest (ties: the lower index), their weights (the scores, optionally renormalized);
-//                 with a `correction` per expert the CHOICE goes by score + correction, the weight stays the score
+//                 with a `correction` per expert the CHOICE goes by score + correction, the weight stays the score;
+//                 with `groups` > 1 the experts form groups of neighbours, ranked by the sum of their two largest
+//                 ranks, and only experts of the best `keep` groups can be chosen; weights times `scale` at the end;
+//                 `always` further choices per token name the experts behind the routed ones, with weight 1 (shared
+//                 experts that ride along in the grouped product)
 //   moe_arrange   the (token, choice) pairs grouped by expert: offsets[E + 1], sorted[p] = pair at place p,
 //                 place[pair] = p
 //   moe_grouped_linear   for every expert e and every place p of it:  out[p] = f(W_e . (s_p * x[row(p)]))
@@ -15,7 +19,8 @@
 //                 sigmoid of one 32-bit number per token
 //
 // Gate activations of the grouped product: 0 silu(g) u, 1 gelu_tanh(g) u, 2 the clamped form
-// g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
+// g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).  Without gate rows the activation
+// is 3, max(v, 0)^2, or none (any other code).
 //
 // The grouped product is a tiled kernel with 32-bit accumulation for float32 and 16-bit storage alike; a block
 // finds its (expert, row tile) from the offsets, so the grid depends only on the step's size.
@@ -26,7 +31,8 @@
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long logits_stride,
                                  const float* __restrict__ correction, int* __restrict__ choice,
                                  float* __restrict__ weight, int tokens, int experts, int top, int softmax_scores,
-                                 int renormalize) {
+                                 int renormalize, int groups, int keep, float scale, int always) {
+  extern __shared__ float rt_smem[];  // per warp: a rank per group (only with groups)
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -40,6 +46,55 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long log
     for (int e = lane; e < experts; e += 32) zsum += expf(z[e] - zmax);
     zsum = warp_sum(zsum);
   }
+  auto score_of = [&](int e) { return softmax_scores ? expf(z[e] - zmax) / zsum : 1.f / (1.f + expf(-z[e])); };
+  // A chosen group's rank becomes +infinity; experts of all others are out.
+  float* g_rank = rt_smem + (threadIdx.x >> 5) * groups;
+  const int per = experts / groups;
+  const bool grouped = keep < groups;
+  if (grouped) {
+    for (int g = 0; g < groups; ++g) {
+      float a = -INFINITY, b = -INFINITY;  // the two largest ranks of this lane's experts
+      for (int i = lane; i < per; i += 32) {
+        const int e = g * per + i;
+        const float s = score_of(e), r = correction != nullptr ? s + correction[e] : s;
+        if (r > a) {
+          b = a;
+          a = r;
+        } else if (r > b) {
+          b = r;
+        }
+      }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+        b = fmaxf(fminf(a, oa), fmaxf(b, ob));
+        a = fmaxf(a, oa);
+      }
+      if (lane == 0) g_rank[g] = a + (per > 1 ? b : 0.f);
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      float best = -INFINITY;
+      int best_g = 0x7fffffff;
+      for (int g = lane; g < groups; g += 32) {
+        const float r = g_rank[g];
+        if (r < INFINITY && (best_g == 0x7fffffff || r > best)) {  // (ascending g: the lower index wins a tie)
+          best = r;
+          best_g = g;
+        }
+      }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+        if (og != 0x7fffffff && (best_g == 0x7fffffff || ob > best || (ob == best && og < best_g))) {
+          best = ob;
+          best_g = og;
+        }
+      }
+      if (lane == 0 && best_g < groups) g_rank[best_g] = INFINITY;
+      __syncwarp();
+    }
+  }
+  const int width = top + always;
   int taken[MOE_MAX_TOP];
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
@@ -48,8 +103,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long log
     for (int e = lane; e < experts; e += 32) {
       bool used = false;
       for (int j = 0; j < k; ++j) used |= taken[j] == e;
-      if (used) continue;
-      const float s = softmax_scores ? expf(z[e] - zmax) / zsum : 1.f / (1.f + expf(-z[e]));
+      if (used || (grouped && g_rank[e / per] < INFINITY)) continue;
+      const float s = score_of(e);
       const float rank = correction != nullptr ? s + correction[e] : s;
       if (rank > best || (rank == best && e < best_e)) {
         best = rank;
@@ -70,12 +125,16 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long log
     taken[k] = best_e;
     total += best_s;
     if (lane == 0) {
-      choice[(long long)t * top + k] = best_e;
-      weight[(long long)t * top + k] = best_s;
+      choice[(long long)t * width + k] = best_e;
+      weight[(long long)t * width + k] = renormalize ? best_s : best_s * scale;
     }
   }
   if (renormalize && lane == 0)
-    for (int k = 0; k < top; ++k) weight[(long long)t * top + k] /= total;
+    for (int k = 0; k < top; ++k) weight[(long long)t * width + k] = weight[(long long)t * width + k] / total * scale;
+  if (lane < always) {
+    choice[(long long)t * width + top + lane] = experts + lane;
+    weight[(long long)t * width + top + lane] = 1.f;
+  }
 }
 
 // One block.  counts in shared memory (experts <= 1024).
@@ -109,6 +168,8 @@ __global__ void moe_arrange_kernel(const int* __restrict__ choice, int pairs, in
       const int at = atomicAdd(&cursor[e], 1);
       sorted[at] = p;
       place[p] = at;
+    } else {
+      place[p] = 0;  // (no expert's row: whoever combines must not find an index that was never written)
     }
   }
 }
@@ -120,6 +181,15 @@ __device__ __forceinline__ float moe_gate_act(int act, float g, float u, float l
     return g / (1.f + expf(-alpha * g)) * (u + 1.f);
   }
   return (act == 0 ? act_silu(g) : act_gelu_tanh(g)) * u;
+}
+
+// the activation of a product without gate rows
+__device__ __forceinline__ float moe_plain_act(int act, float v) {
+  if (act == 3) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return v;
 }
 
 #define MOE_BM 32
@@ -217,7 +287,7 @@ moe_grouped_linear_kernel(const T* __restrict__ x, long long x_stride, const T* 
         const float g = acc[0][i][j] * sc, u = acc[1][i][j] * sc;
         v = moe_gate_act(act, g, u, limit, alpha);
       } else {
-        v = acc[0][i][j] * sc;
+        v = moe_plain_act(act, acc[0][i][j] * sc);
       }
       out[(long long)(p0 + r) * n_out + c] = from_f32<T>(v);
     }
@@ -379,25 +449,11 @@ moe_grouped_mma_kernel(const __nv_bfloat16* __restrict__ x, long long x_stride,
           const float gt = acc[0][t][2 * h + j] * sc, up = acc[NB - 1][t][2 * h + j] * sc;
           v[j] = moe_gate_act(act, gt, up, limit, alpha);
         } else {
-          v[j] = acc[0][t][2 * h + j] * sc;
+          v[j] = moe_plain_act(act, acc[0][t][2 * h + j] * sc);
         }
       }
       *reinterpret_cast<__nv_bfloat162*>(out + (long long)(p0 + r) * n_out + c) = __floats2bfloat162_rn(v[0], v[1]);
     }
-  }
-}
-
-// VEC elements of T from p to 32-bit: one 16-byte load when VEC elements are 16 bytes, else element by element.
-template <typename T, int VEC>
-__device__ __forceinline__ void moe_load_vec(const T* __restrict__ p, float (&out)[VEC]) {
-  if constexpr (VEC * sizeof(T) == 16) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(p);
-    const T* e = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) out[i] = to_f32(e[i]);
-  } else {
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) out[i] = to_f32(p[i]);
   }
 }
 
@@ -420,14 +476,14 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
     const long long pair = t * top + k;
     const bool passes = choice != nullptr && choice[pair] >= experts;  // an expert that is its input
     const T* src = passes ? x + t * x_stride : rows + (long long)place[pair] * cols;
-    moe_load_vec<T, VEC>(src + c0, v);
+    load_vec<T, VEC>(src + c0, v);
     const float w = pair_weight != nullptr ? pair_weight[pair] : 1.f;
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] += w * v[i];
   }
   if (shared_rows != nullptr) {
     const float sg = shared_gate != nullptr ? 1.f / (1.f + expf(-shared_gate[t * gate_stride])) : 1.f;
-    moe_load_vec<T, VEC>(shared_rows + t * cols + c0, v);
+    load_vec<T, VEC>(shared_rows + t * cols + c0, v);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] += sg * v[i];
   }
@@ -444,8 +500,8 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
 }
 
 // The same sum, added to a 32-bit residual stream instead of stored, with a scale per channel, and followed by the
-// RMS norm that reads the stream next:  stream[t] += scale * y[t];  out[t] = w2 * stream[t] / sqrt(mean(stream[t]^2) +
-// eps2).  One block per token; the sum never leaves 32-bit.  `x` (the passing experts' input) and `out` may be the
+// norm that reads the stream next:  stream[t] += scale * y[t];  out[t] = w2 * stream[t] / sqrt(mean(stream[t]^2) +
+// eps2), or with `alpha2` (one number) and `b2`: out[t] = tanh(alpha2 * stream[t]) * w2 + b2.  One block per token; the sum never leaves 32-bit.  `x` (the passing experts' input) and `out` may be the
 // same rows: a block reads its token's row of x before the barrier and writes its row of out behind it.
 template <typename T, int VEC>
 __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const int* __restrict__ place,
@@ -454,7 +510,8 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
                                             long long x_stride, const T* __restrict__ shared_rows,
                                             const float* __restrict__ shared_gate, long long gate_stride,
                                             float* __restrict__ stream, const float* __restrict__ scale,
-                                            const float* __restrict__ w2, float eps2, T* out) {
+                                            const float* __restrict__ w2, float eps2, T* out,
+                                            const float* __restrict__ alpha2, const float* __restrict__ b2) {
   extern __shared__ __align__(16) float mc_row[];
   __shared__ float scratch[33];
   pdl_launch_dependents();
@@ -471,13 +528,13 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
       const long long pair = t * top + k;
       const bool passes = choice != nullptr && choice[pair] >= experts;
       const T* src = passes ? x + t * x_stride : rows + (long long)place[pair] * cols;
-      moe_load_vec<T, VEC>(src + c0, v);
+      load_vec<T, VEC>(src + c0, v);
       const float w = pair_weight != nullptr ? pair_weight[pair] : 1.f;
 #pragma unroll
       for (int i = 0; i < VEC; ++i) acc[i] += w * v[i];
     }
     if (shared_rows != nullptr) {
-      moe_load_vec<T, VEC>(shared_rows + t * cols + c0, v);
+      load_vec<T, VEC>(shared_rows + t * cols + c0, v);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) acc[i] += sg * v[i];
     }
@@ -508,6 +565,20 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
     }
   }
   if (out == nullptr) return;
+  if (alpha2 != nullptr) {
+    // no statistics: a thread reads back what it wrote itself.  (No barrier is needed for x == out either: a thread
+    // overwrites only columns that it alone has read.)
+    const float al = *alpha2;
+    for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+      float v[VEC], g[VEC], d[VEC];
+      load_vec32<VEC>(w2 + c0, g);
+      load_vec32<VEC>(b2 + c0, d);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = tanhf(al * mc_row[c0 + i]) * g[i] + d[i];
+      store_vec<T, VEC>(out + t * cols + c0, v);
+    }
+    return;
+  }
   const float rstd = 1.f / sqrtf(block_sum(sq, scratch) / (float)cols + eps2);
   if constexpr (VEC * sizeof(T) == 16) {
     for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
@@ -527,16 +598,20 @@ static int g_moe_force_plain = 0;
 extern "C" void ullm_moe_force_plain(int on) { g_moe_force_plain = on ? 1 : 0; }
 
 // `logits_stride`: floats between two tokens' rows (the rows may hold further columns behind the experts');
-// `correction` (null: none): added to the scores for the choice only.
+// `correction` (null: none): added to the scores for the choice only.  `groups` / `keep`: 1 / 1 for a choice over all
+// experts.  `choice` and `weight` hold top + `always` entries per token.
 extern "C" int ullm_moe_route(const float* logits, long long logits_stride, const float* correction, int* choice,
                               float* weight, int tokens, int experts, int top, int softmax_scores, int renormalize,
-                              void* stream) {
+                              int groups, int keep, float scale, int always, void* stream) {
   if (tokens < 0 || experts <= 0 || top <= 0 || logits_stride < experts) return ULLM_ERR_BAD_SIZE;
-  if (top > experts || top > MOE_MAX_TOP) return ULLM_ERR_UNSUPPORTED;
+  if (groups < 1 || keep < 1 || keep > groups || experts % groups || always < 0 || always > 32) return ULLM_ERR_BAD_SIZE;
+  if (top > keep * (experts / groups) || top > MOE_MAX_TOP) return ULLM_ERR_UNSUPPORTED;
+  const size_t smem = keep < groups ? (size_t)4 * groups * sizeof(float) : 0;
+  if (smem > 48 * 1024) return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;
-  return ullm_launch_kernel(moe_route_kernel, dim3((tokens + 3) / 4), dim3(128), 0, (cudaStream_t)stream, logits,
+  return ullm_launch_kernel(moe_route_kernel, dim3((tokens + 3) / 4), dim3(128), smem, (cudaStream_t)stream, logits,
                             logits_stride, correction, choice, weight, tokens, experts, top, softmax_scores,
-                            renormalize);
+                            renormalize, groups, keep, scale, always);
 }
 
 extern "C" int ullm_moe_arrange(const int* choice, int pairs, int experts, int* offsets, int* sorted, int* place,
@@ -657,16 +732,18 @@ extern "C" int ullm_moe_combine(int dtype, const void* rows, const int* place, c
 }
 
 // stream (32-bit, [tokens, cols], in place) += scale * (the sum `ullm_moe_combine` forms); `scale` null: 1.  `out` with
-// `w2` (null: none): the RMS norm of the updated rows, in the rows' dtype; `out` may be `x`.
+// `w2` (null: none): the RMS norm of the updated rows (with `alpha2` and `b2`: the tanh norm), in the rows' dtype; `out`
+// may be `x`.
 extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int* place, const float* pair_weight,
                                          int tokens, int top, int cols, const int* choice, int experts, const void* x,
                                          long long x_stride, const void* shared_rows, const float* shared_gate,
                                          long long gate_stride, float* stream_rows, const float* scale,
-                                         const float* w2, float eps2, void* out, void* stream) {
+                                         const float* w2, float eps2, void* out, void* stream, const float* alpha2,
+                                         const float* b2) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || top <= 0 || cols <= 0 || stream_rows == nullptr) return ULLM_ERR_BAD_SIZE;
   if (choice != nullptr && (x == nullptr || x_stride < cols || experts < 0)) return ULLM_ERR_BAD_SIZE;
-  if (out != nullptr && w2 == nullptr) return ULLM_ERR_BAD_SIZE;
+  if (out != nullptr && (w2 == nullptr || (alpha2 == nullptr) != (b2 == nullptr))) return ULLM_ERR_BAD_SIZE;
   const size_t smem = (size_t)cols * sizeof(float);
   if (smem > 160 * 1024) return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;
@@ -674,7 +751,7 @@ extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int*
   const int vec = 16 / esize;
   const bool wide = cols % vec == 0 && x_stride % vec == 0 &&
                     (((uintptr_t)rows | (uintptr_t)x | (uintptr_t)shared_rows | (uintptr_t)stream_rows |
-                      (uintptr_t)scale | (uintptr_t)w2 | (uintptr_t)out) & 15) == 0;
+                      (uintptr_t)scale | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out) & 15) == 0;
   const int per_thread = wide ? vec : 1;
   int threads = 32;
   while (threads < 256 && threads * per_thread < cols) threads <<= 1;
@@ -688,7 +765,7 @@ extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int*
     }                                                                                                                  \
     return ullm_launch_kernel(moe_combine_add_norm_kernel<T, V>, grid, block, smem, st, (const T*)rows, place,         \
                               pair_weight, top, cols, choice, experts, (const T*)x, x_stride, (const T*)shared_rows,   \
-                              shared_gate, gate_stride, stream_rows, scale, w2, eps2, (T*)out);                        \
+                              shared_gate, gate_stride, stream_rows, scale, w2, eps2, (T*)out, alpha2, b2);            \
   }
   if (dtype == ULLM_DTYPE_F32) {
     if (wide) MCA_GO(float, 4);

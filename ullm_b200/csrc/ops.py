@@ -263,8 +263,14 @@ class Kernels:
                                       P, I, LL, P, LL, F, I, P],
             "ullm_paged_attention_generic_ex3": [I, P, LL, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, LL, P, P, I, I,
                                                  F, P, I, I, P, P, P, I, LL, P, LL, F, LL],
-            "ullm_norm_add_norm": [I, P, P, P, I, I, F, F, I, P, P, P, F, I, I, P, P],
-            "ullm_norm_rows": [I, P, P, P, P, I, I, I, F, I, P, P],
+            "ullm_norm_add_norm": [I, P, P, P, I, I, F, F, I, P, P, P, F, I, I, P, P, P, P],
+            "ullm_pair_norm_add_norm": [I, P, P, P, P, I, I, F, F, P, P, P, F, I, P, P, P, P],
+            "ullm_relu2": [I, P, P, LL, P],
+            "ullm_scale_f32": [P, LL, F, P],
+            "ullm_ssd_prepare": [I, P, LL, I, I, I, I, P, I, P, P, P, P, LL, I, P, P, P, I, P, P, P, P, P],
+            "ullm_ssd_recurrence": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
+            "ullm_ssd_gate_norm": [I, P, P, LL, P, P, I, I, I, F, P],
+            "ullm_norm_rows": [I, P, P, P, P, I, I, I, F, I, P, P, P, P],
             "ullm_xielu": [I, P, P, LL, P, P],
             "ullm_kv_shared_prepare": [I, P, LL, I, I, I, P, P, F, P, P, P, LL, P, P],
             "ullm_pool_blocks": [I, P, P, P, P, I, I, LL, P, P, I, I, P, LL, P, P, I, I, P, P],
@@ -275,11 +281,11 @@ class Kernels:
             "ullm_mingru": [I, P, LL, I, I, I, P, P, P, LL, P, P, P, P, LL, F, I, I, I, P, P],
             "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P],
             "ullm_head_norm_gate": [I, P, P, LL, P, P, I, I, I, F, I, I, P],
-            "ullm_moe_route": [P, LL, P, P, P, I, I, I, I, I, P],
+            "ullm_moe_route": [P, LL, P, P, P, I, I, I, I, I, I, I, F, I, P],
             "ullm_moe_arrange": [P, I, I, P, P, P, P],
             "ullm_moe_grouped_linear": [I, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],
             "ullm_moe_combine": [I, P, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P],
-            "ullm_moe_combine_add_norm": [I, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P, P, P, F, P, P],
+            "ullm_moe_combine_add_norm": [I, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P, P, P, F, P, P, P, P],
             "ullm_argmax": [P, LL, I, I, P, P],
             "ullm_sample": [P, LL, I, I, P, P, P, P, P, P, P, P, P, P],
         }
@@ -299,6 +305,8 @@ class Kernels:
         L.ullm_gla_supported.restype = c_int
         L.ullm_gla_state_floats.argtypes = [I, I, I]
         L.ullm_gla_state_floats.restype = c_longlong
+        L.ullm_ssd_supported.argtypes = [I, I, I, I, I]
+        L.ullm_ssd_supported.restype = c_int
         L.ullm_wait_selftest.argtypes = [I, P, P, P]
         L.ullm_wait_selftest.restype = c_int
         L.ullm_decode_attention_supported.argtypes = [I, I, I]
@@ -848,11 +856,34 @@ class Kernels:
                                                   float(alpha), _stream()), "act_mul_clamped")
 
     # -- norms on both sides of a sub-layer, on a 32-bit stream -------------------
+    @staticmethod
+    def _next_norm(what, next_norm, rows: int, cols: int):
+        """(weight, eps, kind, alpha, bias, out) of a `next_norm` argument: None, or `Norm.row_params()` with the
+        output rows behind it.  Kinds: 0 RMS, 1 centred, 2 tanh."""
+        if next_norm is None:
+            return None, 0.0, 0, None, None, None
+        (w, eps, *more), out = next_norm[:-1], next_norm[-1]
+        kind = int(more[0]) if more else 0
+        alpha, bias = more[1:] if len(more) > 1 else (None, None)
+        _need(w, "next norm weight", torch.float32)
+        _need(out, "out")
+        if out.shape != (rows, cols) or w.numel() != cols:
+            raise KernelError(f"{what}: the next norm's shapes differ")
+        if (kind == 2) != (alpha is not None):
+            raise KernelError(f"{what}: the tanh norm comes with a slope and a bias, the others without")
+        if alpha is not None:
+            _need(alpha, "next norm slope", torch.float32)
+            _need(bias, "next norm bias", torch.float32)
+            if alpha.numel() != 1 or bias.numel() != cols:
+                raise KernelError(f"{what}: the next norm's slope is one number, its bias as long as the row")
+        return w, float(eps), kind, alpha, bias, out
+
     @_timed("add_rmsnorm")
     def norm_add_norm(self, stream, a=None, weight=None, eps: float = 0.0, mult: float = 1.0, center: bool = False,
                       extra_rows=None, extra_vec=None, next_norm=None, plain: bool = False):
         """stream (float32, in place) += mult * weight * n(a), then += extra_rows, then += extra_vec (each part
-        optional); `next_norm` = (weight2, eps2, center2, out): out = weight2 * n2(stream) rounded to out's dtype.
+        optional); `next_norm` = (weight2, eps2, center2, out): out = weight2 * n2(stream) rounded to out's dtype, or
+        (weight2, eps2, 2, alpha2, bias2, out): out = tanh(alpha2 * stream) * weight2 + bias2 (see `Norm.row_params`).
         n(v) = v / sqrt(mean(v^2) + eps), with `center` (v - mean) / sqrt(mean((v - mean)^2) + eps); with `plain`
         n(v) = v (a is only scaled channel by channel; `weight` None: not even that)."""
         _need(stream, "stream", torch.float32)
@@ -871,23 +902,16 @@ class Kernels:
             _need(extra_vec, "extra_vec", torch.float32)
             if extra_vec.numel() != cols:
                 raise KernelError("norm_add_norm: the added vector's length differs from the stream's width")
-        w2 = out = None
-        eps2, center2 = 0.0, False
-        if next_norm is not None:
-            w2, eps2, center2, out = next_norm
-            _need(w2, "next norm weight", torch.float32)
-            _need(out, "out")
-            if out.shape != stream.shape or w2.numel() != cols:
-                raise KernelError("norm_add_norm: the next norm's shapes differ")
+        w2, eps2, kind2, alpha2, b2, out = self._next_norm("norm_add_norm", next_norm, rows, cols)
         self._check(self.lib.ullm_norm_add_norm(
             _DT[a.dtype] if a is not None else 0, _ptr(a), _ptr(stream), _ptr(weight), rows, cols, float(eps), float(mult),
-            2 if plain else int(bool(center)), _ptr(extra_rows), _ptr(extra_vec), _ptr(w2), float(eps2), int(bool(center2)),
-            _DT[out.dtype] if out is not None else 0, _ptr(out), _stream()), f"norm_add_norm (row length {cols})")
+            2 if plain else int(bool(center)), _ptr(extra_rows), _ptr(extra_vec), _ptr(w2), float(eps2), kind2,
+            _DT[out.dtype] if out is not None else 0, _ptr(out), _stream(), _ptr(alpha2), _ptr(b2)), f"norm_add_norm (row length {cols})")
 
     @_timed("add_rmsnorm")
-    def norm_rows(self, stream, rows, weight, eps: float, out, center: bool = False):
+    def norm_rows(self, stream, rows, weight, eps: float, out, center: bool = False, alpha=None, bias=None):
         """out[r] = weight * n(stream[rows[r]]) (float32 stream; `rows` int32, or None for all rows in order),
-        rounded to out's dtype; n as in `norm_add_norm`."""
+        rounded to out's dtype; n as in `norm_add_norm`.  With `alpha` and `bias`: tanh(alpha * row) * weight + bias."""
         _need(stream, "stream", torch.float32)
         _need(weight, "weight", torch.float32)
         _need(out, "out")
@@ -898,9 +922,52 @@ class Kernels:
             _need(rows, "rows", torch.int32)
             if rows.numel() < R:
                 raise KernelError("norm_rows: fewer row indices than output rows")
+        if alpha is not None:
+            _need(alpha, "alpha", torch.float32)
+            _need(bias, "bias", torch.float32)
+            if alpha.numel() != 1 or bias.numel() != C:
+                raise KernelError("norm_rows: the slope is one number, the bias as long as the row")
         self._check(self.lib.ullm_norm_rows(_DT[out.dtype], _ptr(stream), _ptr(rows), _ptr(weight), _ptr(out), R, C,
-                                            stream.shape[0], float(eps), int(bool(center)), _ptr(self.status),
-                                            _stream()), f"norm_rows (row length {C})")
+                                            stream.shape[0], float(eps), 2 if alpha is not None else int(bool(center)),
+                                            _ptr(self.status), _stream(), _ptr(alpha), _ptr(bias)),
+                    f"norm_rows (row length {C})")
+
+    @_timed("add_rmsnorm")
+    def pair_norm_add_norm(self, a, b, weight_a, weight_b, eps: float, mult: float, stream=None, rows_out=None,
+                           next_norm=None):
+        """s = mult * (weight_a * n(a) + weight_b * n(b)), n(v) = v / sqrt(mean(v^2) + eps), for two sub-layers' rows
+        [T, W]; stream (float32, in place) += s, and / or rows_out = s (of the stream's sum, when both are given);
+        `next_norm` as in `norm_add_norm`, of the updated stream."""
+        _need(a, "a")
+        _need(b, "b", a.dtype)
+        _need(weight_a, "weight_a", torch.float32)
+        _need(weight_b, "weight_b", torch.float32)
+        T, W = a.shape
+        if b.shape != a.shape or weight_a.numel() != W or weight_b.numel() != W:
+            raise KernelError(f"pair_norm_add_norm: a {tuple(a.shape)}, b {tuple(b.shape)}")
+        if stream is not None:
+            _need(stream, "stream", torch.float32)
+        if rows_out is not None:
+            _need(rows_out, "rows_out", a.dtype)
+        for t in (stream, rows_out):
+            if t is not None and t.shape != a.shape:
+                raise KernelError("pair_norm_add_norm: the rows' shapes differ")
+        w2, eps2, kind2, alpha2, b2, out = self._next_norm("pair_norm_add_norm", next_norm, T, W)
+        if out is not None:
+            _need(out, "out", a.dtype)
+        self._check(self.lib.ullm_pair_norm_add_norm(
+            _DT[a.dtype], _ptr(a), _ptr(b), _ptr(weight_a), _ptr(weight_b), T, W, float(eps), float(mult), _ptr(stream),
+            _ptr(rows_out), _ptr(w2), eps2, kind2, _ptr(alpha2), _ptr(b2), _ptr(out), _stream()),
+            f"pair_norm_add_norm (row length {W})")
+
+    @_timed("act_mul")
+    def relu2(self, x, out):
+        """out = max(x, 0)^2 (`out` may be x)."""
+        _need(x, "x")
+        _need(out, "out", x.dtype)
+        if out.numel() != x.numel():
+            raise KernelError("relu2: shapes differ")
+        self._check(self.lib.ullm_relu2(_DT[x.dtype], _ptr(x), _ptr(out), x.numel(), _stream()), "relu2")
 
     @_timed("act_mul")
     def xielu(self, x, pq, out):
@@ -1069,7 +1136,7 @@ class Kernels:
                            num_kv: int, head_dim: int, v_dim: int, page_size: int, window: int, scale: float, *,
                            slopes=None, pool: int = 0, pooled=None, gate=None, out_scale: float = 1.0,
                            num_requests: int | None = None, workspace=None):
-        """Windowed attention with its further options: in bfloat16, at sizes `ullm_window_attention_supported`
+        """Windowed attention (`window` as in `paged_attention`) with its further options: in bfloat16, at sizes `ullm_window_attention_supported`
         takes and with `num_requests` (the batch rows that `cu_q` describes) given, the tensor-core kernel of
         csrc/attention_window.cu; otherwise (32-bit storage, other sizes) the general kernel.  With a `workspace`
         a step of few rows cuts every row's keys into runs that run side by side (`_window_splits`).  `v_pages` None: a head's values are the first
@@ -1145,12 +1212,12 @@ class Kernels:
     def _window_splits(self, T: int, requests: int, num_q: int, num_kv: int, window: int) -> int:
         """Into how many runs `windowed_attention` cuts a row's key tiles: one while the step's blocks (64 rows of
         a kv head each) fill half of the SMs; otherwise as many as bring two blocks per SM, at most one run per
-        key tile of the window (32 without a window) and 64."""
+        key tile of the window or stretch (32 without a window) and 64."""
         tokens_per_block = max(1, 64 // (num_q // num_kv))
         blocks = (max(requests, -(-T // tokens_per_block))) * num_kv
         if 2 * blocks >= self.sm_count:
             return 1
-        most = -(-window // 64) + 1 if window > 0 else 32
+        most = -(-abs(window) // 64) + 1 if window else 32
         return max(1, min(-(-2 * self.sm_count // blocks), most, 64))
 
     # -- minGRU -------------------------------------------------------------------
@@ -1336,6 +1403,85 @@ class Kernels:
         _need(x, "x", torch.float32)
         self._check(self.lib.ullm_softcap_f32(_ptr(x), x.numel(), float(cap), _stream()), "softcap_f32")
 
+    @_timed("linear_head")
+    def scale_f32(self, x, factor: float):
+        """x (float32, in place) = factor * x."""
+        _need(x, "x", torch.float32)
+        self._check(self.lib.ullm_scale_f32(_ptr(x), x.numel(), float(factor), _stream()), "scale_f32")
+
+    # -- a state-space recurrence with a scalar decay per head (csrc/ssd.cu) ----------------------
+    def ssd_supported(self, heads: int, n_state: int, pdim: int, groups: int, taps: int) -> bool:
+        return bool(self.lib.ullm_ssd_supported(heads, n_state, pdim, groups, taps))
+
+    @_timed("ssd")
+    def ssd_prepare(self, u, xbc_off: int, dt_off: int, conv_w, conv_b, dt_bias, a_log, conv_state, cu_q, token_req,
+                    req_slots, xbc, dt, log_decay):
+        """u [T, *]: the projection's rows, x | B | C from column `xbc_off` and dt from `dt_off`; conv_w [channels, taps],
+        conv_b [channels], dt_bias and a_log [heads] (float32); conv_state: the convolution's columns of the state rows
+        [slots, (taps - 1) * channels] (a view of wider rows).  Out: xbc [T, channels], dt and log_decay [T, heads]."""
+        _need(u, "u", contiguous=False)
+        _need(conv_w, "conv_w", u.dtype)
+        _need(xbc, "xbc", u.dtype)
+        for t_, n_ in ((conv_b, "conv bias"), (dt_bias, "dt_bias"), (a_log, "a_log"), (dt, "dt"), (log_decay, "log_decay")):
+            _need(t_, n_, torch.float32)
+        for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
+            _need(t_, n_, torch.int32)
+        T, heads = u.shape[0], dt_bias.numel()
+        channels, taps = conv_w.shape
+        if (u.stride(1) != 1 or xbc.shape != (T, channels) or dt.shape != (T, heads) or log_decay.shape != (T, heads)
+                or xbc_off + channels > u.shape[1] or dt_off + heads > u.shape[1] or conv_b.numel() != channels
+                or a_log.numel() != heads):
+            raise KernelError(f"ssd_prepare: u {tuple(u.shape)}, xbc {tuple(xbc.shape)}, dt {tuple(dt.shape)}")
+        stride = slots = 0
+        if taps > 1:
+            _need(conv_state, "conv_state", torch.float32, contiguous=False)
+            if conv_state.dim() != 2 or conv_state.stride(1) != 1 or conv_state.shape[1] < (taps - 1) * channels:
+                raise KernelError(f"ssd_prepare: conv_state {tuple(conv_state.shape)} is too small")
+            stride, slots = conv_state.stride(0), conv_state.shape[0]
+        self._check(self.lib.ullm_ssd_prepare(
+            _DT[u.dtype], _ptr(u), u.stride(0), xbc_off, dt_off, channels, heads, _ptr(conv_w), taps, _ptr(conv_b),
+            _ptr(dt_bias), _ptr(a_log), _ptr(conv_state if taps > 1 else None), stride, slots, _ptr(cu_q), _ptr(token_req),
+            _ptr(req_slots), T, _ptr(xbc), _ptr(dt), _ptr(log_decay), _ptr(self.status), _stream()),
+            f"ssd_prepare ({channels} channels, {taps} taps)")
+
+    @_timed("ssd")
+    def ssd_recurrence(self, xbc, b_off: int, c_off: int, dt, log_decay, d_skip, state, cu_q, req_slots, token_req, out,
+                       requests: int, heads: int, n_state: int, pdim: int, groups: int, most_tokens: int = 1 << 30):
+        """The recurrence over the step's tokens, from and into the requests' state rows (float32
+        [slots, >= heads * pdim * n_state]); out [T, heads * pdim] float32.  Requests that bring more than
+        `most_tokens` tokens are left alone."""
+        _need(xbc, "xbc")
+        _need(state, "state", torch.float32, contiguous=False)
+        for t_, n_ in ((dt, "dt"), (log_decay, "log_decay"), (d_skip, "d_skip"), (out, "out")):
+            _need(t_, n_, torch.float32)
+        for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
+            _need(t_, n_, torch.int32)
+        T = xbc.shape[0]
+        if (dt.shape != (T, heads) or log_decay.shape != (T, heads) or out.shape != (T, heads * pdim) or state.dim() != 2
+                or state.stride(1) != 1 or state.shape[1] < heads * pdim * n_state or d_skip.numel() != heads):
+            raise KernelError(f"ssd_recurrence: xbc {tuple(xbc.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+        if max(b_off, c_off) + groups * n_state > xbc.shape[1] or heads * pdim > xbc.shape[1]:
+            raise KernelError("ssd_recurrence: x, B or C lie outside the rows")
+        self._check(self.lib.ullm_ssd_recurrence(
+            _DT[xbc.dtype], _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(state),
+            state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), requests, heads, n_state, pdim,
+            groups, state.shape[0], int(most_tokens), _ptr(self.status), _stream()),
+            f"ssd_recurrence (heads {heads}, state {n_state}, columns {pdim})")
+
+    @_timed("ssd")
+    def ssd_gate_norm(self, y, z, weight, parts: int, eps: float, out):
+        """out = weight * n(y * silu(z)), n over `parts` equal stretches of the row; y [T, inner] float32, z a view
+        [T, inner] of the projection's rows (any row stride)."""
+        _need(y, "y", torch.float32)
+        _need(z, "z", out.dtype, contiguous=False)
+        _need(weight, "weight", torch.float32)
+        _need(out, "out")
+        T, inner = y.shape
+        if z.shape != y.shape or out.shape != y.shape or z.stride(1) != 1 or weight.numel() != inner or inner % parts:
+            raise KernelError(f"ssd_gate_norm: y {tuple(y.shape)}, z {tuple(z.shape)}, {parts} parts")
+        self._check(self.lib.ullm_ssd_gate_norm(_DT[out.dtype], _ptr(y), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), T,
+                                                inner, int(parts), float(eps), _stream()), "ssd_gate_norm")
+
     # -- between an attention's projection and its scores, in general form ----------------
     @_timed("qk_norm_rope_store")
     def qkv_prepare(self, qkv, q_out, num_q, num_kv, head_dim, v_dim, positions, slot_mapping, k_pages, v_pages, *,
@@ -1344,10 +1490,10 @@ class Kernels:
                     norm_last: bool = False, eps: float = 0.0, vmix_mode: int = 0, vmix_lambda=None, v_first=None):
         """See csrc/attention_prep.cu: short convolution (with the requests' state rows), norm, rotation by computed
         angles, unit norm, value mixing, cache stores; q goes to `q_out` [T, num_q * head_dim]."""
-        _need(qkv, "qkv")
+        _need(qkv, "qkv", contiguous=False)
         _need(q_out, "q_out", qkv.dtype)
         T, W = qkv.shape
-        if W != num_q * head_dim + num_kv * (head_dim + v_dim) or q_out.shape != (T, num_q * head_dim):
+        if qkv.stride(1) != 1 or W != num_q * head_dim + num_kv * (head_dim + v_dim) or q_out.shape != (T, num_q * head_dim):
             raise KernelError(f"qkv_prepare: qkv {tuple(qkv.shape)}, q_out {tuple(q_out.shape)}")
         for t_, n_ in ((token_req, "token_req"), (positions, "positions")):
             _need(t_, n_, torch.int32)
@@ -1390,10 +1536,12 @@ class Kernels:
     @_timed("qk_norm_rope_store")
     def conv_state_update(self, qkv, taps: int, conv_state, cu_q, token_req, req_slots, requests: int):
         """After `qkv_prepare` of a step: the requests' state rows take the last taps - 1 projected rows."""
-        _need(qkv, "qkv")
-        _need(conv_state, "conv_state", torch.float32)
+        _need(qkv, "qkv", contiguous=False)
+        _need(conv_state, "conv_state", torch.float32, contiguous=False)
         for t_, n_ in ((cu_q, "cu_q"), (token_req, "token_req"), (req_slots, "req_slots")):
             _need(t_, n_, torch.int32)
+        if (qkv.stride(1) != 1 or conv_state.stride(1) != 1 or conv_state.shape[1] < (taps - 1) * qkv.shape[1]):
+            raise KernelError(f"conv_state_update: rows {tuple(qkv.shape)}, conv_state {tuple(conv_state.shape)}")
         self._check(self.lib.ullm_conv_state_update(_DT[qkv.dtype], _ptr(qkv), qkv.stride(0), qkv.shape[1], int(taps),
                                                     _ptr(conv_state), conv_state.stride(0), _ptr(cu_q), _ptr(token_req),
                                                     _ptr(req_slots), conv_state.shape[0], int(requests), _stream()),
@@ -1414,22 +1562,27 @@ class Kernels:
     # -- routed experts -----------------------------------------------------------
     @_timed("moe")
     def moe_route(self, logits, choice, weight, top: int, softmax_scores: bool = False, renormalize: bool = False,
-                  correction=None, experts: int | None = None):
+                  correction=None, experts: int | None = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
+                  always: int = 0):
         """`experts`: the router's outputs, when the logits' rows hold further columns behind them.  `correction`
-        (float32 [experts]): added to the scores for the choice; the weights stay the scores."""
+        (float32 [experts]): added to the scores for the choice; the weights stay the scores.  `groups` / `keep`: only
+        experts of the `keep` groups of neighbours with the largest sum of two best ranks can be chosen.  `scale`
+        multiplies the weights.  `always` n: choices `top` .. `top + n - 1` of every token are `experts` .. with
+        weight 1 (`choice` and `weight` hold top + n entries per token)."""
         _need(logits, "router logits", torch.float32)
         _need(choice, "choice", torch.int32)
         _need(weight, "weight", torch.float32)
         T = logits.shape[0]
         E = logits.shape[1] if experts is None else int(experts)
-        if choice.numel() < T * top or weight.numel() < T * top or E > logits.shape[1]:
+        if choice.numel() < T * (top + always) or weight.numel() < T * (top + always) or E > logits.shape[1]:
             raise KernelError("moe_route: outputs too small")
         if correction is not None:
             _need(correction, "correction", torch.float32)
             if correction.numel() != E:
                 raise KernelError(f"moe_route: {correction.numel()} corrections for {E} router outputs")
         self._check(self.lib.ullm_moe_route(_ptr(logits), logits.stride(0), _ptr(correction), _ptr(choice), _ptr(weight), T,
-                                            E, top, int(softmax_scores), int(renormalize), _stream()),
+                                            E, top, int(softmax_scores), int(renormalize), int(groups), int(keep),
+                                            float(scale), int(always), _stream()),
                     f"moe_route ({E} experts, top {top})")
 
     @_timed("moe")
@@ -1445,7 +1598,8 @@ class Kernels:
     def moe_grouped_linear(self, x, weights, offsets, sorted_pairs, pair_weight, out, top: int, rows_from_pairs: bool,
                            gated: bool, act: int = 0, limit: float = 0.0, alpha: float = 1.0):
         """out[p] = W_e . x[row(p)] for every place p of every expert e (see csrc/moe.cu); weights
-        [experts, (2 if gated) * n_out, k].  `act` 2: the clamped gate with `limit` and `alpha`."""
+        [experts, (2 if gated) * n_out, k].  `act` 2: the clamped gate with `limit` and `alpha`; without gate rows 3:
+        max(v, 0)^2, anything else: no activation."""
         _need(x, "x")
         _need(weights, "expert weights", x.dtype)
         _need(out, "out", x.dtype)
@@ -1510,8 +1664,8 @@ class Kernels:
     def moe_combine_add_norm(self, rows, place, pair_weight, top: int, stream, scale=None, next_norm=None, passing=None,
                              shared=None) -> bool:
         """stream (float32 [T, cols], in place) += scale * (the sum `moe_combine` forms), the sum kept in 32-bit;
-        `scale` float32 [cols] or None.  `next_norm` = (weight2, eps2, out): out = the RMS norm of the updated rows, in
-        the rows' dtype (it may be the passing experts' x).  False when the kernel does not take the row length
+        `scale` float32 [cols] or None.  `next_norm` (as in `norm_add_norm`, of the kinds without a mean): the norm of
+        the updated rows, in the rows' dtype (its rows may be the passing experts' x).  False when the kernel does not take the row length
         (nothing has run then)."""
         _need(rows, "rows")
         _need(place, "place", torch.int32)
@@ -1525,20 +1679,17 @@ class Kernels:
             _need(scale, "scale", torch.float32)
             if scale.numel() != C:
                 raise KernelError("moe_combine_add_norm: the scale's length differs from the stream's width")
-        w2 = out = None
-        eps2 = 0.0
-        if next_norm is not None:
-            w2, eps2, out = next_norm
-            _need(w2, "next norm weight", torch.float32)
+        w2, eps2, kind2, alpha2, b2, out = self._next_norm("moe_combine_add_norm", next_norm, T, C)
+        if kind2 == 1:
+            return False
+        if out is not None:
             _need(out, "out", rows.dtype)
-            if out.shape != (T, C) or w2.numel() != C:
-                raise KernelError("moe_combine_add_norm: the next norm's shapes differ")
         choice, experts, x, x_stride, s_rows, s_gate, g_stride = self._combine_extras("moe_combine_add_norm", rows, T, C,
                                                                                       top, passing, shared)
         self._check(self.lib.ullm_moe_combine_add_norm(
             _DT[rows.dtype], _ptr(rows), _ptr(place), _ptr(pair_weight), T, top, C, _ptr(choice), experts, _ptr(x),
             x_stride, _ptr(s_rows), _ptr(s_gate), g_stride, _ptr(stream), _ptr(scale), _ptr(w2), float(eps2), _ptr(out),
-            _stream()), "moe_combine_add_norm")
+            _stream(), _ptr(alpha2), _ptr(b2)), "moe_combine_add_norm")
         return True
 
     def check_attention_sizes(self, *a):
@@ -1733,7 +1884,8 @@ class Kernels:
                         v_dim: int | None = None, keep_first: int = 0, softcap: float = 0.0, parts=None,
                         general: bool = False):
         """Attention of every row of the flat batch over its request's pages.
-        `qkv` holds q in its first num_q * head_dim columns.  `fuse` (only after `decode_fusion_applies` said
+        `qkv` holds q in its first num_q * head_dim columns.  `window`: 0 every earlier key is seen; w > 0 the last w;
+        -c the keys of the query's own stretch of c positions (stretches counted from position 0).  `fuse` (only after `decode_fusion_applies` said
         yes): q, k and v are as the projection left them, and the kernel norms, rotates and stores them itself;
         a dict with q_w, k_w (or None), eps, cos, sin, positions, slot_mapping (or None).  `ragged` (decode
         steps): the caller found the requests' lengths very unequal, which picks the batch-balanced kernel."""

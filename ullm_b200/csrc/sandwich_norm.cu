@@ -5,12 +5,16 @@
 //                   stream[t] += extra_rows[t]; stream[t] += extra_vec     (each optional, in this order)
 //                   out[t] = round(w2 * n2(stream[t]))          (optional: the norm that reads the stream next)
 //   norm_rows       out[r] = round(w * n(stream[rows[r]]))      (gathered rows; `rows` null: all in order)
+//   pair_norm_add_norm   stream[t] += mult * (wa * n(a[t]) + wb * n(b[t])) for TWO sub-layers' outputs, each divided by
+//                   its own root mean square; then out as above.  Without a stream: rows_out[t] = round(the sum)
+//   relu2           out = round(max(in, 0)^2)
 //   xielu           out = round(act(in)), act(z) = softplus(p) z^2 + z / 2 for z > 0,
 //                                          (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 otherwise
 //
 // n(v) = v / sqrt(mean(v^2) + eps), or with `center` = 1 (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps): the
 // variance is the mean of the squared deviations, formed in a second pass over the row, which waits in shared
-// memory.  `center` = 2 for the added operand: n(v) = v, so stream[t] += mult * w * a[t] (a scale per channel on a
+// memory.  The norm that reads the stream next may also be `center2` = 2, a norm without statistics:
+// out = tanh(alpha * s) * w2 + b2 with one number alpha and a vector b2.  `center` = 2 for the added operand: n(v) = v, so stream[t] += mult * w * a[t] (a scale per channel on a
 // sub-layer's output; w null: no scale), the arrangement of a pre-norm layer on a 32-bit stream.  Sums, means and the stream are 32-bit; one rounding at each store.  One block per row.
 #include "common.cuh"
 
@@ -39,7 +43,8 @@ template <typename TA, typename TO>
 __global__ void norm_add_norm_kernel(const TA* __restrict__ a, float* __restrict__ stream,
                                      const float* __restrict__ w, int cols, float eps, float mult, int center,
                                      const float* __restrict__ extra_rows, const float* __restrict__ extra_vec,
-                                     const float* __restrict__ w2, float eps2, int center2, TO* __restrict__ out) {
+                                     const float* __restrict__ w2, float eps2, int center2, TO* __restrict__ out,
+                                     const float* __restrict__ alpha2, const float* __restrict__ b2) {
   extern __shared__ float sn_smem[];  // [cols] the operand's row, then [cols] the stream's row
   __shared__ float scratch[33];
   pdl_launch_dependents();
@@ -63,6 +68,12 @@ __global__ void norm_add_norm_kernel(const TA* __restrict__ a, float* __restrict
     row_s[c] = s;
   }
   if (out == nullptr) return;
+  if (center2 == 2) {  // (a thread reads what it wrote itself: no barrier)
+    const float al = *alpha2;
+    for (int c = threadIdx.x; c < cols; c += blockDim.x)
+      out[base + c] = from_f32<TO>(tanhf(al * row_s[c]) * w2[c] + b2[c]);
+    return;
+  }
   __syncthreads();
   float mean2;
   const float rstd2 = row_rstd(row_s, cols, center2 != 0, eps2, scratch, &mean2);
@@ -70,10 +81,90 @@ __global__ void norm_add_norm_kernel(const TA* __restrict__ a, float* __restrict
     out[base + c] = from_f32<TO>((row_s[c] - mean2) * rstd2 * w2[c]);
 }
 
+// Two sub-layers' rows a and b, each divided by its own root mean square and weighted, their sum (times `mult`) added
+// to the stream; then the norm that reads the stream next.  One block per row; VEC neighbouring columns per thread and
+// turn (16-byte pieces where the rows allow), both sums of squares in one set of barriers.
+template <typename T, int VEC>
+__global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __restrict__ b,
+                                          const float* __restrict__ wa, const float* __restrict__ wb, int cols,
+                                          float eps, float mult, float* __restrict__ stream, T* __restrict__ rows_out,
+                                          const float* __restrict__ w2, float eps2, int kind2,
+                                          const float* __restrict__ alpha2, const float* __restrict__ b2,
+                                          T* __restrict__ out) {
+  extern __shared__ __align__(16) float sn_smem[];  // [cols] a, [cols] b; the stream's row takes a's place
+  __shared__ float sums[2][33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long base = (long long)blockIdx.x * cols;
+  float* row_a = sn_smem;
+  float* row_b = sn_smem + cols;
+  float qa = 0.f, qb = 0.f;
+  for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+    float va[VEC], vb[VEC];
+    load_vec<T, VEC>(a + base + c0, va);
+    load_vec<T, VEC>(b + base + c0, vb);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      row_a[c0 + i] = va[i];
+      row_b[c0 + i] = vb[i];
+      qa += va[i] * va[i];
+      qb += vb[i] * vb[i];
+    }
+  }
+  qa = warp_sum(qa);
+  qb = warp_sum(qb);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  if (lane == 0) {
+    sums[0][warp] = qa;
+    sums[1][warp] = qb;
+  }
+  __syncthreads();
+  qa = qb = 0.f;
+  for (int i = 0; i < nwarps; ++i) {  // (every thread adds the warps' sums in the same order)
+    qa += sums[0][i];
+    qb += sums[1][i];
+  }
+  const float ra = mult / sqrtf(qa / (float)cols + eps), rb = mult / sqrtf(qb / (float)cols + eps);
+  const float al = (out != nullptr && kind2 == 2) ? *alpha2 : 0.f;
+  for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+    float s[VEC];
+    if (stream != nullptr) load_vec32<VEC>(stream + base + c0, s);
+    else
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] = 0.f;
+    float ga[VEC], gb[VEC];
+    load_vec32<VEC>(wa + c0, ga);
+    load_vec32<VEC>(wb + c0, gb);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] += row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
+    if (stream != nullptr) store_vec32<VEC>(stream + base + c0, s);
+    if (rows_out != nullptr) store_vec<T, VEC>(rows_out + base + c0, s);
+    if (out == nullptr) continue;
+    if (kind2 == 2) {
+      float g2[VEC], d2[VEC];
+      load_vec32<VEC>(w2 + c0, g2);
+      load_vec32<VEC>(b2 + c0, d2);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] = tanhf(al * s[i]) * g2[i] + d2[i];
+      store_vec<T, VEC>(out + base + c0, s);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) row_a[c0 + i] = s[i];
+    }
+  }
+  if (out == nullptr || kind2 == 2) return;
+  __syncthreads();
+  float mean2;
+  const float rstd2 = row_rstd(row_a, cols, kind2 != 0, eps2, sums[0], &mean2);
+  for (int c = threadIdx.x; c < cols; c += blockDim.x)
+    out[base + c] = from_f32<T>((row_a[c] - mean2) * rstd2 * w2[c]);
+}
+
 template <typename TO>
 __global__ void norm_rows_kernel(const float* __restrict__ stream, const int* __restrict__ rows,
                                  const float* __restrict__ w, TO* __restrict__ out, int cols, int src_rows, float eps,
-                                 int center, int* status) {
+                                 int center, int* status, const float* __restrict__ alpha,
+                                 const float* __restrict__ b) {
   extern __shared__ float sn_smem[];
   __shared__ float scratch[33];
   pdl_launch_dependents();
@@ -85,6 +176,12 @@ __global__ void norm_rows_kernel(const float* __restrict__ stream, const int* __
     r = 0;
   }
   const float* s = stream + (long long)r * cols;
+  if (center == 2) {
+    const float al = *alpha;
+    for (int c = threadIdx.x; c < cols; c += blockDim.x)
+      out[(long long)blockIdx.x * cols + c] = from_f32<TO>(bad ? 0.f : tanhf(al * s[c]) * w[c] + b[c]);
+    return;
+  }
   for (int c = threadIdx.x; c < cols; c += blockDim.x) sn_smem[c] = s[c];
   __syncthreads();
   float mean;
@@ -108,6 +205,24 @@ __global__ void xielu_kernel(const T* __restrict__ in, T* __restrict__ out, long
   }
 }
 
+// out = max(in, 0)^2, VEC elements per thread and turn
+template <typename T, int VEC>
+__global__ void relu2_kernel(const T* in, T* out, long long n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC; i < n;
+       i += (long long)gridDim.x * blockDim.x * VEC) {
+    float v[VEC];
+    load_vec<T, VEC>(in + i, v);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+      const float r = fmaxf(v[k], 0.f);
+      v[k] = r * r;
+    }
+    store_vec<T, VEC>(out + i, v);
+  }
+}
+
 static inline int sn_threads(int cols) {
   int threads = 32;
   while (threads < 512 && threads * 4 < cols) threads <<= 1;
@@ -127,14 +242,15 @@ static int sn_allow_smem(K kernel, size_t smem) {
 template <typename TA, typename TO>
 static int norm_add_norm_launch(const void* a, float* stream, const float* w, int rows, int cols, float eps,
                                 float mult, int center, const float* extra_rows, const float* extra_vec,
-                                const float* w2, float eps2, int center2, void* out, cudaStream_t st) {
+                                const float* w2, float eps2, int center2, void* out, const float* alpha2,
+                                const float* b2, cudaStream_t st) {
   const size_t smem = 2 * (size_t)cols * sizeof(float);
   if (smem > SN_MAX_SMEM) return ULLM_ERR_UNSUPPORTED;
   const int rc = sn_allow_smem(norm_add_norm_kernel<TA, TO>, smem);
   if (rc != ULLM_OK) return rc;
   return ullm_launch_kernel(norm_add_norm_kernel<TA, TO>, dim3(rows), dim3(sn_threads(cols)), smem, st,
                             (const TA*)a, stream, w, cols, eps, mult, center, extra_rows, extra_vec, w2, eps2,
-                            center2, (TO*)out);
+                            center2, (TO*)out, alpha2, b2);
 }
 
 // `a_dtype`: dtype of `a` (the engine's, or 32-bit for a sub-layer that leaves 32-bit rows); `out_dtype`: of `out`.
@@ -142,15 +258,16 @@ static int norm_add_norm_launch(const void* a, float* stream, const float* w, in
 extern "C" int ullm_norm_add_norm(int a_dtype, const void* a, float* stream, const float* w, int rows, int cols,
                                   float eps, float mult, int center, const float* extra_rows,
                                   const float* extra_vec, const float* w2, float eps2, int center2, int out_dtype,
-                                  void* out, void* stream_handle) {
+                                  void* out, void* stream_handle, const float* alpha2, const float* b2) {
   cudaStream_t st = (cudaStream_t)stream_handle;
   if (rows < 0 || cols <= 0) return ULLM_ERR_BAD_SIZE;
   if ((a != nullptr && w == nullptr && center != 2) || (out != nullptr && w2 == nullptr)) return ULLM_ERR_BAD_SIZE;
-  if (center < 0 || center > 2 || center2 < 0 || center2 > 1) return ULLM_ERR_BAD_SIZE;
+  if (center < 0 || center > 2 || center2 < 0 || center2 > 2) return ULLM_ERR_BAD_SIZE;
+  if (out != nullptr && center2 == 2 && (alpha2 == nullptr || b2 == nullptr)) return ULLM_ERR_BAD_SIZE;
   if (rows == 0) return ULLM_OK;
 #define SN_GO(TA, TO)                                                                                              \
   return norm_add_norm_launch<TA, TO>(a, stream, w, rows, cols, eps, mult, center, extra_rows, extra_vec, w2, eps2, \
-                                      center2, out, st)
+                                      center2, out, alpha2, b2, st)
 #define SN_OUT(TA)                                         \
   if (out_dtype == ULLM_DTYPE_F32) SN_GO(TA, float);       \
   if (out_dtype == ULLM_DTYPE_BF16) SN_GO(TA, __nv_bfloat16); \
@@ -166,26 +283,74 @@ extern "C" int ullm_norm_add_norm(int a_dtype, const void* a, float* stream, con
 
 template <typename TO>
 static int norm_rows_launch(const float* stream, const int* rows, const float* w, void* out, int count, int cols,
-                            int src_rows, float eps, int center, int* status, cudaStream_t st) {
+                            int src_rows, float eps, int center, int* status, const float* alpha, const float* b,
+                            cudaStream_t st) {
   const size_t smem = (size_t)cols * sizeof(float);
   if (smem > SN_MAX_SMEM) return ULLM_ERR_UNSUPPORTED;
   const int rc = sn_allow_smem(norm_rows_kernel<TO>, smem);
   if (rc != ULLM_OK) return rc;
   return ullm_launch_kernel(norm_rows_kernel<TO>, dim3(count), dim3(sn_threads(cols)), smem, st, stream, rows, w,
-                            (TO*)out, cols, src_rows, eps, center, status);
+                            (TO*)out, cols, src_rows, eps, center, status, alpha, b);
 }
 
 extern "C" int ullm_norm_rows(int dtype, const float* stream, const int* rows, const float* w, void* out, int count,
-                              int cols, int src_rows, float eps, int center, int* status, void* stream_handle) {
+                              int cols, int src_rows, float eps, int center, int* status, void* stream_handle,
+                              const float* alpha, const float* b) {
   cudaStream_t st = (cudaStream_t)stream_handle;
-  if (count < 0 || cols <= 0 || src_rows < 0) return ULLM_ERR_BAD_SIZE;
+  if (count < 0 || cols <= 0 || src_rows < 0 || center < 0 || center > 2) return ULLM_ERR_BAD_SIZE;
+  if (center == 2 && (alpha == nullptr || b == nullptr)) return ULLM_ERR_BAD_SIZE;
   if (count == 0) return ULLM_OK;
   if (dtype == ULLM_DTYPE_F32)
-    return norm_rows_launch<float>(stream, rows, w, out, count, cols, src_rows, eps, center, status, st);
+    return norm_rows_launch<float>(stream, rows, w, out, count, cols, src_rows, eps, center, status, alpha, b, st);
   if (dtype == ULLM_DTYPE_BF16)
-    return norm_rows_launch<__nv_bfloat16>(stream, rows, w, out, count, cols, src_rows, eps, center, status, st);
+    return norm_rows_launch<__nv_bfloat16>(stream, rows, w, out, count, cols, src_rows, eps, center, status, alpha, b, st);
   if (dtype == ULLM_DTYPE_F16)
-    return norm_rows_launch<__half>(stream, rows, w, out, count, cols, src_rows, eps, center, status, st);
+    return norm_rows_launch<__half>(stream, rows, w, out, count, cols, src_rows, eps, center, status, alpha, b, st);
+  return ULLM_ERR_BAD_DTYPE;
+}
+
+template <typename T>
+static int pair_norm_launch(const void* a, const void* b, const float* wa, const float* wb, int rows, int cols, float eps,
+                            float mult, float* stream, void* rows_out, const float* w2, float eps2, int kind2,
+                            const float* alpha2, const float* b2, void* out, cudaStream_t st) {
+  const size_t smem = 2 * (size_t)cols * sizeof(float);
+  if (smem > SN_MAX_SMEM) return ULLM_ERR_UNSUPPORTED;
+  constexpr int V = 16 / (int)sizeof(T);
+  const bool wide = cols % V == 0 && (((uintptr_t)a | (uintptr_t)b | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)stream |
+                                       (uintptr_t)rows_out | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out) & 15) == 0;
+  int threads = 32;
+  while (threads < 512 && threads * (wide ? V : 1) < cols) threads <<= 1;
+#define PN_GO(VEC)                                                                                                    \
+  {                                                                                                                   \
+    const int rc = sn_allow_smem(pair_norm_add_norm_kernel<T, VEC>, smem);                                            \
+    if (rc != ULLM_OK) return rc;                                                                                     \
+    return ullm_launch_kernel(pair_norm_add_norm_kernel<T, VEC>, dim3(rows), dim3(threads), smem, st, (const T*)a,    \
+                              (const T*)b, wa, wb, cols, eps, mult, stream, (T*)rows_out, w2, eps2, kind2, alpha2, b2, \
+                              (T*)out);                                                                               \
+  }
+  if (wide) PN_GO(V);
+  PN_GO(1);
+#undef PN_GO
+}
+
+// a, b [rows, cols] in the engine's dtype; `stream` (32-bit, updated in place) and `rows_out` (engine's dtype): at least
+// one.  `out` with `w2` (null: none): the next norm of the updated rows; `kind2` 0: RMS, 1: centred, 2: tanh with `alpha2`
+// (one number) and `b2`.
+extern "C" int ullm_pair_norm_add_norm(int dtype, const void* a, const void* b, const float* wa, const float* wb, int rows,
+                                       int cols, float eps, float mult, float* stream, void* rows_out, const float* w2,
+                                       float eps2, int kind2, const float* alpha2, const float* b2, void* out,
+                                       void* stream_handle) {
+  cudaStream_t st = (cudaStream_t)stream_handle;
+  if (rows < 0 || cols <= 0 || a == nullptr || b == nullptr || wa == nullptr || wb == nullptr ||
+      (stream == nullptr && rows_out == nullptr) || (out != nullptr && w2 == nullptr) || kind2 < 0 || kind2 > 2 ||
+      (out != nullptr && kind2 == 2 && (alpha2 == nullptr || b2 == nullptr)))
+    return ULLM_ERR_BAD_SIZE;
+  if (rows == 0) return ULLM_OK;
+#define PN_ARGS a, b, wa, wb, rows, cols, eps, mult, stream, rows_out, w2, eps2, kind2, alpha2, b2, out, st
+  if (dtype == ULLM_DTYPE_F32) return pair_norm_launch<float>(PN_ARGS);
+  if (dtype == ULLM_DTYPE_BF16) return pair_norm_launch<__nv_bfloat16>(PN_ARGS);
+  if (dtype == ULLM_DTYPE_F16) return pair_norm_launch<__half>(PN_ARGS);
+#undef PN_ARGS
   return ULLM_ERR_BAD_DTYPE;
 }
 
@@ -204,5 +369,26 @@ extern "C" int ullm_xielu(int dtype, const void* in, void* out, long long n, con
                               (__nv_bfloat16*)out, n, pq);
   if (dtype == ULLM_DTYPE_F16)
     return ullm_launch_kernel(xielu_kernel<__half>, grid, block, 0, st, (const __half*)in, (__half*)out, n, pq);
+  return ULLM_ERR_BAD_DTYPE;
+}
+
+template <typename T>
+static int relu2_launch(const void* in, void* out, long long n, cudaStream_t st) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const bool wide = n % V == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
+  long long blocks = (n / (wide ? V : 1) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (wide) return ullm_launch_kernel(relu2_kernel<T, V>, dim3((int)blocks), dim3(256), 0, st, (const T*)in, (T*)out, n);
+  return ullm_launch_kernel(relu2_kernel<T, 1>, dim3((int)blocks), dim3(256), 0, st, (const T*)in, (T*)out, n);
+}
+
+// out = max(in, 0)^2 element by element (`out` may be `in`).
+extern "C" int ullm_relu2(int dtype, const void* in, void* out, long long n, void* stream_handle) {
+  cudaStream_t st = (cudaStream_t)stream_handle;
+  if (n < 0) return ULLM_ERR_BAD_SIZE;
+  if (n == 0) return ULLM_OK;
+  if (dtype == ULLM_DTYPE_F32) return relu2_launch<float>(in, out, n, st);
+  if (dtype == ULLM_DTYPE_BF16) return relu2_launch<__nv_bfloat16>(in, out, n, st);
+  if (dtype == ULLM_DTYPE_F16) return relu2_launch<__half>(in, out, n, st);
   return ULLM_ERR_BAD_DTYPE;
 }

@@ -11,6 +11,7 @@
 //   gated_add_f32     stream[t] += sigmoid(g1[t] + b1) * a[t] (+ sigmoid(g2[t] + b2) * f[t]),       copy[t] = round(stream[t])
 //   side_gate_mul     out[t] = gelu_tanh(s[t]) * table[id[t]][offset .. offset + cols)
 //   softcap_f32       x = cap * tanh(x / cap), in place
+//   scale_f32         x = factor * x, in place
 //
 // `copy` is the stream rounded to the engine's dtype, the operand of the next
 // sub-layer's matrix products; with a 32-bit engine it is not needed (null).
@@ -206,6 +207,13 @@ __global__ void softcap_f32_kernel(float* __restrict__ x, long long n, float cap
     x[i] = cap * tanhf(x[i] * inv);
 }
 
+__global__ void scale_f32_kernel(float* __restrict__ x, long long n, float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    x[i] *= factor;
+}
+
 static inline int row_threads(int cols) {
   int threads = 32;
   while (threads < 512 && threads * 4 < cols) threads <<= 1;
@@ -371,6 +379,15 @@ extern "C" int ullm_softcap_f32(float* x, long long n, float cap, void* stream_h
   long long blocks = (n + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   return ullm_launch_kernel(softcap_f32_kernel, dim3((int)blocks), dim3(256), 0, st, x, n, cap);
+}
+
+extern "C" int ullm_scale_f32(float* x, long long n, float factor, void* stream_handle) {
+  cudaStream_t st = (cudaStream_t)stream_handle;
+  if (n < 0) return ULLM_ERR_BAD_SIZE;
+  if (n == 0) return ULLM_OK;
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  return ullm_launch_kernel(scale_f32_kernel, dim3((int)blocks), dim3(256), 0, st, x, n, factor);
 }
 
 extern "C" int ullm_concat_rows_f32(int dtype, const float* a, const float* b, void* out, int rows, int cols_a,

@@ -15,7 +15,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import check_attention_sizes, kernels
-from .base import CacheNeed, Mixer, ParamDecl, StateNeed
+from .base import CacheNeed, Mixer, ParamDecl, SharesInput, StateNeed
 from .linear import linear
 from .registry import build_norm, build_position_encoding, register_mixer
 
@@ -28,7 +28,7 @@ def is_ragged(batch: int, max_kv: int, sum_kv: int) -> bool:
 
 
 @register_mixer("paged_attention")
-class PagedAttention(Mixer):
+class PagedAttention(Mixer, SharesInput):
     def __init__(
         self,
         hidden_size: int,
@@ -53,12 +53,18 @@ class PagedAttention(Mixer):
         whole_norm: bool = False,
         value_unit_norm: bool = False,
         head_temperature: bool = False,
+        chunk: int | None = None,
+        o_bias: bool = False,
+        general: bool = False,
     ):
         """`value_dim`: head size of the values and of the output (default: `head_dim`).  `window` with
         `keep_first`: position i sees j <= i if i - j < window or j < keep_first.  `own_kv` False: the mixer has
         no key / value projections (nor a key norm); it reads the cache of the execution the schedule names
         (`ScheduleEntry.cache_of`) with queries, mask and scale of its own.  `names`: the checkpoint's names of
-        q, k, v, o, q_norm, k_norm behind the mixer's prefix (defaults: `q_proj.weight`, ..., `q_norm.`).
+        q, k, v, o, q_norm, k_norm behind the mixer's prefix (defaults: `q_proj.weight`, ..., `q_norm.`).  `chunk` c
+        (instead of a window): position i sees the j <= i of its own stretch of c positions, floor(j / c) =
+        floor(i / c), stretches being counted from position 0 of the request.  `o_bias`: the output projection has a
+        bias (`qkv_bias`: the other three).  `general`: take the general path below even where no option asks for it.
 
         Further options, all on the general path (csrc/attention_prep.cu, then the tensor-core attention kernels
         where dtype and head sizes allow, else csrc/attention_generic.cu) in prompt and decode steps alike.
@@ -89,6 +95,12 @@ class PagedAttention(Mixer):
         self.head_dim = head_dim
         self.qkv_bias = qkv_bias
         self.window = window
+        self.chunk = None if chunk is None else int(chunk)
+        if self.chunk is not None and (self.chunk <= 0 or window is not None or keep_first):
+            raise ValueError("chunk: a positive size, without a window and without kept first tokens")
+        # what the attention kernels take: 0 every earlier key, w > 0 the last w, -c the stretch of c positions
+        self.mask_arg = -self.chunk if self.chunk else (window or 0)
+        self.o_bias = bool(o_bias)
         self.scale = head_dim ** -0.5 if scale is None else scale
         self.value_dim = head_dim if value_dim is None else value_dim
         self.keep_first = int(keep_first)
@@ -122,7 +134,7 @@ class PagedAttention(Mixer):
             raise ValueError("a mixer without key / value projections has no values to convolve or to mix")
         n = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight", q_bias="q_proj.bias",
                  k_bias="k_proj.bias", v_bias="v_proj.bias", q_norm="q_norm.", k_norm="k_norm.",
-                 q_conv="q_proj.conv", k_conv="k_proj.conv", v_conv="v_proj.conv", talk="talk", vmix="vmix",
+                 o_bias="o_proj.bias", q_conv="q_proj.conv", k_conv="k_proj.conv", v_conv="v_proj.conv", talk="talk", vmix="vmix",
                  temp="temp")
         n.update(names or {})
         self.names = n
@@ -130,6 +142,7 @@ class PagedAttention(Mixer):
         self.kv_size = num_kv_heads * head_dim
         self.v_size = num_kv_heads * self.value_dim
         self.o_size = num_heads * self.value_dim
+        self.w_rows = self.q_size + ((self.kv_size + self.v_size) if self.own_kv else 0)  # of the input product
         if self.whole_norm:
             from dataclasses import replace
 
@@ -145,7 +158,7 @@ class PagedAttention(Mixer):
         self.position = build_position_encoding(position) if position is not None else None
         if getattr(self.position, "interleaved", False) and not self.rows_form:
             raise ValueError("a rotation of neighbouring dimensions needs whole_norm, value_unit_norm or head_temperature")
-        self.general = bool(self.conv_taps or self.score_cap or self.talking_heads or value_mix or self.rows_form
+        self.general = bool(general or self.conv_taps or self.score_cap or self.talking_heads or value_mix or self.rows_form
                             or self.unit_norm_after_rotation or getattr(self.position, "computed", False))
         if self.general and self.position is not None and not getattr(self.position, "computed", False):
             raise ValueError("these attention options take a position encoding of kind 'rope_computed' (or none)")
@@ -163,6 +176,8 @@ class PagedAttention(Mixer):
             if self.own_kv:
                 d[n["k_bias"]] = ParamDecl((self.kv_size,), "bias")
                 d[n["v_bias"]] = ParamDecl((self.v_size,), "bias")
+        if self.o_bias:
+            d[n["o_bias"]] = ParamDecl((H,), "bias")
         if self.conv_taps:
             d[n["q_conv"]] = ParamDecl((self.q_size, self.conv_taps))
             d[n["k_conv"]] = ParamDecl((self.kv_size, self.conv_taps))
@@ -185,8 +200,8 @@ class PagedAttention(Mixer):
 
     def materialize(self, make):
         H, q, kv, n = self.hidden_size, self.q_size, self.kv_size, self.names
-        rows = q + ((kv + self.v_size) if self.own_kv else 0)
-        self.w_qkv = make("qkv_proj.weight", ParamDecl((rows, H)))
+        rows = self.w_rows
+        self.w_qkv = self._make_in(make, "qkv_proj.weight", (rows, H))
         self.tensors[n["q"]] = self.w_qkv[:q]
         if self.own_kv:
             self.tensors[n["k"]] = self.w_qkv[q:q + kv]
@@ -194,11 +209,14 @@ class PagedAttention(Mixer):
         self.tensors[n["o"]] = make("o_proj.weight", ParamDecl((H, self.o_size)))
         self.b_qkv = None
         if self.qkv_bias:
-            self.b_qkv = make("qkv_proj.bias", ParamDecl((rows,), "bias"))
+            self.b_qkv = self._make_in_bias(make, "qkv_proj.bias", rows)
             self.tensors[n["q_bias"]] = self.b_qkv[:q]
             if self.own_kv:
                 self.tensors[n["k_bias"]] = self.b_qkv[q:q + kv]
                 self.tensors[n["v_bias"]] = self.b_qkv[q + kv:]
+        self.w_o_bias = None
+        if self.o_bias:
+            self.w_o_bias = self.tensors[n["o_bias"]] = make(n["o_bias"], ParamDecl((H,), "bias"))
         self.w_conv = None
         if self.conv_taps:
             # the three filters one after the other, as the projection's rows are
@@ -218,7 +236,8 @@ class PagedAttention(Mixer):
     # -- cache ------------------------------------------------------------
     def cache_need(self):
         return CacheNeed(self.num_kv_heads, self.head_dim, self.window,
-                         None if self.value_dim == self.head_dim else self.value_dim, self.keep_first if self.window else 0)
+                         None if self.value_dim == self.head_dim else self.value_dim, self.keep_first if self.window else 0,
+                         chunk=self.chunk)
 
     def state_need(self):
         """The convolution's memory: the last taps - 1 projected rows (q | k | v) of the request, 32-bit."""
@@ -248,13 +267,19 @@ class PagedAttention(Mixer):
         return bool(ctx.decode_only and is_ragged(ctx.num_live_requests, ctx.max_kv_len, ctx.sum_kv_len))
 
     def output_projection(self):
-        return self.tensors[self.names["o"]], None
+        return self.tensors[self.names["o"]], self.w_o_bias
 
     def takes_input_norm(self):
         return not self.general
 
+    def input_width(self):
+        return self.w_rows
+
+    def input_bias(self):
+        return self.qkv_bias
+
     # -- the general path ----------------------------------------------------
-    def _forward_general(self, x, ctx, cache, project_output: bool):
+    def _forward_general(self, x, ctx, cache, project_output: bool, projected=None, out=None):
         """Projection, then csrc/attention_prep.cu (convolution, rotation, norms, value mixing, cache stores), the
         general attention kernel (cap, window, kept tokens), and the mixing of heads if there is any."""
         K = kernels()
@@ -262,8 +287,10 @@ class PagedAttention(Mixer):
         ws = ctx.workspace
         if not self.own_kv:
             raise NotImplementedError("borrowed keys and values beside these attention options")
-        qkv = ws.tokens("attn.qkv", T, self.w_qkv.shape[0], x.dtype)
-        linear(x, self.w_qkv, qkv, self.b_qkv)
+        qkv = projected
+        if qkv is None:
+            qkv = ws.tokens("attn.qkv", T, self.w_qkv.shape[0], x.dtype)
+            linear(x, self.w_qkv, qkv, self.b_qkv)
         g = cache.group
         q = ws.tokens("attn.q", T, self.q_size, x.dtype)
         tables = self.position.tables() if self.position is not None else {}
@@ -290,7 +317,7 @@ class PagedAttention(Mixer):
                 rotary_dim=rotary_dim, interleaved=bool(getattr(self.position, "interleaved", False)),
                 q_head_scale=self.tensors[self.names["temp"]] if self.head_temperature else None,
                 value_unit_norm=self.value_unit_norm)
-            return self._attend(q, x, ctx, cache, project_output)
+            return self._attend(q, x, ctx, cache, project_output, out)
         K.qkv_prepare(
             qkv, q, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, ctx.positions,
             g.slot_mapping if cache.writes else None, cache.k_pages, cache.v_pages,
@@ -303,9 +330,9 @@ class PagedAttention(Mixer):
             vmix_mode=mode, vmix_lambda=self.tensors[self.names["vmix"]] if mode == 2 else None, v_first=v_first)
         if state is not None:
             K.conv_state_update(qkv, self.conv_taps, state, ctx.cu_q, ctx.token_req, ctx.req_slots, ctx.num_requests)
-        return self._attend(q, x, ctx, cache, project_output)
+        return self._attend(q, x, ctx, cache, project_output, out)
 
-    def _attend(self, q, x, ctx, cache, project_output: bool):
+    def _attend(self, q, x, ctx, cache, project_output: bool, out=None):
         """The prepared queries over the pages, then the mixing of heads (if any) and the output projection."""
         K = kernels()
         T = x.shape[0]
@@ -314,36 +341,41 @@ class PagedAttention(Mixer):
         parts = None
         if self.talking_heads:
             parts = ws.tokens("attn.parts", T, self.num_heads * self.num_kv_heads * self.value_dim, torch.float32)
-        if self.rows_form and (self.value_dim != self.head_dim or self.head_dim not in (64, 128)):
+        if (not self.talking_heads and self.score_cap is None and self.keep_first == 0
+                and (self.value_dim != self.head_dim or self.head_dim not in (64, 128))):
             # head sizes the kernels below take only in their general form: the windowed kernel runs multiples of 16
             # on the tensor cores (and falls back to the general kernel itself)
             K.windowed_attention(q, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len,
                                  ctx.token_req, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim,
-                                 g.page_size, self.window or 0, self.scale, num_requests=ctx.num_requests, workspace=ws)
-            if not project_output:
-                return attn
-            out = ws.tokens("mixer.out", T, self.hidden_size, x.dtype)
-            linear(attn, self.tensors[self.names["o"]], out)
-            return out
+                                 g.page_size, self.mask_arg, self.scale, num_requests=ctx.num_requests, workspace=ws)
+            return self._project(attn, ctx, project_output, out)
         K.paged_attention(
             q, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len, ctx.token_req,
-            self.num_heads, self.num_kv_heads, self.head_dim, g.page_size, self.window or 0, self.scale, ctx,
+            self.num_heads, self.num_kv_heads, self.head_dim, g.page_size, self.mask_arg, self.scale, ctx,
             v_dim=self.value_dim, keep_first=self.keep_first if self.window else 0, softcap=self.score_cap or 0.0,
             parts=parts, general=True)
         if parts is not None:
             K.mix_heads(parts, self.tensors[self.names["talk"]], attn, self.num_heads, self.num_kv_heads, self.value_dim)
+        return self._project(attn, ctx, project_output, out)
+
+    def _project(self, attn, ctx, project_output: bool, out=None):
         if not project_output:
-            return attn
-        out = ws.tokens("mixer.out", T, self.hidden_size, x.dtype)
-        linear(attn, self.tensors[self.names["o"]], out)
+            return attn  # (the caller multiplies by `output_projection()` itself)
+        if out is None:
+            out = ctx.workspace.tokens("mixer.out", attn.shape[0], self.hidden_size, attn.dtype)
+        linear(attn, self.tensors[self.names["o"]], out, self.w_o_bias)
         return out
 
     # -- one step ---------------------------------------------------------
-    def forward(self, x, ctx, cache, project_output: bool = True, input_norm=None):
+    def forward(self, x, ctx, cache, project_output: bool = True, input_norm=None, projected=None, out=None):
+        """`projected`: the input product's rows, formed by the caller (only on the general path).  `out`: where the
+        projected output goes (default: the buffer that mixers share)."""
+        if projected is not None and (not self.general or self.rows_form or self.conv_taps):
+            raise NotImplementedError("an input product formed elsewhere beside these attention options")
         if self.general:
             if input_norm is not None:
                 raise RuntimeError("a folded norm was handed to an attention that does not take one")
-            return self._forward_general(x, ctx, cache, project_output)
+            return self._forward_general(x, ctx, cache, project_output, projected, out)
         K = kernels()
         T = x.shape[0]
         ragged = self._ragged(ctx)
@@ -401,11 +433,7 @@ class PagedAttention(Mixer):
             qkv, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len,
             ctx.token_req,
             self.num_heads, self.num_kv_heads, self.head_dim, g.page_size,
-            self.window or 0, self.scale, ctx, ragged=ragged, **({"fuse": fuse} if fuse is not None else {}),
+            self.mask_arg, self.scale, ctx, ragged=ragged, **({"fuse": fuse} if fuse is not None else {}),
             **({} if plain else {"v_dim": self.value_dim, "keep_first": self.keep_first if self.window else 0}),
         )
-        if not project_output:
-            return attn  # (the caller multiplies by `output_projection()` itself)
-        out = ctx.workspace.tokens("mixer.out", T, self.hidden_size, x.dtype)
-        linear(attn, self.tensors[self.names["o"]], out)
-        return out
+        return self._project(attn, ctx, project_output, out)

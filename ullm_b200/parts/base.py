@@ -47,7 +47,8 @@ class CacheNeed:
     """Keys and values this mixer keeps per token: `num_kv_heads` x `head_dim`
     for K and `num_kv_heads` x `value_dim` for V (None: `head_dim`).  `window`:
     None keeps every token, w keeps the last w, and with `keep_first` also the
-    first `keep_first` tokens of the request.  `values_in_keys`: there are no value
+    first `keep_first` tokens of the request; `chunk` c (instead of a window) keeps the tokens of the stretch of c
+    positions, counted from position 0, that the next token lies in.  `values_in_keys`: there are no value
     pages (the mixer reads its values out of the key rows).  `every` n > 1: the
     cache holds one entry per n tokens (entry e is written when token (e + 1) n - 1
     arrives), all of them kept; its pages are counted in entries."""
@@ -59,6 +60,22 @@ class CacheNeed:
     keep_first: int = 0
     values_in_keys: bool = False
     every: int = 1
+    chunk: int | None = None
+
+    @property
+    def keeps_all(self) -> bool:
+        return self.window is None and self.chunk is None
+
+    @property
+    def reach(self) -> int | None:
+        """How many tokens back the farthest one lies that is still kept (None: no limit)."""
+        return self.chunk if self.window is None else self.window
+
+    def first_needed(self, position: int) -> int:
+        """The first position that a token at `position`, or any later one, can still see (kept first tokens aside)."""
+        if self.chunk is not None:
+            return position - position % self.chunk
+        return 0 if self.window is None else max(0, position - self.window + 1)
 
     @property
     def v_dim(self) -> int:
@@ -132,9 +149,10 @@ class Norm(Part):
         raise NotImplementedError
 
     def row_params(self):
-        """(weight, eps, centred) if this norm is w * (x - mean) / sqrt(variance + eps) over the whole row (centred)
-        or w * x / sqrt(mean(x^2) + eps) (not centred), which a block may then hand to a kernel that norms a
-        sub-layer's output, adds it to the stream and applies the next norm at once; None otherwise."""
+        """(weight, eps, 1) if this norm is w * (x - mean) / sqrt(variance + eps) over the whole row, (weight, eps, 0) if
+        it is w * x / sqrt(mean(x^2) + eps), (weight, eps, 2, alpha, bias) if it is tanh(alpha x) * w + bias, which a
+        block may then hand to a kernel that adds a sub-layer's output to the stream and applies the next norm at
+        once; None otherwise."""
         return None
 
     def rms_params(self):
@@ -201,6 +219,12 @@ class Mixer(Part):
         A block may fold that product into a fused kernel."""
         return None
 
+    def forward_add(self, x, ctx, cache, stream, scale=None, next_norm=None) -> bool:
+        """Optional: stream (32-bit, in place) += scale * forward(x) in the mixer's own last kernel (`scale` a 32-bit
+        vector per channel or None), which also leaves `next_norm` (`Norm.row_params()` with the output rows behind
+        it) of the updated rows.  False (the default; nothing has run then): the caller adds `forward(x)` itself."""
+        return False
+
     def operand_dtype(self):
         """The dtype of the rows this mixer's `forward` takes (that of its first matrix)."""
         for t in self.all_tensors().values():
@@ -212,14 +236,39 @@ class Mixer(Part):
         raise NotImplementedError
 
 
+class SharesInput:
+    """What a mixer needs so that a caller can form its input product together with another's (one product for all
+    that reads the same rows): `input_width()` rows of weight, `input_bias()` whether they have a bias, and a `forward`
+    that takes the product's rows as `projected=` (a column range of wider rows).  The caller sets `shared_in` =
+    (weight rows, bias rows or None) before the mixer's parameters are made."""
+
+    shared_in = None
+
+    def input_width(self) -> int:
+        raise NotImplementedError
+
+    def input_bias(self) -> bool:
+        return False
+
+    def _make_in(self, make, name, shape):
+        if self.shared_in is None:
+            return make(name, ParamDecl(shape))
+        if tuple(self.shared_in[0].shape) != tuple(shape):
+            raise ValueError(f"the shared input product has rows {tuple(self.shared_in[0].shape)}, not {tuple(shape)}")
+        return self.shared_in[0]
+
+    def _make_in_bias(self, make, name, rows: int):
+        return make(name, ParamDecl((rows,), "bias")) if self.shared_in is None else self.shared_in[1]
+
+
 class FeedForward(Part):
     def forward(self, x, ctx):
         raise NotImplementedError
 
     def forward_add(self, x, ctx, stream, scale=None, next_norm=None) -> bool:
         """Optional: stream (32-bit, in place) += scale * forward(x) in the part's own last kernel (`scale` a
-        32-bit vector per channel or None), which also leaves the RMS norm `next_norm` = (weight, eps, out) of the
-        updated rows.  False (the default): the caller adds `forward(x)` itself."""
+        32-bit vector per channel or None), which also leaves `next_norm` (`Norm.row_params()`, of a kind without a
+        mean, with the output rows behind it) of the updated rows.  False (the default): the caller adds `forward(x)` itself."""
         return False
 
     def gated_weights(self):

@@ -501,24 +501,25 @@ class PreNormScaledBlock(Block):
         else:
             h = ws.tokens("block.normed", T, W, dt)
             self.mixer_norm.forward_rows(stream, None, h)
-        a = self.mixer.forward(h, ctx, cache)
         nxt = next_norm.row_params() if (next_norm is not None and hasattr(next_norm, "row_params")) else None
         if nxt is not None and nxt[0].numel() != W:
             nxt = None
         # (every reader of h is done when the kernel that overwrites it runs: the rows take its place)
         h2 = ws.tokens("block.normed", T, W, dt)
         s1 = self.tensors[self.names["mixer_scale"]] if self.layer_scale else None
+        behind = self.feed_forward_norm.row_params() if self.feed_forward is not None else nxt
+        behind = (*behind, h2) if behind is not None else None
+        # a mixer whose last kernel can add to the stream itself (and leave the next norm's rows) does so
+        if not self.mixer.forward_add(h, ctx, cache, stream, s1, behind):
+            K.norm_add_norm(stream, self.mixer.forward(h, ctx, cache), s1, plain=True, next_norm=behind)
         if self.feed_forward is not None:
-            K.norm_add_norm(stream, a, s1, plain=True, next_norm=(*self.feed_forward_norm.row_params(), h2))
             s2 = self.tensors[self.names["feed_forward_scale"]] if self.layer_scale else None
             # a feed-forward whose last kernel can add to the stream itself (and leave the next norm's rows) does so
-            takes = nxt is None or not nxt[2]  # (that kernel knows the norm without the mean taken off)
+            takes = nxt is None or nxt[2] != 1  # (that kernel knows the norms without the mean taken off)
             if not (takes and self.feed_forward.forward_add(h2, ctx, stream, s2,
-                                                            (nxt[0], nxt[1], h2) if nxt is not None else None)):
+                                                            (*nxt, h2) if nxt is not None else None)):
                 f = self.feed_forward.forward(h2, ctx)
                 K.norm_add_norm(stream, f, s2, plain=True, next_norm=(*nxt, h2) if nxt is not None else None)
-        else:
-            K.norm_add_norm(stream, a, s1, plain=True, next_norm=(*nxt, h2) if nxt is not None else None)
         if nxt is not None:
             ctx.prepared_norm = (next_norm, h2)
         ctx.stream_operand = None

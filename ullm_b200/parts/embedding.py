@@ -76,15 +76,16 @@ class TokenSideTable(Part):
 
 
 class OutputHead(Part):
-    """logits = h W^T in 32-bit output, then optionally capped: cap * tanh(logits / cap).  `tied_to`, when set, is
+    """logits = h W^T in 32-bit output, times `scale`, then optionally capped: cap * tanh(logits / cap).  `tied_to`, when set, is
     the embedding part whose table is read and no tensor of its own is declared."""
 
     def __init__(self, vocab_size: int, hidden_size: int, tied_to: TokenEmbedding | None = None, param: str = "weight",
-                 softcap: float | None = None):
+                 softcap: float | None = None, scale: float = 1.0):
         super().__init__()
         if softcap is not None and not softcap > 0:
             raise ValueError("a logit cap must be positive")
         self.softcap = softcap
+        self.scale = float(scale)
         self.vocab_size = vocab_size
         self.hidden_size = hidden_size
         self.tied_to = tied_to
@@ -100,6 +101,8 @@ class OutputHead(Part):
 
     def forward(self, h, out_f32):
         kernels().linear_f32_out(h, self.weight(), out_f32)
+        if self.scale != 1.0:
+            kernels().scale_f32(out_f32, self.scale)
         if self.softcap is not None:
             kernels().softcap_f32(out_f32, self.softcap)
         return out_f32

@@ -76,12 +76,17 @@ class DenseMLP(FeedForward):
         z > 0:   softplus(p) z^2 + z / 2
         z <= 0:  (1/2 + softplus(q)) (e^z - 1 - z) + z / 2
 
-    evaluated in 32-bit on the product's rounded output (csrc/sandwich_norm.cu)."""
+    evaluated in 32-bit on the product's rounded output (csrc/sandwich_norm.cu); "relu2", max(z, 0)^2, without a tensor.
+
+    A caller may own the two matrices (`shared_weights` = (up, down), set before the parameters are made): the routed
+    experts stack those of a shared expert of the experts' own size behind the experts'."""
+
+    shared_weights = None
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "xielu", names: dict | None = None):
         super().__init__()
-        if activation != "xielu":
-            raise ValueError(f"activation {activation!r} unknown (have ['xielu'])")
+        if activation not in ("xielu", "relu2"):
+            raise ValueError(f"activation {activation!r} unknown (have ['relu2', 'xielu'])")
         if hidden_size <= 0 or intermediate_size <= 0:
             raise ValueError("sizes must be positive")
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
@@ -91,7 +96,21 @@ class DenseMLP(FeedForward):
 
     def param_decls(self):
         H, I, n = self.hidden_size, self.intermediate_size, self.names
-        return {n["up"]: ParamDecl((I, H)), n["down"]: ParamDecl((H, I)), n["act"]: ParamDecl((2,), "bias32")}
+        d = {n["up"]: ParamDecl((I, H)), n["down"]: ParamDecl((H, I))}
+        if self.activation == "xielu":
+            d[n["act"]] = ParamDecl((2,), "bias32")
+        return d
+
+    def materialize(self, make):
+        n = self.names
+        for name, decl in self.param_decls().items():
+            if self.shared_weights is not None and name in (n["up"], n["down"]):
+                t = self.shared_weights[0 if name == n["up"] else 1]
+                if tuple(t.shape) != decl.shape:
+                    raise ValueError(f"the shared matrix for {name} has shape {tuple(t.shape)}, not {decl.shape}")
+                self.tensors[name] = t
+            else:
+                self.tensors[name] = make(name, decl)
 
     def activation_elems(self):
         return 2 * self.intermediate_size + self.hidden_size
@@ -100,8 +119,12 @@ class DenseMLP(FeedForward):
         T, I, n = x.shape[0], self.intermediate_size, self.names
         u = ctx.workspace.tokens("mlp.up", T, I, x.dtype)
         linear(x, self.tensors[n["up"]], u)
-        a = ctx.workspace.tokens("mlp.act", T, I, x.dtype)
-        kernels().xielu(u, self.tensors[n["act"]], a)
+        if self.activation == "relu2":
+            a = u
+            kernels().relu2(u, a)
+        else:
+            a = ctx.workspace.tokens("mlp.act", T, I, x.dtype)
+            kernels().xielu(u, self.tensors[n["act"]], a)
         out = ctx.workspace.tokens("ffn.out", T, self.hidden_size, x.dtype)
         linear(a, self.tensors[n["down"]], out)
         return out

@@ -38,7 +38,7 @@ class DecoderModel(Part):
         self.final_norm = build_norm(spec.final_norm)
         tied = spec.tie_embeddings and not untie_head
         self.head = OutputHead(spec.vocab_size, spec.hidden_size, self.embedding if tied else None, spec.head_param,
-                               softcap=spec.logit_softcap)
+                               softcap=spec.logit_softcap, scale=spec.logit_scale)
         self.token_side = None
         if spec.token_side is not None:
             self.token_side = TokenSideTable(spec.vocab_size, spec.token_side.dim, spec.token_side.shares)
@@ -175,7 +175,7 @@ class DecoderModel(Part):
                 nxt = (*params, h)
         kernels().norm_add_norm(stream, extra_rows=rows, extra_vec=vec, next_norm=nxt)
         if nxt is not None:
-            ctx.prepared_norm = (block.mixer_norm, nxt[3])
+            ctx.prepared_norm = (block.mixer_norm, nxt[-1])
         ctx.stream_operand = None
 
     def forward(self, ctx, caches):

@@ -1,4 +1,4 @@
-"""RMSNorm, alone or fused with the residual sum.
+"""Norms of rows: RMSNorm, alone or fused with the residual sum; LayerNorm; a tanh norm without statistics.
 
 ullm/layers/layernorm.py:20-34: everything in 32-bit; with a residual the sum
 x + residual is normed unrounded and its rounded value becomes the new
@@ -32,7 +32,7 @@ class RMSNorm(Norm):
         return self.weight, self.eps
 
     def row_params(self):
-        return self.weight, self.eps, False
+        return self.weight, self.eps, 0
 
     def scale_add(self, a, stream, mult: float, copy=None):
         kernels().norm_scale_add(a, stream, self.weight, self.eps, mult, copy)
@@ -72,7 +72,7 @@ class LayerNorm(Norm):
         return self.tensors[self.param]
 
     def row_params(self):
-        return self.weight, self.eps, True
+        return self.weight, self.eps, 1
 
     def scale_add(self, a, stream, mult: float, copy=None):
         if copy is not None:
@@ -82,4 +82,31 @@ class LayerNorm(Norm):
 
     def forward_rows(self, stream, rows, out):
         kernels().norm_rows(stream, rows, self.weight, self.eps, out, center=True)
+        return out
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanh(Norm):
+    """tanh(alpha * x) * weight + bias, element by element: one learned slope for the whole row, no mean and no
+    variance (`eps` is accepted and unused).  32-bit arithmetic on a 32-bit residual stream, one rounding at the store."""
+
+    def __init__(self, size: int, eps: float = 0.0, param: str = "weight", bias_param: str = "bias",
+                 alpha_param: str = "alpha"):
+        super().__init__()
+        self.size = size
+        self.eps = eps
+        self.names = dict(weight=param, bias=bias_param, alpha=alpha_param)
+
+    def param_decls(self):
+        n = self.names
+        return {n["weight"]: ParamDecl((self.size,), "norm"), n["bias"]: ParamDecl((self.size,), "bias32"),
+                n["alpha"]: ParamDecl((), "norm")}
+
+    def row_params(self):
+        n = self.names
+        return self.tensors[n["weight"]], self.eps, 2, self.tensors[n["alpha"]], self.tensors[n["bias"]]
+
+    def forward_rows(self, stream, rows, out):
+        w, eps, _kind, alpha, bias = self.row_params()
+        kernels().norm_rows(stream, rows, w, eps, out, alpha=alpha, bias=bias)
         return out

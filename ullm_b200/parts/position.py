@@ -47,10 +47,15 @@ def scaled_frequencies(rotary_dim: int, theta: float, scaling: dict | None = Non
     """f_i = theta^(-2i / rotary_dim) in 64-bit, i < rotary_dim / 2.  `scaling` (factor, low, high, original)
     rescales by wavelength l = 2 pi / f: waves shorter than original / high stay; waves longer than
     original / low are slowed by `factor`; between the two the slowed and the original frequency are blended
-    linearly in original / l."""
+    linearly in original / l.  With `factor` alone every frequency is slowed by it."""
     i = torch.arange(rotary_dim // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(theta), dtype=torch.float64), -2.0 * i / rotary_dim)
-    if scaling:
+    if scaling and set(scaling) == {"factor"}:
+        factor = float(scaling["factor"])
+        if factor <= 0:
+            raise ValueError("frequency scaling needs factor > 0")
+        f = f / factor
+    elif scaling:
         try:
             factor, low, high, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         except KeyError as e:
