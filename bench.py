@@ -848,6 +848,66 @@ def run_finosun(args) -> dict:
     return out
 
 
+# ---------------------------------------------------------------------------------------------------------
+# `--workload mafarax`: the Mafarax decoder beside the Ludalix decoder with attention, a state layer and routed experts
+# (the closest design the engine has: windowed attention, matrix memory and routed experts on a 32-bit stream)
+# ---------------------------------------------------------------------------------------------------------
+MAFARAX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, window=1024, state_heads=8, state_dim=128, state_vdim=256, experts=16,
+                  top=2, expert_ff=1024, vocab=32768, layers=8),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, window=2048, state_heads=8, state_dim=256, state_vdim=512, experts=32,
+                  top=2, expert_ff=2048, vocab=32768, layers=4),
+}
+
+
+def mafarax_config(width: int, heads: int, kv_heads: int, window: int, state_heads: int, state_dim: int, state_vdim: int,
+                   experts: int, top: int, expert_ff: int, vocab: int, layers: int) -> dict:
+    """`layers` layers of attention inside stretches of `window` positions beside a state-space recurrence with as many
+    state elements as the matrix memory of the given sizes (heads of 64 columns, `state_dim` rows), and routed experts
+    (four groups, two kept) with a shared expert of the same size."""
+    left = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=window),
+                rot=dict(dims=128, base=5e5, scaling=dict(factor=8.0)))
+    right = dict(heads=state_heads * state_vdim // 64, vdim=64, state=state_dim, groups=1, conv=4, norm_groups=1)
+    mlp = dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=expert_ff),
+               router=dict(experts=experts, top=top, scale=1.5, groups=dict(count=4, keep=2)))
+    return dict(architecture="Mafarax", vocab=vocab, width=width, logit_scale=0.5, norm=dict(eps=1e-6), torch_dtype="bfloat16",
+                layers=[dict(type="parallel", mixer=dict(left=left, right=right), mlp=dict(mlp)) for _ in range(layers)])
+
+
+def ludalix_pairs_config(width: int, heads: int, kv_heads: int, window: int, state_heads: int, state_dim: int,
+                         state_vdim: int, experts: int, top: int, expert_ff: int, vocab: int, layers: int) -> dict:
+    """`layers` pairs of a state layer without feed-forward and a windowed attention layer with routed experts: what one
+    Mafarax layer holds, one after the other."""
+    att = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, mask=dict(size=window, keep_first=0), scale=128 ** -0.5)
+    st = dict(heads=state_heads, dim=state_dim, vdim=state_vdim, gate_cap=15.0)
+    moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top))
+    pairs = []
+    for _ in range(layers):
+        pairs += [dict(type="mlstm", mixer=dict(st), mlp=None), dict(type="attention", mixer=dict(att), mlp=dict(moe))]
+    return dict(architecture="Ludalix", vocab=vocab, width=width, residual_mult=0.5, embedding=dict(scale=12.0),
+                norm=dict(eps=1e-6), layers=pairs, torch_dtype="bfloat16")
+
+
+def run_mafarax(args) -> dict:
+    """`--workload mafarax`: prefill (one prompt of 2,048 tokens) and decode (8 requests holding 2,048 tokens each) of the
+    Mafarax decoder at layer sizes that resemble a real model's, random weights, beside the Ludalix decoder with the same
+    mixers and routed experts one after the other; per kernel group the device time of one eager step of each kind.  One
+    JSON object; the default workload and its line are untouched."""
+    T, B, ctx_len = PREFILL_TOKENS, args.batch, START_CONTEXT
+    out = {"workload": "mafarax", "prefill_tokens": T, "decode_batch": B, "decode_context": ctx_len,
+           "data": "synthetic", "dtype": "bf16", "peaks": peaks(), "sizes": {}}
+    names = [args.case] if args.case else list(MAFARAX_SIZES)
+    for name in names:
+        size = MAFARAX_SIZES[name]
+        out["sizes"][name] = {}
+        for label, cfg in (("mafarax", mafarax_config(**size)), ("ludalix_pairs", ludalix_pairs_config(**size))):
+            if args.only_model and args.only_model != label:
+                continue
+            out["sizes"][name][label] = dict(_measure_model(cfg, False, T, B, ctx_len, args.steps, args.warmup),
+                                             layers=len(cfg["layers"]))
+    return out
+
+
 def run_extra_shapes(args, impl: str) -> dict:
     """The two further workloads, each in a process of its own (the 32B shape needs the device to itself), as
     flat entries for `points`."""
@@ -1510,7 +1570,8 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--workload", default="8b", choices=["8b", "32b", "serve-0.6b", "8b-long", "ludalix", "borosun", "pidenex", "finosun"],
+    ap.add_argument("--workload", default="8b", choices=["8b", "32b", "serve-0.6b", "8b-long", "ludalix", "borosun", "pidenex", "finosun",
+                                                           "mafarax"],
                     help="8b: the default line (Qwen3-8B layer sizes); 32b: the same at Qwen3-32B layer sizes; "
                          "serve-0.6b: 256 requests under continuous batching at Qwen3-0.6B layer sizes; 8b-long: "
                          "prefill of 16,384 tokens and decode of 8 requests at that context")
@@ -1524,7 +1585,8 @@ def main() -> int:
                     help="--probe linear: launch only this kernel, eagerly, --steps times (for a profiler)")
     ap.add_argument("--shape", default="gate_up", choices=["qkv", "o", "gate_up", "down", "head"],
                     help="--probe linear --only: which of the decode step's products")
-    ap.add_argument("--only-model", default=None, help="--workload borosun / pidenex / finosun: measure only this model (borosun, pidenex or finosun; ludalix_dense, ludalix_routed)")
+    ap.add_argument("--only-model", default=None, help="--workload borosun / pidenex / finosun / mafarax: measure only this model (borosun, pidenex, finosun or "
+                         "mafarax; ludalix_dense, ludalix_routed, ludalix_pairs)")
     ap.add_argument("--case", default=None, help="run only the case of this name (--probe prefill-attention, decode-attention)")
     ap.add_argument("--context", type=int, default=START_CONTEXT, help="tokens each request holds (--probe)")
     ap.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens of a page (--probe decode-attention)")
@@ -1572,6 +1634,9 @@ def main() -> int:
         return 0
     if args.workload == "finosun":
         print(json.dumps(run_finosun(args)))
+        return 0
+    if args.workload == "mafarax":
+        print(json.dumps(run_mafarax(args)))
         return 0
     out = run_serve(args) if args.workload == "serve-0.6b" else run_ours(args)
     if extra:
