@@ -174,6 +174,59 @@ def test_routing_by_groups_against_the_plain_choice():
             assert (choice[:, top + j] == E + j).all() and (weight[:, top + j] == 1).all()
 
 
+@pytest.mark.parametrize("heads,pdim,n,groups", [(2, 16, 32, 1), (4, 32, 64, 2), (3, 64, 128, 1), (2, 48, 256, 2), (40, 64, 128, 1)])
+def test_the_chunked_recurrence_against_the_plain_one(heads, pdim, n, groups):
+    """Portions of unequal length in one batch (one of them short enough to be left to the token-by-token kernel, one that
+    ends on a chunk's edge, one inside), from states that are not zero, with decays from nearly one to nearly nothing: the
+    chunked form, the token-by-token kernel and the plain recurrence in 64-bit give the same outputs and states."""
+    from ullm_b200.csrc import kernels
+
+    K = kernels()
+    lens, least = (130, 5, 64, 77, 192, 17), 16
+    T, B = sum(lens), len(lens)
+    g = torch.Generator().manual_seed(heads + n)
+    inner, ch = heads * pdim, heads * pdim + 2 * groups * n
+    xbc = (torch.randn(T, ch, generator=g) * 0.7).to(torch.bfloat16)
+    dt = torch.rand(T, heads, generator=g) * 0.5
+    dt[::13] *= 10.0
+    a = -dt * torch.exp(torch.linspace(-5.0, 2.0, heads))
+    D = torch.randn(heads, generator=g)
+    slots = [4, 0, 5, 1, 3, 2]
+    width = heads * pdim * n + 8
+    state0 = torch.randn(B, width, generator=g) * 0.3
+    cu = [0]
+    for k in lens:
+        cu.append(cu[-1] + k)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=device())
+    cu_q, req_slots, token_req = i32(cu), i32(slots), i32([i for i, k in enumerate(lens) for _ in range(k)])
+    dev = [t.to(device()) for t in (xbc, dt, a, D)]
+    ref = torch.zeros(T, inner, dtype=torch.float64)
+    ref_state = state0.double().clone()
+    for i in range(B):
+        S = state0[slots[i], :heads * pdim * n].double().reshape(heads, pdim, n).transpose(1, 2)  # [heads, N, P]
+        for t in range(cu[i], cu[i + 1]):
+            row = xbc[t].double()
+            x = row[:inner].reshape(heads, pdim)
+            Bm, Cm = (row[o:o + groups * n].reshape(groups, n).repeat_interleave(heads // groups, 0) for o in (inner, inner + groups * n))
+            S = torch.exp(a[t].double())[:, None, None] * S + dt[t].double()[:, None, None] * Bm[:, :, None] * x[:, None, :]
+            ref[t] = (torch.einsum("hnp,hn->hp", S, Cm) + D.double()[:, None] * x).reshape(-1)
+        ref_state[slots[i], :heads * pdim * n] = S.transpose(1, 2).reshape(-1)
+    assert K.ssd_chunk_applies(torch.bfloat16, heads, n, pdim, groups)
+    for name in ("chunked", "token by token"):
+        state = state0.to(device())
+        y = torch.full((T, inner), float("nan"), device=device())
+        if name == "chunked":
+            scores = torch.full((K.ssd_chunk_floats(T, groups),), float("nan"), device=device())
+            K.ssd_chunk(dev[0], inner, inner + groups * n, dev[1], dev[2], dev[3], scores, state, cu_q, req_slots, token_req,
+                        y, B, heads, n, pdim, groups, least)
+            assert torch.isnan(y[130:135]).all() and not torch.isnan(y[:130]).any() and not torch.isnan(y[135:]).any()
+        K.ssd_recurrence(dev[0], inner, inner + groups * n, dev[1], dev[2], dev[3], state, cu_q, req_slots, token_req, y, B,
+                         heads, n, pdim, groups, least if name == "chunked" else 1 << 30)
+        K.raise_on_status()
+        close(y, ref.float(), "float32", f"{name}: outputs")
+        close(state, ref_state.float(), "float32", f"{name}: states")
+
+
 def _ctx_for(r, tokens=128):
     from ullm_b200.engine.batch import Workspace
 

@@ -133,7 +133,7 @@ class Kernels:
                 "ULLM_B200_FUSE_DECODE_ROPE", "ULLM_B200_MIXED_DECODE_ROWS", "ULLM_B200_DECODE_TC",
                 "ULLM_B200_DECODE_BALANCED", "ULLM_B200_SMALL_M_LINEAR", "ULLM_B200_STREAM_WEIGHT_MB",
                 "ULLM_B200_FUSED_MLP_ROWS", "ULLM_B200_LT_ROWS", "ULLM_B200_FUSED_TAIL_ROWS",
-                "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC")
+                "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC", "ULLM_B200_SSD_CHUNK")
 
     def apply_switches(self, env) -> None:
         """Sets every kernel choice from `env` (a mapping; the process environment at start-up): a switch that is
@@ -158,6 +158,9 @@ class Kernels:
         self.general_attention_tc = get("ULLM_B200_GENERAL_ATTN_TC", "1") != "0"
         # windowed attention with its further options (values inside the keys, slopes, pooled blocks, a gate) on the
         # tensor-core kernel of csrc/attention_window.cu where the sizes allow; 0: the general kernel always
+        # the state-space recurrence of prompt portions in chunks on the tensor cores where the sizes allow; 0: token by
+        # token always
+        self.ssd_chunk_on = get("ULLM_B200_SSD_CHUNK", "1") != "0"
         self.window_attention_tc = get("ULLM_B200_WINDOW_ATTN_TC", "1") != "0"
         # the splits of a request's keys merge inside a thread-block cluster (at most 8 splits) instead of through
         # scratch arrays and a second kernel
@@ -269,6 +272,7 @@ class Kernels:
             "ullm_scale_f32": [P, LL, F, P],
             "ullm_ssd_prepare": [I, P, LL, I, I, I, I, P, I, P, P, P, P, LL, I, P, P, P, I, P, P, P, P, P],
             "ullm_ssd_recurrence": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
+            "ullm_ssd_chunk": [P, LL, I, I, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P, P],
             "ullm_ssd_gate_norm": [I, P, P, LL, P, P, I, I, I, F, P],
             "ullm_norm_rows": [I, P, P, P, P, I, I, I, F, I, P, P, P, P],
             "ullm_xielu": [I, P, P, LL, P, P],
@@ -307,6 +311,10 @@ class Kernels:
         L.ullm_gla_state_floats.restype = c_longlong
         L.ullm_ssd_supported.argtypes = [I, I, I, I, I]
         L.ullm_ssd_supported.restype = c_int
+        L.ullm_ssd_chunk_supported.argtypes = [I, I, I, I]
+        L.ullm_ssd_chunk_supported.restype = c_int
+        L.ullm_ssd_chunk_tokens.argtypes = []
+        L.ullm_ssd_chunk_tokens.restype = c_int
         L.ullm_wait_selftest.argtypes = [I, P, P, P]
         L.ullm_wait_selftest.restype = c_int
         L.ullm_decode_attention_supported.argtypes = [I, I, I]
@@ -1467,6 +1475,39 @@ class Kernels:
             state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), requests, heads, n_state, pdim,
             groups, state.shape[0], int(most_tokens), _ptr(self.status), _stream()),
             f"ssd_recurrence (heads {heads}, state {n_state}, columns {pdim})")
+
+    def ssd_chunk_applies(self, dtype, heads: int, n_state: int, pdim: int, groups: int) -> bool:
+        """True when `ssd_chunk` takes these sizes (bfloat16; see csrc/ssd_chunk.cu)."""
+        return bool(self.ssd_chunk_on and dtype == torch.bfloat16
+                    and self.lib.ullm_ssd_chunk_supported(heads, n_state, pdim, groups))
+
+    def ssd_chunk_floats(self, tokens: int, groups: int) -> int:
+        return tokens * groups * int(self.lib.ullm_ssd_chunk_tokens())
+
+    @_timed("ssd")
+    def ssd_chunk(self, xbc, b_off: int, c_off: int, dt, log_decay, d_skip, scores, state, cu_q, req_slots, token_req, out,
+                  requests: int, heads: int, n_state: int, pdim: int, groups: int, least: int):
+        """`ssd_recurrence` in its chunked form on the tensor cores, for the requests that bring MORE than `least` tokens
+        (the others are left alone); `scores`: scratch (float32, `ssd_chunk_floats`)."""
+        _need(xbc, "xbc", torch.bfloat16)
+        _need(state, "state", torch.float32, contiguous=False)
+        for t_, n_ in ((dt, "dt"), (log_decay, "log_decay"), (d_skip, "d_skip"), (out, "out"), (scores, "scores")):
+            _need(t_, n_, torch.float32)
+        for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
+            _need(t_, n_, torch.int32)
+        T = xbc.shape[0]
+        if (dt.shape != (T, heads) or log_decay.shape != (T, heads) or out.shape != (T, heads * pdim) or state.dim() != 2
+                or state.stride(1) != 1 or state.shape[1] < heads * pdim * n_state or d_skip.numel() != heads
+                or scores.numel() < self.ssd_chunk_floats(T, groups)):
+            raise KernelError(f"ssd_chunk: xbc {tuple(xbc.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+        if max(b_off, c_off) + groups * n_state > xbc.shape[1] or heads * pdim > xbc.shape[1]:
+            raise KernelError("ssd_chunk: x, B or C lie outside the rows")
+        self._check(self.lib.ullm_ssd_chunk(
+            _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(scores), _ptr(state),
+            state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), T, requests, heads, n_state, pdim,
+            groups, state.shape[0], int(least), _ptr(self.status), _stream()),
+            f"ssd_chunk (heads {heads}, state {n_state}, columns {pdim})")
+        self.launches += 1  # the scores in front of it
 
     @_timed("ssd")
     def ssd_gate_norm(self, y, z, weight, parts: int, eps: float, out):

@@ -24,6 +24,9 @@ from .linear import linear
 from .registry import register_mixer
 
 
+CHUNK_LEAST = 16  # requests that bring more tokens than this take the chunked form
+
+
 def _up4(n: int) -> int:
     return -(-n // 4) * 4
 
@@ -73,7 +76,9 @@ class Mamba2(Mixer, SharesInput):
 
     def activation_elems(self):
         # the input product, the convolved rows, steps and decays and y in 32-bit (two elements each), the gated y, the output
-        return (self.input_width() + self.channels + 4 * self.num_heads + 3 * self.inner + self.hidden_size)
+        # ... and the chunked form's scores
+        return (self.input_width() + self.channels + 4 * self.num_heads + 3 * self.inner + self.hidden_size
+                + 128 * self.groups)
 
     def output_projection(self):
         return self.tensors[self.names["o"]], None
@@ -98,8 +103,15 @@ class Mamba2(Mixer, SharesInput):
             K.conv_state_update(u[:, inner:inner + ch], self.conv_taps, conv_state, ctx.cu_q, ctx.token_req, ctx.req_slots,
                                 ctx.num_requests)
         y = ws.tokens("ssd.y", T, inner, torch.float32)
-        K.ssd_recurrence(xbc, inner, inner + G * S, dt, log_decay, t[n["d"]], cache.state, ctx.cu_q, ctx.req_slots,
-                         ctx.token_req, y, ctx.num_requests, N, S, P, G)
+        # prompt portions in chunks on the tensor cores (16-bit, at the sizes that form takes), the rest token by token
+        chunked = ctx.max_q_len > CHUNK_LEAST and K.ssd_chunk_applies(x.dtype, N, S, P, G)
+        if chunked:
+            scores = ws.tokens("ssd.scores", T, K.ssd_chunk_floats(1, G), torch.float32)
+            K.ssd_chunk(xbc, inner, inner + G * S, dt, log_decay, t[n["d"]], scores, cache.state, ctx.cu_q, ctx.req_slots,
+                        ctx.token_req, y, ctx.num_requests, N, S, P, G, CHUNK_LEAST)
+        if not chunked or ctx.num_requests > 1:
+            K.ssd_recurrence(xbc, inner, inner + G * S, dt, log_decay, t[n["d"]], cache.state, ctx.cu_q, ctx.req_slots,
+                             ctx.token_req, y, ctx.num_requests, N, S, P, G, CHUNK_LEAST if chunked else 1 << 30)
         g = ws.tokens("ssd.gated", T, inner, x.dtype)
         K.ssd_gate_norm(y, u[:, :inner], t[n["norm"]], self.norm_groups, self.eps, g)
         if not project_output:
