@@ -270,7 +270,7 @@ class Kernels:
             "ullm_pair_norm_add_norm": [I, P, P, P, P, I, I, F, F, P, P, P, F, I, P, P, P, P],
             "ullm_relu2": [I, P, P, LL, P],
             "ullm_scale_f32": [P, LL, F, P],
-            "ullm_ssd_prepare": [I, P, LL, I, I, I, I, P, I, P, P, P, P, LL, I, P, P, P, I, P, P, P, P, P],
+            "ullm_ssd_prepare": [I, P, LL, I, I, I, I, P, I, P, P, P, P, LL, I, P, P, P, I, P, P, P, I, P, P],
             "ullm_ssd_recurrence": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
             "ullm_ssd_chunk": [P, LL, I, I, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P, P],
             "ullm_ssd_gate_norm": [I, P, P, LL, P, P, I, I, I, F, P],
@@ -1423,10 +1423,12 @@ class Kernels:
 
     @_timed("ssd")
     def ssd_prepare(self, u, xbc_off: int, dt_off: int, conv_w, conv_b, dt_bias, a_log, conv_state, cu_q, token_req,
-                    req_slots, xbc, dt, log_decay):
+                    req_slots, xbc, dt, log_decay, single: bool = False):
         """u [T, *]: the projection's rows, x | B | C from column `xbc_off` and dt from `dt_off`; conv_w [channels, taps],
         conv_b [channels], dt_bias and a_log [heads] (float32); conv_state: the convolution's columns of the state rows
-        [slots, (taps - 1) * channels] (a view of wider rows).  Out: xbc [T, channels], dt and log_decay [T, heads]."""
+        [slots, (taps - 1) * channels] (a view of wider rows).  Out: xbc [T, channels], dt and log_decay [T, heads].
+        `single`: every request of the step has one token; the convolution's memory is then moved on here (no
+        `conv_state_update`)."""
         _need(u, "u", contiguous=False)
         _need(conv_w, "conv_w", u.dtype)
         _need(xbc, "xbc", u.dtype)
@@ -1449,7 +1451,7 @@ class Kernels:
         self._check(self.lib.ullm_ssd_prepare(
             _DT[u.dtype], _ptr(u), u.stride(0), xbc_off, dt_off, channels, heads, _ptr(conv_w), taps, _ptr(conv_b),
             _ptr(dt_bias), _ptr(a_log), _ptr(conv_state if taps > 1 else None), stride, slots, _ptr(cu_q), _ptr(token_req),
-            _ptr(req_slots), T, _ptr(xbc), _ptr(dt), _ptr(log_decay), _ptr(self.status), _stream()),
+            _ptr(req_slots), T, _ptr(xbc), _ptr(dt), _ptr(log_decay), int(bool(single)), _ptr(self.status), _stream()),
             f"ssd_prepare ({channels} channels, {taps} taps)")
 
     @_timed("ssd")

@@ -11,7 +11,7 @@
 //                   square, times a weight per channel
 //
 // The taps - 1 projected rows in front of a step's first token come from the state row too (zeros for a new request);
-// `conv_state_update` (csrc/attention_prep.cu) moves them on after the step.  The recurrence runs token by token in a
+// in a decode step `ssd_prepare` moves them on itself, otherwise `conv_state_update` (csrc/attention_prep.cu) after it.  The recurrence runs token by token in a
 // fixed order, so a request's result does not depend on how its tokens were cut into steps or on what else is in the
 // batch.  Its parallelism is over requests, heads and the columns of S: a block owns (request, head, a tile of
 // columns); a column's N rows are spread over `rs` neighbouring lanes in pieces of four, which meet in shuffles for
@@ -27,27 +27,28 @@
 
 __device__ __forceinline__ float ssd_softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
-// One thread: VEC neighbouring channels of SSD_TOK tokens in a row (a token's filter is in registers when TAPS > 0).
-// The blocks behind the channels' (blockIdx.x = channel blocks ..) do the step sizes.
-#define SSD_TOK 4
-template <typename T, int VEC, int TAPS>
+// One thread: VEC neighbouring channels of TOK tokens in a row.  With TAPS > 0 (the usual counts as constants) the filter
+// and the taps - 1 rows in front of the current token wait in registers, so every row is read once.  The blocks behind the
+// channels' (blockIdx.x >= channel_blocks) do the step sizes.  `single`: every request of the step has one token; the
+// thread that convolves a channel is then the only reader of its memory and moves it on itself.
+template <typename T, int VEC, int TAPS, int TOK>
 __global__ void ssd_prepare_kernel(const T* __restrict__ u, long long row_stride, int xbc_off, int dt_off, int channels,
                                    int heads, const T* __restrict__ conv_w, int taps_rt,
                                    const float* __restrict__ conv_b, const float* __restrict__ dt_bias,
-                                   const float* __restrict__ a_log, const float* __restrict__ conv_state,
+                                   const float* __restrict__ a_log, float* __restrict__ conv_state,
                                    long long state_stride, int num_slots, const int* __restrict__ cu_q,
                                    const int* __restrict__ token_req, const int* __restrict__ req_slots, int tokens,
                                    T* __restrict__ xbc, float* __restrict__ dt, float* __restrict__ log_decay,
-                                   int channel_blocks, int* status) {
+                                   int channel_blocks, int single, int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const int taps = TAPS > 0 ? TAPS : taps_rt;
-  const int tok0 = blockIdx.y * SSD_TOK;
+  const int tok0 = blockIdx.y * TOK, tok1 = min(tokens, tok0 + TOK);
   if ((int)blockIdx.x >= channel_blocks) {
     const int h = (blockIdx.x - channel_blocks) * blockDim.x + threadIdx.x;
     if (h >= heads) return;
     const float neg_a = -expf(a_log[h]), bias = dt_bias[h];
-    for (int t = tok0; t < min(tokens, tok0 + SSD_TOK); ++t) {
+    for (int t = tok0; t < tok1; ++t) {
       const float d = token_req[t] >= 0 ? ssd_softplus(to_f32(u[(long long)t * row_stride + dt_off + h]) + bias) : 0.f;
       dt[(long long)t * heads + h] = d;
       log_decay[(long long)t * heads + h] = neg_a * d;
@@ -56,52 +57,93 @@ __global__ void ssd_prepare_kernel(const T* __restrict__ u, long long row_stride
   }
   const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
   if (c0 >= channels) return;
-  float w[VEC * (TAPS > 0 ? TAPS : 1)];
+  float cur[TOK][VEC];  // (asked for before anything depends on them)
+#pragma unroll
+  for (int i = 0; i < TOK; ++i)
+    if (tok0 + i < tok1) load_vec<T, VEC>(u + (long long)(tok0 + i) * row_stride + xbc_off + c0, cur[i]);
+  constexpr int TW = TAPS > 0 ? TAPS : 1, BACK = TAPS > 1 ? TAPS - 1 : 1;
+  float w[TW][VEC];  // flat: element i * TAPS + j is channel c0 + i's tap j
   if (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < VEC * TAPS; ++i) w[i] = to_f32(conv_w[(long long)c0 * TAPS + i]);
+    for (int j = 0; j < TW; ++j) load_vec<T, VEC>(conv_w + (long long)c0 * TW + j * VEC, w[j]);
   }
-  float bias[VEC];
+  float bias[VEC], win[BACK][VEC];
+  load_vec32<VEC>(conv_b + c0, bias);
+  int prev = -1, t0 = 0;
+  float* st = nullptr;
 #pragma unroll
-  for (int i = 0; i < VEC; ++i) bias[i] = conv_b != nullptr ? conv_b[c0 + i] : 0.f;
-  for (int t = tok0; t < min(tokens, tok0 + SSD_TOK); ++t) {
+  for (int i = 0; i < TOK; ++i) {
+    const int t = tok0 + i;
+    if (t >= tok1) break;
     const int r = token_req[t];
     float y[VEC];
-    if (r < 0) {
+    if (r < 0) {  // a row that belongs to no request
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) y[i] = 0.f;
+      for (int e = 0; e < VEC; ++e) y[e] = 0.f;
       store_vec<T, VEC>(xbc + (long long)t * channels + c0, y);
+      prev = -1;
       continue;
     }
-    const int t0 = cu_q[r];
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) y[i] = bias[i];
-    auto tap = [&](int j) {
-      const int row = t - (taps - 1 - j);
-      float v[VEC];
-      if (row >= t0) {
-        load_vec<T, VEC>(u + (long long)row * row_stride + xbc_off + c0, v);
+    const bool fresh = r != prev;
+    if (fresh) {
+      prev = r;
+      t0 = cu_q[r];
+      const int slot = req_slots[r];
+      st = nullptr;
+      if (taps > 1 && slot >= 0 && slot < num_slots) st = conv_state + (long long)slot * state_stride + c0;
+      else if (taps > 1) ullm_report(status, ULLM_STATUS_SLOT, t, slot);
+    }
+    auto row_back = [&](int back, float(&v)[VEC]) {  // the projected row `back` >= 1 tokens before t
+      if (t - back >= t0) {
+        load_vec<T, VEC>(u + (long long)(t - back) * row_stride + xbc_off + c0, v);
+      } else if (st != nullptr) {
+        load_vec32<VEC>(st + (long long)(taps - 1 - (t0 - (t - back))) * channels, v);
       } else {
-        const int slot = req_slots[r];
-        if (slot < 0 || slot >= num_slots) {
-          if (threadIdx.x == 0) ullm_report(status, ULLM_STATUS_SLOT, t, slot);
-          return;
-        }
-        const int s = taps - 1 - (t0 - row);  // t0 - row in 1 .. taps - 1
-        load_vec32<VEC>(conv_state + (long long)slot * state_stride + (long long)s * channels + c0, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = 0.f;
+      }
+    };
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y[e] = bias[e];
+    if (TAPS > 0) {
+      if (fresh && TAPS > 1) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) row_back(TAPS - 1 - j, win[j]);
       }
 #pragma unroll
-      for (int i = 0; i < VEC; ++i)
-        y[i] = fmaf(TAPS > 0 ? w[i * (TAPS > 0 ? TAPS : 1) + j] : to_f32(conv_w[(long long)(c0 + i) * taps + j]), v[i], y[i]);
-    };
-    if (TAPS > 0) {
+      for (int j = 0; j < TAPS; ++j) {
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) tap(j);
+        for (int e = 0; e < VEC; ++e) {
+          const int f = e * TW + j;  // (f / VEC, f % VEC: constants after unrolling)
+          y[e] = fmaf(w[f / VEC][f % VEC], j < TAPS - 1 ? win[j < BACK ? j : 0][e] : cur[i][e], y[e]);
+        }
+      }
+      if (TAPS > 1) {
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS - 1; ++j)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) win[j][e] = win[j + 1][e];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) win[BACK - 1][e] = cur[i][e];
+        if (single && st != nullptr) {
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) store_vec32<VEC>(st + (long long)j * channels, win[j]);
+        }
+      }
     } else {
-      for (int j = 0; j < taps; ++j) tap(j);
+      float v[VEC];
+      for (int j = 0; j < taps - 1; ++j) {
+        row_back(taps - 1 - j, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(to_f32(conv_w[(long long)(c0 + e) * taps + j]), v[e], y[e]);
+        if (single && st != nullptr && j > 0) store_vec32<VEC>(st + (long long)(j - 1) * channels, v);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = fmaf(to_f32(conv_w[(long long)(c0 + e) * taps + taps - 1]), cur[i][e], y[e]);
+      if (single && st != nullptr) store_vec32<VEC>(st + (long long)(taps - 2) * channels, cur[i]);
     }
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) y[i] = act_silu(y[i]);
+    for (int e = 0; e < VEC; ++e) y[e] = act_silu(y[e]);
     store_vec<T, VEC>(xbc + (long long)t * channels + c0, y);
   }
 }
@@ -336,47 +378,56 @@ extern "C" int ullm_ssd_supported(int heads, int n_state, int pdim, int groups, 
 template <typename T>
 static int prepare_go(const void* u, long long row_stride, int xbc_off, int dt_off, int channels, int heads,
                       const void* conv_w, int taps, const float* conv_b, const float* dt_bias, const float* a_log,
-                      const float* conv_state, long long state_stride, int num_slots, const int* cu_q,
+                      float* conv_state, long long state_stride, int num_slots, const int* cu_q,
                       const int* token_req, const int* req_slots, int tokens, void* xbc, float* dt, float* log_decay,
-                      int* status, cudaStream_t st) {
+                      int single, int* status, cudaStream_t st) {
   constexpr int V = 16 / (int)sizeof(T);
   const bool wide = channels % V == 0 && xbc_off % V == 0 && row_stride % V == 0 && state_stride % 4 == 0 &&
-                    (((uintptr_t)u | (uintptr_t)xbc | (uintptr_t)conv_state) & 15) == 0;
+                    (((uintptr_t)u | (uintptr_t)xbc | (uintptr_t)conv_state | (uintptr_t)conv_w | (uintptr_t)conv_b) & 15) == 0;
   const int vec = wide ? V : 1;
-  const int threads = 128;
+  // steps of few tokens: a token per thread, small blocks; prompts: four tokens share a thread's filter and rows
+  const int tok = tokens >= 512 ? 4 : 1, threads = tokens >= 512 ? 128 : 64;
   const int cb = (channels + threads * vec - 1) / (threads * vec), hb = (heads + threads - 1) / threads;
-  const dim3 grid(cb + hb, (tokens + SSD_TOK - 1) / SSD_TOK), block(threads);
+  const dim3 grid(cb + hb, (tokens + tok - 1) / tok), block(threads);
   if (grid.y > 65535) return ULLM_ERR_BAD_SIZE;
-#define SP_GO(VEC, TAPS)                                                                                              \
-  return ullm_launch_kernel(ssd_prepare_kernel<T, VEC, TAPS>, grid, block, 0, st, (const T*)u, row_stride, xbc_off,   \
-                            dt_off, channels, heads, (const T*)conv_w, taps, conv_b, dt_bias, a_log, conv_state,      \
-                            state_stride, num_slots, cu_q, token_req, req_slots, tokens, (T*)xbc, dt, log_decay, cb,  \
-                            status)
-  if (wide) {
-    if (taps == 4) SP_GO(V, 4);
-    SP_GO(V, 0);
+#define SP_GO(VEC, TAPS, TOK)                                                                                         \
+  return ullm_launch_kernel(ssd_prepare_kernel<T, VEC, TAPS, TOK>, grid, block, 0, st, (const T*)u, row_stride,       \
+                            xbc_off, dt_off, channels, heads, (const T*)conv_w, taps, conv_b, dt_bias, a_log,         \
+                            conv_state, state_stride, num_slots, cu_q, token_req, req_slots, tokens, (T*)xbc, dt,     \
+                            log_decay, cb, single, status)
+#define SP_TOK(VEC, TAPS)              \
+  {                                    \
+    if (tok == 4) SP_GO(VEC, TAPS, 4); \
+    SP_GO(VEC, TAPS, 1);               \
   }
-  if (taps == 4) SP_GO(1, 4);
-  SP_GO(1, 0);
+  if (wide) {
+    if (taps == 4) SP_TOK(V, 4);
+    if (taps == 3) SP_TOK(V, 3);
+    if (taps == 2) SP_TOK(V, 2);
+    SP_TOK(V, 0);
+  }
+  SP_TOK(1, 0);
+#undef SP_TOK
 #undef SP_GO
 }
 
 // u: rows of the projection, x | B | C (`channels` columns) from column xbc_off, dt (heads columns) from dt_off;
 // conv_w [channels][taps], the last column meets the current token; conv_state: the convolution's part of the requests'
-// state rows.  xbc [tokens, channels]; dt, log_decay [tokens, heads] 32-bit.
+// state rows.  xbc [tokens, channels]; dt, log_decay [tokens, heads] 32-bit.  `single`: every request has one token (a
+// decode step); the convolution's memory is then moved on here, and `ullm_conv_state_update` is not needed.
 extern "C" int ullm_ssd_prepare(int dtype, const void* u, long long row_stride, int xbc_off, int dt_off, int channels,
                                 int heads, const void* conv_w, int taps, const float* conv_b, const float* dt_bias,
-                                const float* a_log, const float* conv_state, long long state_stride, int num_slots,
+                                const float* a_log, float* conv_state, long long state_stride, int num_slots,
                                 const int* cu_q, const int* token_req, const int* req_slots, int tokens, void* xbc,
-                                float* dt, float* log_decay, int* status, void* stream) {
+                                float* dt, float* log_decay, int single, int* status, void* stream) {
   cudaStream_t st = (cudaStream_t)stream;
-  if (tokens < 0 || channels <= 0 || heads <= 0 || taps < 1 || (taps > 1 && (conv_state == nullptr || num_slots <= 0)))
+  if (tokens < 0 || channels <= 0 || heads <= 0 || taps < 1 || conv_b == nullptr || (taps > 1 && (conv_state == nullptr || num_slots <= 0)))
     return ULLM_ERR_BAD_SIZE;
   if (taps > SSD_MAX_TAPS) return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;
 #define SP_ARGS                                                                                                       \
   u, row_stride, xbc_off, dt_off, channels, heads, conv_w, taps, conv_b, dt_bias, a_log, conv_state, state_stride,    \
-      num_slots, cu_q, token_req, req_slots, tokens, xbc, dt, log_decay, status, st
+      num_slots, cu_q, token_req, req_slots, tokens, xbc, dt, log_decay, single, status, st
   if (dtype == ULLM_DTYPE_F32) return prepare_go<float>(SP_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return prepare_go<__nv_bfloat16>(SP_ARGS);
   if (dtype == ULLM_DTYPE_F16) return prepare_go<__half>(SP_ARGS);

@@ -124,10 +124,13 @@ ssd_scores_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, i
   }
 }
 
-// PT: columns of S a block owns (16 or 32); n_state = 32 * NT.  Warp w finishes the chunk's rows 16 w .. 16 w + 15 of y and
-// keeps the columns w N / 4 .. of S^T [PT][N].
-template <int PT, int NT>
-__global__ void __launch_bounds__(SSC_THREADS)
+// PT: columns of S a block owns (16 or 32); n_state = 32 * NT.  Two sets of four warps work on a chunk side by side: set 0
+// forms its y (warp w the rows 16 w .. 16 w + 15) from the state in front of it, which waits in shared memory as two bfloat16
+// terms; set 1 keeps S^T [PT][N] in accumulators (warp w the columns w N / 4 ..), adds the chunk to it, and fetches the next
+// chunk's rows and decays meanwhile.  SB: buffers of the state's terms (with two, one barrier of the block per chunk; with
+// one, where two do not fit, a second barrier stands in front of their renewal).
+template <int PT, int NT, int SB>
+__global__ void __launch_bounds__(2 * SSC_THREADS)
 ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, int b_off, int c_off,
                  const float* __restrict__ dt, const float* __restrict__ log_decay, const float* __restrict__ d_skip,
                  const float* __restrict__ scores, float* __restrict__ state, long long state_stride,
@@ -138,27 +141,112 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
   constexpr int RS = N * 2 + 16;              // bytes between rows of B, C and S
   constexpr int XS = PT * 2 + 16;             // ... of x
   constexpr int BC = SSC_Q * RS, XB = SSC_Q * XS, GB = SSC_Q * SSC_G_STRIDE * 4;
-  constexpr int STAGE = 2 * BC + XB + GB;
+  constexpr int STAGE = 2 * BC + XB + GB, ST = PT * RS;
   constexpr int MT = PT / 16, PN = PT / 8;
   extern __shared__ __align__(16) unsigned char sc_smem[];
-  __shared__ float s_cum[SSC_Q], s_dt[SSC_Q], s_e[SSC_Q], s_w[SSC_Q];
-  __shared__ float s_total;
+  __shared__ float s_cum[2][SSC_Q], s_dt[2][SSC_Q], s_e[2][SSC_Q], s_w[2][SSC_Q];
+  __shared__ float s_total[2];
   pdl_launch_dependents();
   pdl_wait();
   const int req = blockIdx.z, head = blockIdx.y, p0 = blockIdx.x * PT;
   const int t0 = cu_q[req], n = cu_q[req + 1] - t0;
   if (n <= least || token_req[t0] < 0) return;
   const int slot = req_slots[req];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x & (SSC_THREADS - 1), warp = tid >> 5, lane = tid & 31;
+  const bool keeper = threadIdx.x >= SSC_THREADS;  // set 1
   if (slot < 0 || slot >= num_slots) {
-    if (tid == 0) ullm_report(status, ULLM_STATUS_SLOT, req, slot);
+    if (threadIdx.x == 0) ullm_report(status, ULLM_STATUS_SLOT, req, slot);
     return;
   }
   const int group = head / per_group;
-  unsigned char* sh_s = sc_smem + 2 * STAGE;  // S^T rounded, [PT][N]
-  unsigned char* sl_s = sh_s + PT * RS;       // ... the rests
-  unsigned char* xh_s = sl_s + PT * RS;       // weighted x rounded, [SSC_Q][PT]
+  unsigned char* s_terms = sc_smem + 2 * STAGE;  // [SB]: S^T rounded [PT][N], then the rests
+  unsigned char* xh_s = s_terms + SB * 2 * ST;   // weighted x rounded, [SSC_Q][PT]
   unsigned char* xl_s = xh_s + XB;
+  const int mat = lane >> 3;
+  const int chunks = (n + SSC_Q - 1) / SSC_Q;
+
+  if (!keeper) {
+    const float skip = d_skip[head];
+    __syncthreads();  // chunk 0, its decays and the first state's terms are there
+    for (int c = 0; c < chunks; ++c) {
+      const int cn = min(SSC_Q, n - c * SSC_Q), cb = c & 1;
+      const unsigned char* stg = sc_smem + cb * STAGE;
+      const unsigned char* sh_s = s_terms + (SB == 2 ? cb : 0) * 2 * ST;
+      const unsigned char* sl_s = sh_s + ST;
+      const unsigned char* x_s = stg + 2 * BC;
+      const int tr = warp * 16;  // the warp's rows of y
+      if (tr < cn) {
+        float y[PN][4], yi[PN][4];
+#pragma unroll
+        for (int j = 0; j < PN; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[j][e] = yi[j][e] = 0.f;
+        // what the state in front of the chunk gives
+#pragma unroll(4)
+        for (int k = 0; k < N / 16; ++k) {
+          unsigned a[4];
+          ssc_ldsm4(a, stg + (tr + (mat & 1) * 8 + (lane & 7)) * RS + (k * 16 + (mat >> 1) * 8) * 2);
+#pragma unroll
+          for (int j = 0; j < PN; j += 2) {
+            const int off = (j * 8 + (mat >> 1) * 8 + (lane & 7)) * RS + (k * 16 + (mat & 1) * 8) * 2;
+            unsigned bh[4], bl[4];
+            ssc_ldsm4(bh, sh_s + off);
+            ssc_ldsm4(bl, sl_s + off);
+            ssc_mma(yi[j], a, bh[0], bh[1]);
+            ssc_mma(yi[j + 1], a, bh[2], bh[3]);
+            ssc_mma(yi[j], a, bl[0], bl[1]);
+            ssc_mma(yi[j + 1], a, bl[2], bl[3]);
+          }
+        }
+        // what the tokens of this chunk leave to one another
+        const float* g_s = reinterpret_cast<const float*>(stg + 2 * BC + XB);
+        const int r0 = tr + (lane >> 2);
+        const float cr[2] = {s_cum[cb][r0], s_cum[cb][r0 + 8]};
+#pragma unroll
+        for (int ks = 0; ks < SSC_Q / 16; ++ks) {
+          if (ks > warp) continue;
+          unsigned ah[4], al[4];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {  // the fragment's four register pairs: rows + 8 (q & 1), columns + 8 (q >> 1)
+            const int row = r0 + (q & 1) * 8, s = ks * 16 + (q >> 1) * 8 + (lane & 3) * 2;
+            const float2 g = *reinterpret_cast<const float2*>(g_s + row * SSC_G_STRIDE + s);
+            const float2 cs = *reinterpret_cast<const float2*>(&s_cum[cb][s]);
+            const float2 ds = *reinterpret_cast<const float2*>(&s_dt[cb][s]);
+            const float v0 = s <= row ? g.x * (__expf(cr[q & 1] - cs.x) * ds.x) : 0.f;
+            const float v1 = s + 1 <= row ? g.y * (__expf(cr[q & 1] - cs.y) * ds.y) : 0.f;
+            ssc_split(v0, v1, ah[q], al[q]);
+          }
+#pragma unroll
+          for (int j = 0; j < PN; j += 2) {
+            unsigned b[4];
+            ssc_ldsm4t(b, x_s + (ks * 16 + (mat & 1) * 8 + (lane & 7)) * XS + (j * 8 + (mat >> 1) * 8) * 2);
+            ssc_mma(y[j], ah, b[0], b[1]);
+            ssc_mma(y[j + 1], ah, b[2], b[3]);
+            ssc_mma(y[j], al, b[0], b[1]);
+            ssc_mma(y[j + 1], al, b[2], b[3]);
+          }
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int row = r0 + 8 * h;
+          if (row >= cn) continue;
+          const float e = s_e[cb][row];
+          float* dst = out + ((long long)(t0 + c * SSC_Q + row) * heads + head) * pdim + p0 + (lane & 3) * 2;
+#pragma unroll
+          for (int j = 0; j < PN; ++j) {
+            const __nv_bfloat162 xv =
+                *reinterpret_cast<const __nv_bfloat162*>(x_s + row * XS + (j * 8 + (lane & 3) * 2) * 2);
+            *reinterpret_cast<float2*>(dst + j * 8) =
+                make_float2(fmaf(e, yi[j][2 * h], y[j][2 * h]) + skip * __bfloat162float(xv.x),
+                            fmaf(e, yi[j][2 * h + 1], y[j][2 * h + 1]) + skip * __bfloat162float(xv.y));
+          }
+        }
+      }
+      if (SB == 1) __syncthreads();  // the state's terms have been read
+      __syncthreads();               // the chunk is done, the next one is there
+    }
+    return;
+  }
 
   auto issue = [&](int chunk) {
     unsigned char* st = sc_smem + (chunk & 1) * STAGE;
@@ -184,6 +272,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
       ssc_cp_async_16(st + 2 * BC + XB + row * (SSC_G_STRIDE * 4) + ch * 16,
                       scores + ((long long)group * tokens + c0 + (ok ? row : 0)) * SSC_Q + ch * 4, ok);
     }
+    ssc_commit();
   };
   float pa[2] = {0.f, 0.f}, pd[2] = {0.f, 0.f};  // warp 0: decays and steps of tokens 2 lane, 2 lane + 1, a chunk ahead
   auto fetch = [&](int chunk) {
@@ -194,9 +283,43 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
       pd[i] = t < n ? dt[(long long)(t0 + t) * heads + head] : 0.f;
     }
   };
+  auto weigh = [&](int buf) {  // warp 0: the chunk's running sums and weights from what `fetch` brought
+    float run = pa[0] + pa[1];  // the inclusive sum over the lanes
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += v;
+    }
+    const float total = __shfl_sync(0xffffffffu, run, 31);
+    const float cu[2] = {run - pa[1], run};
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      s_cum[buf][2 * lane + i] = cu[i];
+      s_dt[buf][2 * lane + i] = pd[i];
+      s_e[buf][2 * lane + i] = expf(cu[i]);
+      s_w[buf][2 * lane + i] = expf(total - cu[i]) * pd[i];
+    }
+    if (lane == 0) s_total[buf] = expf(total);
+  };
 
   // S^T fragments: rows p = 16 m + lane / 4 (+ 8), columns n = warp * NW + 8 j + 2 (lane % 4) (+ 1)
   float S[MT][NT][4];
+  auto put_terms = [&](int buf) {
+    unsigned char* sh_s = s_terms + (SB == 2 ? buf : 0) * 2 * ST;
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          unsigned hi, lo;
+          ssc_split(S[m][j][2 * h], S[m][j][2 * h + 1], hi, lo);
+          const int off = (16 * m + (lane >> 2) + 8 * h) * RS + (warp * NW + 8 * j + (lane & 3) * 2) * 2;
+          *reinterpret_cast<unsigned*>(sh_s + off) = hi;
+          *reinterpret_cast<unsigned*>(sh_s + ST + off) = lo;
+        }
+  };
+  issue(0);
   float* st_head = state + (long long)slot * state_stride + ((long long)head * pdim + p0) * N;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -209,133 +332,31 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
         S[m][j][2 * h] = v.x;
         S[m][j][2 * h + 1] = v.y;
       }
-  const float skip = d_skip[head];
-  const int chunks = (n + SSC_Q - 1) / SSC_Q;
-  issue(0);
-  ssc_commit();
-  if (warp == 0) fetch(0);
-
+  if (warp == 0) {
+    fetch(0);
+    weigh(0);
+    if (chunks > 1) fetch(1);
+  }
+  put_terms(0);
+  ssc_wait<0>();
+  __syncthreads();
   for (int c = 0; c < chunks; ++c) {
-    const int cn = min(SSC_Q, n - c * SSC_Q);
-    unsigned char* stg = sc_smem + (c & 1) * STAGE;
+    const int cb = c & 1;
+    unsigned char* stg = sc_smem + cb * STAGE;
     if (c + 1 < chunks) issue(c + 1);
-    ssc_commit();
-    if (warp == 0) {
-      float run = pa[0] + pa[1];  // the inclusive sum over the lanes
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float v = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += v;
-      }
-      const float total = __shfl_sync(0xffffffffu, run, 31);
-      const float cu[2] = {run - pa[1], run};
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        s_cum[2 * lane + i] = cu[i];
-        s_dt[2 * lane + i] = pd[i];
-        s_e[2 * lane + i] = expf(cu[i]);
-        s_w[2 * lane + i] = expf(total - cu[i]) * pd[i];
-      }
-      if (lane == 0) s_total = expf(total);
-      if (c + 1 < chunks) fetch(c + 1);
-    }
-    // the state in front of this chunk, as two terms
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int j = 0; j < NT; ++j)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          unsigned hi, lo;
-          ssc_split(S[m][j][2 * h], S[m][j][2 * h + 1], hi, lo);
-          const int off = (16 * m + (lane >> 2) + 8 * h) * RS + (warp * NW + 8 * j + (lane & 3) * 2) * 2;
-          *reinterpret_cast<unsigned*>(sh_s + off) = hi;
-          *reinterpret_cast<unsigned*>(sl_s + off) = lo;
-        }
-    ssc_wait<1>();
-    __syncthreads();
-    const unsigned char* x_s = stg + 2 * BC;
     // x weighted by its step and by what is left of it at the chunk's end, as two terms
+    const unsigned char* x_s = stg + 2 * BC;
     for (int i = tid; i < SSC_Q * PT / 2; i += SSC_THREADS) {
       const int row = i / (PT / 2), q = i - row * (PT / 2);
       const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(x_s + row * XS + q * 4);
-      const float w = s_w[row];
+      const float w = s_w[cb][row];
       unsigned hi, lo;
       ssc_split(__bfloat162float(v.x) * w, __bfloat162float(v.y) * w, hi, lo);
       *reinterpret_cast<unsigned*>(xh_s + row * XS + q * 4) = hi;
       *reinterpret_cast<unsigned*>(xl_s + row * XS + q * 4) = lo;
     }
-    const int mat = lane >> 3;
-    const int tr = warp * 16;  // the warp's rows of y
-    if (tr < cn) {
-      float y[PN][4], yi[PN][4];
-#pragma unroll
-      for (int j = 0; j < PN; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) y[j][e] = yi[j][e] = 0.f;
-      // what the tokens of this chunk leave to one another
-      const float* g_s = reinterpret_cast<const float*>(stg + 2 * BC + XB);
-      const int r0 = tr + (lane >> 2);
-      const float cr[2] = {s_cum[r0], s_cum[r0 + 8]};
-#pragma unroll
-      for (int ks = 0; ks < SSC_Q / 16; ++ks) {
-        if (ks > warp) continue;
-        unsigned ah[4], al[4];
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {  // the fragment's four register pairs: rows + 8 (q & 1), columns + 8 (q >> 1)
-          const int row = r0 + (q & 1) * 8, s = ks * 16 + (q >> 1) * 8 + (lane & 3) * 2;
-          const float2 g = *reinterpret_cast<const float2*>(g_s + row * SSC_G_STRIDE + s);
-          const float2 cs = *reinterpret_cast<const float2*>(s_cum + s);
-          const float2 ds = *reinterpret_cast<const float2*>(s_dt + s);
-          const float v0 = s <= row ? g.x * (__expf(cr[q & 1] - cs.x) * ds.x) : 0.f;
-          const float v1 = s + 1 <= row ? g.y * (__expf(cr[q & 1] - cs.y) * ds.y) : 0.f;
-          ssc_split(v0, v1, ah[q], al[q]);
-        }
-#pragma unroll
-        for (int j = 0; j < PN; j += 2) {
-          unsigned b[4];
-          ssc_ldsm4t(b, x_s + (ks * 16 + (mat & 1) * 8 + (lane & 7)) * XS + (j * 8 + (mat >> 1) * 8) * 2);
-          ssc_mma(y[j], ah, b[0], b[1]);
-          ssc_mma(y[j], al, b[0], b[1]);
-          ssc_mma(y[j + 1], ah, b[2], b[3]);
-          ssc_mma(y[j + 1], al, b[2], b[3]);
-        }
-      }
-      // what the state in front of the chunk gives
-#pragma unroll(4)
-      for (int k = 0; k < N / 16; ++k) {
-        unsigned a[4];
-        ssc_ldsm4(a, stg + (tr + (mat & 1) * 8 + (lane & 7)) * RS + (k * 16 + (mat >> 1) * 8) * 2);
-#pragma unroll
-        for (int j = 0; j < PN; j += 2) {
-          const int off = (j * 8 + (mat >> 1) * 8 + (lane & 7)) * RS + (k * 16 + (mat & 1) * 8) * 2;
-          unsigned bh[4], bl[4];
-          ssc_ldsm4(bh, sh_s + off);
-          ssc_ldsm4(bl, sl_s + off);
-          ssc_mma(yi[j], a, bh[0], bh[1]);
-          ssc_mma(yi[j], a, bl[0], bl[1]);
-          ssc_mma(yi[j + 1], a, bh[2], bh[3]);
-          ssc_mma(yi[j + 1], a, bl[2], bl[3]);
-        }
-      }
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int row = r0 + 8 * h;
-        if (row >= cn) continue;
-        const float e = s_e[row];
-        float* dst = out + ((long long)(t0 + c * SSC_Q + row) * heads + head) * pdim + p0 + (lane & 3) * 2;
-#pragma unroll
-        for (int j = 0; j < PN; ++j) {
-          const __nv_bfloat162 xv =
-              *reinterpret_cast<const __nv_bfloat162*>(x_s + row * XS + (j * 8 + (lane & 3) * 2) * 2);
-          *reinterpret_cast<float2*>(dst + j * 8) =
-              make_float2(fmaf(e, yi[j][2 * h], y[j][2 * h]) + skip * __bfloat162float(xv.x),
-                          fmaf(e, yi[j][2 * h + 1], y[j][2 * h + 1]) + skip * __bfloat162float(xv.y));
-        }
-      }
-    }
-    __syncthreads();  // the weighted x is complete
-    const float total = s_total;
+    asm volatile("bar.sync 1, %0;" ::"n"(SSC_THREADS) : "memory");  // (set 1 alone)
+    const float total = s_total[cb];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -359,17 +380,23 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           ssc_mma(S[m][j], ah[m], b[0], b[1]);
+          if (NT > 1) ssc_mma(S[m][NT > 1 ? j + 1 : j], ah[m], b[2], b[3]);
           ssc_mma(S[m][j], al[m], b[0], b[1]);
-          if (NT > 1) {
-            ssc_mma(S[m][NT > 1 ? j + 1 : j], ah[m], b[2], b[3]);
-            ssc_mma(S[m][NT > 1 ? j + 1 : j], al[m], b[2], b[3]);
-          }
+          if (NT > 1) ssc_mma(S[m][NT > 1 ? j + 1 : j], al[m], b[2], b[3]);
         }
       }
     }
-    __syncthreads();  // this chunk's rows, weights and state terms have been read
+    if (SB == 1) __syncthreads();  // set 0 has read the state's terms
+    if (c + 1 < chunks) {
+      put_terms(cb ^ 1);
+      if (warp == 0) {
+        weigh(cb ^ 1);
+        if (c + 2 < chunks) fetch(c + 2);
+      }
+      ssc_wait<0>();
+    }
+    __syncthreads();
   }
-  ssc_wait<0>();
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -393,18 +420,20 @@ static int chunk_go(const void* xbc, long long row_stride, int b_off, int c_off,
                     const int* req_slots, const int* token_req, float* out, int tokens, int requests, int heads, int pdim,
                     int groups, int num_slots, int least, int* status, cudaStream_t st) {
   constexpr int N = 32 * NT, RS = N * 2 + 16, XS = PT * 2 + 16;
-  constexpr size_t smem = 2 * (2 * SSC_Q * RS + SSC_Q * XS + SSC_Q * SSC_G_STRIDE * 4) + 2 * PT * RS + 2 * SSC_Q * XS;
-  static_assert(smem <= 227 * 1024, "a chunk's stages fit the shared memory");
+  constexpr size_t stages = 2 * (2 * SSC_Q * RS + SSC_Q * XS + SSC_Q * SSC_G_STRIDE * 4) + 2 * SSC_Q * XS;
+  constexpr int SB = stages + 4 * PT * RS + 2304 <= 227 * 1024 ? 2 : 1;  // (2304: more than the static arrays)
+  constexpr size_t smem = stages + SB * 2 * PT * RS;
+  static_assert(smem + 2304 <= 227 * 1024, "a chunk's stages fit the shared memory");
   static int attr_set = 0;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(ssd_chunk_kernel<PT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(ssd_chunk_kernel<PT, NT, SB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       cudaGetLastError();
       return ULLM_ERR_LAUNCH;
     }
-    cudaFuncSetAttribute(ssd_chunk_kernel<PT, NT>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    cudaFuncSetAttribute(ssd_chunk_kernel<PT, NT, SB>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     attr_set = 1;
   }
-  return ullm_launch_kernel(ssd_chunk_kernel<PT, NT>, dim3(pdim / PT, heads, requests), dim3(SSC_THREADS), smem, st,
+  return ullm_launch_kernel(ssd_chunk_kernel<PT, NT, SB>, dim3(pdim / PT, heads, requests), dim3(2 * SSC_THREADS), smem, st,
                             (const __nv_bfloat16*)xbc, row_stride, b_off, c_off, dt, log_decay, d_skip, scores, state,
                             state_stride, cu_q, req_slots, token_req, out, heads, pdim, heads / groups, tokens, num_slots,
                             least, status);
@@ -440,8 +469,13 @@ extern "C" int ullm_ssd_chunk(const void* xbc, long long row_stride, int b_off, 
   if (rc != ULLM_OK) return rc;
   int sms = 148, dev = 0;
   if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-  // 32 columns per block where there are blocks enough (fewer blocks read the same B, C and scores), else 16
-  const bool wide = pdim % 32 == 0 && (long long)(pdim / 32) * heads * requests >= sms;
+  // 16 or 32 columns per block, by (waves of blocks) x (a chunk's cost, which grows slowly with the columns)
+  const int per_sm = n_state <= 64 ? 3 : (n_state == 128 ? 2 : 1);
+  const long long b16 = (long long)(pdim / 16) * heads * requests, b32 = (long long)(pdim / 32) * heads * requests;
+  const double places = (double)per_sm * sms;
+  const double c16 = b16 <= sms ? 1.0 : (double)((long long)((b16 + places - 1) / places)) * per_sm;
+  const double c32 = (b32 <= sms ? 1.0 : (double)((long long)((b32 + places - 1) / places)) * per_sm) * 1.5;
+  const bool wide = pdim % 32 == 0 && c32 < c16;
 #define SSC_GO(PT, NT)                                                                                               \
   return chunk_go<PT, NT>(xbc, row_stride, b_off, c_off, dt, log_decay, d_skip, scores, state, state_stride, cu_q,    \
                           req_slots, token_req, out, tokens, requests, heads, pdim, groups, num_slots, least, status, st)

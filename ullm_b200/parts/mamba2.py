@@ -98,8 +98,8 @@ class Mamba2(Mixer, SharesInput):
         dt = ws.tokens("ssd.dt", T, N, torch.float32)
         log_decay = ws.tokens("ssd.log_decay", T, N, torch.float32)
         K.ssd_prepare(u, inner, inner + ch, t[n["conv"]], t[n["conv_bias"]], t[n["dt_bias"]], t[n["a_log"]], conv_state,
-                      ctx.cu_q, ctx.token_req, ctx.req_slots, xbc, dt, log_decay)
-        if self.conv_taps > 1:
+                      ctx.cu_q, ctx.token_req, ctx.req_slots, xbc, dt, log_decay, single=ctx.max_q_len == 1)
+        if self.conv_taps > 1 and ctx.max_q_len > 1:
             K.conv_state_update(u[:, inner:inner + ch], self.conv_taps, conv_state, ctx.cu_q, ctx.token_req, ctx.req_slots,
                                 ctx.num_requests)
         y = ws.tokens("ssd.y", T, inner, torch.float32)
