@@ -143,7 +143,8 @@ def attention_reference(q, kf, vf, block_table, req_slots, q_lens, kv_lens, Hq, 
     for r, (ql, kl) in enumerate(zip(q_lens, kv_lens)):
         for j in range(ql):
             pos = kl - ql + j
-            lo = max(0, pos - window + 1) if window else 0
+            # (a negative window: stretches of -window positions, counted from position 0)
+            lo = pos // -window * -window if window < 0 else max(0, pos - window + 1) if window else 0
             keys = torch.arange(lo, pos + 1)
             slots = block_table[req_slots[r]][keys // page] * page + keys % page
             for h in range(Hq):
@@ -157,7 +158,7 @@ def attention_reference(q, kf, vf, block_table, req_slots, q_lens, kv_lens, Hq, 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("Hq,Hkv,D,page,window", [
     (4, 2, 16, 4, 0), (9, 3, 32, 16, 0), (6, 1, 48, 16, 24), (5, 5, 80, 8, 0), (8, 2, 128, 16, 0),
-    (8, 2, 128, 16, 33), (2, 1, 256, 32, 0), (3, 3, 64, 16, 7),
+    (8, 2, 128, 16, 33), (2, 1, 256, 32, 0), (3, 3, 64, 16, 7), (4, 2, 40, 8, -29), (8, 2, 128, 16, -64),
 ])
 def test_paged_attention_ragged_batch(dtype, Hq, Hkv, D, page, window):
     q_lens = [1, 37, 1, 2, 64]
@@ -342,6 +343,7 @@ class _DecodeCtx:
 @pytest.mark.parametrize("Hq,Hkv,D,page,window", [
     (32, 8, 128, 16, 0), (8, 8, 128, 16, 0), (16, 1, 64, 16, 0), (12, 3, 64, 8, 0), (6, 2, 128, 32, 0),
     (32, 8, 128, 16, 100), (4, 2, 64, 4, 37), (9, 3, 128, 1, 0), (24, 2, 128, 8, 0), (16, 1, 128, 128, 300),
+    (32, 8, 128, 16, -100), (4, 2, 64, 4, -64), (8, 2, 128, 16, -1000),
 ])
 @pytest.mark.parametrize("batch", [1, 3, 24, 40])  # (24 requests x 8 kv heads: the pairs that run unsplit in one wave)
 @pytest.mark.parametrize("mode", ["split", "split-merge-kernel", "balanced", "tcgen05"])
@@ -426,6 +428,7 @@ class _MixedCtx(_DecodeCtx):
 @pytest.mark.parametrize("Hq,Hkv,D,page,window", [
     (32, 8, 128, 16, 0), (8, 8, 128, 16, 0), (16, 1, 64, 16, 0), (9, 3, 64, 8, 0), (6, 2, 128, 32, 0),
     (8, 2, 128, 16, 100), (4, 2, 64, 4, 37), (12, 4, 128, 1, 0), (5, 1, 64, 16, 0),
+    (8, 2, 128, 16, -100), (4, 2, 64, 4, -32), (9, 3, 64, 8, -7),
 ])
 def test_prefill_attention_bf16_mixed_batch(Hq, Hkv, D, page, window):
     """The tensor-core kernel for batches with prompt portions: whole prompts,
@@ -823,7 +826,7 @@ def test_small_m_linear_refuses_what_it_does_not_take():
 @pytest.mark.parametrize("mode", ["pair", "single"])
 @pytest.mark.parametrize("Hq,Hkv,page,window", [(32, 8, 16, 0), (8, 8, 16, 0), (16, 1, 16, 0), (8, 2, 32, 0),
                                                  (4, 2, 8, 0), (8, 2, 16, 100), (4, 1, 64, 37), (8, 4, 128, 0),
-                                                 (4, 4, 16, 300)])
+                                                 (4, 4, 16, 300), (8, 2, 16, -100), (4, 1, 64, -128), (32, 8, 16, -300), (4, 2, 8, -9)])
 def test_prefill_attention_tcgen05_mixed_batch(Hq, Hkv, page, window, mode):
     """The two tcgen05/TMA attention kernels (head size 128; two query tiles per block, and one) on the same ragged
     batch as the mma.sync kernel: whole prompts, portions that continue a context, two-token portions, single
@@ -931,7 +934,7 @@ def test_library_product_inside_a_stream_capture_takes_an_untimed_shape_without_
 
 @pytest.mark.parametrize("Hq,Hkv,D,page,window,with_norm", [
     (32, 8, 128, 16, 0, True), (8, 8, 128, 16, 0, True), (12, 3, 64, 8, 0, True), (6, 2, 128, 32, 40, False),
-    (16, 1, 64, 16, 0, True),
+    (16, 1, 64, 16, 0, True), (8, 2, 128, 16, -50, True),
 ])
 @pytest.mark.parametrize("batch", [1, 3, 40])
 def test_decode_attention_that_prepares_q_k_and_v_itself(Hq, Hkv, D, page, window, with_norm, batch):
