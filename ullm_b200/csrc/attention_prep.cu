@@ -15,7 +15,8 @@
 //      in `v_first`, every later one computes v <- (1 - lambda) v + lambda v_first;
 //   6. k and v go to their cache slots, q to `q_out` [T, heads * head_dim].
 //
-// One warp per (token, head) over the q heads, the k heads and the v heads.  All arithmetic is 32-bit; a value is
+// One warp per (token, head) over the q heads, the k heads and the v heads; rotation and stores alone (nothing of 1, 2, 4
+// and 5) at sizes that allow 16-byte pieces run one block per token.  All arithmetic is 32-bit; a value is
 // rounded once, when it is stored.
 #include "common.cuh"
 
@@ -145,6 +146,72 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, long long row_stri
   }
 }
 
+// The usual case without convolution, norms and value mixing: rotation and stores alone.  One block per token: its sines
+// and cosines are formed once, in shared memory, for all heads; a thread then moves 8 + 8 elements of a head's rotated part
+// (dimensions i .. i + 7 and their partners) or 8 elements that only pass, in 16-byte pieces (`VEC` elements each).
+template <typename T, int VEC>
+__global__ void qkv_rotate_store_kernel(const T* __restrict__ qkv, long long row_stride, int num_q, int num_kv,
+                                        int head_dim, int v_dim, const int* __restrict__ positions,
+                                        const float* __restrict__ inv_freq, int rotary_dim,
+                                        const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
+                                        T* __restrict__ v_cache, long long num_slots, T* __restrict__ q_out, int* status) {
+  extern __shared__ __align__(16) float rot_sm[];  // [half] cosines, [half] sines
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int half = rotary_dim >> 1;
+  if (half > 0) {
+    const float p = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * inv_freq[i], &rot_sm[half + i], &rot_sm[i]);
+  }
+  const int slot = slot_mapping != nullptr ? slot_mapping[t] : -1;
+  if (slot_mapping != nullptr && slot >= num_slots && threadIdx.x == 0) ullm_report(status, ULLM_STATUS_SLOT, t, slot);
+  const bool store = slot >= 0 && slot < num_slots;
+  __syncthreads();
+  const int rot_items = half / VEC, per_head = rot_items + (head_dim - rotary_dim) / VEC, v_items = v_dim / VEC;
+  const int qk_heads = num_q + num_kv;
+  const int qk_total = qk_heads * per_head, total = qk_total + num_kv * v_items;
+  const T* row = qkv + (long long)t * row_stride;
+  for (int i = threadIdx.x; i < total; i += blockDim.x) {
+    float a[VEC];
+    if (i >= qk_total) {  // a value
+      if (!store) continue;
+      const int c = (i - qk_total) * VEC;
+      load_vec<T, VEC>(row + qk_heads * head_dim + c, a);
+      store_vec<T, VEC>(v_cache + (long long)slot * num_kv * v_dim + c, a);
+      continue;
+    }
+    const int h = i / per_head, e = i - h * per_head;
+    T* dst;
+    if (h < num_q) {
+      dst = q_out + ((long long)t * num_q + h) * head_dim;
+    } else {
+      if (!store) continue;
+      dst = k_cache + ((long long)slot * num_kv + (h - num_q)) * head_dim;
+    }
+    const T* src = row + (long long)h * head_dim;
+    if (e < rot_items) {
+      const int d = e * VEC;
+      float b[VEC], cs[VEC], sn[VEC], x[VEC];
+      load_vec<T, VEC>(src + d, a);
+      load_vec<T, VEC>(src + half + d, b);
+      load_vec32<VEC>(rot_sm + d, cs);
+      load_vec32<VEC>(rot_sm + half + d, sn);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        x[j] = a[j] * cs[j] - b[j] * sn[j];
+        b[j] = b[j] * cs[j] + a[j] * sn[j];
+      }
+      store_vec<T, VEC>(dst + d, x);
+      store_vec<T, VEC>(dst + half + d, b);
+    } else {
+      const int d = rotary_dim + (e - rot_items) * VEC;
+      load_vec<T, VEC>(src + d, a);
+      store_vec<T, VEC>(dst + d, a);
+    }
+  }
+}
+
 // After a step: the state row of every request of the step holds the last taps - 1 projected rows.  One thread
 // per (request, channel); rows are moved in ascending order, so a request that brought fewer than taps - 1 tokens
 // shifts its old rows down before it appends (row s takes old row s + n: always a row not yet written).
@@ -182,6 +249,19 @@ static int prepare_launch(const void* qkv, long long row_stride, int tokens, int
                           const float* k_w, int norm_first, int norm_last, float eps, int vmix_mode,
                           const float* vmix_lambda, void* v_first, const int* slot_mapping, void* k_cache,
                           void* v_cache, long long num_slots, void* q_out, int* status, cudaStream_t st) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const bool plain = conv_w == nullptr && !norm_first && !norm_last && vmix_mode == 0 && head_dim % V == 0 &&
+                     v_dim % V == 0 && rotary_dim % (2 * V) == 0 && row_stride % V == 0 &&
+                     (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
+  if (plain) {
+    const int rot = inv_freq != nullptr ? rotary_dim : 0;
+    const int items = (num_q + num_kv) * (head_dim - rot / 2) / V + num_kv * v_dim / V;
+    int threads = 64;
+    while (threads < 256 && threads < items) threads <<= 1;
+    return ullm_launch_kernel(qkv_rotate_store_kernel<T, V>, dim3(tokens), dim3(threads), (size_t)rot * sizeof(float), st,
+                              (const T*)qkv, row_stride, num_q, num_kv, head_dim, v_dim, positions, inv_freq, rot,
+                              slot_mapping, (T*)k_cache, (T*)v_cache, num_slots, (T*)q_out, status);
+  }
   const long long units = (long long)tokens * (num_q + 2 * num_kv);
   const long long blocks = (units + PREP_WARPS - 1) / PREP_WARPS;
   if (blocks > 0x7fffffffLL) return ULLM_ERR_BAD_SIZE;

@@ -385,8 +385,8 @@ static int prepare_go(const void* u, long long row_stride, int xbc_off, int dt_o
   const bool wide = channels % V == 0 && xbc_off % V == 0 && row_stride % V == 0 && state_stride % 4 == 0 &&
                     (((uintptr_t)u | (uintptr_t)xbc | (uintptr_t)conv_state | (uintptr_t)conv_w | (uintptr_t)conv_b) & 15) == 0;
   const int vec = wide ? V : 1;
-  // steps of few tokens: a token per thread, small blocks; prompts: four tokens share a thread's filter and rows
-  const int tok = tokens >= 512 ? 4 : 1, threads = tokens >= 512 ? 128 : 64;
+  // steps of few tokens: a token per thread; prompts: four tokens share a thread's filter and rows (2 and 8: 10 % slower)
+  const int tok = tokens >= 512 ? 4 : 1, threads = 64;
   const int cb = (channels + threads * vec - 1) / (threads * vec), hb = (heads + threads - 1) / threads;
   const dim3 grid(cb + hb, (tokens + tok - 1) / tok), block(threads);
   if (grid.y > 65535) return ULLM_ERR_BAD_SIZE;
