@@ -866,11 +866,11 @@ def mafarax_config(width: int, heads: int, kv_heads: int, window: int, state_hea
     state elements as the matrix memory of the given sizes (heads of 64 columns, `state_dim` rows), and routed experts
     (four groups, two kept) with a shared expert of the same size."""
     left = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=window),
-                rot=dict(dims=128, base=5e5, scaling=dict(factor=8.0)))
+                rot=dict(dims=128, base=1e6, scaling=dict(factor=4.0)))
     right = dict(heads=state_heads * state_vdim // 64, vdim=64, state=state_dim, groups=1, conv=4, norm_groups=1)
     mlp = dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=expert_ff),
-               router=dict(experts=experts, top=top, scale=1.5, groups=dict(count=4, keep=2)))
-    return dict(architecture="Mafarax", vocab=vocab, width=width, logit_scale=0.5, norm=dict(eps=1e-6), torch_dtype="bfloat16",
+               router=dict(experts=experts, top=top, scale=2.0, groups=dict(count=4, keep=2)))
+    return dict(architecture="Mafarax", vocab=vocab, width=width, logit_scale=0.25, norm=dict(eps=1e-5), torch_dtype="bfloat16",
                 layers=[dict(type="parallel", mixer=dict(left=left, right=right), mlp=dict(mlp)) for _ in range(layers)])
 
 

@@ -71,13 +71,13 @@ CFG_D = config(48, 61, [
     (left(2, 1, 15, 9, 0.25, 6, rot_dims=6, base=11.0), right(3, 4, 5, 3, 6, 1), moe(4, 4, 16, groups=(2, 2), shared=8)),
 ])
 # E: sizes the tensor-core kernels of the 16-bit path take: heads of 64 and 128 with stretches longer than a key tile,
-# heads of 64 with values of 128, heads of 32 with values of 48; states of 64 and 128 rows
+# heads of 64 with values of 112, heads of 32 with values of 48; states of 64 and 128 rows
 CFG_E = config(96, 150, [
     (left(4, 2, 64, 64, 0.125, 70, rot_dims=32, factor=2.0), right(4, 64, 64, 1, 4, 1), moe(4, 2, 64, groups=(2, 1), shared=64)),
     (left(4, 1, 128, 128, 0.09, 40, rot_dims=64, base=500.0, factor=3.0), right(2, 32, 128, 2, 4, 2), None),
-    (left(8, 1, 64, 128, 0.11, 90, rot_dims=64, factor=8.0), right(6, 16, 32, 3, 4, 1), moe(8, 4, 32, groups=(2, 2), scale=1.5, shared=32)),
+    (left(6, 1, 64, 112, 0.11, 90, rot_dims=48, factor=5.0), right(6, 16, 32, 3, 4, 1), moe(8, 4, 32, groups=(2, 2), scale=1.4, shared=32)),
     (left(2, 2, 32, 48, 0.2, 33, rot_dims=8, factor=1.5), right(2, 128, 16, 1, 4, 2), None),
-], logit_scale=0.5)
+], logit_scale=0.45)
 
 CONFIGS = {"A": (CFG_A, 8), "B": (CFG_B, 4), "C": (CFG_C, 16), "D": (CFG_D, 8), "E": (CFG_E, 16)}  # config, page size
 

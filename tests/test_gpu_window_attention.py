@@ -90,7 +90,7 @@ CASES = [
     (16, 2, 64, 64, False, 1, 1, False, True, [5, 1], [5, 66]),                  # window of one, blocks of one
     (64, 1, 32, 32, False, 9, 2, False, False, [3, 1], [30, 11]),                # a token's heads fill a block
     # negative: stretches of positions
-    (8, 1, 64, 128, True, -120, 0, False, False, [130, 1, 2, 61], [130, 240, 242, 300]),
+    (6, 1, 64, 112, True, -100, 0, False, False, [130, 1, 2, 61], [130, 200, 202, 300]),
     (5, 1, 48, 32, True, -20, 0, True, False, [1, 1, 1], [97, 20, 21]),
     (4, 4, 32, 48, True, -64, 0, False, True, [64, 65, 1], [64, 130, 193]),
     (2, 1, 208, 176, True, -1, 0, False, False, [9, 1], [30, 8]),
