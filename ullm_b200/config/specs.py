@@ -96,6 +96,18 @@ class TokenSideSpec:
     shares: int
 
 
+@dataclass(frozen=True)
+class PairEmbeddingSpec:
+    """A second embedding table [buckets + 1, hidden] whose row (previous token * mul_prev + token * mul_cur) mod buckets is
+    added to the token's; a request's first token adds the last row.  The previous token is a part of the request's
+    state.  `name`: the table's tensor name."""
+
+    name: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
 @dataclass
 class ModelSpec:
     architecture: str
@@ -118,6 +130,8 @@ class ModelSpec:
     # x0 = table[id] * embedding_scale (+ an absolute position encoding that is added to the embedding)
     embedding_scale: float = 1.0
     embedding_position: PositionSpec | None = None
+    # a second table that neighbouring tokens choose the row of together; needs stream_dtype="float32"
+    embedding_pairs: PairEmbeddingSpec | None = None
     # "engine": the residual stream has the engine's dtype; "float32": it is kept in 32-bit whatever the engine's
     # dtype (the blocks of such a model take and return a 32-bit stream)
     stream_dtype: str = "engine"

@@ -39,7 +39,10 @@
 //                 entry b of the request sits in the pooled pages pk / pv ([*, page, kv heads, head_dim / v_dim],
 //                 pv null: the first v_dim elements of pk's rows) through a block table of their own; they are
 //                 visited first, in groups of 32 of their own, and share the softmax
-//   gate          [tokens][heads x v_dim] (row stride gate_stride): out *= sigmoid(gate) before the one rounding
+//   gate          [tokens][heads x v_dim] (row stride gate_stride): out *= sigmoid(gate) before the one rounding;
+//                 gate_heads: [tokens][heads], one number per head
+//   dist_bias     [heads][dist_len] 32-bit: the score of (query at i, key at j) gains dist_bias[h][min(i - j, dist_len - 1)]
+//                 (token keys only)
 //   out_scale     multiplies the output (0 = 1); out_stride: elements between output rows (0: heads x v_dim)
 struct AttExtras {
   const float* slopes;
@@ -54,6 +57,9 @@ struct AttExtras {
   long long gate_stride;
   float out_scale;
   long long out_stride;
+  int gate_heads;
+  const float* dist_bias;
+  int dist_len;
 };
 
 template <typename T, int OREGS>
@@ -111,6 +117,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, long lon
   const long long v_row = ex.v_row > 0 ? ex.v_row : (long long)num_kv * v_dim;
   const long long v_head = ex.v_head > 0 ? ex.v_head : (long long)v_dim;
   const float slope = ex.slopes != nullptr ? ex.slopes[h] : 0.f;
+  const float* bias = ex.dist_bias != nullptr ? ex.dist_bias + (long long)h * ex.dist_len : nullptr;
   // three stretches of keys: the pooled blocks that lie wholly before the window, the kept first positions that
   // lie below the window, then the window
   const int kept = min(keep_first, lo);
@@ -143,6 +150,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, long lon
         s = d * scale;
         if (softcap > 0.f) s = softcap * tanhf(s * inv_cap);
         if (part >= 0) s -= slope * (float)(pos - key);
+        if (bias != nullptr && part >= 0) s += bias[min(pos - key, ex.dist_len - 1)];
       }
     }
     const float m_new = fmaxf(m, warp_max(s));
@@ -167,13 +175,14 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, long lon
   }
   }
   const float inv = (l > 0.f ? 1.f / l : 0.f) * (ex.out_scale != 0.f ? ex.out_scale : 1.f);
-  const T* gate = ex.gate != nullptr ? (const T*)ex.gate + (long long)t * ex.gate_stride + (long long)hu * v_dim : nullptr;
+  const T* gate = ex.gate != nullptr ? (const T*)ex.gate + (long long)t * ex.gate_stride +
+                                           (ex.gate_heads ? (long long)hu : (long long)hu * v_dim) : nullptr;
 #pragma unroll
   for (int i = 0; i < OREGS; ++i) {
     const int e = lane + 32 * i;
     if (e < v_dim) {
       float o = acc[i] * inv;
-      if (gate != nullptr) o /= 1.f + expf(-to_f32(gate[e]));
+      if (gate != nullptr) o /= 1.f + expf(-to_f32(gate[ex.gate_heads ? 0 : e]));
       if (o32 != nullptr) o32[e] = o;
       else o_ptr[e] = from_f32<T>(o);
     }
@@ -309,7 +318,8 @@ extern "C" int ullm_paged_attention_generic_ex2(int dtype, const void* q, long l
 }
 
 // The general kernel with the further options of `AttExtras` (see there): distance slopes, values inside the key
-// rows (`values_in_keys`), pooled blocks behind the window, an output gate, a scale and a row stride of the output.
+// rows (`values_in_keys`), pooled blocks behind the window, an output gate, a scale and a row stride of the output, a
+// learned bias per head and distance.
 extern "C" int ullm_paged_attention_generic_ex3(int dtype, const void* q, long long q_row_stride, void* out,
                                                 const void* k_cache, const void* v_cache, const int* block_table,
                                                 int max_pages, const int* req_slots, const int* cu_q,
@@ -320,7 +330,8 @@ extern "C" int ullm_paged_attention_generic_ex3(int dtype, const void* q, long l
                                                 int values_in_keys, int pool, const void* pk, const void* pv,
                                                 const int* p_block_table, int p_max_pages, long long p_num_pages,
                                                 const void* gate, long long gate_stride, float out_scale,
-                                                long long out_stride) {
+                                                long long out_stride, int gate_heads, const float* dist_bias,
+                                                int dist_len) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || page_size <= 0 || max_pages <= 0)
     return ULLM_ERR_BAD_SIZE;
@@ -332,6 +343,7 @@ extern "C" int ullm_paged_attention_generic_ex3(int dtype, const void* q, long l
                    slopes != nullptr))
     return ULLM_ERR_UNSUPPORTED;
   if (out_stride != 0 && out_stride < (long long)num_q * v_dim) return ULLM_ERR_BAD_SIZE;
+  if (dist_bias != nullptr && dist_len <= 0) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
   AttExtras ex = {};
   ex.slopes = slopes;
@@ -350,6 +362,9 @@ extern "C" int ullm_paged_attention_generic_ex3(int dtype, const void* q, long l
   ex.gate_stride = gate_stride;
   ex.out_scale = out_scale;
   ex.out_stride = out_stride;
+  ex.gate_heads = gate_heads;
+  ex.dist_bias = dist_bias;
+  ex.dist_len = dist_len;
   if (dtype == ULLM_DTYPE_F32)
     return launch_generic<float>(q, q_row_stride, out, k_cache, v_cache, block_table, max_pages, req_slots, cu_q,
                                  kv_len, token_req, tokens, num_q, num_kv, head_dim, page_size, window, scale, num_pages,

@@ -13,6 +13,7 @@
 //   4. optionally the unit RMS norm of q and k AFTER the rotation (no weight);
 //   5. optionally value mixing across layers: the first layer that mixes leaves its values of the step's tokens
 //      in `v_first`, every later one computes v <- (1 - lambda) v + lambda v_first;
+//      optionally every query is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p;
 //   6. k and v go to their cache slots, q to `q_out` [T, heads * head_dim].
 //
 // One warp per (token, head) over the q heads, the k heads and the v heads; rotation and stores alone (nothing of 1, 2, 4
@@ -35,7 +36,8 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, long long row_stri
                                    int norm_first, int norm_last, float eps, int vmix_mode,
                                    const float* __restrict__ vmix_lambda, T* __restrict__ v_first,
                                    const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
-                                   T* __restrict__ v_cache, long long num_slots, T* __restrict__ q_out, int* status) {
+                                   T* __restrict__ v_cache, long long num_slots, T* __restrict__ q_out, int* status,
+                                   float temp_coef, int temp_every) {
   __shared__ float buf[PREP_WARPS][PREP_MAX_DIM];
   pdl_launch_dependents();
   pdl_wait();
@@ -134,6 +136,7 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, long long row_stri
   }
   // 6. stores
   if (kind == 0) {
+    if (temp_every > 0) mult *= 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1));
     T* dst = q_out + ((long long)t * num_q + head) * head_dim;
     for (int e = lane; e < dim; e += 32) dst[e] = from_f32<T>(x[e] * mult);
   } else {
@@ -248,9 +251,10 @@ static int prepare_launch(const void* qkv, long long row_stride, int tokens, int
                           const int* positions, const float* inv_freq, int rotary_dim, const float* q_w,
                           const float* k_w, int norm_first, int norm_last, float eps, int vmix_mode,
                           const float* vmix_lambda, void* v_first, const int* slot_mapping, void* k_cache,
-                          void* v_cache, long long num_slots, void* q_out, int* status, cudaStream_t st) {
+                          void* v_cache, long long num_slots, void* q_out, int* status, float temp_coef, int temp_every,
+                          cudaStream_t st) {
   constexpr int V = 16 / (int)sizeof(T);
-  const bool plain = conv_w == nullptr && !norm_first && !norm_last && vmix_mode == 0 && head_dim % V == 0 &&
+  const bool plain = conv_w == nullptr && !norm_first && !norm_last && vmix_mode == 0 && temp_every <= 0 && head_dim % V == 0 &&
                      v_dim % V == 0 && rotary_dim % (2 * V) == 0 && row_stride % V == 0 &&
                      (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
   if (plain) {
@@ -269,9 +273,10 @@ static int prepare_launch(const void* qkv, long long row_stride, int tokens, int
                             row_stride, tokens, num_q, num_kv, head_dim, v_dim, (const T*)conv_w, taps, conv_state,
                             state_stride, cu_q, token_req, req_slots, num_state_slots, positions, inv_freq, rotary_dim,
                             q_w, k_w, norm_first, norm_last, eps, vmix_mode, vmix_lambda, (T*)v_first, slot_mapping,
-                            (T*)k_cache, (T*)v_cache, num_slots, (T*)q_out, status);
+                            (T*)k_cache, (T*)v_cache, num_slots, (T*)q_out, status, temp_coef, temp_every);
 }
 
+// `temp_every` > 0: the queries' temperature (with `positions`), 0: none.
 // `conv_w`: [row width][taps] in the engine's dtype (the q, k and v filters one after the other) or null.
 // `vmix_mode`: 0 none, 1 this layer leaves its values in `v_first`, 2 it mixes them in with *vmix_lambda.
 extern "C" int ullm_qkv_prepare(int dtype, const void* qkv, long long row_stride, int tokens, int num_q, int num_kv,
@@ -281,7 +286,7 @@ extern "C" int ullm_qkv_prepare(int dtype, const void* qkv, long long row_stride
                                 const float* q_w, const float* k_w, int norm_first, int norm_last, float eps,
                                 int vmix_mode, const float* vmix_lambda, void* v_first, const int* slot_mapping,
                                 void* k_cache, void* v_cache, long long num_slots, void* q_out, int* status,
-                                void* stream) {
+                                void* stream, float temp_coef, int temp_every) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || v_dim <= 0) return ULLM_ERR_BAD_SIZE;
   if (head_dim > PREP_MAX_DIM || v_dim > PREP_MAX_DIM || rotary_dim < 0 || rotary_dim > head_dim || (rotary_dim & 1))
@@ -291,12 +296,13 @@ extern "C" int ullm_qkv_prepare(int dtype, const void* qkv, long long row_stride
   if (vmix_mode < 0 || vmix_mode > 2 || (vmix_mode != 0 && v_first == nullptr) ||
       (vmix_mode == 2 && vmix_lambda == nullptr))
     return ULLM_ERR_BAD_SIZE;
+  if (temp_every > 0 && positions == nullptr) return ULLM_ERR_BAD_SIZE;
   if (rotary_dim > 0 && (inv_freq == nullptr || positions == nullptr)) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
 #define PREP_ARGS                                                                                                   \
   qkv, row_stride, tokens, num_q, num_kv, head_dim, v_dim, conv_w, taps, conv_state, state_stride, cu_q, token_req,  \
       req_slots, num_state_slots, positions, inv_freq, rotary_dim, q_w, k_w, norm_first, norm_last, eps, vmix_mode, \
-      vmix_lambda, v_first, slot_mapping, k_cache, v_cache, num_slots, q_out, status, st
+      vmix_lambda, v_first, slot_mapping, k_cache, v_cache, num_slots, q_out, status, temp_coef, temp_every, st
   if (dtype == ULLM_DTYPE_F32) return prepare_launch<float>(PREP_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return prepare_launch<__nv_bfloat16>(PREP_ARGS);
   if (dtype == ULLM_DTYPE_F16) return prepare_launch<__half>(PREP_ARGS);

@@ -18,7 +18,9 @@
 // rows can see (entry b stands for positions bP .. bP + P - 1 and is seen by a row at position i when
 // bP + P - 1 <= i - window), then the keys from the first one that its first token
 // sees (the window's start, or the start of its stretch of positions) to its last token.  All
-// stretches share one online softmax.  For steps of few rows the tiles of a block are cut into runs (grid.y)
+// stretches share one online softmax.  A learned bias per head and distance (`dist_bias`, constant from some distance on)
+// is staged per key tile: the distances between the block's tokens and the tile's keys are tokens + 63 numbers per head of
+// the group; tiles that lie wholly beyond the last distinct distance take one number per row instead.  For steps of few rows the tiles of a block are cut into runs (grid.y)
 // whose unnormalised results a second kernel merges.  The only waits are cp.async groups and block barriers.
 #include "common.cuh"
 
@@ -56,6 +58,9 @@ struct WinArgs {
   // [token x head][nsplit][dv + 2], and `window_merge_kernel` forms the output rows
   int nsplit;
   float* parts;
+  int gate_heads;  // the gate has one number per head
+  const float* dist_bias;  // [num_q][dist_len] or null
+  int dist_len;
   int ksplit;  // the column groups of a row group share the steps of Q K^T (needs the exchange buffer)
 };
 
@@ -106,6 +111,8 @@ static inline long long win_smem_bytes(int dk, int dv, bool v_own) {
   const long long qs = dk * 2 + 16, vs = dv * 2 + 16;
   return 16LL * win_row_groups(dv) * qs + 2LL * WIN_N * qs + (v_own ? 1LL * WIN_N * vs : 0) + 2LL * WIN_N * 8;
 }
+// the biases of two key tiles: [2][heads of the group][tokens of the block + 63]
+static inline long long win_bias_bytes(int group) { return 2LL * group * (64 / group + WIN_N - 1) * 4; }
 // the partial scores that the column groups of a row group exchange: [row group][column group][32 registers][lane]
 static inline long long win_exchange_bytes(int dv) {
   return win_col_groups(dv) > 1 ? 4096LL * win_row_groups(dv) * win_col_groups(dv) : 0;
@@ -113,7 +120,8 @@ static inline long long win_exchange_bytes(int dv) {
 
 // DKT > 0: the key rows are DKT wide and the values DVW x CW, known to the compiler (strides, piece counts and the
 // steps of Q K^T become constants and the loops unroll); DKT = 0: both are read from the arguments.
-template <int DVW, int CW, int RW, int DKT>
+// BIAS: with a distance bias.
+template <int DVW, int CW, int RW, int DKT, bool BIAS>
 __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attention_kernel(const WinArgs a) {
   extern __shared__ __align__(128) unsigned char smem[];
   pdl_launch_dependents();
@@ -129,13 +137,15 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
   unsigned char* k_s = q_s + WIN_M * qs;
   unsigned char* v_s = k_s + 2 * WIN_N * qs;
   long long* slot_s = reinterpret_cast<long long*>(v_s + (v_own ? WIN_N * vs : 0));
-  float* exch_s = reinterpret_cast<float*>(slot_s + 2 * WIN_N);  // only with `ksplit`
 
   // consecutive blocks are the same token tile of all kv heads, the last tiles (most keys) first
   const int num_kv = a.num_kv;
   const int kh = (int)(blockIdx.x % num_kv);
   const int G = a.num_q / num_kv;
   const int tpt = WIN_M / G;  // tokens per block
+  const int span = tpt + WIN_N - 1;
+  float* bias_s = reinterpret_cast<float*>(slot_s + 2 * WIN_N);  // only with BIAS: [2][G][span]
+  float* exch_s = bias_s + (BIAS ? 2 * G * span : 0);            // only with `ksplit`
   const int tile_id = (int)(gridDim.x / num_kv) - 1 - (int)(blockIdx.x / num_kv);
   int r = -1, first = 0, q_len = 0, q_begin = 0;
   {
@@ -230,6 +240,17 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
       }
       slots[tid] = s;
     }
+    if (BIAS && !pooled) {
+      const int d0 = p0 - (key0 + (tile - ptiles) * WIN_N) - (WIN_N - 1);  // the distance that entry 0 stands for
+      if (d0 < a.dist_len - 1) {
+        float* dst = bias_s + st * G * span;
+        const float* src = a.dist_bias + (long long)kh * G * a.dist_len;
+        for (int i = tid; i < G * span; i += THREADS) {
+          const int h = i / span, d = d0 + i - h * span;
+          dst[i] = src[(long long)h * a.dist_len + max(0, min(d, a.dist_len - 1))] * 1.4426950408889634f;
+        }
+      }
+    }
     __syncthreads();
     // a thread's 16-byte pieces are THREADS apart: (row, piece) steps by the quotient and remainder found once
     const __nv_bfloat16* kc = (pooled ? a.pk : a.k_cache) + (long long)kh * dk;
@@ -251,6 +272,8 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
   const float log2e = 1.4426950408889634f;
   int pos[2], lo[2], nblk[2];
   float slope[2], slope_pos[2];
+  int b_off[2];     // BIAS: the row's entry for the tile's first key
+  float b_far[2];   // ... and its bias at every distance beyond the table
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int row = wrow + (lane >> 2) + h * 8;
@@ -260,6 +283,8 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
     nblk[h] = (valid && a.pool > 0 && W > 0 && lo[h] > 0) ? lo[h] / a.pool : 0;
     slope[h] = (valid && a.slopes != nullptr) ? a.slopes[kh * G + row % G] * log2e : 0.f;
     slope_pos[h] = -slope[h] * (float)pos[h];
+    b_off[h] = valid ? (row % G) * span + row / G + WIN_N - 1 : WIN_N - 1;
+    b_far[h] = (BIAS && valid) ? a.dist_bias[((long long)kh * G + row % G + 1) * a.dist_len - 1] * log2e : 0.f;
   }
   const bool has_slopes = a.slopes != nullptr;
   const bool warp_live = wrow < rows_valid;
@@ -341,7 +366,30 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
       }
       // ---- scale, distance bias, mask: scores in units of log2 from here on ------------------
       const bool edge = pooled || !warp_full || kb + WIN_N - 1 > wp_min || kb < wp_lo_last;
-      if (has_slopes && !pooled) {
+      if (BIAS && !pooled) {
+        if (p0 - kb - (WIN_N - 1) < a.dist_len - 1) {
+          const float* bt_s = bias_s + (it & 1) * G * span - (lane & 3) * 2;
+#pragma unroll
+          for (int t = 0; t < NT_S; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              sc[t][e] = fmaf(sc[t][e], a.scale_log2, bt_s[b_off[e >> 1] - (t * 8 + (e & 1))]);
+        } else {
+#pragma unroll
+          for (int t = 0; t < NT_S; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[t][e] = fmaf(sc[t][e], a.scale_log2, b_far[e >> 1]);
+        }
+        if (edge) {
+#pragma unroll
+          for (int t = 0; t < NT_S; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int key = kb + t * 8 + (lane & 3) * 2 + (e & 1), h = e >> 1;
+              if (!(key <= pos[h] && key >= lo[h])) sc[t][e] = -INFINITY;
+            }
+        }
+      } else if (has_slopes && !pooled) {
         // score * scale - slope (pos - key), as two multiply-adds per score
         const float kf = (float)(kb + (lane & 3) * 2);
 #pragma unroll
@@ -459,7 +507,7 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
     float ls = l[h];
     ls += __shfl_xor_sync(0xffffffffu, ls, 1);
     ls += __shfl_xor_sync(0xffffffffu, ls, 2);
-    const float inv = (ls > 0.f ? 1.f / ls : 0.f) * out_scale;
+    float inv = (ls > 0.f ? 1.f / ls : 0.f) * out_scale;
     const int row = wrow + (lane >> 2) + h * 8;
     if (row < rows_valid && nsplit > 1) {
       float* pp = a.parts + (((long long)(q_begin + first + row / G) * a.num_q + kh * G + row % G) * nsplit + split) * (dv + 2);
@@ -474,7 +522,9 @@ __global__ void __launch_bounds__(RW * CW * 32, CW == 1 ? 3 : 1) window_attentio
       const long long tok = q_begin + first + row / G;
       const long long col = (long long)(kh * G + row % G) * dv + c0 + c;
       __nv_bfloat16* op = a.out + tok * a.out_stride + col;
-      const __nv_bfloat16* gp = a.gate != nullptr ? a.gate + tok * a.gate_stride + col : nullptr;
+      const __nv_bfloat16* gp = a.gate != nullptr && !a.gate_heads ? a.gate + tok * a.gate_stride + col : nullptr;
+      if (a.gate != nullptr && a.gate_heads)
+        inv /= 1.f + expf(-__bfloat162float(a.gate[tok * a.gate_stride + kh * G + row % G]));
 #pragma unroll
       for (int j = 0; j < NT_O; ++j) {
         if (c0 + j * 8 < dv) {
@@ -518,12 +568,14 @@ __global__ void __launch_bounds__(128) window_merge_kernel(const WinArgs a) {
   const long long tok = th / a.num_q;
   const int head = (int)(th - tok * a.num_q);
   __nv_bfloat16* op = a.out + tok * a.out_stride + (long long)head * dv;
-  const __nv_bfloat16* gp = a.gate != nullptr ? a.gate + tok * a.gate_stride + (long long)head * dv : nullptr;
+  const __nv_bfloat16* gp = a.gate != nullptr && !a.gate_heads ? a.gate + tok * a.gate_stride + (long long)head * dv : nullptr;
+  const float head_gate =
+      a.gate != nullptr && a.gate_heads ? 1.f / (1.f + expf(-__bfloat162float(a.gate[tok * a.gate_stride + head]))) : 1.f;
   for (int e = tid; e < dv; e += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < nsplit; ++s)
       if (w_s[s] > 0.f) acc += w_s[s] * pp[(long long)s * (dv + 2) + e];
-    acc *= inv_s;
+    acc *= inv_s * head_gate;
     if (gp != nullptr) acc /= 1.f + expf(-__bfloat162float(gp[e]));
     op[e] = __float2bfloat16_rn(acc);
   }
@@ -532,18 +584,19 @@ __global__ void __launch_bounds__(128) window_merge_kernel(const WinArgs a) {
 #define WIN_SMEM_LIMIT (227 * 1024)
 #define WIN_MAX_SPLITS 64
 
-template <int DVW, int CW, int RW, int DKT = 0>
-static int launch_window(WinArgs a, int tokens, long long smem, cudaStream_t st) {
+template <int DVW, int CW, int RW, int DKT, bool BIAS>
+static int launch_window_as(WinArgs a, int tokens, long long smem, cudaStream_t st) {
+  if (BIAS) smem += win_bias_bytes(a.num_q / a.num_kv);
   if (CW > 1 && smem + win_exchange_bytes(a.dv) <= WIN_SMEM_LIMIT) {
     a.ksplit = 1;
     smem += win_exchange_bytes(a.dv);
   }
   static long long attr_bytes = 0;  // (one per instantiation) the largest size the attribute was set for
   if (smem > attr_bytes) {
-    if (cudaFuncSetAttribute(window_attention_kernel<DVW, CW, RW, DKT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) !=
+    if (cudaFuncSetAttribute(window_attention_kernel<DVW, CW, RW, DKT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) !=
         cudaSuccess)
       return ULLM_ERR_LAUNCH;
-    cudaFuncSetAttribute(window_attention_kernel<DVW, CW, RW, DKT>, cudaFuncAttributePreferredSharedMemoryCarveout,
+    cudaFuncSetAttribute(window_attention_kernel<DVW, CW, RW, DKT, BIAS>, cudaFuncAttributePreferredSharedMemoryCarveout,
                          cudaSharedmemCarveoutMaxShared);
     attr_bytes = smem;
   }
@@ -551,23 +604,31 @@ static int launch_window(WinArgs a, int tokens, long long smem, cudaStream_t st)
   // at most ceil(tokens / tpt) + num_requests token tiles exist, however the tokens are spread
   const long long blocks = ((long long)(tokens + tpt - 1) / tpt + a.num_requests) * a.num_kv;
   if (blocks > 0x7fffffffLL) return ULLM_ERR_BAD_SIZE;
-  const int rc = ullm_launch_kernel(window_attention_kernel<DVW, CW, RW, DKT>, dim3((unsigned)blocks, (unsigned)a.nsplit),
+  const int rc = ullm_launch_kernel(window_attention_kernel<DVW, CW, RW, DKT, BIAS>, dim3((unsigned)blocks, (unsigned)a.nsplit),
                                     dim3(RW * CW * 32), (size_t)smem, st, a);
   if (rc != ULLM_OK || a.nsplit <= 1) return rc;
   return ullm_launch_kernel(window_merge_kernel, dim3((unsigned)((long long)tokens * a.num_q)), dim3(128), 0, st, a);
 }
 
+template <int DVW, int CW, int RW, int DKT = 0>
+static int launch_window(const WinArgs& a, int tokens, long long smem, cudaStream_t st) {
+  if (a.dist_bias != nullptr) return launch_window_as<DVW, CW, RW, DKT, true>(a, tokens, smem, st);
+  return launch_window_as<DVW, CW, RW, DKT, false>(a, tokens, smem, st);
+}
+
 // Sizes this kernel takes (bfloat16): key rows and values multiples of 16, values up to 512, at most 64 query
 // heads per kv head, and tiles that fit the shared memory (key rows up to 576 with values inside them).
-extern "C" int ullm_window_attention_supported(int dk, int dv, int num_q, int num_kv, int values_in_keys) {
+// `biased`: with a distance bias, whose staged pieces take shared memory too.
+extern "C" int ullm_window_attention_supported(int dk, int dv, int num_q, int num_kv, int values_in_keys, int biased) {
   if (dk <= 0 || dv <= 0 || num_q <= 0 || num_kv <= 0 || num_q % num_kv) return 0;
   if (dk % 16 || dv % 16 || dv > 512 || num_q / num_kv > WIN_MAX_GROUP) return 0;
   if (values_in_keys && dv > dk) return 0;
-  return win_smem_bytes(dk, dv, !values_in_keys) <= WIN_SMEM_LIMIT;
+  return win_smem_bytes(dk, dv, !values_in_keys) + (biased ? win_bias_bytes(num_q / num_kv) : 0) <= WIN_SMEM_LIMIT;
 }
 
 // `v_cache` null: values inside the key rows (and then `pv` null too).  `slopes` (32-bit [num_q]) or null;
-// `pool` > 0 with the pooled pages `pk` (`pv`) and their block table; `gate` or null; `out_scale` 0 = 1.
+// `pool` > 0 with the pooled pages `pk` (`pv`) and their block table; `gate` or null (`gate_heads`: one number per head); `out_scale` 0 = 1.
+// `dist_bias` (32-bit [num_q][dist_len]) or null: added to the scaled score at distance min(i - j, dist_len - 1).
 // `nsplit` > 1 (at most 64) with `parts` (32-bit, tokens x num_q x nsplit x (dv + 2)): a block's key tiles are
 // cut into nsplit runs that run side by side and are merged by a second launch (steps of few rows).
 // q rows, page rows, `out` and `gate` rows must start on 16- (q, pages) and 4-byte (out) boundaries.
@@ -578,11 +639,12 @@ extern "C" int ullm_window_attention(const void* q, long long q_row_stride, void
                                      float scale, long long num_pages, int* status, void* stream, const float* slopes,
                                      int pool, const void* pk, const void* pv, const int* p_block_table,
                                      int p_max_pages, long long p_num_pages, const void* gate, long long gate_stride,
-                                     float out_scale, int nsplit, float* parts) {
+                                     float out_scale, int nsplit, float* parts, int gate_heads, const float* dist_bias,
+                                     int dist_len) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_requests <= 0 || page_size <= 0 || max_pages <= 0 || pool < 0)
     return ULLM_ERR_BAD_SIZE;
-  if (!ullm_window_attention_supported(dk, dv, num_q, num_kv, v_cache == nullptr)) return ULLM_ERR_UNSUPPORTED;
+  if (!ullm_window_attention_supported(dk, dv, num_q, num_kv, v_cache == nullptr, dist_bias != nullptr)) return ULLM_ERR_UNSUPPORTED;
   if (pool > 0 && (window <= 0 || pk == nullptr || p_block_table == nullptr || p_max_pages <= 0 || slopes != nullptr ||
                    (pv == nullptr) != (v_cache == nullptr)))
     return ULLM_ERR_UNSUPPORTED;
@@ -592,6 +654,7 @@ extern "C" int ullm_window_attention(const void* q, long long q_row_stride, void
   if (nsplit < 1 || nsplit > WIN_MAX_SPLITS || (nsplit > 1 && parts == nullptr) || ((uintptr_t)parts & 7))
     return ULLM_ERR_BAD_SIZE;
   if ((long long)tokens * num_q > 0x7fffffffLL) return ULLM_ERR_BAD_SIZE;
+  if (dist_bias != nullptr && (dist_len <= 0 || slopes != nullptr)) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
   WinArgs a = {};
   a.q = (const __nv_bfloat16*)q;
@@ -627,6 +690,9 @@ extern "C" int ullm_window_attention(const void* q, long long q_row_stride, void
   a.status = status;
   a.nsplit = nsplit;
   a.parts = parts;
+  a.gate_heads = gate_heads;
+  a.dist_bias = dist_bias;
+  a.dist_len = dist_len;
   const long long smem = win_smem_bytes(dk, dv, v_cache != nullptr);
   // the sizes of the usual head shapes (64, 128; latents of 384 + 64 and 512 + 64) as constants
   if (dk == 64 && dv == 64) return launch_window<64, 1, 4, 64>(a, tokens, smem, st);

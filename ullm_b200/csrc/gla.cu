@@ -3,8 +3,10 @@
 // floats, kept in the request's state row between steps:
 //
 //   alpha_t = exp(logsigmoid(z_t + b) / tau)          decay per key channel, z: a 32-bit projection
+//             or decays that the caller brings
 //   S_t = diag(alpha_t) S_{t-1} + k_t v_t^T
 //   o_t = S_t^T q_t,   q_t = q_scale * (projected query)
+//             or, with a bonus u: o_t = (S_{t-1} + diag(u) k_t v_t^T)^T q_t   (the current token through u alone)
 //
 // The recurrence runs token by token, so a request's result does not depend on how its tokens were cut into steps
 // or on what else is in the batch.  The parallelism is over requests, heads and the columns of S: a block owns
@@ -43,13 +45,15 @@ __global__ void gla_decay_kernel(float* __restrict__ z, long long stride, const 
 // 128 .. 255 stage the next chunk (q scaled, k, the decays, the tile's v; 32-bit) in the other half.  A staged row
 // is padded to RPT * rs entries with q = k = decay = 0, so the row loop has no bounds checks: the padded rows of S
 // stay zero.  CPT: neighbouring value columns a thread holds; the q, k and decay it reads serve all of them.
-template <typename T, int RPT, int CPT>
+// BONUS: the form with the bonus `u` [heads * dim] for the current token.
+template <typename T, int RPT, int CPT, bool BONUS>
 __global__ void __launch_bounds__(2 * GLA_THREADS)
 gla_recurrence_kernel(const T* __restrict__ qkv, long long row_stride, int q_off, int k_off, int v_off,
                       const float* __restrict__ decay, long long decay_stride, float q_scale,
                       float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                       const int* __restrict__ req_slots, const int* __restrict__ token_req, float* __restrict__ out,
-                      int heads, int dim, int vdim, int rs, int chunk, int num_slots, int* status) {
+                      int heads, int dim, int vdim, int rs, int chunk, int num_slots, int* status,
+                      const float* __restrict__ bonus) {
   extern __shared__ __align__(16) float sm[];
   pdl_launch_dependents();
   pdl_wait();
@@ -160,6 +164,14 @@ gla_recurrence_kernel(const T* __restrict__ qkv, long long row_stride, int q_off
   };
 
   float S[RPT][CPT];
+  float u[BONUS ? RPT : 1];
+  if (BONUS && !loader) {
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int r = ((i >> 2) * rs + lane_row) * 4 + (i & 3);
+      u[BONUS ? i : 0] = r < dim ? bonus[head * dim + r] : 0.f;
+    }
+  }
   if (!loader) {
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
@@ -207,8 +219,10 @@ gla_recurrence_kernel(const T* __restrict__ qkv, long long row_stride, int q_off
               for (int e = 0; e < 4; ++e) {
 #pragma unroll
                 for (int c = 0; c < CPT; ++c) {
-                  S[4 * g + e][c] = fmaf(ar[e], S[4 * g + e][c], kr[e] * v[c]);
-                  acc[j][c] = fmaf(S[4 * g + e][c], qr[e], acc[j][c]);
+                  const float kv = kr[e] * v[c];
+                  if (BONUS) acc[j][c] = fmaf(fmaf(u[BONUS ? 4 * g + e : 0], kv, S[4 * g + e][c]), qr[e], acc[j][c]);
+                  S[4 * g + e][c] = fmaf(ar[e], S[4 * g + e][c], kv);
+                  if (!BONUS) acc[j][c] = fmaf(S[4 * g + e][c], qr[e], acc[j][c]);
                 }
               }
             }
@@ -261,9 +275,10 @@ template <typename T>
 static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_off, int v_off, float* z,
                       long long z_stride, const float* z_bias, float inv_tau, float q_scale, float* state,
                       long long state_stride, const int* cu_q, const int* req_slots, const int* token_req, float* out,
-                      int tokens, int requests, int heads, int dim, int vdim, int num_slots, int* status, cudaStream_t st) {
+                      int tokens, int requests, int heads, int dim, int vdim, int num_slots, int* status,
+                      const float* bonus, cudaStream_t st) {
   const long long total = (long long)tokens * heads * dim;
-  if (total > 0) {
+  if (total > 0 && inv_tau > 0.f) {
     const long long blocks = (total + 255) / 256;
     if (blocks > 0x7fffffffLL) return ULLM_ERR_BAD_SIZE;
     const int rc = ullm_launch_kernel(gla_decay_kernel, dim3((int)blocks), dim3(256), 0, st, z, z_stride, z_bias,
@@ -297,10 +312,15 @@ static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_of
   chunk = chunk < 1 ? 1 : (chunk > 32 ? 32 : chunk);
   const size_t smem = (size_t)2 * chunk * (3 * dimp + cpb) * sizeof(float);
   const dim3 grid((vdim + cpb - 1) / cpb, heads, requests), block(2 * GLA_THREADS);
-#define GLA_GO(RPT, CPT)                                                                                              \
-  return ullm_launch_kernel(gla_recurrence_kernel<T, RPT, CPT>, grid, block, smem, st, (const T*)qkv, row_stride,      \
-                            q_off, k_off, v_off, (const float*)z, z_stride, q_scale, state, state_stride, cu_q,        \
-                            req_slots, token_req, out, heads, dim, vdim, rs, chunk, num_slots, status)
+#define GLA_AS(RPT, CPT, BONUS)                                                                                       \
+  return ullm_launch_kernel(gla_recurrence_kernel<T, RPT, CPT, BONUS>, grid, block, smem, st, (const T*)qkv,           \
+                            row_stride, q_off, k_off, v_off, (const float*)z, z_stride, q_scale, state, state_stride,  \
+                            cu_q, req_slots, token_req, out, heads, dim, vdim, rs, chunk, num_slots, status, bonus)
+#define GLA_GO(RPT, CPT)                         \
+  {                                              \
+    if (bonus != nullptr) GLA_AS(RPT, CPT, true); \
+    GLA_AS(RPT, CPT, false);                     \
+  }
   if (rpt == 4) {
     if (cpt == 4) GLA_GO(4, 4);
     if (cpt == 2) GLA_GO(4, 2);
@@ -313,16 +333,18 @@ static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_of
   }
   GLA_GO(GLA_RPT, 1);
 #undef GLA_GO
+#undef GLA_AS
 }
 
 // qkv [tokens, *]: q and k (heads x dim) and v (heads x vdim) at the given column offsets of rows `row_stride`
 // apart; z [tokens, heads * dim] 32-bit (rows `z_stride` apart), `z_bias` [heads * dim] or null: the decay's
-// projection, REPLACED by the decays; out [tokens, heads * vdim] 32-bit.
+// projection, REPLACED by the decays (`inv_tau` 0: z holds the decays already); `bonus` [heads * dim] or null; out [tokens, heads * vdim] 32-bit.
 extern "C" int ullm_gla_recurrence(int dtype, const void* qkv, long long row_stride, int q_off, int k_off, int v_off,
                                    float* z, long long z_stride, const float* z_bias, float inv_tau,
                                    float q_scale, float* state, long long state_stride, const int* cu_q,
                                    const int* req_slots, const int* token_req, float* out, int tokens, int requests,
-                                   int heads, int dim, int vdim, int num_slots, int* status, void* stream) {
+                                   int heads, int dim, int vdim, int num_slots, int* status, void* stream,
+                                   const float* bonus) {
   cudaStream_t st = (cudaStream_t)stream;
   if (requests < 0 || tokens < 0 || heads <= 0 || dim <= 0 || vdim <= 0 || num_slots <= 0) return ULLM_ERR_BAD_SIZE;
   if (dim > GLA_MAX_DIM || heads > 65535 || requests > 65535) return ULLM_ERR_UNSUPPORTED;
@@ -330,7 +352,7 @@ extern "C" int ullm_gla_recurrence(int dtype, const void* qkv, long long row_str
   if (requests == 0) return ULLM_OK;
 #define GLA_ARGS                                                                                                     \
   qkv, row_stride, q_off, k_off, v_off, z, z_stride, z_bias, inv_tau, q_scale, state, state_stride, cu_q, req_slots, \
-      token_req, out, tokens, requests, heads, dim, vdim, num_slots, status, st
+      token_req, out, tokens, requests, heads, dim, vdim, num_slots, status, bonus, st
   if (dtype == ULLM_DTYPE_F32) return gla_launch<float>(GLA_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return gla_launch<__nv_bfloat16>(GLA_ARGS);
   if (dtype == ULLM_DTYPE_F16) return gla_launch<__half>(GLA_ARGS);

@@ -24,6 +24,8 @@
 //     thread-block cluster around one unit, each takes a range of K, and ranks 1.. put their sums into rank 0's
 //     shared memory (distributed shared memory, released by an arrival at rank 0's barrier); rank 0 adds them in
 //     rank order and writes the result.
+//   * Several products whose operands have a row set each (mixes of the same rows, say) are one launch: the weights are
+//     stacked, the row sets too, and a unit takes the row set of its group (groups are whole numbers of units).
 //   * Every mbarrier wait is bounded; a wait that runs out records ULLM_STATUS_TIMEOUT, the block stops
 //     computing but keeps arriving at its barriers, waits (bounded) for the copies it still has in flight, and
 //     returns.
@@ -55,6 +57,7 @@ struct LsParams {
   int sq_count;
   float sq_inv_cols, sq_eps;      // 1 / (columns of the normed row), the norm's eps
   int* status;
+  int group_units;                // > 0: unit u meets rows (u / group_units) * M .. of x (row sets stacked); 0: rows 0 ..
 };
 
 // ---- cluster helpers: a block's rank, a peer's shared-memory address, remote stores and barrier arrivals ------
@@ -141,10 +144,11 @@ __global__ void __launch_bounds__(LS_THREADS, 2) linear_stream_kernel(const __gr
       // One thread's instruction stream is what paces the ring: no division per stage.  The position in the list
       // of stages (unit, k block) and in the ring (slot, round) is carried along and stepped.
       struct Pos {
-        int u, kb, slot, round;
+        int u, kb, slot, round, x_row;
       };
+      auto x_row_of = [&](int u) { return p.group_units > 0 ? u / p.group_units * p.M : 0; };
       auto step = [&](Pos& q) {
-        if (++q.kb == nkb) q.kb = 0, q.u += ncl;
+        if (++q.kb == nkb) q.kb = 0, q.u += ncl, q.x_row = x_row_of(q.u);
         if (++q.slot == p.stages) q.slot = 0, ++q.round;
       };
       auto issue_w = [&](const Pos& q) {
@@ -172,15 +176,15 @@ __global__ void __launch_bounds__(LS_THREADS, 2) linear_stream_kernel(const __gr
         unsigned char* st = ring + q.slot * STAGE_BYTES + LS_W_STAGE_BYTES;
         const int kb = kb0 + q.kb;
         if (p.chunked)
-          tma_load_3d(st, &x_map, &full_bar[q.slot], 0, 0, kb * 4);
+          tma_load_3d(st, &x_map, &full_bar[q.slot], 0, q.x_row, kb * 4);
         else
-          tma_load_2d(st + kc * X_BOX_BYTES, &x_map, &full_bar[q.slot], kb * LS_BK + kc * 64, 0);
+          tma_load_2d(st + kc * X_BOX_BYTES, &x_map, &full_bar[q.slot], kb * LS_BK + kc * 64, q.x_row);
       };
       const int first = total_it < p.stages ? total_it : p.stages;
-      Pos w = {cid, 0, 0, 0};
+      Pos w = {cid, 0, 0, 0, x_row_of(cid)};
       for (int it = 0; it < first; ++it, step(w)) issue_w(w);  // the weights: before the kernel in front has finished
       pdl_wait();
-      Pos x = {cid, 0, 0, 0};
+      Pos x = {cid, 0, 0, 0, x_row_of(cid)};
       for (int it = 0; it < first; ++it, step(x)) issue_x(x);  // the batch rows: what that kernel wrote
       for (int it = first; it < total_it; ++it, step(w)) {
         if (!mbar_wait(&empty_bar[w.slot], (w.round - 1) & 1)) {
@@ -519,10 +523,30 @@ extern "C" int ullm_linear_stream(const void* x, const void* w, const void* bias
                                  0, 0.f, status, stream);
 }
 
+static int ls_run(const void* x, const void* w, const void* bias, const void* residual, void* out, int M, int N, int K,
+                  int out_f32, int act, const float* pre_w, void* pre_out, float* sq_out, const float* sq_in, int sq_count,
+                  int sq_cols, float sq_eps, int groups, int group_units, int* status, void* stream);
+
 extern "C" int ullm_linear_stream_norm(const void* x, const void* w, const void* bias, const void* residual, void* out,
                                        int M, int N, int K, int out_f32, int act, const float* pre_w, void* pre_out,
                                        float* sq_out, const float* sq_in, int sq_count, int sq_cols, float sq_eps,
                                        int* status, void* stream) {
+  return ls_run(x, w, bias, residual, out, M, N, K, out_f32, act, pre_w, pre_out, sq_out, sq_in, sq_count, sq_cols, sq_eps, 1,
+                0, status, stream);
+}
+
+// Products with a row set each: rows g * group_rows .. of w [N, K] meet x[g] of x [groups][M][K] (group_rows a multiple of
+// 32; the last group may have fewer rows); out [M, N] bfloat16.
+extern "C" int ullm_linear_stream_grouped(const void* x, const void* w, void* out, int M, int N, int K, int group_rows,
+                                          int* status, void* stream) {
+  if (group_rows <= 0 || group_rows % LS_UNIT_ROWS) return ULLM_ERR_UNSUPPORTED;
+  return ls_run(x, w, nullptr, nullptr, out, M, N, K, 0, 0, nullptr, nullptr, nullptr, nullptr, 0, 0, 0.f,
+                (N + group_rows - 1) / group_rows, group_rows / LS_UNIT_ROWS, status, stream);
+}
+
+static int ls_run(const void* x, const void* w, const void* bias, const void* residual, void* out, int M, int N, int K,
+                  int out_f32, int act, const float* pre_w, void* pre_out, float* sq_out, const float* sq_in, int sq_count,
+                  int sq_cols, float sq_eps, int groups, int group_units, int* status, void* stream) {
   if ((pre_w != nullptr) != (pre_out != nullptr) || (pre_w != nullptr) != (sq_out != nullptr)) return ULLM_ERR_BAD_SIZE;
   if (pre_w != nullptr && (act != 0 || M > 16)) return ULLM_ERR_UNSUPPORTED;
   if (sq_in != nullptr && (sq_count <= 0 || sq_cols <= 0 || M > 16)) return ULLM_ERR_BAD_SIZE;
@@ -537,12 +561,13 @@ extern "C" int ullm_linear_stream_norm(const void* x, const void* w, const void*
   const int NT = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
   CUtensorMap wm, wm32, xm;
   const int chunked = K % 64 == 0;
-  // x as a matrix of exactly M rows: boxes of 8 NT rows read zeros past them
+  // x as a matrix of exactly M rows (per row set): boxes of 8 NT rows read zeros past them, or rows of the next set that
+  // nothing is made of
   if (chunked) {
     if (!ls_chunked_map(w, N, K, 16, &wm) || !ls_chunked_map(w, N, K, 32, &wm32) ||
-        !ls_chunked_map(x, M, K, 8 * NT, &xm))
+        !ls_chunked_map(x, (long long)groups * M, K, 8 * NT, &xm))
       return ULLM_ERR_LAUNCH;
-  } else if (!get_map(w, N, K, 16, &wm) || !get_map(w, N, K, 32, &wm32) || !get_map(x, M, K, 8 * NT, &xm)) {
+  } else if (!get_map(w, N, K, 16, &wm) || !get_map(w, N, K, 32, &wm32) || !get_map(x, groups * M, K, 8 * NT, &xm)) {
     return ULLM_ERR_LAUNCH;
   }
   LsParams p;
@@ -566,6 +591,7 @@ extern "C" int ullm_linear_stream_norm(const void* x, const void* w, const void*
   p.sq_inv_cols = sq_cols > 0 ? 1.f / (float)sq_cols : 0.f;
   p.sq_eps = sq_eps;
   p.status = status;
+  p.group_units = group_units;
   if (NT == 1) return ls_launch<1>(0, wm, wm32, xm, p, (cudaStream_t)stream);
   if (NT == 2) return ls_launch<2>(1, wm, wm32, xm, p, (cudaStream_t)stream);
   return ls_launch<4>(2, wm, wm32, xm, p, (cudaStream_t)stream);

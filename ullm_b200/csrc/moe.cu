@@ -105,7 +105,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long log
       for (int j = 0; j < k; ++j) used |= taken[j] == e;
       if (used || (grouped && g_rank[e / per] < INFINITY)) continue;
       const float s = score_of(e);
-      const float rank = correction != nullptr ? s + correction[e] : s;
+      // (a softmax keeps the logits' order, and far below the largest one only the logits still show it)
+      const float rank = correction != nullptr ? s + correction[e] : (softmax_scores ? z[e] : s);
       if (rank > best || (rank == best && e < best_e)) {
         best = rank;
         best_s = s;
@@ -501,7 +502,8 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
 
 // The same sum, added to a 32-bit residual stream instead of stored, with a scale per channel, and followed by the
 // norm that reads the stream next:  stream[t] += scale * y[t];  out[t] = w2 * stream[t] / sqrt(mean(stream[t]^2) +
-// eps2), or with `alpha2` (one number) and `b2`: out[t] = tanh(alpha2 * stream[t]) * w2 + b2.  One block per token; the sum never leaves 32-bit.  `x` (the passing experts' input) and `out` may be the
+// eps2), or with `alpha2` (one number) and `b2`: out[t] = tanh(alpha2 * stream[t]) * w2 + b2, or with w2 null the stream's
+// row as it is, rounded.  With an outer norm `wo`: stream[t] += scale * wo * y[t] / sqrt(mean(y[t]^2) + eps_o).  One block per token; the sum never leaves 32-bit.  `x` (the passing experts' input) and `out` may be the
 // same rows: a block reads its token's row of x before the barrier and writes its row of out behind it.
 template <typename T, int VEC>
 __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const int* __restrict__ place,
@@ -511,7 +513,8 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
                                             const float* __restrict__ shared_gate, long long gate_stride,
                                             float* __restrict__ stream, const float* __restrict__ scale,
                                             const float* __restrict__ w2, float eps2, T* out,
-                                            const float* __restrict__ alpha2, const float* __restrict__ b2) {
+                                            const float* __restrict__ alpha2, const float* __restrict__ b2,
+                                            const float* __restrict__ wo, float eps_o) {
   extern __shared__ __align__(16) float mc_row[];
   __shared__ float scratch[33];
   pdl_launch_dependents();
@@ -537,6 +540,12 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
       load_vec<T, VEC>(shared_rows + t * cols + c0, v);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) acc[i] += sg * v[i];
+    }
+    if (wo != nullptr) {
+      store_vec32<VEC>(mc_row + c0, acc);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) sq += acc[i] * acc[i];
+      continue;
     }
     if constexpr (VEC % 4 == 0) {
       // (c0 is a multiple of VEC, cols too: 16-byte pieces of the stream, the scale and the row in shared memory)
@@ -564,7 +573,32 @@ __global__ void moe_combine_add_norm_kernel(const T* __restrict__ rows, const in
       }
     }
   }
+  if (wo != nullptr) {  // (from here on a thread touches only the columns it formed)
+    const float ro = 1.f / sqrtf(block_sum(sq, scratch) / (float)cols + eps_o);
+    sq = 0.f;
+    for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+      float v[VEC], g[VEC], s[VEC];
+      load_vec32<VEC>(mc_row + c0, v);
+      load_vec32<VEC>(wo + c0, g);
+      load_vec32<VEC>(stream + t * cols + c0, s);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        s[i] += (scale != nullptr ? scale[c0 + i] : 1.f) * (v[i] * ro * g[i]);
+        sq += s[i] * s[i];
+      }
+      store_vec32<VEC>(stream + t * cols + c0, s);
+      store_vec32<VEC>(mc_row + c0, s);
+    }
+  }
   if (out == nullptr) return;
+  if (w2 == nullptr) {
+    for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+      float v[VEC];
+      load_vec32<VEC>(mc_row + c0, v);
+      store_vec<T, VEC>(out + t * cols + c0, v);
+    }
+    return;
+  }
   if (alpha2 != nullptr) {
     // no statistics: a thread reads back what it wrote itself.  (No barrier is needed for x == out either: a thread
     // overwrites only columns that it alone has read.)
@@ -731,19 +765,19 @@ extern "C" int ullm_moe_combine(int dtype, const void* rows, const int* place, c
   return ULLM_ERR_BAD_DTYPE;
 }
 
-// stream (32-bit, [tokens, cols], in place) += scale * (the sum `ullm_moe_combine` forms); `scale` null: 1.  `out` with
-// `w2` (null: none): the RMS norm of the updated rows (with `alpha2` and `b2`: the tanh norm), in the rows' dtype; `out`
-// may be `x`.
+// stream (32-bit, [tokens, cols], in place) += scale * (the sum `ullm_moe_combine` forms); `scale` null: 1.  `out`
+// (null: none): the RMS norm of the updated rows with `w2` (with `alpha2` and `b2`: the tanh norm; `w2` null: the rows as
+// they are), in the rows' dtype; `out` may be `x`.  `wo` (null: none): the sum is normed before it is added.
 extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int* place, const float* pair_weight,
                                          int tokens, int top, int cols, const int* choice, int experts, const void* x,
                                          long long x_stride, const void* shared_rows, const float* shared_gate,
                                          long long gate_stride, float* stream_rows, const float* scale,
                                          const float* w2, float eps2, void* out, void* stream, const float* alpha2,
-                                         const float* b2) {
+                                         const float* b2, const float* wo, float eps_o) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || top <= 0 || cols <= 0 || stream_rows == nullptr) return ULLM_ERR_BAD_SIZE;
   if (choice != nullptr && (x == nullptr || x_stride < cols || experts < 0)) return ULLM_ERR_BAD_SIZE;
-  if (out != nullptr && (w2 == nullptr || (alpha2 == nullptr) != (b2 == nullptr))) return ULLM_ERR_BAD_SIZE;
+  if (out != nullptr && ((alpha2 == nullptr) != (b2 == nullptr) || (w2 == nullptr && alpha2 != nullptr))) return ULLM_ERR_BAD_SIZE;
   const size_t smem = (size_t)cols * sizeof(float);
   if (smem > 160 * 1024) return ULLM_ERR_UNSUPPORTED;
   if (tokens == 0) return ULLM_OK;
@@ -751,7 +785,7 @@ extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int*
   const int vec = 16 / esize;
   const bool wide = cols % vec == 0 && x_stride % vec == 0 &&
                     (((uintptr_t)rows | (uintptr_t)x | (uintptr_t)shared_rows | (uintptr_t)stream_rows |
-                      (uintptr_t)scale | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out) & 15) == 0;
+                      (uintptr_t)scale | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out | (uintptr_t)wo) & 15) == 0;
   const int per_thread = wide ? vec : 1;
   int threads = 32;
   while (threads < 256 && threads * per_thread < cols) threads <<= 1;
@@ -765,7 +799,7 @@ extern "C" int ullm_moe_combine_add_norm(int dtype, const void* rows, const int*
     }                                                                                                                  \
     return ullm_launch_kernel(moe_combine_add_norm_kernel<T, V>, grid, block, smem, st, (const T*)rows, place,         \
                               pair_weight, top, cols, choice, experts, (const T*)x, x_stride, (const T*)shared_rows,   \
-                              shared_gate, gate_stride, stream_rows, scale, w2, eps2, (T*)out, alpha2, b2);            \
+                              shared_gate, gate_stride, stream_rows, scale, w2, eps2, (T*)out, alpha2, b2, wo, eps_o); \
   }
   if (dtype == ULLM_DTYPE_F32) {
     if (wide) MCA_GO(float, 4);

@@ -246,7 +246,7 @@ class Kernels:
             "ullm_paged_attention_generic_ex": [I, P, LL, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, LL, P, P, I, I],
             "ullm_qk_norm_rope_store_ex": [I, P, I, I, I, I, P, P, F, P, P, I, I, P, P, P, P, LL, P, P, I, I],
             "ullm_act_mul_clamped": [I, P, P, I, I, F, F, P],
-            "ullm_embed_scaled": [I, P, P, P, P, I, I, I, F, P, P, P, P, P, P, P],
+            "ullm_embed_scaled": [I, P, P, P, P, I, I, I, F, P, P, P, P, P, P, P, P, I, LL, LL, P, LL, I, P],
             "ullm_norm_scale_add": [I, P, P, P, P, I, I, F, F, P],
             "ullm_norm_scale_add_norm": [I, P, P, P, I, I, F, F, P, F, P, P],
             "ullm_rmsnorm_rows_f32": [I, P, P, P, P, I, I, I, F, P, P],
@@ -257,23 +257,24 @@ class Kernels:
             "ullm_side_gate_mul": [I, P, P, P, LL, I, P, I, I, I, P, P, P, P, P],
             "ullm_softcap_f32": [P, LL, F, P],
             "ullm_qkv_prepare": [I, P, LL, I, I, I, I, I, P, I, P, LL, P, P, P, I, P, P, I, P, P, I, I, F, I, P, P, P, P,
-                                 P, LL, P, P, P],
+                                 P, LL, P, P, P, F, I],
             "ullm_conv_state_update": [I, P, LL, I, I, P, LL, P, P, P, I, I, P],
             "ullm_paged_attention_generic_ex2": [I, P, LL, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, LL, P, P, I, I,
                                                  F, P],
             "ullm_mix_heads": [I, P, P, P, I, I, I, I, P],
             "ullm_window_attention": [P, LL, P, LL, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, LL, P, P, P, I, P, P,
-                                      P, I, LL, P, LL, F, I, P],
+                                      P, I, LL, P, LL, F, I, P, I, P, I],
             "ullm_paged_attention_generic_ex3": [I, P, LL, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, LL, P, P, I, I,
-                                                 F, P, I, I, P, P, P, I, LL, P, LL, F, LL],
+                                                 F, P, I, I, P, P, P, I, LL, P, LL, F, LL, I, P, I],
             "ullm_norm_add_norm": [I, P, P, P, I, I, F, F, I, P, P, P, F, I, I, P, P, P, P],
-            "ullm_pair_norm_add_norm": [I, P, P, P, P, I, I, F, F, P, P, P, F, I, P, P, P, P],
+            "ullm_pair_norm_add_norm": [I, P, P, P, P, I, I, F, F, P, P, P, F, I, P, P, P, P, F, F, P],
+            "ullm_act_rows": [I, I, P, LL, P, LL, I, I, P],
             "ullm_relu2": [I, P, P, LL, P],
             "ullm_scale_f32": [P, LL, F, P],
             "ullm_ssd_prepare": [I, P, LL, I, I, I, I, P, I, P, P, P, P, LL, I, P, P, P, I, P, P, P, I, P, P],
-            "ullm_ssd_recurrence": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
-            "ullm_ssd_chunk": [P, LL, I, I, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P, P],
-            "ullm_ssd_gate_norm": [I, P, P, LL, P, P, I, I, I, F, P],
+            "ullm_ssd_recurrence": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P, LL, I],
+            "ullm_ssd_chunk": [P, LL, I, I, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P, P, LL],
+            "ullm_ssd_gate_norm": [I, P, P, LL, P, P, I, I, I, F, P, I],
             "ullm_norm_rows": [I, P, P, P, P, I, I, I, F, I, P, P, P, P],
             "ullm_xielu": [I, P, P, LL, P, P],
             "ullm_kv_shared_prepare": [I, P, LL, I, I, I, P, P, F, P, P, P, LL, P, P],
@@ -283,13 +284,16 @@ class Kernels:
             "ullm_concat_rows_f32": [I, P, P, P, I, I, I, P],
             "ullm_sigmoid_gate": [I, P, P, LL, I, I, P],
             "ullm_mingru": [I, P, LL, I, I, I, P, P, P, LL, P, P, P, P, LL, F, I, I, I, P, P],
-            "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P],
+            "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, P],
+            "ullm_token_shift_mix": [I, P, LL, P, I, I, P, P, LL, I, P, P, P, I, I, P, P],
+            "ullm_low_rank_decay": [I, P, LL, I, I, P, P, P, I, I, I, P],
+            "ullm_linear_stream_grouped": [P, P, P, I, I, I, I, P, P],
             "ullm_head_norm_gate": [I, P, P, LL, P, P, I, I, I, F, I, I, P],
             "ullm_moe_route": [P, LL, P, P, P, I, I, I, I, I, I, I, F, I, P],
             "ullm_moe_arrange": [P, I, I, P, P, P, P],
             "ullm_moe_grouped_linear": [I, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],
             "ullm_moe_combine": [I, P, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P],
-            "ullm_moe_combine_add_norm": [I, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P, P, P, F, P, P, P, P],
+            "ullm_moe_combine_add_norm": [I, P, P, P, I, I, I, P, I, P, LL, P, P, LL, P, P, P, F, P, P, P, P, P, F],
             "ullm_argmax": [P, LL, I, I, P, P],
             "ullm_sample": [P, LL, I, I, P, P, P, P, P, P, P, P, P, P],
         }
@@ -339,7 +343,7 @@ class Kernels:
         L.ullm_lt_available.restype = c_int
         L.ullm_lt_last_choice.argtypes = [P, P, P, P]
         L.ullm_lt_last_choice.restype = None
-        L.ullm_window_attention_supported.argtypes = [I, I, I, I, I]
+        L.ullm_window_attention_supported.argtypes = [I, I, I, I, I, I]
         L.ullm_window_attention_supported.restype = c_int
         L.ullm_prefill_attention_supported.argtypes = [I, I, I]
         L.ullm_prefill_attention_supported.restype = c_int
@@ -768,10 +772,13 @@ class Kernels:
     # -- a residual stream kept in 32-bit ---------------------------------------
     @_timed("embedding")
     def embed_scaled(self, ids, table, stream, copy=None, scale: float = 1.0, inv_freq=None, positions=None,
-                     last_tokens=None, token_req=None, req_slots=None):
+                     last_tokens=None, token_req=None, req_slots=None, pairs=None):
         """stream[t] (float32) = table[ids[t]] * scale, plus the sinusoid of positions[t] when `inv_freq`
         (float32 [ceil(hidden / 2)]) is given; `copy` (the table's dtype, optional) gets the rounded stream.
-        An id of -1 is the request's last sampled token, as in `embedding`."""
+        An id of -1 is the request's last sampled token, as in `embedding`.  `pairs` = (table2 [buckets + 1, hidden],
+        mul_prev, mul_cur, state int32 [slots, 1], cu_q): row (previous id * mul_prev + id * mul_cur) mod buckets of
+        table2 is added, for a request's first token the last row; the state keeps the previous id (+ 1; 0: none) from
+        step to step and is moved on here."""
         _need(ids, "ids", torch.int32)
         _need(table, "table")
         _need(stream, "stream", torch.float32)
@@ -790,10 +797,23 @@ class Kernels:
         if last_tokens is not None:
             for t_, n_ in ((last_tokens, "last_tokens"), (token_req, "token_req"), (req_slots, "req_slots")):
                 _need(t_, n_, torch.int32)
+        table2 = p_state = cu_q = None
+        mul_prev = mul_cur = 0
+        if pairs is not None:
+            table2, mul_prev, mul_cur, p_state, cu_q = pairs
+            _need(table2, "pair table", table.dtype)
+            _need(p_state, "pair state", torch.int32, contiguous=False)
+            for t_, n_ in ((cu_q, "cu_q"), (token_req, "token_req"), (req_slots, "req_slots")):
+                _need(t_, n_, torch.int32)
+            if table2.dim() != 2 or table2.shape[1] != H or table2.shape[0] < 2:
+                raise KernelError(f"embed_scaled: the pair table {tuple(table2.shape)} does not fit rows of {H}")
         self._check(self.lib.ullm_embed_scaled(_DT[table.dtype], _ptr(ids), _ptr(table), _ptr(stream), _ptr(copy), T, H,
                                                table.shape[0], float(scale), _ptr(inv_freq), _ptr(positions),
                                                _ptr(last_tokens), _ptr(token_req), _ptr(req_slots), _ptr(self.status),
-                                               _stream()), "embed_scaled")
+                                               _stream(), _ptr(table2), table2.shape[0] - 1 if table2 is not None else 0,
+                                               int(mul_prev), int(mul_cur), _ptr(p_state),
+                                               p_state.stride(0) if p_state is not None else 0,
+                                               p_state.shape[0] if p_state is not None else 0, _ptr(cu_q)), "embed_scaled")
 
     @_timed("add_rmsnorm")
     def norm_scale_add(self, a, stream, weight, eps: float, mult: float, copy=None, next_norm=None):
@@ -867,15 +887,16 @@ class Kernels:
     @staticmethod
     def _next_norm(what, next_norm, rows: int, cols: int):
         """(weight, eps, kind, alpha, bias, out) of a `next_norm` argument: None, or `Norm.row_params()` with the
-        output rows behind it.  Kinds: 0 RMS, 1 centred, 2 tanh."""
+        output rows behind it.  Kinds: 0 RMS, 1 centred, 2 tanh, 3 none (the rows as they are; weight None)."""
         if next_norm is None:
             return None, 0.0, 0, None, None, None
         (w, eps, *more), out = next_norm[:-1], next_norm[-1]
         kind = int(more[0]) if more else 0
         alpha, bias = more[1:] if len(more) > 1 else (None, None)
-        _need(w, "next norm weight", torch.float32)
+        if kind != 3:
+            _need(w, "next norm weight", torch.float32)
         _need(out, "out")
-        if out.shape != (rows, cols) or w.numel() != cols:
+        if out.shape != (rows, cols) or (kind == 3) != (w is None) or (w is not None and w.numel() != cols):
             raise KernelError(f"{what}: the next norm's shapes differ")
         if (kind == 2) != (alpha is not None):
             raise KernelError(f"{what}: the tanh norm comes with a slope and a bias, the others without")
@@ -942,10 +963,11 @@ class Kernels:
 
     @_timed("add_rmsnorm")
     def pair_norm_add_norm(self, a, b, weight_a, weight_b, eps: float, mult: float, stream=None, rows_out=None,
-                           next_norm=None):
+                           next_norm=None, outer_norm=None):
         """s = mult * (weight_a * n(a) + weight_b * n(b)), n(v) = v / sqrt(mean(v^2) + eps), for two sub-layers' rows
         [T, W]; stream (float32, in place) += s, and / or rows_out = s (of the stream's sum, when both are given);
-        `next_norm` as in `norm_add_norm`, of the updated stream."""
+        `next_norm` as in `norm_add_norm`, of the updated stream.  `outer_norm` = (weight, eps, mult): the sum s passes
+        mult * weight * n(s) before it is added."""
         _need(a, "a")
         _need(b, "b", a.dtype)
         _need(weight_a, "weight_a", torch.float32)
@@ -963,9 +985,15 @@ class Kernels:
         w2, eps2, kind2, alpha2, b2, out = self._next_norm("pair_norm_add_norm", next_norm, T, W)
         if out is not None:
             _need(out, "out", a.dtype)
+        wo, eps_o, mult_o = outer_norm if outer_norm is not None else (None, 0.0, 1.0)
+        if wo is not None:
+            _need(wo, "outer norm weight", torch.float32)
+            if wo.numel() != W:
+                raise KernelError("pair_norm_add_norm: the outer norm's weight differs from the row's length")
         self._check(self.lib.ullm_pair_norm_add_norm(
             _DT[a.dtype], _ptr(a), _ptr(b), _ptr(weight_a), _ptr(weight_b), T, W, float(eps), float(mult), _ptr(stream),
-            _ptr(rows_out), _ptr(w2), eps2, kind2, _ptr(alpha2), _ptr(b2), _ptr(out), _stream()),
+            _ptr(rows_out), _ptr(w2), eps2, kind2, _ptr(alpha2), _ptr(b2), _ptr(out), _ptr(wo), float(eps_o), float(mult_o),
+            _stream()),
             f"pair_norm_add_norm (row length {W})")
 
     @_timed("act_mul")
@@ -976,6 +1004,17 @@ class Kernels:
         if out.numel() != x.numel():
             raise KernelError("relu2: shapes differ")
         self._check(self.lib.ullm_relu2(_DT[x.dtype], _ptr(x), _ptr(out), x.numel(), _stream()), "relu2")
+
+    @_timed("act_mul")
+    def act_rows(self, act: str, x, out):
+        """out = act(x) element by element for rows [T, n] (column ranges of wider rows are fine; `out` may be x); `act`:
+        "silu" or "gelu" (the exact one)."""
+        _need(x, "x", contiguous=False)
+        _need(out, "out", x.dtype, contiguous=False)
+        if x.dim() != 2 or out.shape != x.shape or x.stride(1) != 1 or out.stride(1) != 1:
+            raise KernelError(f"act_rows: x {tuple(x.shape)}, out {tuple(out.shape)}")
+        self._check(self.lib.ullm_act_rows(_DT[x.dtype], {"silu": 0, "gelu": 1}[act], _ptr(x), x.stride(0), _ptr(out),
+                                           out.stride(0), x.shape[0], x.shape[1], _stream()), f"act_rows ({act})")
 
     @_timed("act_mul")
     def xielu(self, x, pq, out):
@@ -1142,7 +1181,7 @@ class Kernels:
     @_timed("attention")
     def windowed_attention(self, q, out, k_pages, v_pages, block_table, req_slots, cu_q, kv_len, token_req, num_q: int,
                            num_kv: int, head_dim: int, v_dim: int, page_size: int, window: int, scale: float, *,
-                           slopes=None, pool: int = 0, pooled=None, gate=None, out_scale: float = 1.0,
+                           slopes=None, pool: int = 0, pooled=None, gate=None, out_scale: float = 1.0, dist_bias=None,
                            num_requests: int | None = None, workspace=None):
         """Windowed attention (`window` as in `paged_attention`) with its further options: in bfloat16, at sizes `ullm_window_attention_supported`
         takes and with `num_requests` (the batch rows that `cu_q` describes) given, the tensor-core kernel of
@@ -1151,7 +1190,9 @@ class Kernels:
         `v_dim` elements of its key rows.  `slopes` (float32 [num_q]): score(i, j) -= slopes[h] (i - j).  `pool` P
         with `pooled` = (pooled key pages, pooled value pages or None, their block table): blocks of P positions
         that lie wholly before the window are seen through one mean key / value each.  `gate` [T, num_q x v_dim]
-        (row stride free): out *= sigmoid(gate).  `out` [T, num_q x v_dim] may be a column range of wider rows."""
+        (row stride free): out *= sigmoid(gate); a gate [T, num_q] has one number per head.  `dist_bias` (float32
+        [num_q, n]): score(i, j) += dist_bias[h][min(i - j, n - 1)].  `out` [T, num_q x v_dim] may be a column range of
+        wider rows."""
         _need(q, "q", contiguous=False)
         _need(out, "out", q.dtype, contiguous=False)
         _need(k_pages, "k_pages", q.dtype)
@@ -1184,13 +1225,20 @@ class Kernels:
                 _need(pv, "pooled value pages", q.dtype)
         if gate is not None:
             _need(gate, "gate", q.dtype, contiguous=False)
-            if gate.stride(1) != 1 or gate.shape != (T, num_q * v_dim):
+            if gate.stride(1) != 1 or gate.shape not in ((T, num_q * v_dim), (T, num_q)):
                 raise KernelError(f"windowed_attention: gate {tuple(gate.shape)}")
+        gate_heads = int(gate is not None and v_dim != 1 and gate.shape[1] == num_q)
+        if dist_bias is not None:
+            _need(dist_bias, "distance bias", torch.float32)
+            if dist_bias.dim() != 2 or dist_bias.shape[0] != num_q or slopes is not None:
+                raise KernelError(f"windowed_attention: distance bias {tuple(dist_bias.shape)} for {num_q} heads")
+        bias_len = dist_bias.shape[1] if dist_bias is not None else 0
         num_pages = k_pages.numel() // (page_size * num_kv * head_dim)
         p_pages = pk.numel() // (page_size * num_kv * head_dim) if pk is not None else 0
         if (self.window_attention_tc and q.dtype == torch.bfloat16 and num_requests and q.stride(0) % 8 == 0
                 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and q.data_ptr() % 16 == 0
-                and self.lib.ullm_window_attention_supported(head_dim, v_dim, num_q, num_kv, int(v_pages is None))):
+                and self.lib.ullm_window_attention_supported(head_dim, v_dim, num_q, num_kv, int(v_pages is None),
+                                                             int(dist_bias is not None))):
             self.attention_path = "window_mma"
             splits = self._window_splits(T, int(num_requests), num_q, num_kv, int(window)) if workspace is not None else 1
             parts = None
@@ -1203,7 +1251,8 @@ class Kernels:
                 block_table.shape[1], _ptr(req_slots), _ptr(cu_q), _ptr(kv_len), T, int(num_requests), num_q, num_kv,
                 head_dim, v_dim, page_size, int(window), float(scale), num_pages, _ptr(self.status), _stream(),
                 _ptr(slopes), int(pool), _ptr(pk), _ptr(pv), _ptr(pbt), pbt.shape[1] if pbt is not None else 0, p_pages,
-                _ptr(gate), gate.stride(0) if gate is not None else 0, float(out_scale), splits, _ptr(parts)),
+                _ptr(gate), gate.stride(0) if gate is not None else 0, float(out_scale), splits, _ptr(parts), gate_heads,
+                _ptr(dist_bias), bias_len),
                 f"window_attention (key rows {head_dim}, values {v_dim}, pool {pool})")
             return
         self.attention_path = "generic"
@@ -1214,7 +1263,8 @@ class Kernels:
             _stream(), v_dim, 0, 0.0, _ptr(slopes), int(v_pages is None), int(pool), _ptr(pk), _ptr(pv), _ptr(pbt),
             pbt.shape[1] if pbt is not None else 0,
             pk.numel() // (page_size * num_kv * head_dim) if pk is not None else 0, _ptr(gate),
-            gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0)),
+            gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), gate_heads, _ptr(dist_bias),
+            bias_len),
             f"windowed_attention (head_dim {head_dim}, values {v_dim}, pool {pool})")
 
     def _window_splits(self, T: int, requests: int, num_q: int, num_kv: int, window: int) -> int:
@@ -1336,14 +1386,19 @@ class Kernels:
 
     @_timed("gla")
     def gla_recurrence(self, qkv, q_off, k_off, v_off, z, z_bias, inv_tau, q_scale, state, cu_q, req_slots, token_req,
-                       out, requests, heads, dim, vdim):
+                       out, requests, heads, dim, vdim, bonus=None):
         """The recurrence of csrc/gla.cu over the step's tokens, from and into the requests' state rows.
         qkv [T, *]: q, k, v at the given column offsets; z [T, heads * dim] float32 (the decay's projection, a view
-        with any row stride; the kernel REPLACES it by the decays), `z_bias` float32 [heads * dim] or None;
+        with any row stride; the kernel REPLACES it by the decays; `inv_tau` 0: z holds the decays already), `z_bias` float32
+        [heads * dim] or None; `bonus` float32 [heads, dim] or None: the current token through it alone;
         out [T, heads * vdim] float32."""
         _need(qkv, "qkv")
         _need(z, "z", torch.float32, contiguous=False)
-        _need(state, "state", torch.float32)
+        _need(state, "state", torch.float32, contiguous=False)
+        if bonus is not None:
+            _need(bonus, "bonus", torch.float32)
+            if bonus.numel() != heads * dim:
+                raise KernelError("gla_recurrence: the bonus has the wrong length")
         _need(out, "out", torch.float32)
         if z_bias is not None:
             _need(z_bias, "decay bias", torch.float32)
@@ -1352,6 +1407,8 @@ class Kernels:
         T = qkv.shape[0]
         if z.shape != (T, heads * dim) or z.stride(1) != 1 or out.shape != (T, heads * vdim) or state.dim() != 2:
             raise KernelError(f"gla_recurrence: qkv {tuple(qkv.shape)}, z {tuple(z.shape)}, out {tuple(out.shape)}")
+        if state.stride(1) != 1 or state.shape[1] < heads * vdim * dim:
+            raise KernelError(f"gla_recurrence: state {tuple(state.shape)}")
         if max(q_off, k_off) + heads * dim > qkv.shape[1] or v_off + heads * vdim > qkv.shape[1]:
             raise KernelError("gla_recurrence: q, k or v lie outside the rows")
         if z_bias is not None and z_bias.numel() != heads * dim:
@@ -1359,8 +1416,74 @@ class Kernels:
         self._check(self.lib.ullm_gla_recurrence(
             _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), q_off, k_off, v_off, _ptr(z), z.stride(0), _ptr(z_bias),
             float(inv_tau), float(q_scale), _ptr(state), state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req),
-            _ptr(out), T, requests, heads, dim, vdim, state.shape[0], _ptr(self.status), _stream()),
+            _ptr(out), T, requests, heads, dim, vdim, state.shape[0], _ptr(self.status), _stream(), _ptr(bonus)),
             f"gla_recurrence (heads {heads}, dim {dim}, vdim {vdim})")
+
+    # -- mixes of a row with the row before it; low-rank decays ---------------------------
+    @_timed("token_shift")
+    def token_shift_mix(self, h, mu, out, state, cu_q, token_req, req_slots, requests: int, single: bool = False):
+        """out[g, t] = h[t] + (h[t - 1] - h[t]) * mu[g] for G mixes at once: h [T, W], mu float32 [G, W], out [G, T, W].
+        The row in front of a request's first token of the step comes from its state (float32 [slots, W], a view of wider
+        rows; zeros for a new request), which is moved on to the step's last row: here when `single` (every request has
+        one token), else by `conv_state_update` behind it."""
+        _need(h, "h")
+        _need(mu, "mu", torch.float32)
+        _need(out, "out", h.dtype)
+        _need(state, "state", torch.float32, contiguous=False)
+        for t_, n_ in ((cu_q, "cu_q"), (token_req, "token_req"), (req_slots, "req_slots")):
+            _need(t_, n_, torch.int32)
+        T, W = h.shape
+        G = mu.shape[0]
+        if mu.shape != (G, W) or out.shape != (G, T, W) or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < W:
+            raise KernelError(f"token_shift_mix: h {tuple(h.shape)}, mu {tuple(mu.shape)}, out {tuple(out.shape)}")
+        self._check(self.lib.ullm_token_shift_mix(
+            _DT[h.dtype], _ptr(h), h.stride(0), _ptr(mu), G, W, _ptr(out), _ptr(state), state.stride(0), state.shape[0],
+            _ptr(cu_q), _ptr(token_req), _ptr(req_slots), T, int(bool(single)), _ptr(self.status), _stream()),
+            f"token_shift_mix ({G} mixes of {W})")
+        if not single:
+            self.conv_state_update(h, 2, state[:, :W], cu_q, token_req, req_slots, requests)
+
+    @_timed("gla")
+    def low_rank_decay(self, a, w2, w0, out, log: bool = False):
+        """out[t, c] = exp(-exp(w2[c] . tanh(a[t]) + w0[c])), or with `log` its logarithm: a [T, R] (any row stride), w2
+        [n, R] in a's dtype, w0 float32 [n], out float32 [T, n]; 32-bit arithmetic."""
+        _need(a, "a", contiguous=False)
+        _need(w2, "w2", a.dtype)
+        _need(w0, "w0", torch.float32)
+        _need(out, "out", torch.float32)
+        T, R = a.shape
+        n = w2.shape[0]
+        if a.stride(1) != 1 or w2.shape != (n, R) or w0.numel() != n or out.shape != (T, n):
+            raise KernelError(f"low_rank_decay: a {tuple(a.shape)}, w2 {tuple(w2.shape)}, out {tuple(out.shape)}")
+        self._check(self.lib.ullm_low_rank_decay(_DT[a.dtype], _ptr(a), a.stride(0), T, R, _ptr(w2), _ptr(w0), _ptr(out), n,
+                                                 n, int(bool(log)), _stream()), f"low_rank_decay (rank {R})")
+
+    @_timed("linear", lambda x, weight, *rest: weight.numel() * weight.element_size())
+    def grouped_linear(self, x, weight, out, group_rows: int):
+        """Products with an operand each: rows g * group_rows .. of the stacked `weight` [N, K] meet x[g] of x [G, T, K]
+        (the last group may have fewer rows); out [T, N].  Few bfloat16 rows: the weight-streaming kernel, one launch;
+        otherwise the library's batched product for the full groups and a product for the rest."""
+        _need(x, "x")
+        _need(out, "out", x.dtype)
+        G, T, K = x.shape
+        N = weight.shape[0]
+        full = min(N // group_rows, G)
+        if weight.shape[1] != K or out.shape != (T, N) or not (G - 1) * group_rows < N <= G * group_rows:
+            raise KernelError(f"grouped_linear: x {tuple(x.shape)}, weight {tuple(weight.shape)}, groups of {group_rows}")
+        if (x.dtype == torch.bfloat16 and self.small_m_mode in ("auto", "stream") and T <= self.stream_all_rows
+                and group_rows % 32 == 0 and weight.is_contiguous() and weight.dtype == x.dtype
+                and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0
+                and self.lib.ullm_linear_stream_supported(T, N, K)):
+            self._check(self.lib.ullm_linear_stream_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, group_rows,
+                                                            _ptr(self.status), _stream()),
+                        f"linear_stream_grouped ({G} x {T}x{K} . {N}x{K})")
+            return out
+        n = full * group_rows
+        torch.bmm(x[:full], weight[:n].view(full, group_rows, K).transpose(1, 2),
+                  out=out[:, :n].view(T, full, group_rows).transpose(0, 1))
+        if n < N:
+            torch.mm(x[full], weight[n:].t(), out=out[:, n:])
+        return out
 
     # -- sub-layers added to a 32-bit stream through gates; a per-token side input ----------
     @_timed("add_rmsnorm")
@@ -1456,10 +1579,12 @@ class Kernels:
 
     @_timed("ssd")
     def ssd_recurrence(self, xbc, b_off: int, c_off: int, dt, log_decay, d_skip, state, cu_q, req_slots, token_req, out,
-                       requests: int, heads: int, n_state: int, pdim: int, groups: int, most_tokens: int = 1 << 30):
+                       requests: int, heads: int, n_state: int, pdim: int, groups: int, most_tokens: int = 1 << 30,
+                       silu_in: bool = False):
         """The recurrence over the step's tokens, from and into the requests' state rows (float32
         [slots, >= heads * pdim * n_state]); out [T, heads * pdim] float32.  Requests that bring more than
-        `most_tokens` tokens are left alone."""
+        `most_tokens` tokens are left alone.  dt and log_decay may have ONE row that serves all tokens; `silu_in`: x, B
+        and C pass a silu as they are read."""
         _need(xbc, "xbc")
         _need(state, "state", torch.float32, contiguous=False)
         for t_, n_ in ((dt, "dt"), (log_decay, "log_decay"), (d_skip, "d_skip"), (out, "out")):
@@ -1467,7 +1592,8 @@ class Kernels:
         for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
             _need(t_, n_, torch.int32)
         T = xbc.shape[0]
-        if (dt.shape != (T, heads) or log_decay.shape != (T, heads) or out.shape != (T, heads * pdim) or state.dim() != 2
+        if (dt.shape not in ((T, heads), (1, heads)) or log_decay.shape != dt.shape or out.shape != (T, heads * pdim)
+                or state.dim() != 2
                 or state.stride(1) != 1 or state.shape[1] < heads * pdim * n_state or d_skip.numel() != heads):
             raise KernelError(f"ssd_recurrence: xbc {tuple(xbc.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
         if max(b_off, c_off) + groups * n_state > xbc.shape[1] or heads * pdim > xbc.shape[1]:
@@ -1475,7 +1601,8 @@ class Kernels:
         self._check(self.lib.ullm_ssd_recurrence(
             _DT[xbc.dtype], _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(state),
             state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), requests, heads, n_state, pdim,
-            groups, state.shape[0], int(most_tokens), _ptr(self.status), _stream()),
+            groups, state.shape[0], int(most_tokens), _ptr(self.status), _stream(), heads if dt.shape[0] == T else 0,
+            int(bool(silu_in))),
             f"ssd_recurrence (heads {heads}, state {n_state}, columns {pdim})")
 
     def ssd_chunk_applies(self, dtype, heads: int, n_state: int, pdim: int, groups: int) -> bool:
@@ -1498,7 +1625,8 @@ class Kernels:
         for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
             _need(t_, n_, torch.int32)
         T = xbc.shape[0]
-        if (dt.shape != (T, heads) or log_decay.shape != (T, heads) or out.shape != (T, heads * pdim) or state.dim() != 2
+        if (dt.shape not in ((T, heads), (1, heads)) or log_decay.shape != dt.shape or out.shape != (T, heads * pdim)
+                or state.dim() != 2
                 or state.stride(1) != 1 or state.shape[1] < heads * pdim * n_state or d_skip.numel() != heads
                 or scores.numel() < self.ssd_chunk_floats(T, groups)):
             raise KernelError(f"ssd_chunk: xbc {tuple(xbc.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
@@ -1507,13 +1635,14 @@ class Kernels:
         self._check(self.lib.ullm_ssd_chunk(
             _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(scores), _ptr(state),
             state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), T, requests, heads, n_state, pdim,
-            groups, state.shape[0], int(least), _ptr(self.status), _stream()),
+            groups, state.shape[0], int(least), _ptr(self.status), _stream(), heads if dt.shape[0] == T else 0),
             f"ssd_chunk (heads {heads}, state {n_state}, columns {pdim})")
         self.launches += 1  # the scores in front of it
 
     @_timed("ssd")
-    def ssd_gate_norm(self, y, z, weight, parts: int, eps: float, out):
-        """out = weight * n(y * silu(z)), n over `parts` equal stretches of the row; y [T, inner] float32, z a view
+    def ssd_gate_norm(self, y, z, weight, parts: int, eps: float, out, gate_behind: bool = False):
+        """out = weight * n(y * silu(z)), n over `parts` equal stretches of the row, or with `gate_behind`
+        weight * n(y) * sigmoid(z); y [T, inner] float32, z a view
         [T, inner] of the projection's rows (any row stride)."""
         _need(y, "y", torch.float32)
         _need(z, "z", out.dtype, contiguous=False)
@@ -1523,16 +1652,19 @@ class Kernels:
         if z.shape != y.shape or out.shape != y.shape or z.stride(1) != 1 or weight.numel() != inner or inner % parts:
             raise KernelError(f"ssd_gate_norm: y {tuple(y.shape)}, z {tuple(z.shape)}, {parts} parts")
         self._check(self.lib.ullm_ssd_gate_norm(_DT[out.dtype], _ptr(y), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), T,
-                                                inner, int(parts), float(eps), _stream()), "ssd_gate_norm")
+                                                inner, int(parts), float(eps), _stream(), int(bool(gate_behind))),
+                    "ssd_gate_norm")
 
     # -- between an attention's projection and its scores, in general form ----------------
     @_timed("qk_norm_rope_store")
     def qkv_prepare(self, qkv, q_out, num_q, num_kv, head_dim, v_dim, positions, slot_mapping, k_pages, v_pages, *,
                     conv_w=None, taps: int = 0, conv_state=None, cu_q=None, token_req=None, req_slots=None,
                     inv_freq=None, rotary_dim: int = 0, q_w=None, k_w=None, norm_first: bool = False,
-                    norm_last: bool = False, eps: float = 0.0, vmix_mode: int = 0, vmix_lambda=None, v_first=None):
+                    norm_last: bool = False, eps: float = 0.0, vmix_mode: int = 0, vmix_lambda=None, v_first=None,
+                    q_temp=None):
         """See csrc/attention_prep.cu: short convolution (with the requests' state rows), norm, rotation by computed
-        angles, unit norm, value mixing, cache stores; q goes to `q_out` [T, num_q * head_dim]."""
+        angles, unit norm, value mixing, cache stores; q goes to `q_out` [T, num_q * head_dim].  `q_temp` = (coef, every): every
+        query times 1 + coef ln(floor((p + 1) / every) + 1) at its position p."""
         _need(qkv, "qkv", contiguous=False)
         _need(q_out, "q_out", qkv.dtype)
         T, W = qkv.shape
@@ -1548,8 +1680,8 @@ class Kernels:
             for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots")):
                 _need(t_, n_, torch.int32)
             if taps > 1:
-                _need(conv_state, "conv_state", torch.float32)
-                if conv_state.dim() != 2 or conv_state.shape[1] < (taps - 1) * W:
+                _need(conv_state, "conv_state", torch.float32, contiguous=False)
+                if conv_state.dim() != 2 or conv_state.stride(1) != 1 or conv_state.shape[1] < (taps - 1) * W:
                     raise KernelError(f"qkv_prepare: conv_state {tuple(conv_state.shape)} is too small")
                 state_stride, state_slots = conv_state.stride(0), conv_state.shape[0]
         for t_, n_ in ((inv_freq, "inv_freq"), (q_w, "q norm weight"), (k_w, "k norm weight"), (vmix_lambda, "vmix")):
@@ -1574,7 +1706,8 @@ class Kernels:
             _ptr(conv_state), state_stride, _ptr(cu_q), _ptr(token_req), _ptr(req_slots), state_slots, _ptr(positions),
             _ptr(inv_freq), int(rotary_dim), _ptr(q_w), _ptr(k_w), int(norm_first), int(norm_last), float(eps),
             int(vmix_mode), _ptr(vmix_lambda), _ptr(v_first), _ptr(slot_mapping), _ptr(k_pages), _ptr(v_pages), num_slots,
-            _ptr(q_out), _ptr(self.status), _stream()), f"qkv_prepare (head_dim {head_dim})")
+            _ptr(q_out), _ptr(self.status), _stream(), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0),
+            f"qkv_prepare (head_dim {head_dim})")
 
     @_timed("qk_norm_rope_store")
     def conv_state_update(self, qkv, taps: int, conv_state, cu_q, token_req, req_slots, requests: int):
@@ -1705,11 +1838,12 @@ class Kernels:
 
     @_timed("moe")
     def moe_combine_add_norm(self, rows, place, pair_weight, top: int, stream, scale=None, next_norm=None, passing=None,
-                             shared=None) -> bool:
+                             shared=None, outer_norm=None) -> bool:
         """stream (float32 [T, cols], in place) += scale * (the sum `moe_combine` forms), the sum kept in 32-bit;
         `scale` float32 [cols] or None.  `next_norm` (as in `norm_add_norm`, of the kinds without a mean): the norm of
         the updated rows, in the rows' dtype (its rows may be the passing experts' x).  False when the kernel does not take the row length
-        (nothing has run then)."""
+        (nothing has run then).  `outer_norm` = (weight, eps): the sum s passes weight * s / sqrt(mean(s^2) + eps) before it
+        is added."""
         _need(rows, "rows")
         _need(place, "place", torch.int32)
         _need(stream, "stream", torch.float32)
@@ -1725,6 +1859,11 @@ class Kernels:
         w2, eps2, kind2, alpha2, b2, out = self._next_norm("moe_combine_add_norm", next_norm, T, C)
         if kind2 == 1:
             return False
+        wo, eps_o = outer_norm if outer_norm is not None else (None, 0.0)
+        if wo is not None:
+            _need(wo, "outer norm weight", torch.float32)
+            if wo.numel() != C:
+                raise KernelError("moe_combine_add_norm: the outer norm's weight differs from the row's length")
         if out is not None:
             _need(out, "out", rows.dtype)
         choice, experts, x, x_stride, s_rows, s_gate, g_stride = self._combine_extras("moe_combine_add_norm", rows, T, C,
@@ -1732,7 +1871,7 @@ class Kernels:
         self._check(self.lib.ullm_moe_combine_add_norm(
             _DT[rows.dtype], _ptr(rows), _ptr(place), _ptr(pair_weight), T, top, C, _ptr(choice), experts, _ptr(x),
             x_stride, _ptr(s_rows), _ptr(s_gate), g_stride, _ptr(stream), _ptr(scale), _ptr(w2), float(eps2), _ptr(out),
-            _stream(), _ptr(alpha2), _ptr(b2)), "moe_combine_add_norm")
+            _stream(), _ptr(alpha2), _ptr(b2), _ptr(wo), float(eps_o)), "moe_combine_add_norm")
         return True
 
     def check_attention_sizes(self, *a):

@@ -7,14 +7,17 @@
 //   norm_rows       out[r] = round(w * n(stream[rows[r]]))      (gathered rows; `rows` null: all in order)
 //   pair_norm_add_norm   stream[t] += mult * (wa * n(a[t]) + wb * n(b[t])) for TWO sub-layers' outputs, each divided by
 //                   its own root mean square; then out as above.  Without a stream: rows_out[t] = round(the sum)
+//                   With an outer norm: stream[t] += mult_o * wo * n(s) for s = the sum of the two
 //   relu2           out = round(max(in, 0)^2)
+//   act_rows        out = round(act(in)) on a column range of wider rows: silu or the exact gelu
 //   xielu           out = round(act(in)), act(z) = softplus(p) z^2 + z / 2 for z > 0,
 //                                          (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 otherwise
 //
 // n(v) = v / sqrt(mean(v^2) + eps), or with `center` = 1 (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps): the
 // variance is the mean of the squared deviations, formed in a second pass over the row, which waits in shared
 // memory.  The norm that reads the stream next may also be `center2` = 2, a norm without statistics:
-// out = tanh(alpha * s) * w2 + b2 with one number alpha and a vector b2.  `center` = 2 for the added operand: n(v) = v, so stream[t] += mult * w * a[t] (a scale per channel on a
+// out = tanh(alpha * s) * w2 + b2 with one number alpha and a vector b2, or `center2` = 3, no norm at all: out is the
+// stream rounded.  `center` = 2 for the added operand: n(v) = v, so stream[t] += mult * w * a[t] (a scale per channel on a
 // sub-layer's output; w null: no scale), the arrangement of a pre-norm layer on a 32-bit stream.  Sums, means and the stream are 32-bit; one rounding at each store.  One block per row.
 #include "common.cuh"
 
@@ -65,9 +68,13 @@ __global__ void norm_add_norm_kernel(const TA* __restrict__ a, float* __restrict
     if (extra_rows != nullptr) s += extra_rows[base + c];
     if (extra_vec != nullptr) s += extra_vec[c];
     stream[base + c] = s;
-    row_s[c] = s;
+    if (center2 == 3) {
+      if (out != nullptr) out[base + c] = from_f32<TO>(s);
+    } else {
+      row_s[c] = s;
+    }
   }
-  if (out == nullptr) return;
+  if (out == nullptr || center2 == 3) return;
   if (center2 == 2) {  // (a thread reads what it wrote itself: no barrier)
     const float al = *alpha2;
     for (int c = threadIdx.x; c < cols; c += blockDim.x)
@@ -90,7 +97,7 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
                                           float eps, float mult, float* __restrict__ stream, T* __restrict__ rows_out,
                                           const float* __restrict__ w2, float eps2, int kind2,
                                           const float* __restrict__ alpha2, const float* __restrict__ b2,
-                                          T* __restrict__ out) {
+                                          T* __restrict__ out, const float* __restrict__ wo, float eps_o, float mult_o) {
   extern __shared__ __align__(16) float sn_smem[];  // [cols] a, [cols] b; the stream's row takes a's place
   __shared__ float sums[2][33];
   pdl_launch_dependents();
@@ -125,6 +132,28 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
     qb += sums[1][i];
   }
   const float ra = mult / sqrtf(qa / (float)cols + eps), rb = mult / sqrtf(qb / (float)cols + eps);
+  float ro = 1.f;
+  if (wo != nullptr) {  // the weighted sum takes b's place and is normed as one row
+    float qo = 0.f;
+    for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
+      float ga[VEC], gb[VEC];
+      load_vec32<VEC>(wa + c0, ga);
+      load_vec32<VEC>(wb + c0, gb);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const float v = row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
+        row_b[c0 + i] = v;
+        qo += v * v;
+      }
+    }
+    qo = warp_sum(qo);
+    __syncthreads();  // the two sums have been read
+    if (lane == 0) sums[0][warp] = qo;
+    __syncthreads();
+    qo = 0.f;
+    for (int i = 0; i < nwarps; ++i) qo += sums[0][i];
+    ro = mult_o / sqrtf(qo / (float)cols + eps_o);
+  }
   const float al = (out != nullptr && kind2 == 2) ? *alpha2 : 0.f;
   for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
     float s[VEC];
@@ -133,14 +162,22 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
 #pragma unroll
       for (int i = 0; i < VEC; ++i) s[i] = 0.f;
     float ga[VEC], gb[VEC];
-    load_vec32<VEC>(wa + c0, ga);
-    load_vec32<VEC>(wb + c0, gb);
+    if (wo != nullptr) {
+      load_vec32<VEC>(wo + c0, ga);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) s[i] += row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
+      for (int i = 0; i < VEC; ++i) s[i] += row_b[c0 + i] * ro * ga[i];
+    } else {
+      load_vec32<VEC>(wa + c0, ga);
+      load_vec32<VEC>(wb + c0, gb);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] += row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
+    }
     if (stream != nullptr) store_vec32<VEC>(stream + base + c0, s);
     if (rows_out != nullptr) store_vec<T, VEC>(rows_out + base + c0, s);
     if (out == nullptr) continue;
-    if (kind2 == 2) {
+    if (kind2 == 3) {
+      store_vec<T, VEC>(out + base + c0, s);
+    } else if (kind2 == 2) {
       float g2[VEC], d2[VEC];
       load_vec32<VEC>(w2 + c0, g2);
       load_vec32<VEC>(b2 + c0, d2);
@@ -152,7 +189,7 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
       for (int i = 0; i < VEC; ++i) row_a[c0 + i] = s[i];
     }
   }
-  if (out == nullptr || kind2 == 2) return;
+  if (out == nullptr || kind2 >= 2) return;
   __syncthreads();
   float mean2;
   const float rstd2 = row_rstd(row_a, cols, kind2 != 0, eps2, sums[0], &mean2);
@@ -223,6 +260,24 @@ __global__ void relu2_kernel(const T* in, T* out, long long n) {
   }
 }
 
+// out[r][c] = act(in[r][c]) for a column range of wider rows (strides in elements; `out` may be `in`): ACT 0 silu,
+// 1 the exact gelu z (1 + erf(z / sqrt 2)) / 2
+template <typename T, int VEC, int ACT>
+__global__ void act_rows_kernel(const T* in, long long in_stride, T* out, long long out_stride, long long pieces,
+                                int per_row) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < pieces; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / per_row;
+    const int c = (int)(i - r * per_row) * VEC;
+    float v[VEC];
+    load_vec<T, VEC>(in + r * in_stride + c, v);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = ACT == 0 ? act_silu(v[k]) : 0.5f * v[k] * (1.f + erff(v[k] * 0.70710678118654752f));
+    store_vec<T, VEC>(out + r * out_stride + c, v);
+  }
+}
+
 static inline int sn_threads(int cols) {
   int threads = 32;
   while (threads < 512 && threads * 4 < cols) threads <<= 1;
@@ -261,8 +316,8 @@ extern "C" int ullm_norm_add_norm(int a_dtype, const void* a, float* stream, con
                                   void* out, void* stream_handle, const float* alpha2, const float* b2) {
   cudaStream_t st = (cudaStream_t)stream_handle;
   if (rows < 0 || cols <= 0) return ULLM_ERR_BAD_SIZE;
-  if ((a != nullptr && w == nullptr && center != 2) || (out != nullptr && w2 == nullptr)) return ULLM_ERR_BAD_SIZE;
-  if (center < 0 || center > 2 || center2 < 0 || center2 > 2) return ULLM_ERR_BAD_SIZE;
+  if ((a != nullptr && w == nullptr && center != 2) || (out != nullptr && w2 == nullptr && center2 != 3)) return ULLM_ERR_BAD_SIZE;
+  if (center < 0 || center > 2 || center2 < 0 || center2 > 3) return ULLM_ERR_BAD_SIZE;
   if (out != nullptr && center2 == 2 && (alpha2 == nullptr || b2 == nullptr)) return ULLM_ERR_BAD_SIZE;
   if (rows == 0) return ULLM_OK;
 #define SN_GO(TA, TO)                                                                                              \
@@ -312,12 +367,14 @@ extern "C" int ullm_norm_rows(int dtype, const float* stream, const int* rows, c
 template <typename T>
 static int pair_norm_launch(const void* a, const void* b, const float* wa, const float* wb, int rows, int cols, float eps,
                             float mult, float* stream, void* rows_out, const float* w2, float eps2, int kind2,
-                            const float* alpha2, const float* b2, void* out, cudaStream_t st) {
+                            const float* alpha2, const float* b2, void* out, const float* wo, float eps_o, float mult_o,
+                            cudaStream_t st) {
   const size_t smem = 2 * (size_t)cols * sizeof(float);
   if (smem > SN_MAX_SMEM) return ULLM_ERR_UNSUPPORTED;
   constexpr int V = 16 / (int)sizeof(T);
   const bool wide = cols % V == 0 && (((uintptr_t)a | (uintptr_t)b | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)stream |
-                                       (uintptr_t)rows_out | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out) & 15) == 0;
+                                       (uintptr_t)rows_out | (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out |
+                                       (uintptr_t)wo) & 15) == 0;
   int threads = 32;
   while (threads < 512 && threads * (wide ? V : 1) < cols) threads <<= 1;
 #define PN_GO(VEC)                                                                                                    \
@@ -326,7 +383,7 @@ static int pair_norm_launch(const void* a, const void* b, const float* wa, const
     if (rc != ULLM_OK) return rc;                                                                                     \
     return ullm_launch_kernel(pair_norm_add_norm_kernel<T, VEC>, dim3(rows), dim3(threads), smem, st, (const T*)a,    \
                               (const T*)b, wa, wb, cols, eps, mult, stream, (T*)rows_out, w2, eps2, kind2, alpha2, b2, \
-                              (T*)out);                                                                               \
+                              (T*)out, wo, eps_o, mult_o);                                                                               \
   }
   if (wide) PN_GO(V);
   PN_GO(1);
@@ -335,18 +392,18 @@ static int pair_norm_launch(const void* a, const void* b, const float* wa, const
 
 // a, b [rows, cols] in the engine's dtype; `stream` (32-bit, updated in place) and `rows_out` (engine's dtype): at least
 // one.  `out` with `w2` (null: none): the next norm of the updated rows; `kind2` 0: RMS, 1: centred, 2: tanh with `alpha2`
-// (one number) and `b2`.
+// (one number) and `b2`, 3: the rows as they are, rounded.  `wo` (null: none): the outer norm of the sum.
 extern "C" int ullm_pair_norm_add_norm(int dtype, const void* a, const void* b, const float* wa, const float* wb, int rows,
                                        int cols, float eps, float mult, float* stream, void* rows_out, const float* w2,
                                        float eps2, int kind2, const float* alpha2, const float* b2, void* out,
-                                       void* stream_handle) {
+                                       const float* wo, float eps_o, float mult_o, void* stream_handle) {
   cudaStream_t st = (cudaStream_t)stream_handle;
   if (rows < 0 || cols <= 0 || a == nullptr || b == nullptr || wa == nullptr || wb == nullptr ||
-      (stream == nullptr && rows_out == nullptr) || (out != nullptr && w2 == nullptr) || kind2 < 0 || kind2 > 2 ||
+      (stream == nullptr && rows_out == nullptr) || (out != nullptr && w2 == nullptr && kind2 != 3) || kind2 < 0 || kind2 > 3 ||
       (out != nullptr && kind2 == 2 && (alpha2 == nullptr || b2 == nullptr)))
     return ULLM_ERR_BAD_SIZE;
   if (rows == 0) return ULLM_OK;
-#define PN_ARGS a, b, wa, wb, rows, cols, eps, mult, stream, rows_out, w2, eps2, kind2, alpha2, b2, out, st
+#define PN_ARGS a, b, wa, wb, rows, cols, eps, mult, stream, rows_out, w2, eps2, kind2, alpha2, b2, out, wo, eps_o, mult_o, st
   if (dtype == ULLM_DTYPE_F32) return pair_norm_launch<float>(PN_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return pair_norm_launch<__nv_bfloat16>(PN_ARGS);
   if (dtype == ULLM_DTYPE_F16) return pair_norm_launch<__half>(PN_ARGS);
@@ -390,5 +447,37 @@ extern "C" int ullm_relu2(int dtype, const void* in, void* out, long long n, voi
   if (dtype == ULLM_DTYPE_F32) return relu2_launch<float>(in, out, n, st);
   if (dtype == ULLM_DTYPE_BF16) return relu2_launch<__nv_bfloat16>(in, out, n, st);
   if (dtype == ULLM_DTYPE_F16) return relu2_launch<__half>(in, out, n, st);
+  return ULLM_ERR_BAD_DTYPE;
+}
+
+template <typename T, int ACT>
+static int act_rows_launch(const void* in, long long in_stride, void* out, long long out_stride, int rows, int cols,
+                           cudaStream_t st) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const bool wide = cols % V == 0 && in_stride % V == 0 && out_stride % V == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
+  const int per_row = wide ? cols / V : cols;
+  const long long pieces = (long long)rows * per_row;
+  long long blocks = (pieces + 127) / 128;
+  if (blocks > 148 * 32) blocks = 148 * 32;
+  if (wide)
+    return ullm_launch_kernel(act_rows_kernel<T, V, ACT>, dim3((int)blocks), dim3(128), 0, st, (const T*)in, in_stride,
+                              (T*)out, out_stride, pieces, per_row);
+  return ullm_launch_kernel(act_rows_kernel<T, 1, ACT>, dim3((int)blocks), dim3(128), 0, st, (const T*)in, in_stride,
+                            (T*)out, out_stride, pieces, per_row);
+}
+
+// `act` 0: silu, 1: the exact gelu; rows of `cols` elements, strides in elements, `out` may be `in`.
+extern "C" int ullm_act_rows(int dtype, int act, const void* in, long long in_stride, void* out, long long out_stride,
+                             int rows, int cols, void* stream_handle) {
+  cudaStream_t st = (cudaStream_t)stream_handle;
+  if (rows < 0 || cols <= 0 || in_stride < cols || out_stride < cols || act < 0 || act > 1) return ULLM_ERR_BAD_SIZE;
+  if (rows == 0) return ULLM_OK;
+#define AR_GO(T)                                                                                         \
+  return act == 0 ? act_rows_launch<T, 0>(in, in_stride, out, out_stride, rows, cols, st)                \
+                  : act_rows_launch<T, 1>(in, in_stride, out, out_stride, rows, cols, st)
+  if (dtype == ULLM_DTYPE_F32) AR_GO(float);
+  if (dtype == ULLM_DTYPE_BF16) AR_GO(__nv_bfloat16);
+  if (dtype == ULLM_DTYPE_F16) AR_GO(__half);
+#undef AR_GO
   return ULLM_ERR_BAD_DTYPE;
 }

@@ -8,7 +8,10 @@
 //                     S_t = exp(-exp(A_log) dt_t) S_{t-1} + dt_t B_t x_t^T,    y_t = S_t^T C_t + D x_t
 //                   (head h reads B and C of group h / (heads / groups))
 //   ssd_gate_norm   y <- y * silu(z), then every one of `parts` equal stretches of the row divided by its own root mean
-//                   square, times a weight per channel
+//                   square, times a weight per channel; or the norm first and sigmoid(z) behind it
+//
+// Steps and decays that do not depend on the token (a linear attention with a fixed decay per head: x = v, B = k, C = q,
+// dt = 1) come as one row with a row stride of 0; `silu_in` puts a silu on x, B and C as they are read.
 //
 // The taps - 1 projected rows in front of a step's first token come from the state row too (zeros for a new request);
 // in a decode step `ssd_prepare` moves them on itself, otherwise `conv_state_update` (csrc/attention_prep.cu) after it.  The recurrence runs token by token in a
@@ -158,7 +161,7 @@ ssd_recurrence_kernel(const T* __restrict__ xbc, long long row_stride, int b_off
                       float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                       const int* __restrict__ req_slots, const int* __restrict__ token_req, float* __restrict__ out,
                       int heads, int n_state, int pdim, int per_group, int rs, int chunk, int num_slots, int most_tokens,
-                      int* status) {
+                      int* status, long long dt_stride, int silu_in) {
   extern __shared__ __align__(16) float sm[];
   pdl_launch_dependents();
   pdl_wait();
@@ -205,6 +208,13 @@ ssd_recurrence_kernel(const T* __restrict__ xbc, long long row_stride, int b_off
         if (r < n_state) {
           load_vec<T, 8>(xbc + (long long)(c0 + t) * row_stride + bg + r, vb);
           load_vec<T, 8>(xbc + (long long)(c0 + t) * row_stride + cg + r, vc);
+          if (silu_in) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              vb[i] = act_silu(vb[i]);
+              vc[i] = act_silu(vc[i]);
+            }
+          }
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i) vb[i] = vc[i] = 0.f;
@@ -216,17 +226,23 @@ ssd_recurrence_kernel(const T* __restrict__ xbc, long long row_stride, int b_off
       for (int i = tid; i < cn * dimp; i += SSD_THREADS) {
         const int t = i / dimp, r = i - t * dimp;
         const T* row = xbc + (long long)(c0 + t) * row_stride;
-        sb[i] = r < n_state ? to_f32(row[bg + r]) : 0.f;
-        sc[i] = r < n_state ? to_f32(row[cg + r]) : 0.f;
+        float b = r < n_state ? to_f32(row[bg + r]) : 0.f, c = r < n_state ? to_f32(row[cg + r]) : 0.f;
+        if (silu_in) {  // (silu(0) = 0: the padding stays zero)
+          b = act_silu(b);
+          c = act_silu(c);
+        }
+        sb[i] = b;
+        sc[i] = c;
       }
     }
     for (int i = tid; i < cn * cols_per_block; i += SSD_THREADS) {
       const int t = i / cols_per_block, c = i - t * cols_per_block;
-      sx[i] = col0 + c < pdim ? to_f32(xbc[(long long)(c0 + t) * row_stride + x_off + col0 + c]) : 0.f;
+      const float x = col0 + c < pdim ? to_f32(xbc[(long long)(c0 + t) * row_stride + x_off + col0 + c]) : 0.f;
+      sx[i] = silu_in ? act_silu(x) : x;
     }
     for (int t = tid; t < cn; t += SSD_THREADS) {
-      ss[t * 4] = expf(log_decay[(long long)(c0 + t) * heads + head]);
-      ss[t * 4 + 1] = dt[(long long)(c0 + t) * heads + head];
+      ss[t * 4] = expf(log_decay[(long long)(c0 + t) * dt_stride + head]);
+      ss[t * 4 + 1] = dt[(long long)(c0 + t) * dt_stride + head];
     }
   };
 
@@ -340,7 +356,7 @@ ssd_recurrence_kernel(const T* __restrict__ xbc, long long row_stride, int b_off
 template <typename T, int VEC>
 __global__ void ssd_gate_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, long long z_stride,
                                      const float* __restrict__ w, T* __restrict__ out, int inner, int part_size,
-                                     float eps) {
+                                     float eps, int gate_behind) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float scratch[33];
   pdl_launch_dependents();
@@ -354,7 +370,7 @@ __global__ void ssd_gate_norm_kernel(const float* __restrict__ y, const T* __res
     load_vec<T, VEC>(z + t * z_stride + p0 + c, zv);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) {
-      g[i] *= act_silu(zv[i]);
+      if (!gate_behind) g[i] *= act_silu(zv[i]);
       sq += g[i] * g[i];
     }
     store_vec32<VEC>(sm + c, g);
@@ -366,6 +382,12 @@ __global__ void ssd_gate_norm_kernel(const float* __restrict__ y, const T* __res
     load_vec32<VEC>(w + p0 + c, wv);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) g[i] *= rstd * wv[i];
+    if (gate_behind) {
+      float zv[VEC];
+      load_vec<T, VEC>(z + t * z_stride + p0 + c, zv);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) g[i] /= 1.f + expf(-zv[i]);
+    }
     store_vec<T, VEC>(out + t * inner + p0 + c, g);
   }
 }
@@ -439,7 +461,8 @@ template <typename T>
 static int recurrence_go(const void* xbc, long long row_stride, int b_off, int c_off, const float* dt,
                          const float* log_decay, const float* d_skip, float* state, long long state_stride,
                          const int* cu_q, const int* req_slots, const int* token_req, float* out, int requests, int heads,
-                         int n_state, int pdim, int groups, int num_slots, int most_tokens, int* status, cudaStream_t st) {
+                         int n_state, int pdim, int groups, int num_slots, int most_tokens, int* status,
+                         long long dt_stride, int silu_in, cudaStream_t st) {
   int rs = 1;  // lanes that share a column: as many as leave a thread about 8 rows, at most a warp
   while (rs < 32 && rs * 8 < n_state) rs <<= 1;
   const int col_groups = SSD_THREADS / rs;
@@ -469,7 +492,7 @@ static int recurrence_go(const void* xbc, long long row_stride, int b_off, int c
 #define SSD_GO(RPT, CPT)                                                                                              \
   return ullm_launch_kernel(ssd_recurrence_kernel<T, RPT, CPT>, grid, block, smem, st, (const T*)xbc, row_stride, b_off, \
                             c_off, dt, log_decay, d_skip, state, state_stride, cu_q, req_slots, token_req, out, heads, \
-                            n_state, pdim, heads / groups, rs, chunk, num_slots, most_tokens, status)
+                            n_state, pdim, heads / groups, rs, chunk, num_slots, most_tokens, status, dt_stride, silu_in)
   if (rpt == 4) {
     if (cpt == 4) SSD_GO(4, 4);
     if (cpt == 2) SSD_GO(4, 2);
@@ -485,12 +508,13 @@ static int recurrence_go(const void* xbc, long long row_stride, int b_off, int c
 }
 
 // xbc [tokens, row_stride]: x in columns 0 .. heads * pdim - 1, B and C (groups * n_state each) from b_off and c_off.
-// Requests that bring more than `most_tokens` tokens are left alone.
+// Requests that bring more than `most_tokens` tokens are left alone.  `dt_stride`: floats between two tokens' steps and
+// decays (heads, or 0 for one row that serves all tokens); `silu_in`: x, B and C pass a silu as they are read.
 extern "C" int ullm_ssd_recurrence(int dtype, const void* xbc, long long row_stride, int b_off, int c_off,
                                    const float* dt, const float* log_decay, const float* d_skip, float* state,
                                    long long state_stride, const int* cu_q, const int* req_slots, const int* token_req,
                                    float* out, int requests, int heads, int n_state, int pdim, int groups, int num_slots,
-                                   int most_tokens, int* status, void* stream) {
+                                   int most_tokens, int* status, void* stream, long long dt_stride, int silu_in) {
   cudaStream_t st = (cudaStream_t)stream;
   if (requests < 0 || num_slots <= 0 || !ullm_ssd_supported(heads, n_state, pdim, groups, 1)) return ULLM_ERR_BAD_SIZE;
   if (requests > 65535) return ULLM_ERR_UNSUPPORTED;
@@ -498,7 +522,7 @@ extern "C" int ullm_ssd_recurrence(int dtype, const void* xbc, long long row_str
   if (requests == 0) return ULLM_OK;
 #define SR_ARGS                                                                                                    \
   xbc, row_stride, b_off, c_off, dt, log_decay, d_skip, state, state_stride, cu_q, req_slots, token_req, out,      \
-      requests, heads, n_state, pdim, groups, num_slots, most_tokens, status, st
+      requests, heads, n_state, pdim, groups, num_slots, most_tokens, status, dt_stride, silu_in, st
   if (dtype == ULLM_DTYPE_F32) return recurrence_go<float>(SR_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return recurrence_go<__nv_bfloat16>(SR_ARGS);
   if (dtype == ULLM_DTYPE_F16) return recurrence_go<__half>(SR_ARGS);
@@ -508,7 +532,7 @@ extern "C" int ullm_ssd_recurrence(int dtype, const void* xbc, long long row_str
 
 template <typename T>
 static int gate_norm_go(const float* y, const void* z, long long z_stride, const float* w, void* out, int tokens,
-                        int inner, int parts, float eps, cudaStream_t st) {
+                        int inner, int parts, float eps, int gate_behind, cudaStream_t st) {
   const int part = inner / parts;
   const size_t smem = (size_t)part * sizeof(float);
   if (smem > 160 * 1024) return ULLM_ERR_UNSUPPORTED;
@@ -525,21 +549,22 @@ static int gate_norm_go(const float* y, const void* z, long long z_stride, const
       return ULLM_ERR_LAUNCH;                                                                                         \
     }                                                                                                                 \
     return ullm_launch_kernel(ssd_gate_norm_kernel<T, VEC>, dim3(tokens, parts), dim3(threads), smem, st, y,          \
-                              (const T*)z, z_stride, w, (T*)out, inner, part, eps);                                   \
+                              (const T*)z, z_stride, w, (T*)out, inner, part, eps, gate_behind);                                   \
   }
   if (wide) SG_GO(V);
   SG_GO(1);
 #undef SG_GO
 }
 
-// out [tokens, inner] = norm of y * silu(z) over `parts` equal stretches, times w; y 32-bit, z rows z_stride apart.
+// out [tokens, inner] = norm of y * silu(z) over `parts` equal stretches, times w, or with `gate_behind` norm of y times w
+// times sigmoid(z); y 32-bit, z rows z_stride apart.
 extern "C" int ullm_ssd_gate_norm(int dtype, const float* y, const void* z, long long z_stride, const float* w, void* out,
-                                  int tokens, int inner, int parts, float eps, void* stream) {
+                                  int tokens, int inner, int parts, float eps, void* stream, int gate_behind) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || inner <= 0 || parts <= 0 || inner % parts || parts > 65535 || z_stride < inner) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
-  if (dtype == ULLM_DTYPE_F32) return gate_norm_go<float>(y, z, z_stride, w, out, tokens, inner, parts, eps, st);
-  if (dtype == ULLM_DTYPE_BF16) return gate_norm_go<__nv_bfloat16>(y, z, z_stride, w, out, tokens, inner, parts, eps, st);
-  if (dtype == ULLM_DTYPE_F16) return gate_norm_go<__half>(y, z, z_stride, w, out, tokens, inner, parts, eps, st);
+  if (dtype == ULLM_DTYPE_F32) return gate_norm_go<float>(y, z, z_stride, w, out, tokens, inner, parts, eps, gate_behind, st);
+  if (dtype == ULLM_DTYPE_BF16) return gate_norm_go<__nv_bfloat16>(y, z, z_stride, w, out, tokens, inner, parts, eps, gate_behind, st);
+  if (dtype == ULLM_DTYPE_F16) return gate_norm_go<__half>(y, z, z_stride, w, out, tokens, inner, parts, eps, gate_behind, st);
   return ULLM_ERR_BAD_DTYPE;
 }

@@ -136,7 +136,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
                  const float* __restrict__ scores, float* __restrict__ state, long long state_stride,
                  const int* __restrict__ cu_q, const int* __restrict__ req_slots, const int* __restrict__ token_req,
                  float* __restrict__ out, int heads, int pdim, int per_group, int tokens, int num_slots, int least,
-                 int* status) {
+                 int* status, long long dt_stride) {
   constexpr int N = 32 * NT, NW = N / 4;      // a warp's columns of S^T
   constexpr int RS = N * 2 + 16;              // bytes between rows of B, C and S
   constexpr int XS = PT * 2 + 16;             // ... of x
@@ -279,8 +279,8 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, long long row_stride, in
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int t = chunk * SSC_Q + 2 * lane + i;
-      pa[i] = t < n ? log_decay[(long long)(t0 + t) * heads + head] : 0.f;
-      pd[i] = t < n ? dt[(long long)(t0 + t) * heads + head] : 0.f;
+      pa[i] = t < n ? log_decay[(long long)(t0 + t) * dt_stride + head] : 0.f;
+      pd[i] = t < n ? dt[(long long)(t0 + t) * dt_stride + head] : 0.f;
     }
   };
   auto weigh = [&](int buf) {  // warp 0: the chunk's running sums and weights from what `fetch` brought
@@ -418,7 +418,7 @@ template <int PT, int NT>
 static int chunk_go(const void* xbc, long long row_stride, int b_off, int c_off, const float* dt, const float* log_decay,
                     const float* d_skip, const float* scores, float* state, long long state_stride, const int* cu_q,
                     const int* req_slots, const int* token_req, float* out, int tokens, int requests, int heads, int pdim,
-                    int groups, int num_slots, int least, int* status, cudaStream_t st) {
+                    int groups, int num_slots, int least, int* status, long long dt_stride, cudaStream_t st) {
   constexpr int N = 32 * NT, RS = N * 2 + 16, XS = PT * 2 + 16;
   constexpr size_t stages = 2 * (2 * SSC_Q * RS + SSC_Q * XS + SSC_Q * SSC_G_STRIDE * 4) + 2 * SSC_Q * XS;
   constexpr int SB = stages + 4 * PT * RS + 2304 <= 227 * 1024 ? 2 : 1;  // (2304: more than the static arrays)
@@ -436,7 +436,7 @@ static int chunk_go(const void* xbc, long long row_stride, int b_off, int c_off,
   return ullm_launch_kernel(ssd_chunk_kernel<PT, NT, SB>, dim3(pdim / PT, heads, requests), dim3(2 * SSC_THREADS), smem, st,
                             (const __nv_bfloat16*)xbc, row_stride, b_off, c_off, dt, log_decay, d_skip, scores, state,
                             state_stride, cu_q, req_slots, token_req, out, heads, pdim, heads / groups, tokens, num_slots,
-                            least, status);
+                            least, status, dt_stride);
 }
 
 // Arguments as `ullm_ssd_recurrence`; `scores`: scratch of groups * tokens * SSC_Q floats.  Runs the requests that bring
@@ -445,7 +445,7 @@ extern "C" int ullm_ssd_chunk(const void* xbc, long long row_stride, int b_off, 
                               const float* log_decay, const float* d_skip, float* scores, float* state,
                               long long state_stride, const int* cu_q, const int* req_slots, const int* token_req, float* out,
                               int tokens, int requests, int heads, int n_state, int pdim, int groups, int num_slots,
-                              int least, int* status, void* stream) {
+                              int least, int* status, void* stream, long long dt_stride) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || requests < 0 || num_slots <= 0 || scores == nullptr) return ULLM_ERR_BAD_SIZE;
   if (!ullm_ssd_chunk_supported(heads, n_state, pdim, groups) || requests > 65535 || groups > 65535) return ULLM_ERR_UNSUPPORTED;
@@ -478,7 +478,7 @@ extern "C" int ullm_ssd_chunk(const void* xbc, long long row_stride, int b_off, 
   const bool wide = pdim % 32 == 0 && c32 < c16;
 #define SSC_GO(PT, NT)                                                                                               \
   return chunk_go<PT, NT>(xbc, row_stride, b_off, c_off, dt, log_decay, d_skip, scores, state, state_stride, cu_q,    \
-                          req_slots, token_req, out, tokens, requests, heads, pdim, groups, num_slots, least, status, st)
+                          req_slots, token_req, out, tokens, requests, heads, pdim, groups, num_slots, least, status, dt_stride, st)
   switch (n_state) {
     case 32:
       if (wide) SSC_GO(32, 1);

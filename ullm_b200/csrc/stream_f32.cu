@@ -1,7 +1,8 @@
 // A residual stream kept in 32-bit whatever the engine's dtype, for
 // arrangements that norm a sub-layer's OUTPUT and add it to the stream:
 //
-//   embed_scaled      stream[t] = table[id[t]] * scale (+ sinusoid of the position), copy[t] = round(stream[t])
+//   embed_scaled      stream[t] = table[id[t]] * scale (+ sinusoid of the position) (+ a row of a second table that the
+//                     token and the one before it choose), copy[t] = round(stream[t])
 //   norm_scale_add    stream[t] += mult * w * a[t] / sqrt(mean(a[t]^2) + eps),       copy[t] = round(stream[t])
 //   norm_scale_add_norm   the same, and out[t] = the NEXT norm of the updated stream[t]
 //   rmsnorm_rows_f32  out[r] = round(w * s / sqrt(mean(s^2) + eps)), s = stream[rows[r]]
@@ -21,13 +22,28 @@
 // Position term: column c of position p is sin(p f_i) for even c and cos(p f_i) for odd c, i = c / 2, with
 // f_i = base^(-2 i / width) read from a 32-bit table the host built in 64-bit.  The angle is the 32-bit
 // product; sinf / cosf are the accurate forms (full range reduction).
+//
+// Pair term: with a second table `pairs` of `buckets` + 1 rows, row (previous id * mul_prev + id * mul_cur) mod buckets is
+// added, for a request's first token row `buckets`.  The id in front of a step's first token comes from the request's
+// state (id + 1; 0: there is none), which the block of that token moves on to the step's last one: no other block of the
+// step touches it.
+struct PairEmbedding {
+  const void* table;
+  long long mul_prev, mul_cur;
+  int buckets;
+  int* state;  // [slots], `state_stride` ints apart
+  long long state_stride;
+  int num_slots;
+  const int* cu_q;
+};
+
 template <typename T, typename TAB>
 __global__ void embed_scaled_kernel(const int* __restrict__ ids, const TAB* __restrict__ table,
                                     float* __restrict__ stream, T* __restrict__ copy, int hidden, int vocab,
                                     float scale, const float* __restrict__ inv_freq,
                                     const int* __restrict__ positions, const int* __restrict__ last_tokens,
                                     const int* __restrict__ token_req, const int* __restrict__ req_slots,
-                                    int* status) {
+                                    int* status, PairEmbedding pe) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -39,6 +55,29 @@ __global__ void embed_scaled_kernel(const int* __restrict__ ids, const TAB* __re
   const bool bad = id < 0 || id >= vocab;
   if (bad && threadIdx.x == 0) ullm_report(status, ULLM_STATUS_TOKEN_ID, t, id);
   const TAB* row = table + (long long)(bad ? 0 : id) * hidden;
+  const TAB* pair = nullptr;
+  if (pe.table != nullptr) {
+    const int b = token_req[t];
+    long long bucket = pe.buckets;
+    if (b >= 0 && !bad) {
+      const int t0 = pe.cu_q[b], slot = req_slots[b];
+      const bool slot_ok = slot >= 0 && slot < pe.num_slots;
+      if (!slot_ok && threadIdx.x == 0) ullm_report(status, ULLM_STATUS_SLOT, t, slot);
+      int prev = -1;
+      if (t > t0) prev = ids[t - 1];
+      else if (slot_ok) prev = pe.state[slot * pe.state_stride] - 1;
+      if (prev >= 0) {
+        bucket = ((long long)prev * pe.mul_prev + (long long)id * pe.mul_cur) % pe.buckets;
+        if (bucket < 0) bucket += pe.buckets;
+      }
+      if (t == t0) {
+        __syncthreads();  // the state has been read
+        const int last = pe.cu_q[b + 1] - 1;
+        if (threadIdx.x == 0 && slot_ok) pe.state[slot * pe.state_stride] = (last == t ? id : ids[last]) + 1;
+      }
+    }
+    pair = (const TAB*)pe.table + bucket * hidden;
+  }
   const float p = inv_freq != nullptr ? (float)positions[t] : 0.f;
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
     float v = bad ? 0.f : to_f32(row[c]) * scale;
@@ -46,6 +85,7 @@ __global__ void embed_scaled_kernel(const int* __restrict__ ids, const TAB* __re
       const float ang = p * inv_freq[c >> 1];
       v += (c & 1) ? cosf(ang) : sinf(ang);
     }
+    if (pair != nullptr) v += to_f32(pair[c]);
     stream[(long long)t * hidden + c] = v;
     if (copy != nullptr) copy[(long long)t * hidden + c] = from_f32<T>(v);
   }
@@ -224,32 +264,39 @@ template <typename T, typename TAB>
 static int embed_scaled_launch(const int* ids, const void* table, float* stream, void* copy, int tokens, int hidden,
                                int vocab, float scale, const float* inv_freq, const int* positions,
                                const int* last_tokens, const int* token_req, const int* req_slots, int* status,
-                               cudaStream_t st) {
+                               const PairEmbedding& pe, cudaStream_t st) {
   return ullm_launch_kernel(embed_scaled_kernel<T, TAB>, dim3(tokens), dim3(row_threads(hidden)), 0, st, ids,
                             (const TAB*)table, stream, (T*)copy, hidden, vocab, scale, inv_freq, positions,
-                            last_tokens, token_req, req_slots, status);
+                            last_tokens, token_req, req_slots, status, pe);
 }
 
-// `dtype`: the engine's dtype = the table's and the copy's.  `copy` may be null.
+// `dtype`: the engine's dtype = the table's and the copy's.  `copy` may be null.  `pairs` (null: none): the second table
+// [buckets + 1, hidden] (see PairEmbedding), with the requests' state and `cu_q`, `token_req` and `req_slots` given.
 extern "C" int ullm_embed_scaled(int dtype, const int* ids, const void* table, float* stream, void* copy, int tokens,
                                  int hidden, int vocab, float scale, const float* inv_freq, const int* positions,
                                  const int* last_tokens, const int* token_req, const int* req_slots, int* status,
-                                 void* stream_handle) {
+                                 void* stream_handle, const void* pairs, int buckets, long long mul_prev,
+                                 long long mul_cur, int* pair_state, long long pair_stride, int num_slots,
+                                 const int* cu_q) {
   cudaStream_t st = (cudaStream_t)stream_handle;
   if (tokens < 0 || hidden <= 0 || vocab <= 0) return ULLM_ERR_BAD_SIZE;
+  if (pairs != nullptr && (buckets <= 0 || pair_state == nullptr || num_slots <= 0 || cu_q == nullptr ||
+                           token_req == nullptr || req_slots == nullptr))
+    return ULLM_ERR_BAD_SIZE;
+  const PairEmbedding pe = {pairs, mul_prev, mul_cur, buckets, pair_state, pair_stride, num_slots, cu_q};
   if (inv_freq != nullptr && positions == nullptr) return ULLM_ERR_BAD_SIZE;
   if (last_tokens != nullptr && (token_req == nullptr || req_slots == nullptr)) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
   if (dtype == ULLM_DTYPE_F32)
     return embed_scaled_launch<float, float>(ids, table, stream, copy, tokens, hidden, vocab, scale, inv_freq,
-                                             positions, last_tokens, token_req, req_slots, status, st);
+                                             positions, last_tokens, token_req, req_slots, status, pe, st);
   if (dtype == ULLM_DTYPE_BF16)
     return embed_scaled_launch<__nv_bfloat16, __nv_bfloat16>(ids, table, stream, copy, tokens, hidden, vocab, scale,
                                                              inv_freq, positions, last_tokens, token_req, req_slots,
-                                                             status, st);
+                                                             status, pe, st);
   if (dtype == ULLM_DTYPE_F16)
     return embed_scaled_launch<__half, __half>(ids, table, stream, copy, tokens, hidden, vocab, scale, inv_freq,
-                                               positions, last_tokens, token_req, req_slots, status, st);
+                                               positions, last_tokens, token_req, req_slots, status, pe, st);
   return ULLM_ERR_BAD_DTYPE;
 }
 

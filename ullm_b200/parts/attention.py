@@ -17,6 +17,7 @@ import torch
 from ..csrc import check_attention_sizes, kernels
 from .base import CacheNeed, Mixer, ParamDecl, SharesInput, StateNeed
 from .linear import linear
+from .position import distance_buckets
 from .registry import build_norm, build_position_encoding, register_mixer
 
 
@@ -56,6 +57,9 @@ class PagedAttention(Mixer, SharesInput):
         chunk: int | None = None,
         o_bias: bool = False,
         general: bool = False,
+        q_temperature: tuple[float, int] | None = None,
+        distance_bias: tuple[int, int] | None = None,
+        head_gate: bool = False,
     ):
         """`value_dim`: head size of the values and of the output (default: `head_dim`).  `window` with
         `keep_first`: position i sees j <= i if i - j < window or j < keep_first.  `own_kv` False: the mixer has
@@ -84,7 +88,15 @@ class PagedAttention(Mixer, SharesInput):
         weight per channel (`q_norm` [heads * head_dim], `k_norm` [kv heads * head_dim]), before the rotation.
         `value_unit_norm`: every head's value is divided by its root mean square (eps `norm_eps`, no weight); the
         cache holds it so.  `head_temperature`: the scores of head h are multiplied by the learned number `temp`[h]
-        (it is folded into the prepared queries in 32-bit).  With any of them a `rope_computed` position may say
+        (it is folded into the prepared queries in 32-bit).
+
+        Three on either.  `q_temperature` = (coef, every): the query at position p is multiplied by
+        1 + coef ln(floor((p + 1) / every) + 1).  `distance_bias` = (rows, most): the scaled score of query i and key j
+        gains `rel`[bucket(i - j), head], `rel` [rows, heads] (`distance_buckets` in parts/position.py).  `head_gate`: the
+        output of head h is multiplied by sigmoid(W_g x)_h, `gate` [heads, hidden], whose rows ride behind q, k and v in
+        the input product.
+
+        With any of them a `rope_computed` position may say
         `interleaved=True` (neighbouring dimensions turn together)."""
         super().__init__()
         if num_heads % num_kv_heads:
@@ -122,6 +134,16 @@ class PagedAttention(Mixer, SharesInput):
                                or not own_kv or keep_first):
             raise ValueError("whole_norm / value_unit_norm / head_temperature do not combine with the convolution, value "
                              "mixing, the norm behind the rotation, mixed heads, biases, kept tokens or borrowed keys")
+        self.q_temperature = (float(q_temperature[0]), int(q_temperature[1])) if q_temperature is not None else None
+        if self.q_temperature is not None and self.q_temperature[1] <= 0:
+            raise ValueError("q_temperature: `every` must be positive")
+        self.distance_bias = (int(distance_bias[0]), int(distance_bias[1])) if distance_bias is not None else None
+        self.head_gate = bool(head_gate)
+        if (self.q_temperature or self.distance_bias or self.head_gate) and (
+                self.rows_form or talking_heads or score_cap or keep_first or not own_kv):
+            raise ValueError("q_temperature / distance_bias / head_gate do not combine with mixed heads, capped scores, kept "
+                             "tokens, borrowed keys or the forms of the whole-projection norm")
+        self.bias_table = None  # [heads, distances] 32-bit, made of `rel` when the weights are there
         if self.whole_norm and qk_norm is None:
             raise ValueError("whole_norm needs the norm's spec (qk_norm)")
         if self.conv_taps < 0 or self.conv_taps > 32:
@@ -135,14 +157,15 @@ class PagedAttention(Mixer, SharesInput):
         n = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight", q_bias="q_proj.bias",
                  k_bias="k_proj.bias", v_bias="v_proj.bias", q_norm="q_norm.", k_norm="k_norm.",
                  o_bias="o_proj.bias", q_conv="q_proj.conv", k_conv="k_proj.conv", v_conv="v_proj.conv", talk="talk", vmix="vmix",
-                 temp="temp")
+                 temp="temp", rel="rel", gate="gate_proj.weight")
         n.update(names or {})
         self.names = n
         self.q_size = num_heads * head_dim
         self.kv_size = num_kv_heads * head_dim
         self.v_size = num_kv_heads * self.value_dim
         self.o_size = num_heads * self.value_dim
-        self.w_rows = self.q_size + ((self.kv_size + self.v_size) if self.own_kv else 0)  # of the input product
+        self.qkv_rows = self.q_size + ((self.kv_size + self.v_size) if self.own_kv else 0)
+        self.w_rows = self.qkv_rows + (num_heads if self.head_gate else 0)  # of the input product
         if self.whole_norm:
             from dataclasses import replace
 
@@ -158,7 +181,7 @@ class PagedAttention(Mixer, SharesInput):
         self.position = build_position_encoding(position) if position is not None else None
         if getattr(self.position, "interleaved", False) and not self.rows_form:
             raise ValueError("a rotation of neighbouring dimensions needs whole_norm, value_unit_norm or head_temperature")
-        self.general = bool(general or self.conv_taps or self.score_cap or self.talking_heads or value_mix or self.rows_form
+        self.general = bool(general or self.q_temperature or self.distance_bias or self.head_gate or self.conv_taps or self.score_cap or self.talking_heads or value_mix or self.rows_form
                             or self.unit_norm_after_rotation or getattr(self.position, "computed", False))
         if self.general and self.position is not None and not getattr(self.position, "computed", False):
             raise ValueError("these attention options take a position encoding of kind 'rope_computed' (or none)")
@@ -188,6 +211,10 @@ class PagedAttention(Mixer, SharesInput):
             d[n["vmix"]] = ParamDecl((), "bias32")
         if self.head_temperature:
             d[n["temp"]] = ParamDecl((self.num_heads,), "norm")
+        if self.distance_bias is not None:
+            d[n["rel"]] = ParamDecl((self.distance_bias[0], self.num_heads), "bias32")
+        if self.head_gate:
+            d[n["gate"]] = ParamDecl((self.num_heads, H))
         return d
 
     def subparts(self):
@@ -205,7 +232,9 @@ class PagedAttention(Mixer, SharesInput):
         self.tensors[n["q"]] = self.w_qkv[:q]
         if self.own_kv:
             self.tensors[n["k"]] = self.w_qkv[q:q + kv]
-            self.tensors[n["v"]] = self.w_qkv[q + kv:]
+            self.tensors[n["v"]] = self.w_qkv[q + kv:self.qkv_rows]
+        if self.head_gate:
+            self.tensors[n["gate"]] = self.w_qkv[self.qkv_rows:]
         self.tensors[n["o"]] = make("o_proj.weight", ParamDecl((H, self.o_size)))
         self.b_qkv = None
         if self.qkv_bias:
@@ -213,14 +242,15 @@ class PagedAttention(Mixer, SharesInput):
             self.tensors[n["q_bias"]] = self.b_qkv[:q]
             if self.own_kv:
                 self.tensors[n["k_bias"]] = self.b_qkv[q:q + kv]
-                self.tensors[n["v_bias"]] = self.b_qkv[q + kv:]
+                self.tensors[n["v_bias"]] = self.b_qkv[q + kv:self.qkv_rows]
+            self.b_qkv[self.qkv_rows:].zero_()  # (the gate has none)
         self.w_o_bias = None
         if self.o_bias:
             self.w_o_bias = self.tensors[n["o_bias"]] = make(n["o_bias"], ParamDecl((H,), "bias"))
         self.w_conv = None
         if self.conv_taps:
             # the three filters one after the other, as the projection's rows are
-            self.w_conv = make("qkv_proj.conv", ParamDecl((rows, self.conv_taps)))
+            self.w_conv = make("qkv_proj.conv", ParamDecl((self.qkv_rows, self.conv_taps)))
             self.tensors[n["q_conv"]] = self.w_conv[:q]
             self.tensors[n["k_conv"]] = self.w_conv[q:q + kv]
             self.tensors[n["v_conv"]] = self.w_conv[q + kv:]
@@ -230,8 +260,16 @@ class PagedAttention(Mixer, SharesInput):
             self.tensors[n["vmix"]] = make(n["vmix"], ParamDecl((), "bias32"))
         if self.head_temperature:
             self.tensors[n["temp"]] = make(n["temp"], ParamDecl((self.num_heads,), "norm"))
+        if self.distance_bias is not None:
+            self.tensors[n["rel"]] = make(n["rel"], ParamDecl((self.distance_bias[0], self.num_heads), "bias32"))
         if self.position is not None:
             self.position.build_tables(self.w_qkv.device)
+
+    def weights_loaded(self):
+        if self.distance_bias is not None:
+            rel = self.tensors[self.names["rel"]]
+            rows = torch.tensor(distance_buckets(*self.distance_bias), dtype=torch.long, device=rel.device)
+            self.bias_table = rel[rows].t().contiguous()
 
     # -- cache ------------------------------------------------------------
     def cache_need(self):
@@ -291,6 +329,9 @@ class PagedAttention(Mixer, SharesInput):
         if qkv is None:
             qkv = ws.tokens("attn.qkv", T, self.w_qkv.shape[0], x.dtype)
             linear(x, self.w_qkv, qkv, self.b_qkv)
+        gate = None
+        if self.head_gate:
+            qkv, gate = qkv[:, :self.qkv_rows], qkv[:, self.qkv_rows:]
         g = cache.group
         q = ws.tokens("attn.q", T, self.q_size, x.dtype)
         tables = self.position.tables() if self.position is not None else {}
@@ -327,12 +368,13 @@ class PagedAttention(Mixer, SharesInput):
             k_w=self.k_norm.weight if self.k_norm is not None else None, norm_first=self.q_norm is not None,
             norm_last=self.unit_norm_after_rotation,
             eps=self.q_norm.eps if self.q_norm is not None else self.norm_eps,
-            vmix_mode=mode, vmix_lambda=self.tensors[self.names["vmix"]] if mode == 2 else None, v_first=v_first)
+            vmix_mode=mode, vmix_lambda=self.tensors[self.names["vmix"]] if mode == 2 else None, v_first=v_first,
+            **({"q_temp": self.q_temperature} if self.q_temperature else {}))
         if state is not None:
             K.conv_state_update(qkv, self.conv_taps, state, ctx.cu_q, ctx.token_req, ctx.req_slots, ctx.num_requests)
-        return self._attend(q, x, ctx, cache, project_output, out)
+        return self._attend(q, x, ctx, cache, project_output, out, gate)
 
-    def _attend(self, q, x, ctx, cache, project_output: bool, out=None):
+    def _attend(self, q, x, ctx, cache, project_output: bool, out=None, gate=None):
         """The prepared queries over the pages, then the mixing of heads (if any) and the output projection."""
         K = kernels()
         T = x.shape[0]
@@ -341,13 +383,16 @@ class PagedAttention(Mixer, SharesInput):
         parts = None
         if self.talking_heads:
             parts = ws.tokens("attn.parts", T, self.num_heads * self.num_kv_heads * self.value_dim, torch.float32)
-        if (not self.talking_heads and self.score_cap is None and self.keep_first == 0
+        if gate is not None or self.distance_bias is not None or (
+                not self.talking_heads and self.score_cap is None and self.keep_first == 0
                 and (self.value_dim != self.head_dim or self.head_dim not in (64, 128))):
             # head sizes the kernels below take only in their general form: the windowed kernel runs multiples of 16
-            # on the tensor cores (and falls back to the general kernel itself)
+            # on the tensor cores (and falls back to the general kernel itself); it alone has the distance bias and the gate
             K.windowed_attention(q, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len,
                                  ctx.token_req, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim,
-                                 g.page_size, self.mask_arg, self.scale, num_requests=ctx.num_requests, workspace=ws)
+                                 g.page_size, self.mask_arg, self.scale, num_requests=ctx.num_requests, workspace=ws,
+                                 **({"gate": gate, "dist_bias": self.bias_table}
+                                    if gate is not None or self.distance_bias is not None else {}))
             return self._project(attn, ctx, project_output, out)
         K.paged_attention(
             q, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len, ctx.token_req,
@@ -370,7 +415,7 @@ class PagedAttention(Mixer, SharesInput):
     def forward(self, x, ctx, cache, project_output: bool = True, input_norm=None, projected=None, out=None):
         """`projected`: the input product's rows, formed by the caller (only on the general path).  `out`: where the
         projected output goes (default: the buffer that mixers share)."""
-        if projected is not None and (not self.general or self.rows_form or self.conv_taps):
+        if projected is not None and (not self.general or self.rows_form):
             raise NotImplementedError("an input product formed elsewhere beside these attention options")
         if self.general:
             if input_norm is not None:

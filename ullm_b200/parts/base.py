@@ -110,6 +110,10 @@ class Part:
         """Nested parts by tensor-name prefix."""
         return {}
 
+    def weights_loaded(self) -> None:
+        """Called once the parameters hold their values (read from files or random): what the part derives from them
+        (a table, a sum) is formed here."""
+
     def activation_elems(self) -> int:
         """Elements per token that this part (with its sub-parts) keeps in the step's workspace while it
         runs; the engine sets that much memory aside before it sizes the cache pool.  A part that takes
@@ -127,6 +131,11 @@ class Part:
         self.materialize(lambda n, d: make(prefix + n, d))
         for sub_prefix, sub in self.subparts().items():
             sub.materialize_all(make, prefix + sub_prefix)
+
+    def all_weights_loaded(self) -> None:
+        self.weights_loaded()
+        for sub in self.subparts().values():
+            sub.all_weights_loaded()
 
     def all_tensors(self, prefix: str = "") -> dict[str, torch.Tensor]:
         out = {prefix + n: t for n, t in self.tensors.items()}
@@ -152,7 +161,8 @@ class Norm(Part):
         """(weight, eps, 1) if this norm is w * (x - mean) / sqrt(variance + eps) over the whole row, (weight, eps, 0) if
         it is w * x / sqrt(mean(x^2) + eps), (weight, eps, 2, alpha, bias) if it is tanh(alpha x) * w + bias, which a
         block may then hand to a kernel that adds a sub-layer's output to the stream and applies the next norm at
-        once; None otherwise."""
+        once; None otherwise.  (In the place of a next norm's parameters (None, 0, 3) stands for no norm: the rows of the
+        stream as they are, rounded.)"""
         return None
 
     def rms_params(self):
@@ -225,6 +235,12 @@ class Mixer(Part):
         it) of the updated rows.  False (the default; nothing has run then): the caller adds `forward(x)` itself."""
         return False
 
+    def forward_norm_add(self, x, ctx, cache, stream, norm, mult: float, copy=None) -> bool:
+        """Optional: stream (32-bit, in place) += mult * norm(forward(x)) in the mixer's own last kernel, for an arrangement
+        that norms its sub-layers' outputs (`norm`: (weight, eps) of an RMS norm); `copy` (may be x) receives the updated
+        rows, rounded.  False (the default; nothing has run then): the caller does it itself."""
+        return False
+
     def operand_dtype(self):
         """The dtype of the rows this mixer's `forward` takes (that of its first matrix)."""
         for t in self.all_tensors().values():
@@ -269,6 +285,10 @@ class FeedForward(Part):
         """Optional: stream (32-bit, in place) += scale * forward(x) in the part's own last kernel (`scale` a
         32-bit vector per channel or None), which also leaves `next_norm` (`Norm.row_params()`, of a kind without a
         mean, with the output rows behind it) of the updated rows.  False (the default): the caller adds `forward(x)` itself."""
+        return False
+
+    def forward_norm_add(self, x, ctx, stream, norm, mult: float, copy=None) -> bool:
+        """Optional: as `Mixer.forward_norm_add`."""
         return False
 
     def gated_weights(self):

@@ -202,11 +202,16 @@ class OutputNormResidualBlock(Block):
                 h = ctx.workspace.tokens("model.stream_copy", T, H, engine_dtype)
                 kernels().cast_rows_f32(stream, h)
         copy = None if h is stream else h
-        a = self.mixer.forward(h, ctx, cache)
-        self.mixer_norm.scale_add(a, stream, self.residual_mult, copy)
+        # (a sub-layer whose last kernel can norm its output and add it to the stream itself does so)
+        norm = self.mixer_norm.rms_params()
+        if norm is None or not self.mixer.forward_norm_add(h, ctx, cache, stream, norm, self.residual_mult, copy):
+            a = self.mixer.forward(h, ctx, cache)
+            self.mixer_norm.scale_add(a, stream, self.residual_mult, copy)
         if self.feed_forward is not None:
-            y = self.feed_forward.forward(h, ctx)
-            self.feed_forward_norm.scale_add(y, stream, self.residual_mult, copy)
+            norm = self.feed_forward_norm.rms_params()
+            if norm is None or not self.feed_forward.forward_norm_add(h, ctx, stream, norm, self.residual_mult, copy):
+                y = self.feed_forward.forward(h, ctx)
+                self.feed_forward_norm.scale_add(y, stream, self.residual_mult, copy)
         ctx.stream_operand = h
         return None, stream
 

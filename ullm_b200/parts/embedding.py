@@ -5,8 +5,10 @@ vocabulary size.  A tied head reads the embedding table."""
 
 from __future__ import annotations
 
+import torch
+
 from ..csrc import kernels
-from .base import ParamDecl, Part
+from .base import ParamDecl, Part, StateNeed
 
 
 class TokenEmbedding(Part):
@@ -37,13 +39,17 @@ class TokenEmbedding(Part):
     def plain(self) -> bool:
         return self.scale == 1.0 and self.position is None
 
-    def forward_stream(self, token_ids, stream, copy, ctx):
-        """stream [T, hidden] float32 = table[id] * scale (+ the added position encoding); copy (the table's dtype,
-        or None) = the rounded stream."""
+    def forward_stream(self, token_ids, stream, copy, ctx, pairs=None):
+        """stream [T, hidden] float32 = table[id] * scale (+ the added position encoding) (+ the row that `pairs` = (the
+        model's `PairTable`, its state rows) adds); copy (the table's dtype, or None) = the rounded stream."""
+        more = {}
+        if pairs is not None:
+            part, state = pairs
+            more["pairs"] = (part.table, part.mul_prev, part.mul_cur, state, ctx.cu_q)
         inv = self.position.tables()["inv_freq"] if self.position is not None else None
         kernels().embed_scaled(token_ids, self.table, stream, copy, self.scale, inv, ctx.positions if inv is not None else None,
-                               ctx.last_tokens, ctx.token_req if ctx.last_tokens is not None else None,
-                               ctx.req_slots if ctx.last_tokens is not None else None)
+                               ctx.last_tokens, ctx.token_req if ctx.last_tokens is not None or pairs else None,
+                               ctx.req_slots if ctx.last_tokens is not None or pairs else None, **more)
         return stream
 
     def forward(self, token_ids, out, ctx=None):
@@ -69,6 +75,28 @@ class TokenSideTable(Part):
 
     def param_decls(self):
         return {self.param: ParamDecl((self.vocab_size, self.shares * self.dim))}
+
+    @property
+    def table(self):
+        return self.tensors[self.param]
+
+
+class PairTable(Part):
+    """A second table [buckets + 1, hidden]; the row (previous token * mul_prev + token * mul_cur) mod buckets is added to the
+    token's embedding, for a request's first token the last row.  The previous token of every request (+ 1; 0: none) is a
+    state row of the model."""
+
+    def __init__(self, buckets: int, hidden_size: int, mul_prev: int, mul_cur: int, param: str = ""):
+        super().__init__()
+        if min(buckets, hidden_size) <= 0:
+            raise ValueError("a pair table needs positive sizes")
+        self.buckets, self.hidden_size, self.mul_prev, self.mul_cur, self.param = buckets, hidden_size, mul_prev, mul_cur, param
+
+    def param_decls(self):
+        return {self.param: ParamDecl((self.buckets + 1, self.hidden_size))}
+
+    def state_need(self):
+        return StateNeed((1,), torch.int32)
 
     @property
     def table(self):

@@ -76,7 +76,8 @@ class DenseMLP(FeedForward):
         z > 0:   softplus(p) z^2 + z / 2
         z <= 0:  (1/2 + softplus(q)) (e^z - 1 - z) + z / 2
 
-    evaluated in 32-bit on the product's rounded output (csrc/sandwich_norm.cu); "relu2", max(z, 0)^2, without a tensor.
+    evaluated in 32-bit on the product's rounded output (csrc/sandwich_norm.cu); "relu2", max(z, 0)^2, and "gelu", the
+    exact one z (1 + erf(z / sqrt 2)) / 2, without a tensor.
 
     A caller may own the two matrices (`shared_weights` = (up, down), set before the parameters are made): the routed
     experts stack those of a shared expert of the experts' own size behind the experts'."""
@@ -85,8 +86,8 @@ class DenseMLP(FeedForward):
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "xielu", names: dict | None = None):
         super().__init__()
-        if activation not in ("xielu", "relu2"):
-            raise ValueError(f"activation {activation!r} unknown (have ['relu2', 'xielu'])")
+        if activation not in ("xielu", "relu2", "gelu"):
+            raise ValueError(f"activation {activation!r} unknown (have ['gelu', 'relu2', 'xielu'])")
         if hidden_size <= 0 or intermediate_size <= 0:
             raise ValueError("sizes must be positive")
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
@@ -122,6 +123,9 @@ class DenseMLP(FeedForward):
         if self.activation == "relu2":
             a = u
             kernels().relu2(u, a)
+        elif self.activation == "gelu":
+            a = u
+            kernels().act_rows("gelu", u, a)
         else:
             a = ctx.workspace.tokens("mlp.act", T, I, x.dtype)
             kernels().xielu(u, self.tensors[n["act"]], a)

@@ -13,7 +13,7 @@ import torch
 from ..config.specs import ModelSpec
 from ..csrc import kernels
 from .base import ParamDecl, Part
-from .embedding import OutputHead, TokenEmbedding, TokenSideTable
+from .embedding import OutputHead, PairTable, TokenEmbedding, TokenSideTable
 from .registry import build_block, build_norm, build_position_encoding
 
 
@@ -42,6 +42,12 @@ class DecoderModel(Part):
         self.token_side = None
         if spec.token_side is not None:
             self.token_side = TokenSideTable(spec.vocab_size, spec.token_side.dim, spec.token_side.shares)
+        self.pair_table = None
+        if spec.embedding_pairs is not None:
+            p = spec.embedding_pairs
+            if not self.stream_f32:
+                raise ValueError("an embedding of token pairs needs stream_dtype='float32'")
+            self.pair_table = PairTable(p.buckets, spec.hidden_size, p.mul_prev, p.mul_cur)
         self.schedule = list(spec.schedule)
         self._keeps_input = any(e.add_input or e.project_input for e in self.schedule)
         # one mixer of each group answers `graph_key` for all of its kind
@@ -61,6 +67,8 @@ class DecoderModel(Part):
         s[self.spec.head_name] = self.head
         if self.token_side is not None:
             s[self.spec.token_side.name] = self.token_side
+        if self.pair_table is not None:
+            s[self.spec.embedding_pairs.name] = self.pair_table
         return s
 
     def param_decls(self):
@@ -74,11 +82,14 @@ class DecoderModel(Part):
 
     # -- what the cache manager needs to know ------------------------------
     def cache_needs(self):
-        """Per schedule entry: (CacheNeed | None, StateNeed | None, cache_of, second CacheNeed | None)."""
+        """Per schedule entry: (CacheNeed | None, StateNeed | None, cache_of, second CacheNeed | None); behind them one more
+        for the state of the embedding, if it has any."""
         out = []
         for e in self.schedule:
             m = self.blocks[e.layer].mixer
             out.append((m.cache_need(), m.state_need(), e.cache_of, m.aux_cache_need()))
+        if self.pair_table is not None:
+            out.append((None, self.pair_table.state_need(), None, None))
         return out
 
     def graph_key(self, ctx) -> tuple:
@@ -112,7 +123,11 @@ class DecoderModel(Part):
             copy = None
             if self.dtype != torch.float32:
                 copy = ctx.workspace.tokens("model.stream_copy", T, self.spec.hidden_size, self.dtype)
-            self.embedding.forward_stream(ctx.token_ids, x, copy, ctx)
+            if self.pair_table is not None:
+                self.embedding.forward_stream(ctx.token_ids, x, copy, ctx,
+                                              pairs=(self.pair_table, caches[len(self.schedule)].state))
+            else:
+                self.embedding.forward_stream(ctx.token_ids, x, copy, ctx)
             ctx.stream_operand = copy if copy is not None else x
         else:
             x = ctx.workspace.tokens("model.hidden", T, self.spec.hidden_size, self.dtype)

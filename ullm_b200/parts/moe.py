@@ -145,7 +145,13 @@ class RoutedExperts(FeedForward):
         self._run(x, ctx, (stream, scale, next_norm))
         return True
 
-    def _run(self, x, ctx, add):
+    def forward_norm_add(self, x, ctx, stream, norm, mult: float, copy=None) -> bool:
+        if self.weight_on != "output" or mult != 1.0 or stream.shape[1] * 4 > 160 * 1024:
+            return False
+        self._run(x, ctx, (stream, None, (None, 0.0, 3, copy) if copy is not None else None), norm)
+        return True
+
+    def _run(self, x, ctx, add, outer_norm=None):
         K = kernels()
         T = x.shape[0]
         always = 1 if (self.rides and T <= RIDE_ROWS) else 0  # the shared expert as one more choice of every token
@@ -176,7 +182,7 @@ class RoutedExperts(FeedForward):
         if add is not None:
             stream, scale, next_norm = add
             if not K.moe_combine_add_norm(rows, place, None if on_input else weight, top, stream, scale, next_norm,
-                                          passing=passing, shared=shared):
+                                          passing=passing, shared=shared, **({"outer_norm": outer_norm} if outer_norm else {})):
                 raise RuntimeError("the combining kernel refused a row length that had been accepted")
             return None
         # (a buffer of its own: the shared expert's output may lie in "ffn.out")

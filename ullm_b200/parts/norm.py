@@ -14,18 +14,30 @@ from .registry import register_norm
 
 @register_norm("rmsnorm")
 class RMSNorm(Norm):
-    def __init__(self, size: int, eps: float, param: str = "weight"):
-        """`param`: the name of the weight behind the norm's prefix (may be empty: the prefix is the name)."""
+    def __init__(self, size: int, eps: float, param: str = "weight", around_zero: bool = False):
+        """`param`: the name of the weight behind the norm's prefix (may be empty: the prefix is the name).
+        `around_zero`: the checkpoint stores the weight minus one; 1 + w is formed once, in 32-bit, when the weights are
+        there."""
         super().__init__()
         self.size = size
         self.eps = eps
         self.param = param
+        self.around_zero = bool(around_zero)
+        self._one_plus = None
 
     def param_decls(self):
-        return {self.param: ParamDecl((self.size,), "norm")}
+        return {self.param: ParamDecl((self.size,), "bias32" if self.around_zero else "norm")}
+
+    def weights_loaded(self):
+        if self.around_zero:
+            self._one_plus = self.tensors[self.param] + 1.0
 
     @property
     def weight(self):
+        if self.around_zero:
+            if self._one_plus is None:
+                raise RuntimeError("a norm's weights are used before they were loaded (Part.weights_loaded)")
+            return self._one_plus
         return self.tensors[self.param]
 
     def rms_params(self):

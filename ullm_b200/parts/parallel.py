@@ -6,7 +6,7 @@ ONE product with the two projections' weights side by side [hidden, left width +
 At most one of the two keeps pages and at most one keeps state rows; each finds them in the execution's cache.
 
 `parallel_normed_mixers`: result = mult * (RMSnorm(left(h)) + RMSnorm(right(h))), each norm over the model width with a
-weight of its own.  The norms stand between the output projections and the sum, so there are two projections; but both
+weight of its own.  Both may keep state: their rows lie side by side in the execution's.  The norms stand between the output projections and the sum, so there are two projections; but both
 mixers read the same rows, so their input projections are ONE product (rows left | right), of which each gets its
 column range.  Norms, sum and the addition to a 32-bit stream are one kernel, which also leaves the rows of the norm
 that reads the stream next (`forward_add`).
@@ -14,10 +14,12 @@ that reads the stream next (`forward_add`).
 
 from __future__ import annotations
 
+from dataclasses import replace
+
 import torch
 
 from ..csrc import kernels
-from .base import Mixer, ParamDecl, SharesInput
+from .base import Mixer, ParamDecl, SharesInput, StateNeed
 from .linear import linear
 from .registry import build_mixer, register_mixer
 from .window_attention import _ProjectsOutput
@@ -104,7 +106,14 @@ class ParallelNormedMixers(Mixer):
         for m in (self.left, self.right):
             if not isinstance(m, SharesInput):
                 raise ValueError(f"{type(m).__name__} cannot take its input product from a caller")
-        _check_caches(self.left, self.right)
+        if self.left.cache_need() is not None and self.right.cache_need() is not None:
+            raise ValueError("at most one of two mixers side by side keeps pages")
+        sl, sr = self.left.state_need(), self.right.state_need()
+        self.left_state = 0  # floats of the left mixer's part of the state row, where both keep one
+        if sl is not None and sr is not None:
+            if len(sl.shape) != 1 or len(sr.shape) != 1 or sl.dtype != sr.dtype:
+                raise ValueError("two mixers side by side keep flat state rows of one dtype")
+            self.left_state = -(-sl.shape[0] // 4) * 4
         n = dict(left="left.", right="right.", left_norm="left_norm.weight", right_norm="right_norm.weight")
         n.update(names or {})
         self.names = n
@@ -125,7 +134,7 @@ class ParallelNormedMixers(Mixer):
         wl, wr, lc = self.left.input_width(), self.right.input_width(), self.left_cols
         self.w_in = make("in_proj.weight", ParamDecl((self.in_cols, self.hidden_size)))
         self.w_in[wl:lc].zero_()
-        self.w_in[lc + wr:].zero_()
+        self.w_in[lc + wr:].zero_()  # (so are the parts of the bias that a mixer leaves out)
         self.b_in = None
         if self.left.input_bias() or self.right.input_bias():
             self.b_in = make("in_proj.bias", ParamDecl((self.in_cols,), "bias"))
@@ -140,7 +149,10 @@ class ParallelNormedMixers(Mixer):
         return self.left.aux_cache_need() or self.right.aux_cache_need()
 
     def state_need(self):
-        return self.left.state_need() or self.right.state_need()
+        sl, sr = self.left.state_need(), self.right.state_need()
+        if self.left_state:
+            return StateNeed((self.left_state + -(-sr.shape[0] // 4) * 4,), sl.dtype)
+        return sl or sr
 
     def graph_key(self, ctx):
         return (self.left.graph_key(ctx), self.right.graph_key(ctx))
@@ -161,8 +173,12 @@ class ParallelNormedMixers(Mixer):
         a = ws.tokens("parallel.left", T, self.hidden_size, x.dtype)
         b = ws.tokens("parallel.right", T, self.hidden_size, x.dtype)
         lc = self.left_cols
-        self.left.forward(x, ctx, cache, projected=both[:, :self.left.input_width()], out=a)
-        self.right.forward(x, ctx, cache, projected=both[:, lc:lc + self.right.input_width()], out=b)
+        left_cache = right_cache = cache
+        if self.left_state and cache.state is not None:
+            left_cache = replace(cache, state=cache.state[:, :self.left_state])
+            right_cache = replace(cache, state=cache.state[:, self.left_state:])
+        self.left.forward(x, ctx, left_cache, projected=both[:, :self.left.input_width()], out=a)
+        self.right.forward(x, ctx, right_cache, projected=both[:, lc:lc + self.right.input_width()], out=b)
         return a, b
 
     def forward(self, x, ctx, cache):
@@ -180,4 +196,14 @@ class ParallelNormedMixers(Mixer):
         n = self.names
         kernels().pair_norm_add_norm(a, b, self.tensors[n["left_norm"]], self.tensors[n["right_norm"]], self.eps, self.mult,
                                      stream=stream, next_norm=next_norm)
+        return True
+
+    def forward_norm_add(self, x, ctx, cache, stream, norm, mult, copy=None):
+        if stream.dtype != torch.float32:
+            return False
+        a, b = self._sides(x, ctx, cache)
+        n = self.names
+        kernels().pair_norm_add_norm(a, b, self.tensors[n["left_norm"]], self.tensors[n["right_norm"]], self.eps, self.mult,
+                                     stream=stream, next_norm=(None, 0.0, 3, copy) if copy is not None else None,
+                                     outer_norm=(*norm, mult))
         return True

@@ -140,3 +140,22 @@ class AddedSinusoid(PositionEncoding):
 
     def tables(self):
         return self._tables
+
+
+def distance_buckets(rows: int, most: int) -> list[int]:
+    """Which of `rows` table rows a distance n = 0, 1, .. takes: one row per distance below h = rows // 2, then
+    h + floor(ln(n / h) / ln(most / h) * (rows - h)), at most rows - 1.  The list ends with the first distance of the last
+    row, which every longer distance takes too.  Where the ratio of the logarithms is a whole number in exact arithmetic the
+    floor takes that number, whatever the logarithms' last bit says."""
+    h = rows // 2
+    if rows < 2 or most <= h:
+        raise ValueError(f"distance buckets: {rows} rows up to a distance of {most} (at least 2 rows, more than rows // 2)")
+    out = list(range(h))
+    n = h
+    while not out or out[-1] < rows - 1:
+        v = math.log(n / h) / math.log(most / h) * (rows - h)
+        if abs(v - round(v)) < 1e-9:
+            v = round(v)
+        out.append(min(rows - 1, h + math.floor(v)))
+        n += 1
+    return out

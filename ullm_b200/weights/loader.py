@@ -72,6 +72,7 @@ def load_weights(model, model_dir: str, progress=None) -> dict[str, str]:
                 dst.copy_(src)  # converts on the way; float32 -> bfloat16 rounds to nearest even
             if progress is not None:
                 progress(i + 1, len(targets), n)
+        model.all_weights_loaded()
         return seen
     finally:
         for f in files:

@@ -94,3 +94,4 @@ def fill_random_(model, seed: int = 0, std: float = 0.02, norm_std: float = 0.0)
         else:
             tmp = torch.empty(t.shape, dtype=t.dtype, device=t.device).normal_(0.0, 1.0, generator=g)
             t.copy_(1.0 + tmp * norm_std if d.role == "norm" else tmp * std)
+    model.all_weights_loaded()
