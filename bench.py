@@ -908,6 +908,60 @@ def run_mafarax(args) -> dict:
     return out
 
 
+# ---------------------------------------------------------------------------------------------------------
+# `--workload ninelix`: the Ninelix decoder beside the Mafarax decoder (attention beside a state-space recurrence in every
+# layer, routed experts) and the Borosun decoder (linear attention with data-dependent decays, dense feed-forwards)
+# ---------------------------------------------------------------------------------------------------------
+NINELIX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, ff=8192, wkv_heads=32, lin_heads=16, experts=16, top=2, expert_ff=1024,
+                  vocab=32768, groups=2),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, ff=12288, wkv_heads=64, lin_heads=32, experts=32, top=2, expert_ff=2048,
+                  vocab=32768, groups=1),
+}
+
+
+def ninelix_config(width: int, heads: int, kv_heads: int, ff: int, wkv_heads: int, lin_heads: int, experts: int, top: int,
+                   expert_ff: int, vocab: int, groups: int) -> dict:
+    """Per group four layers: linear attention with fixed decays (heads of 128) and a dense feed-forward, attention beside a
+    state-space recurrence (heads of 64 columns, 128 rows) with routed experts, time mixing (heads of 64) with a dense
+    feed-forward, and the second kind once more."""
+    left = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, conv=4, bias_max=512,
+                q_temp=dict(coef=0.25, every=1024))
+    right = dict(heads=width // 64, vdim=64, state=128, groups=1, conv=4, norm_groups=1)
+    lin = dict(heads=lin_heads, dim=128, vdim=128, decay=[1.0 - 2.0 ** (-1 - 8.0 * h / lin_heads) for h in range(lin_heads)])
+    wkv = dict(heads=wkv_heads, dim=64)
+    dense = dict(kind="dense", ff=ff)
+    moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top))
+    kinds = [("lightning", lin, dense), ("parallel", dict(left=left, right=right), moe), ("wkv", wkv, dense),
+             ("parallel", dict(left=left, right=right), moe)]
+    return dict(architecture="Ninelix", vocab=vocab, width=width, logit_scale=0.25, norm=dict(eps=1e-5), torch_dtype="bfloat16",
+                embedding=dict(bigram=dict(buckets=65521, mul_prev=31, mul_cur=7)),
+                layers=[dict(type=t, mixer=dict(m), mlp=dict(f)) for _ in range(groups) for t, m, f in kinds])
+
+
+def run_ninelix(args) -> dict:
+    """`--workload ninelix`: prefill (one prompt of 2,048 tokens) and decode (8 requests holding 2,048 tokens each) of the
+    Ninelix decoder at layer sizes that resemble a real model's, random weights, beside the Mafarax and the Borosun decoder
+    (its linear attention) of the same width, heads and experts; per kernel group the device time of one eager step of each
+    kind.  One JSON object; the default workload and its line are untouched."""
+    T, B, ctx_len = PREFILL_TOKENS, args.batch, START_CONTEXT
+    out = {"workload": "ninelix", "prefill_tokens": T, "decode_batch": B, "decode_context": ctx_len,
+           "data": "synthetic", "dtype": "bf16", "peaks": peaks(), "sizes": {}}
+    names = [args.case] if args.case else list(NINELIX_SIZES)
+    for name in names:
+        size = NINELIX_SIZES[name]
+        out["sizes"][name] = {}
+        maf = dict(MAFARAX_SIZES[name], layers=4 * size["groups"])
+        bor = dict(BOROSUN_SIZES[name], groups=size["groups"])
+        for label, cfg in (("ninelix", ninelix_config(**size)), ("mafarax", mafarax_config(**maf)),
+                           ("borosun", borosun_config(**bor))):
+            if args.only_model and args.only_model != label:
+                continue
+            out["sizes"][name][label] = dict(_measure_model(cfg, False, T, B, ctx_len, args.steps, args.warmup),
+                                             layers=len(cfg["layers"]))
+    return out
+
+
 def run_extra_shapes(args, impl: str) -> dict:
     """The two further workloads, each in a process of its own (the 32B shape needs the device to itself), as
     flat entries for `points`."""
@@ -1571,7 +1625,7 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--workload", default="8b", choices=["8b", "32b", "serve-0.6b", "8b-long", "ludalix", "borosun", "pidenex", "finosun",
-                                                           "mafarax"],
+                                                           "mafarax", "ninelix"],
                     help="8b: the default line (Qwen3-8B layer sizes); 32b: the same at Qwen3-32B layer sizes; "
                          "serve-0.6b: 256 requests under continuous batching at Qwen3-0.6B layer sizes; 8b-long: "
                          "prefill of 16,384 tokens and decode of 8 requests at that context")
@@ -1585,8 +1639,8 @@ def main() -> int:
                     help="--probe linear: launch only this kernel, eagerly, --steps times (for a profiler)")
     ap.add_argument("--shape", default="gate_up", choices=["qkv", "o", "gate_up", "down", "head"],
                     help="--probe linear --only: which of the decode step's products")
-    ap.add_argument("--only-model", default=None, help="--workload borosun / pidenex / finosun / mafarax: measure only this model (borosun, pidenex, finosun or "
-                         "mafarax; ludalix_dense, ludalix_routed, ludalix_pairs)")
+    ap.add_argument("--only-model", default=None, help="--workload borosun / pidenex / finosun / mafarax / ninelix: measure only this model (borosun, pidenex, finosun, "
+                         "mafarax or ninelix; ludalix_dense, ludalix_routed, ludalix_pairs)")
     ap.add_argument("--case", default=None, help="run only the case of this name (--probe prefill-attention, decode-attention)")
     ap.add_argument("--context", type=int, default=START_CONTEXT, help="tokens each request holds (--probe)")
     ap.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens of a page (--probe decode-attention)")
@@ -1637,6 +1691,9 @@ def main() -> int:
         return 0
     if args.workload == "mafarax":
         print(json.dumps(run_mafarax(args)))
+        return 0
+    if args.workload == "ninelix":
+        print(json.dumps(run_ninelix(args)))
         return 0
     out = run_serve(args) if args.workload == "serve-0.6b" else run_ours(args)
     if extra:

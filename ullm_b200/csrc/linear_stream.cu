@@ -57,7 +57,7 @@ struct LsParams {
   int sq_count;
   float sq_inv_cols, sq_eps;      // 1 / (columns of the normed row), the norm's eps
   int* status;
-  int group_units;                // > 0: unit u meets rows (u / group_units) * M .. of x (row sets stacked); 0: rows 0 ..
+  int group_units, groups;        // > 0: unit u meets row set min(u / group_units, groups - 1) of M rows of x (stacked)
 };
 
 // ---- cluster helpers: a block's rank, a peer's shared-memory address, remote stores and barrier arrivals ------
@@ -146,7 +146,7 @@ __global__ void __launch_bounds__(LS_THREADS, 2) linear_stream_kernel(const __gr
       struct Pos {
         int u, kb, slot, round, x_row;
       };
-      auto x_row_of = [&](int u) { return p.group_units > 0 ? u / p.group_units * p.M : 0; };
+      auto x_row_of = [&](int u) { return p.group_units > 0 ? min(u / p.group_units, p.groups - 1) * p.M : 0; };
       auto step = [&](Pos& q) {
         if (++q.kb == nkb) q.kb = 0, q.u += ncl, q.x_row = x_row_of(q.u);
         if (++q.slot == p.stages) q.slot = 0, ++q.round;
@@ -536,12 +536,12 @@ extern "C" int ullm_linear_stream_norm(const void* x, const void* w, const void*
 }
 
 // Products with a row set each: rows g * group_rows .. of w [N, K] meet x[g] of x [groups][M][K] (group_rows a multiple of
-// 32; the last group may have fewer rows); out [M, N] bfloat16.
-extern "C" int ullm_linear_stream_grouped(const void* x, const void* w, void* out, int M, int N, int K, int group_rows,
-                                          int* status, void* stream) {
-  if (group_rows <= 0 || group_rows % LS_UNIT_ROWS) return ULLM_ERR_UNSUPPORTED;
+// 32; the last group takes what is left); out [M, N] bfloat16.
+extern "C" int ullm_linear_stream_grouped(const void* x, const void* w, void* out, int M, int N, int K, int groups,
+                                          int group_rows, int* status, void* stream) {
+  if (groups <= 0 || group_rows <= 0 || group_rows % LS_UNIT_ROWS) return ULLM_ERR_UNSUPPORTED;
   return ls_run(x, w, nullptr, nullptr, out, M, N, K, 0, 0, nullptr, nullptr, nullptr, nullptr, 0, 0, 0.f,
-                (N + group_rows - 1) / group_rows, group_rows / LS_UNIT_ROWS, status, stream);
+                groups, group_rows / LS_UNIT_ROWS, status, stream);
 }
 
 static int ls_run(const void* x, const void* w, const void* bias, const void* residual, void* out, int M, int N, int K,
@@ -592,6 +592,7 @@ static int ls_run(const void* x, const void* w, const void* bias, const void* re
   p.sq_eps = sq_eps;
   p.status = status;
   p.group_units = group_units;
+  p.groups = groups;
   if (NT == 1) return ls_launch<1>(0, wm, wm32, xm, p, (cudaStream_t)stream);
   if (NT == 2) return ls_launch<2>(1, wm, wm32, xm, p, (cudaStream_t)stream);
   return ls_launch<4>(2, wm, wm32, xm, p, (cudaStream_t)stream);

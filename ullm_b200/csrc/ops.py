@@ -287,7 +287,7 @@ class Kernels:
             "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, P],
             "ullm_token_shift_mix": [I, P, LL, P, I, I, P, P, LL, I, P, P, P, I, I, P, P],
             "ullm_low_rank_decay": [I, P, LL, I, I, P, P, P, I, I, I, P],
-            "ullm_linear_stream_grouped": [P, P, P, I, I, I, I, P, P],
+            "ullm_linear_stream_grouped": [P, P, P, I, I, I, I, I, P, P],
             "ullm_head_norm_gate": [I, P, P, LL, P, P, I, I, I, F, I, I, P],
             "ullm_moe_route": [P, LL, P, P, P, I, I, I, I, I, I, I, F, I, P],
             "ullm_moe_arrange": [P, I, I, P, P, P, P],
@@ -1461,20 +1461,20 @@ class Kernels:
     @_timed("linear", lambda x, weight, *rest: weight.numel() * weight.element_size())
     def grouped_linear(self, x, weight, out, group_rows: int):
         """Products with an operand each: rows g * group_rows .. of the stacked `weight` [N, K] meet x[g] of x [G, T, K]
-        (the last group may have fewer rows); out [T, N].  Few bfloat16 rows: the weight-streaming kernel, one launch;
+        (the last group takes what is left, more rows or fewer); out [T, N].  Few bfloat16 rows: the weight-streaming kernel, one launch;
         otherwise the library's batched product for the full groups and a product for the rest."""
         _need(x, "x")
         _need(out, "out", x.dtype)
         G, T, K = x.shape
         N = weight.shape[0]
-        full = min(N // group_rows, G)
-        if weight.shape[1] != K or out.shape != (T, N) or not (G - 1) * group_rows < N <= G * group_rows:
+        full = G if N == G * group_rows else G - 1
+        if weight.shape[1] != K or out.shape != (T, N) or N <= (G - 1) * group_rows:
             raise KernelError(f"grouped_linear: x {tuple(x.shape)}, weight {tuple(weight.shape)}, groups of {group_rows}")
         if (x.dtype == torch.bfloat16 and self.small_m_mode in ("auto", "stream") and T <= self.stream_all_rows
                 and group_rows % 32 == 0 and weight.is_contiguous() and weight.dtype == x.dtype
                 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0
                 and self.lib.ullm_linear_stream_supported(T, N, K)):
-            self._check(self.lib.ullm_linear_stream_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, group_rows,
+            self._check(self.lib.ullm_linear_stream_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, G, group_rows,
                                                             _ptr(self.status), _stream()),
                         f"linear_stream_grouped ({G} x {T}x{K} . {N}x{K})")
             return out
