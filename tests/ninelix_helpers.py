@@ -144,3 +144,32 @@ def make_runner(tmp_path, cfg, w, page, dtype, num_pages=64, max_requests=4, nam
 def oracle(ids, w, cfg) -> torch.Tensor:
     """Logits at every position, 64-bit arithmetic on the weights as given (rounded ones stay rounded)."""
     return pn.forward(cfg, {n: t.double() for n, t in w.items()}, ids).float()
+
+
+def assert_model_close(got, ids, w, cfg, dtype: str, what: str = "") -> None:
+    """A whole model's logits at every position against the plain model.  32-bit: the fixed limits of tests/helpers.py.
+    16-bit: a read-out that nearly vanishes is divided by its own root mean square, and every sub-layer's output is normed
+    once more, so roundings are amplified at some positions; how far is taken from the plain model with nothing but its
+    sub-layers' inputs and outputs rounded, or moved by as much at random (the largest of five runs).  Rows may err by the fixed rms limit or three times that model's own error, there
+    or over all rows (one in 25 by twice as much), all rows together by the fixed rms limit or twice its error."""
+    from helpers import TOL_RMS, assert_close
+
+    ref = oracle(ids, w, cfg)
+    if dtype == "float32":
+        return assert_close(got, ref, dtype, what)
+    assert got.shape == ref.shape and torch.isfinite(got.float()).all(), f"{what}: shape or non-finite values"
+    wd, td = {n: t.double() for n, t in w.items()}, getattr(torch, dtype)
+    g = torch.Generator().manual_seed(1)
+    unit = torch.finfo(td).eps / 2  # (the largest relative error of a rounding)
+    moved = lambda v: v * (1.0 + unit * (2.0 * torch.rand(v.shape, generator=g, dtype=v.dtype) - 1.0))
+    own = [pn.forward(cfg, wd, ids, rounded=r).float() - ref for r in [lambda v: v.to(td).double()] + [moved] * 4]
+    scale = max(ref.abs().max().item(), 1e-6)
+    rms = lambda d: d.pow(2).mean(-1).sqrt() / scale
+    err, floor = rms(got.detach().float().cpu() - ref), torch.stack([rms(d) for d in own]).amax(0)
+    own_all = float(floor.pow(2).mean().sqrt())
+    limit = (3 * floor).clamp(min=max(3 * own_all, TOL_RMS[dtype]))
+    total, allowed = err.pow(2).mean().sqrt(), max(TOL_RMS[dtype], 2 * own_all)
+    over = int((err > limit).sum())
+    assert total <= allowed, f"{what}: rms {total:.3e} (limit {allowed:.3e}) of scale"
+    assert over <= max(1, len(err) // 25) and (err <= 2 * limit).all(), (
+        f"{what}: {over} of {len(err)} rows over their limit, worst {float((err / limit).max()):.2f} times")

@@ -241,22 +241,23 @@ def feed_forward(h, f, w, pre):
 # ---------------------------------------------------------------------------------------------------------
 # the model
 # ---------------------------------------------------------------------------------------------------------
-def layer(x, i, cfg, w):
+def layer(x, i, cfg, w, rounded=lambda v: v):
     L, eps, pre = cfg["layers"][i], cfg["norm"]["eps"], f"l{i}."
-    x = x + rms_norm_one_plus(mixer(x, L, w, pre + "mix.", eps), w[pre + "norm1"], eps)
+    x = x + rms_norm_one_plus(rounded(mixer(rounded(x), L, w, pre + "mix.", eps)), w[pre + "norm1"], eps)
     if L.get("mlp") is not None:
-        x = x + rms_norm_one_plus(feed_forward(x, L["mlp"], w, pre + "mlp."), w[pre + "norm2"], eps)
+        x = x + rms_norm_one_plus(rounded(feed_forward(rounded(x), L["mlp"], w, pre + "mlp.")), w[pre + "norm2"], eps)
     return x
 
 
-def forward(cfg, w, ids, return_layers: bool = False):
-    """Logits [n, vocab] of one sequence (and the stream after every layer, if asked)."""
+def forward(cfg, w, ids, return_layers: bool = False, rounded=lambda v: v):
+    """Logits [n, vocab] of one sequence (and the stream after every layer, if asked).  `rounded`: what happens to the
+    sub-layers' inputs and outputs (a rounding to 16 bits shows how far such roundings alone carry)."""
     x = embed(list(ids), w, cfg)
     seen = []
     for i in range(len(cfg["layers"])):
-        x = layer(x, i, cfg, w)
+        x = layer(x, i, cfg, w, rounded)
         seen.append(x)
-    logits = (rms_norm_one_plus(x, w["final.norm"], cfg["norm"]["eps"]) @ w["head"].T) * cfg["logit_scale"]
+    logits = (rounded(rms_norm_one_plus(x, w["final.norm"], cfg["norm"]["eps"])) @ w["head"].T) * cfg["logit_scale"]
     return (logits, torch.stack(seen)) if return_layers else logits
 
 

@@ -5,6 +5,8 @@ that remember one token from hundreds of positions back, the first tokens, long 
 entry point and the scheduler."""
 
 import copy
+import os
+from types import SimpleNamespace
 
 import pytest
 import torch
@@ -13,7 +15,7 @@ import plain_ninelix as pn
 from conftest import device
 from helpers import TOL, assert_close, errors, random_ids
 from ludalix_helpers import assert_rows_close
-from ninelix_helpers import (CONFIGS, TENSOR_SIZES, cast, config, dense, every_expert_chosen, left, lightning, make_runner,
+from ninelix_helpers import (CONFIGS, assert_model_close, cast, config, dense, every_expert_chosen, left, lightning, make_runner,
                              model_for, moe, oracle, parallel, replay, right, weights_for, wkv, write_model)
 
 pytestmark = [pytest.mark.gpu, pytest.mark.needs_cuda]
@@ -461,18 +463,67 @@ def test_attention_with_distance_biases_and_head_gates(dtype, heads, kv, dim, vd
                 s = torch.einsum("jhd,hd->hj", kb[:i + 1], q[t].double()) * scale + bias.double()[:, dist]
                 ref[t] = torch.einsum("hj,jhv->hv", torch.softmax(s, -1), vb[:i + 1])
         gated = ref * torch.sigmoid(gate[:, :heads].double())[..., None]
-        for use_gate, ws in ((False, None), (True, None), (True, Workspace(device()))):
+        ws_ = Workspace(device())
+        ctx = SimpleNamespace(decode_only=False, num_requests=B + 1, workspace=ws_)
+        for use_gate, ws, step in ((False, None, None), (True, None, None), (True, ws_, None), (True, ws_, ctx), (False, ws_, ctx)):
             out = torch.full((T, heads * vdim), 7.0, dtype=td, device=device())
+            K.pair_biased_rows = 1  # (short steps too)
             K.windowed_attention(q.view(T, -1).to(device()), out, k.view(-1, page, kv, dim).to(device()),
                                  v.view(-1, page, kv, vdim).to(device()), table, i32([0, 1, 2, 3, 0]), i32(cu + [T]),
                                  i32(list(held) + [0]), i32([b for b in range(B) for _ in range(new[b])] + [-1]), heads, kv, dim,
                                  vdim, page, 0, scale, gate=gate.to(device())[:, :heads] if use_gate else None,
-                                 dist_bias=bias.to(device()), num_requests=B + 1, workspace=ws)
+                                 dist_bias=bias.to(device()), num_requests=B + 1, workspace=ws, ctx=step)
             K.raise_on_status()
-            assert K.attention_path == ("window_mma" if dtype == "bfloat16" and dim % 16 == 0 and vdim % 16 == 0 else "generic")
+            K.apply_switches(os.environ)
+            path = "window_mma" if dtype == "bfloat16" and dim % 16 == 0 and vdim % 16 == 0 else "generic"
+            if step is not None and dtype == "bfloat16" and dim == vdim == 128:
+                path = "prefill_tcgen05"
+            assert K.attention_path == path
             assert not out[T - 1].any()
             close(out[:T - 1], (gated if use_gate else ref)[:T - 1].reshape(T - 1, -1).float(), dtype,
                   f"biases to distance {length}, gate {use_gate}, runs {ws is not None}")
+
+
+@pytest.mark.parametrize("heads,kv,dim,page", [(4, 2, 64, 16), (16, 1, 128, 8), (3, 3, 128, 16), (8, 4, 64, 4)])
+def test_decode_attention_with_distance_biases_and_head_gates(heads, kv, dim, page):
+    """Steps of single tokens on the split decode kernel, merged inside a cluster, by the second kernel, and unsplit."""
+    from ullm_b200.csrc import kernels
+    from ullm_b200.engine.batch import Workspace
+
+    K = kernels()
+    g = torch.Generator().manual_seed(heads + dim)
+    held = (600, 1, 64, 257, 33)
+    B, per = len(held), -(-max(held) // page)
+    T = B + 1
+    pages = torch.randperm(B * per, generator=g).view(B, per)
+    k, v = (torch.randn(B * per * page, kv, dim, generator=g).to(torch.bfloat16) for _ in range(2))
+    q = (torch.randn(T, heads, dim, generator=g) * 1.5).to(torch.bfloat16)
+    gate = torch.randn(T, heads + 2, generator=g).to(torch.bfloat16)
+    scale = 0.7 / dim ** 0.5
+    ctx = SimpleNamespace(decode_only=True, num_requests=T, workspace=Workspace(device()))
+    for length in (1, 40, 300):
+        bias = torch.randn(heads, length, generator=g) * 2
+        ref = torch.zeros(B, heads, dim, dtype=torch.float64)
+        for b in range(B):
+            slots = (pages[b][:, None] * page + torch.arange(page)).reshape(-1)[:held[b]]
+            kb, vb = (x.double()[slots].repeat_interleave(heads // kv, 1) for x in (k, v))
+            dist = (held[b] - 1 - torch.arange(held[b])).clamp(max=length - 1)
+            s = torch.einsum("jhd,hd->hj", kb, q[b].double()) * scale + bias.double()[:, dist]
+            ref[b] = torch.einsum("hj,jhv->hv", torch.softmax(s, -1), vb)
+        for merge in (True, False, "one"):
+            K.decode_cluster_merge, K.decode_split_target = (merge, 400) if merge != "one" else (False, 1)
+            for use_gate in (True, False):
+                out = torch.full((T, heads * dim), 7.0, dtype=torch.bfloat16, device=device())
+                K.windowed_attention(q.view(T, -1).to(device()), out, k.view(-1, page, kv, dim).to(device()),
+                                     v.view(-1, page, kv, dim).to(device()), pages.to(torch.int32).to(device()),
+                                     i32([0, 1, 2, 3, 4, 0]), i32(list(range(T + 1))), i32(list(held) + [0]), i32([0, 1, 2, 3, 4, -1]),
+                                     heads, kv, dim, dim, page, 0, scale, gate=gate.to(device())[:, :heads] if use_gate else None,
+                                     dist_bias=bias.to(device()), num_requests=T, workspace=ctx.workspace, ctx=ctx)
+                K.raise_on_status()
+                assert K.attention_path == "decode" and not out[B].any()
+                want = ref * torch.sigmoid(gate[:B, :heads].double())[..., None] if use_gate else ref
+                close(out[:B], want.reshape(B, -1).float(), "bfloat16", f"biases to distance {length}, merge {merge}, gate {use_gate}")
+            K.apply_switches(os.environ)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -524,7 +575,6 @@ def test_whole_decode_and_portions_agree_with_the_plain_model(tmp_path, dtype, t
     r = make_runner(tmp_path, cfg, w, page, dtype, num_pages=64)
     n = 75 if tag not in ("E", "F") else 190
     ids = random_ids(cfg["vocab"], n, 11)
-    ref = oracle(ids, w, cfg)
     plans = {
         "whole": [[("a", n)]],
         "decode": [[("b", 3)]] + [[("b", 1)] for _ in range(n - 3)],
@@ -535,11 +585,10 @@ def test_whole_decode_and_portions_agree_with_the_plain_model(tmp_path, dtype, t
     for name, plan in plans.items():
         rid = plan[0][0][0]
         got = replay(r, {rid: ids}, plan)[rid]
-        assert_rows_close(got, ref, dtype, f"{tag} {name}")
+        assert_model_close(got, ids, w, cfg, dtype, f"{tag} {name}")
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("tag", ["A", "E"])
+@pytest.mark.parametrize("tag,dtype", [("A", "float32"), ("F", "float32"), ("E", "float32"), ("E", "bfloat16")])
 def test_unequal_batches_with_pages_and_slots_used_again(tmp_path, dtype, tag):
     """Three request slots and a pool that cannot hold all requests at once: six requests of unequal length come
     and go, portions of some beside single tokens of others; every request equals itself run alone."""
@@ -559,7 +608,7 @@ def test_unequal_batches_with_pages_and_slots_used_again(tmp_path, dtype, tag):
     ]
     got = replay(r, reqs, plan)
     for k in reqs:
-        assert_rows_close(got[k], oracle(reqs[k], w, cfg), dtype, f"request {k}")
+        assert_model_close(got[k], reqs[k], w, cfg, dtype, f"request {k}")
     assert not r.cache.requests
     assert all(r.cache.num_free_pages(g) == n for g, n in enumerate(r.cache.group_pages))
 
@@ -695,7 +744,7 @@ def test_the_first_tokens_alone_and_in_pairs(tmp_path, dtype):
         reqs = {k: random_ids(cfg["vocab"], n, 7 + n) for k, n in dict(a=1, b=2, c=3, d=2).items()}
         got = replay(r, reqs, [[("a", 1)], [("b", 2), ("c", 1)], [("c", 2), ("d", 1)], [("d", 1)]])
         for k in reqs:
-            assert_rows_close(got[k], oracle(reqs[k], w, cfg), dtype, f"{tag} request {k}")
+            assert_model_close(got[k], reqs[k], w, cfg, dtype, f"{tag} request {k}")
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -705,7 +754,7 @@ def test_long_decoding(tmp_path, dtype):
     r = make_runner(tmp_path, cfg, w, page, dtype, num_pages=160)
     ids = random_ids(cfg["vocab"], 301, 17)
     got = replay(r, {"a": ids}, [[("a", 1)] for _ in range(301)])["a"]
-    assert_rows_close(got, oracle(ids, w, cfg), dtype, "long decoding")
+    assert_model_close(got, ids, w, cfg, dtype, "long decoding")
 
 
 # ---------------------------------------------------------------------------------------------------------

@@ -52,7 +52,17 @@ struct DecFuse {
   // applied to the values of any kv head, and the 32-bit results go to parts [request][head][value head][D]
   // (what mixing the softmax weights across heads needs); `out` is not written
   float* parts;
+  // a learned bias per head and distance ([num_q][dist_len] 32-bit, added to the scaled score; the last one serves every
+  // longer distance) and a gate per head ([batch][num_q], row stride gate_stride): out *= sigmoid(gate); null: none
+  const float* dist_bias;
+  int dist_len;
+  const __nv_bfloat16* gate;
+  long long gate_stride;
 };
+
+__device__ __forceinline__ float dec_head_gate(const __nv_bfloat16* gate, long long stride, long long b, int h) {
+  return gate != nullptr ? 1.f / (1.f + expf(-__bfloat162float(gate[b * stride + h]))) : 1.f;
+}
 
 // 2^x by the hardware's unit alone (exp2f adds a range fix-up around the same instruction)
 __device__ __forceinline__ float dec_ex2(float x) {
@@ -295,6 +305,17 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
   float o[NT_O][4];
 #pragma unroll
   for (int j = 0; j < NT_O; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  // the two rows' biases: their table rows, and the number of every distance beyond the table
+  const float log2e = 1.4426950408889634f;
+  const float* brow[2] = {nullptr, nullptr};
+  float b_far[2] = {0.f, 0.f};
+  if (fu.dist_bias != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      brow[r] = fu.dist_bias + (long long)(kh * group + min((lane >> 2) + 8 * r, group - 1)) * fu.dist_len;
+      b_far[r] = brow[r][fu.dist_len - 1] * log2e;
+    }
+  }
 
   if (!early) {
 #pragma unroll
@@ -346,12 +367,30 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
     // ---- mask, online softmax -------------------------------------------------------
     const int base = w_begin + it * DEC_TILE;
     float mx[2] = {m[0], m[1]};
+    if (fu.dist_bias != nullptr) {
+      // (key number -> distance: the keys behind the kept ones are lo .. pos in order)
+      const int d0 = n_keys - 1 - base;
+      const bool far = d0 - (DEC_TILE - 1) >= fu.dist_len - 1 && base >= kept;
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float bias = b_far[e >> 1];
+          if (!far) {
+            const int key = base + t * 8 + (lane & 3) * 2 + (e & 1);
+            const int dist = key < kept ? pos - key : n_keys - 1 - key;
+            bias = __ldg(brow[e >> 1] + max(0, min(dist, fu.dist_len - 1))) * log2e;
+          }
+          sc[t][e] = fmaf(sc[t][e], scale_log2, bias);
+        }
+    }
+    const float mult = fu.dist_bias != nullptr ? 1.f : scale_log2;
 #pragma unroll
     for (int t = 0; t < 2; ++t) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = base + t * 8 + (lane & 3) * 2 + (e & 1);
-        const float raw = fu.cap_pre > 0.f ? dec_tanh(sc[t][e] * fu.cap_pre) * fu.cap_post : sc[t][e] * scale_log2;
+        const float raw = fu.cap_pre > 0.f ? dec_tanh(sc[t][e] * fu.cap_pre) * fu.cap_post : sc[t][e] * mult;
         const float v = key < w_end ? raw : -INFINITY;
         sc[t][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -447,7 +486,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
     if (num_splits == 1) {
       const float val = ll > 0.f ? acc / ll : 0.f;
       if (fu.parts != nullptr) fu.parts[orow * D + d] = val;
-      else out[orow * D + d] = __float2bfloat16_rn(val);
+      else out[orow * D + d] = __float2bfloat16_rn(val * dec_head_gate(fu.gate, fu.gate_stride, b, h));
     } else if (CL) {
       cm[r * (D + 2) + d] = acc;
       if (d == 0) {
@@ -497,7 +536,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
       const long long orow = ((long long)b * num_q + kh * group + r) * o_rep + (fu.parts != nullptr ? vh : 0);
       const float val = ll > 0.f ? acc / ll : 0.f;
       if (fu.parts != nullptr) fu.parts[orow * D + d] = val;
-      else out[orow * D + d] = __float2bfloat16_rn(val);
+      else out[orow * D + d] = __float2bfloat16_rn(val * dec_head_gate(fu.gate, fu.gate_stride, b, kh * group + r));
     }
     cluster.sync();  // no block leaves while a peer may still read its partial
   }
@@ -506,7 +545,8 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_str
 // out[b, h, :] = sum_s O_s 2^(m_s - M) / sum_s l_s 2^(m_s - M)
 template <int D>
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    __nv_bfloat16* __restrict__ out, int num_splits, float* __restrict__ out_f32) {
+                                    __nv_bfloat16* __restrict__ out, int num_splits, float* __restrict__ out_f32,
+                                    const __nv_bfloat16* __restrict__ gate, long long gate_stride, int num_q) {
   pdl_launch_dependents();
   pdl_wait();
   const long long bh = blockIdx.x;
@@ -543,7 +583,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   }
   const float val = ll > 0.f ? acc / ll : 0.f;
   if (out_f32 != nullptr) out_f32[bh * D + d] = val;  // (rows then count (request, head, value head))
-  else out[bh * D + d] = __float2bfloat16_rn(val);
+  else out[bh * D + d] = __float2bfloat16_rn(val * dec_head_gate(gate, gate_stride, bh / num_q, (int)(bh % num_q)));
 }
 
 static int g_decode_attr_set[2] = {0, 0};
@@ -609,7 +649,7 @@ static int launch_decode(int which, const void* q, long long q_row_stride, const
   if (rc != ULLM_OK) return rc;
   if (num_splits > 1)
     rc = ullm_launch_kernel(decode_merge_kernel<D>, dim3(batch * num_q * o_rep), dim3(D), 0, st, (const float*)part_o,
-                            (const float*)part_ml, (__nv_bfloat16*)out, num_splits, fu.parts);
+                            (const float*)part_ml, (__nv_bfloat16*)out, num_splits, fu.parts, fu.gate, fu.gate_stride, num_q);
   return rc;
 }
 
@@ -684,6 +724,26 @@ extern "C" int ullm_decode_attention_capped(const void* q, long long q_row_strid
   fu.keep_first = window > 0 ? keep_first : 0;
   fu.cap_pre = scale / softcap;
   fu.cap_post = softcap * 1.4426950408889634f;
+  return decode_attention_impl(q, q_row_stride, k_cache, v_cache, block_table, max_pages, req_slots, kv_len, out, scratch,
+                               batch, num_q, num_kv, head_dim, page_size, window, scale, num_splits, num_pages, status,
+                               stream, fu);
+}
+
+// With a learned bias per head and distance (32-bit [num_q][dist_len]; the last one serves every longer distance; null: none)
+// and a gate per head ([batch][num_q], row stride `gate_stride`; null: none).
+extern "C" int ullm_decode_attention_biased(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
+                                            const int* block_table, int max_pages, const int* req_slots,
+                                            const int* kv_len, void* out, float* scratch, int batch, int num_q,
+                                            int num_kv, int head_dim, int page_size, int window, float scale,
+                                            int num_splits, long long num_pages, int* status, void* stream,
+                                            const float* dist_bias, int dist_len, const void* gate,
+                                            long long gate_stride) {
+  if ((dist_bias != nullptr && dist_len <= 0) || (gate != nullptr && gate_stride < num_q)) return ULLM_ERR_BAD_SIZE;
+  DecFuse fu = {};
+  fu.dist_bias = dist_bias;
+  fu.dist_len = dist_len;
+  fu.gate = (const __nv_bfloat16*)gate;
+  fu.gate_stride = gate_stride;
   return decode_attention_impl(q, q_row_stride, k_cache, v_cache, block_table, max_pages, req_slots, kv_len, out, scratch,
                                batch, num_q, num_kv, head_dim, page_size, window, scale, num_splits, num_pages, status,
                                stream, fu);

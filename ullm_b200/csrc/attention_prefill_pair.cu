@@ -27,6 +27,9 @@
 // a page past the request's length are zeroed in shared memory before V is used (they may hold anything).  Every
 // load is issued by the block that uses it.
 //
+// A learned bias per head and distance (BIAS) is added to the scores as they are read: element by element where distances
+// differ, as one number per row in key tiles that lie wholly beyond the last distinct distance.
+//
 // Every wait on an mbarrier is bounded; a wait that runs out records ULLM_STATUS_TIMEOUT, and the block stops
 // waiting, frees its tensor memory and returns.
 #include <cuda.h>
@@ -215,12 +218,19 @@ struct TpParams {
   // PARTS: the grid counts (token block, key head, VALUE head); the weights of the key head's query heads meet the
   // values of any kv head, and the 32-bit results go here, [token][head][value head][128] (`out` is not written)
   float* parts;
+  // BIAS: [num_q][dist_len] 32-bit, added to the scaled score at distance min(i - j, dist_len - 1); a gate per head
+  // ([tokens][num_q], row stride gate_stride; null: none): out *= sigmoid(gate)
+  const float* dist_bias;
+  const __nv_bfloat16* gate;
+  long long gate_stride;
+  int dist_len;
+  float inv_scale;
 };
 
 // tanh by one exponential and one division of the hardware's units: 1 - 2 / (e^(2x) + 1)
 __device__ __forceinline__ float tp_tanh(float x) { return 1.f - __fdividef(2.f, tp_ex2(x * 2.8853900817779268f) + 1.f); }
 
-template <bool CAP, bool PARTS>
+template <bool CAP, bool PARTS, bool BIAS>
 __global__ void __launch_bounds__(TP_THREADS, 1)
 prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                               const __grid_constant__ CUtensorMap map_v, const TpParams p) {
@@ -486,6 +496,11 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
     const int pos = row_ok ? pf + row / G : -1;
     const int lo = first_seen(pos, p.window);
     const int lo_last = first_seen(pl, p.window);  // what the tile's last token sees first
+    // BIAS: the head's row of the table, in units of the unscaled score; a row that does not exist reads what the tile's
+    // first token would
+    const float* brow = BIAS ? p.dist_bias + (long long)(kh * G + (row_ok ? row % G : 0)) * p.dist_len : nullptr;
+    const int bpos = row_ok ? pos : pf;
+    const float far = BIAS ? brow[p.dist_len - 1] * p.inv_scale : 0.f;
     const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t tmem_s = tmem + i * TP_KEYS + lane_base;
     const uint32_t tmem_o = tmem + 2 * TP_KEYS + i * TP_D + lane_base;
@@ -525,6 +540,22 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
           for (int k = 0; k < TP_KEYS; ++k) sr[k] = __float_as_uint(tp_tanh(__uint_as_float(sr[k])));
         }
       }
+      float add = 0.f;  // BIAS: what every score of the row gets (a tile beyond the last distinct distance)
+      if (BIAS) {
+        if (pf - key0 - (TP_KEYS - 1) >= p.dist_len - 1) {
+          add = far;
+        } else if (pl - key0 <= p.dist_len - 1 && pf - key0 - (TP_KEYS - 1) >= 0) {
+          const float* bp = brow + (bpos - key0);
+#pragma unroll
+          for (int k = 0; k < TP_KEYS; ++k) sr[k] = __float_as_uint(fmaf(__ldg(bp - k), p.inv_scale, __uint_as_float(sr[k])));
+        } else {
+#pragma unroll
+          for (int k = 0; k < TP_KEYS; ++k) {
+            const int d = max(0, min(bpos - key0 - k, p.dist_len - 1));
+            sr[k] = __float_as_uint(fmaf(__ldg(brow + d), p.inv_scale, __uint_as_float(sr[k])));
+          }
+        }
+      }
       const bool need_mask = rows_valid < TP_ROWS || key0 + TP_KEYS - 1 > pf || key0 < lo_last;
       if (need_mask) {
 #pragma unroll
@@ -537,7 +568,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
 #pragma unroll
       for (int k = 0; k < TP_KEYS / 2; ++k)
         mx[k & 3] = tp_max3(mx[k & 3], __uint_as_float(sr[2 * k]), __uint_as_float(sr[2 * k + 1]));
-      const float row_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      const float row_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) + add;
       // The reference point of the exponents only moves when the row's maximum grows by more than 2^8:
       // until then P is at most 256 (exact in bf16 range, sums in 32-bit), and O and l, which share the
       // reference, need no rescaling.  The result O / l does not depend on the reference.
@@ -547,7 +578,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
       const float alpha = m == -INFINITY ? 1.f : tp_ex2(m - m_use);  // (no key seen yet: O and l are still zero)
       m = m_new;
       float sum[4] = {0.f, 0.f, 0.f, 0.f};
-      const float neg_m = -m_use;
+      const float neg_m = BIAS ? fmaf(add, p.scale_log2, -m_use) : -m_use;
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         uint32_t pk[32];
@@ -602,7 +633,10 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
         ok = false;
       }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (BIAS && p.gate != nullptr && row_ok)
+        inv /= 1.f + expf(-__bfloat162float(
+                              p.gate[(long long)(q_begin + first + i * tpt + row / G) * p.gate_stride + kh * G + row % G]));
       const long long th = (long long)(q_begin + first + i * tpt + row / G) * p.num_q + kh * G + row % G;
       __nv_bfloat16* op = p.out + th * TP_D;
       float* pp = PARTS ? p.parts + (th * p.num_kv + vh) * TP_D : nullptr;
@@ -694,11 +728,13 @@ extern "C" int ullm_prefill_attention_pair_supported(int head_dim, int num_q, in
   return page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64 || page_size == 128;
 }
 
-template <bool CAP, bool PARTS>
+template <bool CAP, bool PARTS, bool BIAS = false>
 static int tp_launch(const void* q, long long q_row_stride, void* out, const void* k_cache, const void* v_cache,
                      const int* block_table, int max_pages, const int* req_slots, const int* cu_q, const int* kv_len,
                      int tokens, int num_requests, int num_q, int num_kv, int head_dim, int page_size, int window,
-                     float scale, long long num_pages, int* status, void* stream, float softcap, float* parts) {
+                     float scale, long long num_pages, int* status, void* stream, float softcap, float* parts,
+                     const float* dist_bias = nullptr, int dist_len = 0, const void* gate = nullptr,
+                     long long gate_stride = 0) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || num_requests <= 0 || max_pages <= 0) return ULLM_ERR_BAD_SIZE;
   if (CAP && !(softcap > 0.f)) return ULLM_ERR_BAD_SIZE;
@@ -716,7 +752,7 @@ static int tp_launch(const void* q, long long q_row_stride, void* out, const voi
     return ULLM_ERR_LAUNCH;
   static int attr_set = 0;  // (one flag per instantiation)
   if (!attr_set) {
-    if (cudaFuncSetAttribute(prefill_attention_pair_kernel<CAP, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(prefill_attention_pair_kernel<CAP, PARTS, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              TP_SMEM) != cudaSuccess)
       return ULLM_ERR_LAUNCH;
     attr_set = 1;
@@ -739,9 +775,14 @@ static int tp_launch(const void* q, long long q_row_stride, void* out, const voi
   p.cap_pre = CAP ? scale / softcap : 0.f;
   p.num_pages = num_pages;
   p.parts = PARTS ? parts : nullptr;
+  p.dist_bias = dist_bias;
+  p.dist_len = dist_len;
+  p.gate = (const __nv_bfloat16*)gate;
+  p.gate_stride = gate_stride;
+  p.inv_scale = 1.f / scale;
   const int tpb = 2 * (TP_ROWS / G);
   dim3 grid(((tokens + tpb - 1) / tpb + num_requests) * num_kv * (PARTS ? num_kv : 1));
-  return ullm_launch_kernel(prefill_attention_pair_kernel<CAP, PARTS>, grid, dim3(TP_THREADS), (size_t)TP_SMEM, st, mq, mk,
+  return ullm_launch_kernel(prefill_attention_pair_kernel<CAP, PARTS, BIAS>, grid, dim3(TP_THREADS), (size_t)TP_SMEM, st, mq, mk,
                             mv, p);
 }
 
@@ -765,6 +806,21 @@ extern "C" int ullm_prefill_attention_pair_capped(const void* q, long long q_row
   return tp_launch<true, false>(q, q_row_stride, out, k_cache, v_cache, block_table, max_pages, req_slots, cu_q,
                                 kv_len, tokens, num_requests, num_q, num_kv, head_dim, page_size, window, scale,
                                 num_pages, status, stream, softcap, nullptr);
+}
+
+// With a learned bias per head and distance (32-bit [num_q][dist_len]; the last one serves every longer distance) and a gate
+// per head ([tokens][num_q], row stride `gate_stride`; null: none).  The scale must be positive.
+extern "C" int ullm_prefill_attention_pair_biased(const void* q, long long q_row_stride, void* out, const void* k_cache,
+                                                  const void* v_cache, const int* block_table, int max_pages,
+                                                  const int* req_slots, const int* cu_q, const int* kv_len, int tokens,
+                                                  int num_requests, int num_q, int num_kv, int head_dim, int page_size,
+                                                  int window, float scale, long long num_pages, int* status, void* stream,
+                                                  const float* dist_bias, int dist_len, const void* gate,
+                                                  long long gate_stride) {
+  if (dist_bias == nullptr || dist_len <= 0 || !(scale > 0.f) || (gate != nullptr && gate_stride < num_q)) return ULLM_ERR_BAD_SIZE;
+  return tp_launch<false, false, true>(q, q_row_stride, out, k_cache, v_cache, block_table, max_pages, req_slots, cu_q, kv_len,
+                                       tokens, num_requests, num_q, num_kv, head_dim, page_size, window, scale, num_pages,
+                                       status, stream, 0.f, nullptr, dist_bias, dist_len, gate, gate_stride);
 }
 
 // Every head's softmax weights applied to EVERY kv head's values, unrounded, into `parts` (32-bit,

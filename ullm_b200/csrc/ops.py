@@ -133,7 +133,8 @@ class Kernels:
                 "ULLM_B200_FUSE_DECODE_ROPE", "ULLM_B200_MIXED_DECODE_ROWS", "ULLM_B200_DECODE_TC",
                 "ULLM_B200_DECODE_BALANCED", "ULLM_B200_SMALL_M_LINEAR", "ULLM_B200_STREAM_WEIGHT_MB",
                 "ULLM_B200_FUSED_MLP_ROWS", "ULLM_B200_LT_ROWS", "ULLM_B200_FUSED_TAIL_ROWS",
-                "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC", "ULLM_B200_SSD_CHUNK")
+                "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC", "ULLM_B200_SSD_CHUNK",
+                "ULLM_B200_PAIR_BIASED_ROWS")
 
     def apply_switches(self, env) -> None:
         """Sets every kernel choice from `env` (a mapping; the process environment at start-up): a switch that is
@@ -161,6 +162,8 @@ class Kernels:
         # the state-space recurrence of prompt portions in chunks on the tensor cores where the sizes allow; 0: token by
         # token always
         self.ssd_chunk_on = get("ULLM_B200_SSD_CHUNK", "1") != "0"
+        # rows from which a step with distance biases (heads of 128) takes the tcgen05 prompt kernel
+        self.pair_biased_rows = int(get("ULLM_B200_PAIR_BIASED_ROWS", "128"))
         self.window_attention_tc = get("ULLM_B200_WINDOW_ATTN_TC", "1") != "0"
         # the splits of a request's keys merge inside a thread-block cluster (at most 8 splits) instead of through
         # scratch arrays and a second kernel
@@ -235,6 +238,8 @@ class Kernels:
             "ullm_prefill_attention_pair": [P, LL, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, LL, P, P],
             "ullm_prefill_attention_pair_capped": [P, LL, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, LL, P, P, F],
             "ullm_prefill_attention_pair_parts": [P, LL, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, LL, P, P],
+            "ullm_prefill_attention_pair_biased": [P, LL, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, LL, P, P, P, I, P, LL],
+            "ullm_decode_attention_biased": [P, LL, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, I, LL, P, P, P, I, P, LL],
             "ullm_linear_tcgen05": [P, P, P, P, I, I, I, I, I, P, LL, P, I, P, P],
             "ullm_linear_skinny": [P, P, P, P, I, I, I, I, I, P],
             "ullm_linear_stream": [P, P, P, P, P, I, I, I, I, I, P, P],
@@ -1182,7 +1187,7 @@ class Kernels:
     def windowed_attention(self, q, out, k_pages, v_pages, block_table, req_slots, cu_q, kv_len, token_req, num_q: int,
                            num_kv: int, head_dim: int, v_dim: int, page_size: int, window: int, scale: float, *,
                            slopes=None, pool: int = 0, pooled=None, gate=None, out_scale: float = 1.0, dist_bias=None,
-                           num_requests: int | None = None, workspace=None):
+                           num_requests: int | None = None, workspace=None, ctx=None):
         """Windowed attention (`window` as in `paged_attention`) with its further options: in bfloat16, at sizes `ullm_window_attention_supported`
         takes and with `num_requests` (the batch rows that `cu_q` describes) given, the tensor-core kernel of
         csrc/attention_window.cu; otherwise (32-bit storage, other sizes) the general kernel.  With a `workspace`
@@ -1191,7 +1196,8 @@ class Kernels:
         with `pooled` = (pooled key pages, pooled value pages or None, their block table): blocks of P positions
         that lie wholly before the window are seen through one mean key / value each.  `gate` [T, num_q x v_dim]
         (row stride free): out *= sigmoid(gate); a gate [T, num_q] has one number per head.  `dist_bias` (float32
-        [num_q, n]): score(i, j) += dist_bias[h][min(i - j, n - 1)].  `out` [T, num_q x v_dim] may be a column range of
+        [num_q, n]): score(i, j) += dist_bias[h][min(i - j, n - 1)]; with the step's `ctx` such calls take the split decode
+        kernel (steps of single tokens, heads of 64 or 128) and the tcgen05 prompt kernel (heads of 128) where they can.  `out` [T, num_q x v_dim] may be a column range of
         wider rows."""
         _need(q, "q", contiguous=False)
         _need(out, "out", q.dtype, contiguous=False)
@@ -1234,6 +1240,24 @@ class Kernels:
                 raise KernelError(f"windowed_attention: distance bias {tuple(dist_bias.shape)} for {num_q} heads")
         bias_len = dist_bias.shape[1] if dist_bias is not None else 0
         num_pages = k_pages.numel() // (page_size * num_kv * head_dim)
+        if (ctx is not None and self.window_attention_tc and q.dtype == torch.bfloat16 and v_pages is not None
+                and v_dim == head_dim and (dist_bias is not None or gate_heads) and (gate is None or gate_heads) and not pool
+                and slopes is None and out_scale == 1.0 and q.is_contiguous() and out.is_contiguous() and scale > 0):
+            if (ctx.decode_only and T == ctx.num_requests
+                    and self.lib.ullm_decode_attention_supported(head_dim, num_q, num_kv)):
+                self._decode_rows(q, out, k_pages, v_pages, block_table, req_slots, kv_len, num_q, num_kv, head_dim, page_size,
+                                  window, scale, num_pages, False, ctx, dist_bias=dist_bias, head_gate=gate)
+                return
+            if (T >= self.pair_biased_rows and dist_bias is not None and self.use_tcgen05_attention
+                    and self.lib.ullm_prefill_attention_pair_supported(head_dim, num_q, num_kv, page_size)):
+                self._check(self.lib.ullm_prefill_attention_pair_biased(
+                    _ptr(q), q.stride(0), _ptr(out), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
+                    _ptr(req_slots), _ptr(cu_q), _ptr(kv_len), T, ctx.num_requests, num_q, num_kv, head_dim, page_size,
+                    int(window), float(scale), num_pages, _ptr(self.status), _stream(), _ptr(dist_bias), bias_len, _ptr(gate),
+                    gate.stride(0) if gate is not None else 0), f"prefill_attention_pair (head_dim {head_dim}, distance bias)")
+                self.prefill_attention_kernel = "pair"
+                self.attention_path = "prefill_tcgen05"
+                return
         p_pages = pk.numel() // (page_size * num_kv * head_dim) if pk is not None else 0
         if (self.window_attention_tc and q.dtype == torch.bfloat16 and num_requests and q.stride(0) % 8 == 0
                 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and q.data_ptr() % 16 == 0
@@ -1960,14 +1984,14 @@ class Kernels:
 
     def _decode_rows(self, qkv, out, k_pages, v_pages, block_table, req_slots, kv_len, num_q, num_kv, head_dim,
                      page_size, window, scale, num_pages, ragged, ctx, fuse=None, keep_first: int = 0,
-                     softcap: float = 0.0, parts=None) -> None:
+                     softcap: float = 0.0, parts=None, dist_bias=None, head_gate=None) -> None:
         """Decode attention of T one-token rows (row i belongs to request row i): streams the pages once.
         `keep_first` > 0 (with a window), `softcap` > 0 (capped scores) or `parts` (every head's weights on every
-        kv head's values, 32-bit [T, num_q * num_kv * head_dim]; `out` unused): the per-request split kernel, the
-        one that takes them."""
+        kv head's values, 32-bit [T, num_q * num_kv * head_dim]; `out` unused), `dist_bias` or `head_gate`: the per-request
+        split kernel, the one that takes them."""
         T = qkv.shape[0]
         choice = self._decode_choice(T, ragged, num_q, num_kv, head_dim, page_size, qkv.stride(0))
-        if keep_first > 0 or softcap > 0 or parts is not None:
+        if keep_first > 0 or softcap > 0 or parts is not None or dist_bias is not None or head_gate is not None:
             choice = "split"
         if fuse is not None and choice != "split":
             raise KernelError("decode attention: q and k were left unprepared for a kernel that does not prepare them")
@@ -2031,6 +2055,14 @@ class Kernels:
                 _ptr(fuse["cos"]), _ptr(fuse["sin"]), fuse["cos"].shape[0], _ptr(fuse["positions"]),
                 _ptr(fuse["slot_mapping"]), _ptr(self.status), _stream()),
                 f"decode_attention_fused (head_dim {head_dim})")
+        elif dist_bias is not None or head_gate is not None:
+            self._check(self.lib.ullm_decode_attention_biased(
+                _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
+                _ptr(req_slots), _ptr(kv_len), _ptr(out), _ptr(scratch), T, num_q, num_kv, head_dim, page_size,
+                int(window), float(scale), splits, num_pages, _ptr(self.status), _stream(), _ptr(dist_bias),
+                dist_bias.shape[1] if dist_bias is not None else 0, _ptr(head_gate),
+                head_gate.stride(0) if head_gate is not None else 0),
+                f"decode_attention (head_dim {head_dim}, distance bias)")
         elif parts is not None:
             self._check(self.lib.ullm_decode_attention_parts(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],

@@ -391,7 +391,7 @@ class PagedAttention(Mixer, SharesInput):
             K.windowed_attention(q, attn, cache.k_pages, cache.v_pages, g.block_table, g.req_slots, ctx.cu_q, g.kv_len,
                                  ctx.token_req, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim,
                                  g.page_size, self.mask_arg, self.scale, num_requests=ctx.num_requests, workspace=ws,
-                                 **({"gate": gate, "dist_bias": self.bias_table}
+                                 **({"gate": gate, "dist_bias": self.bias_table, "ctx": ctx}
                                     if gate is not None or self.distance_bias is not None else {}))
             return self._project(attn, ctx, project_output, out)
         K.paged_attention(
