@@ -346,6 +346,7 @@ def test_recurrence_with_a_bonus_against_the_plain_one(dtype, heads, dim):
     """Portions of unequal length in one batch, from states that are not zero, with decays from nearly one to nearly nothing:
     outputs and states of every form against 64-bit."""
     from ullm_b200.csrc import kernels
+    from ullm_b200.engine.batch import Workspace
 
     K, td = kernels(), getattr(torch, dtype)
     lens, slots = (130, 5, 64, 1, 77), [4, 0, 1, 3, 2]
@@ -366,11 +367,56 @@ def test_recurrence_with_a_bonus_against_the_plain_one(dtype, heads, dim):
             ref[t] = torch.einsum("hkv,hk->hv", S_ + u.double()[:, :, None] * kv, r)
             S_ = log[t].double().exp().view(heads, dim, 1) * S_ + kv
         ref_state[slots[i], :heads * dim * dim] = S_.transpose(1, 2).reshape(-1)
-    state, out = state0.to(device()), torch.empty(T, S, device=device())
-    K.gla_recurrence(qkv.to(device()), 0, S, 2 * S, log.exp().to(device()), None, 0.0, 1.0, state, cu_q, req_slots, token_req, out,
-                     len(lens), heads, dim, dim, bonus=u.to(device()))
+    names = ["token by token"] + (["in chunks"] if K.gla_chunk_applies(td, heads, dim, dim) else [])
+    assert len(names) == 1 + (dtype == "bfloat16" and dim % 16 == 0)
+    qd, wd, ud = qkv.to(device()), log.exp().to(device()), u.to(device())
+    for name in names:
+        state, out = state0.to(device()), torch.full((T, S), float("nan"), device=device())
+        most = 1 << 30
+        if name == "in chunks":
+            most = 16
+            K.gla_chunk(qd, 0, S, 2 * S, wd, 1.0, K.gla_chunk_scratch(Workspace(device()), T, len(lens), heads, dim, dim), state,
+                        cu_q, req_slots, token_req, out, len(lens), heads, dim, dim, 16, bonus=ud)
+            assert torch.isnan(out[130:135]).all() and torch.isnan(out[199]).all() and not torch.isnan(out[:130]).any()
+        K.gla_recurrence(qd, 0, S, 2 * S, wd.clone(), None, 0.0, 1.0, state, cu_q, req_slots, token_req, out, len(lens), heads,
+                         dim, dim, bonus=ud, most_tokens=most)
+        K.raise_on_status()
+        close(out, ref.reshape(T, S).float(), "float32", f"{name}: outputs")
+        close(state, ref_state.float(), "float32", f"{name}: states")
+
+
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 64, 32), (1, 128, 256), (3, 16, 48), (2, 96, 16), (1, 256, 64)])
+def test_chunked_recurrence_without_a_bonus(heads, dim, vdim):
+    """Queries with a factor, values of another width, the current token behind its own decay's step."""
+    from ullm_b200.csrc import kernels
+    from ullm_b200.engine.batch import Workspace
+
+    K = kernels()
+    lens, slots = (70, 17, 9, 128), [3, 1, 0, 2]
+    g = torch.Generator().manual_seed(dim + vdim)
+    T, S, V = sum(lens), heads * dim, heads * vdim
+    qkv = (torch.randn(T, 2 * S + V + 8, generator=g) * 0.7).to(torch.bfloat16)
+    w = torch.exp(-torch.exp(torch.randn(T, S, generator=g) * 2 - 3))
+    w[::17] = 0.0
+    cu, cu_q, req_slots, token_req, state0 = _recurrence_batch(lens, slots, heads * dim * vdim + 8, g)
+    ref = torch.zeros(T, heads, vdim, dtype=torch.float64)
+    ref_state = state0.double().clone()
+    for i in range(len(lens)):
+        S_ = state0[slots[i], :S * vdim].double().view(heads, vdim, dim)
+        for t in range(cu[i], cu[i + 1]):
+            q, k = (qkv[t, o * S:(o + 1) * S].double().view(heads, dim) for o in range(2))
+            v = qkv[t, 2 * S:2 * S + V].double().view(heads, vdim)
+            S_ = w[t].double().view(heads, 1, dim) * S_ + v[:, :, None] * k[:, None, :]
+            ref[t] = torch.einsum("hvk,hk->hv", S_, q) * 0.3
+        ref_state[slots[i], :S * vdim] = S_.reshape(-1)
+    state, out = state0.to(device()), torch.full((T, V), float("nan"), device=device())
+    qd, wd = qkv.to(device()), w.to(device())
+    K.gla_chunk(qd, 0, S, 2 * S, wd, 0.3, K.gla_chunk_scratch(Workspace(device()), T, 4, heads, dim, vdim), state, cu_q, req_slots,
+                token_req, out, 4, heads, dim, vdim, 16)
+    K.gla_recurrence(qd, 0, S, 2 * S, wd.clone(), None, 0.0, 0.3, state, cu_q, req_slots, token_req, out, 4, heads, dim, vdim,
+                     most_tokens=16)
     K.raise_on_status()
-    close(out, ref.reshape(T, S).float(), "float32", "outputs")
+    close(out, ref.reshape(T, V).float(), "float32", "outputs")
     close(state, ref_state.float(), "float32", "states")
 
 

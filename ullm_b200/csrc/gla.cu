@@ -53,7 +53,7 @@ gla_recurrence_kernel(const T* __restrict__ qkv, long long row_stride, int q_off
                       float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                       const int* __restrict__ req_slots, const int* __restrict__ token_req, float* __restrict__ out,
                       int heads, int dim, int vdim, int rs, int chunk, int num_slots, int* status,
-                      const float* __restrict__ bonus) {
+                      const float* __restrict__ bonus, int most_tokens) {
   extern __shared__ __align__(16) float sm[];
   pdl_launch_dependents();
   pdl_wait();
@@ -68,7 +68,7 @@ gla_recurrence_kernel(const T* __restrict__ qkv, long long row_stride, int q_off
   const int col = col0 + group * CPT;        // the thread's first column
   const int dimp = RPT * rs;                 // a staged row, padded
   const int t0 = cu_q[req], t1 = cu_q[req + 1];
-  if (t1 <= t0) return;
+  if (t1 <= t0 || t1 - t0 > most_tokens) return;  // (longer portions are another kernel's)
   if (token_req[t0] < 0) {  // a row that belongs to no request: zeros out, no state touched
     if (!loader && lane_row == 0)
       for (int t = t0; t < t1; ++t)
@@ -276,7 +276,7 @@ static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_of
                       long long z_stride, const float* z_bias, float inv_tau, float q_scale, float* state,
                       long long state_stride, const int* cu_q, const int* req_slots, const int* token_req, float* out,
                       int tokens, int requests, int heads, int dim, int vdim, int num_slots, int* status,
-                      const float* bonus, cudaStream_t st) {
+                      const float* bonus, int most_tokens, cudaStream_t st) {
   const long long total = (long long)tokens * heads * dim;
   if (total > 0 && inv_tau > 0.f) {
     const long long blocks = (total + 255) / 256;
@@ -315,7 +315,8 @@ static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_of
 #define GLA_AS(RPT, CPT, BONUS)                                                                                       \
   return ullm_launch_kernel(gla_recurrence_kernel<T, RPT, CPT, BONUS>, grid, block, smem, st, (const T*)qkv,           \
                             row_stride, q_off, k_off, v_off, (const float*)z, z_stride, q_scale, state, state_stride,  \
-                            cu_q, req_slots, token_req, out, heads, dim, vdim, rs, chunk, num_slots, status, bonus)
+                            cu_q, req_slots, token_req, out, heads, dim, vdim, rs, chunk, num_slots, status, bonus, \
+                            most_tokens)
 #define GLA_GO(RPT, CPT)                         \
   {                                              \
     if (bonus != nullptr) GLA_AS(RPT, CPT, true); \
@@ -338,13 +339,14 @@ static int gla_launch(const void* qkv, long long row_stride, int q_off, int k_of
 
 // qkv [tokens, *]: q and k (heads x dim) and v (heads x vdim) at the given column offsets of rows `row_stride`
 // apart; z [tokens, heads * dim] 32-bit (rows `z_stride` apart), `z_bias` [heads * dim] or null: the decay's
-// projection, REPLACED by the decays (`inv_tau` 0: z holds the decays already); `bonus` [heads * dim] or null; out [tokens, heads * vdim] 32-bit.
+// projection, REPLACED by the decays (`inv_tau` 0: z holds the decays already); `bonus` [heads * dim] or null; requests that bring more than
+// `most_tokens` tokens are left alone; out [tokens, heads * vdim] 32-bit.
 extern "C" int ullm_gla_recurrence(int dtype, const void* qkv, long long row_stride, int q_off, int k_off, int v_off,
                                    float* z, long long z_stride, const float* z_bias, float inv_tau,
                                    float q_scale, float* state, long long state_stride, const int* cu_q,
                                    const int* req_slots, const int* token_req, float* out, int tokens, int requests,
                                    int heads, int dim, int vdim, int num_slots, int* status, void* stream,
-                                   const float* bonus) {
+                                   const float* bonus, int most_tokens) {
   cudaStream_t st = (cudaStream_t)stream;
   if (requests < 0 || tokens < 0 || heads <= 0 || dim <= 0 || vdim <= 0 || num_slots <= 0) return ULLM_ERR_BAD_SIZE;
   if (dim > GLA_MAX_DIM || heads > 65535 || requests > 65535) return ULLM_ERR_UNSUPPORTED;
@@ -352,7 +354,7 @@ extern "C" int ullm_gla_recurrence(int dtype, const void* qkv, long long row_str
   if (requests == 0) return ULLM_OK;
 #define GLA_ARGS                                                                                                     \
   qkv, row_stride, q_off, k_off, v_off, z, z_stride, z_bias, inv_tau, q_scale, state, state_stride, cu_q, req_slots, \
-      token_req, out, tokens, requests, heads, dim, vdim, num_slots, status, bonus, st
+      token_req, out, tokens, requests, heads, dim, vdim, num_slots, status, bonus, most_tokens, st
   if (dtype == ULLM_DTYPE_F32) return gla_launch<float>(GLA_ARGS);
   if (dtype == ULLM_DTYPE_BF16) return gla_launch<__nv_bfloat16>(GLA_ARGS);
   if (dtype == ULLM_DTYPE_F16) return gla_launch<__half>(GLA_ARGS);

@@ -134,7 +134,7 @@ class Kernels:
                 "ULLM_B200_DECODE_BALANCED", "ULLM_B200_SMALL_M_LINEAR", "ULLM_B200_STREAM_WEIGHT_MB",
                 "ULLM_B200_FUSED_MLP_ROWS", "ULLM_B200_LT_ROWS", "ULLM_B200_FUSED_TAIL_ROWS",
                 "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC", "ULLM_B200_SSD_CHUNK",
-                "ULLM_B200_PAIR_BIASED_ROWS")
+                "ULLM_B200_PAIR_BIASED_ROWS", "ULLM_B200_GLA_CHUNK")
 
     def apply_switches(self, env) -> None:
         """Sets every kernel choice from `env` (a mapping; the process environment at start-up): a switch that is
@@ -162,6 +162,8 @@ class Kernels:
         # the state-space recurrence of prompt portions in chunks on the tensor cores where the sizes allow; 0: token by
         # token always
         self.ssd_chunk_on = get("ULLM_B200_SSD_CHUNK", "1") != "0"
+        # the same for the recurrence with a decay per key channel
+        self.gla_chunk_on = get("ULLM_B200_GLA_CHUNK", "1") != "0"
         # rows from which a step with distance biases (heads of 128) takes the tcgen05 prompt kernel
         self.pair_biased_rows = int(get("ULLM_B200_PAIR_BIASED_ROWS", "128"))
         self.window_attention_tc = get("ULLM_B200_WINDOW_ATTN_TC", "1") != "0"
@@ -289,7 +291,8 @@ class Kernels:
             "ullm_concat_rows_f32": [I, P, P, P, I, I, I, P],
             "ullm_sigmoid_gate": [I, P, P, LL, I, I, P],
             "ullm_mingru": [I, P, LL, I, I, I, P, P, P, LL, P, P, P, P, LL, F, I, I, I, P, P],
-            "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, P],
+            "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, P, I],
+            "ullm_gla_chunk": [P, LL, I, I, I, P, LL, P, F, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
             "ullm_token_shift_mix": [I, P, LL, P, I, I, P, P, LL, I, P, P, P, I, I, P, P],
             "ullm_low_rank_decay": [I, P, LL, I, I, P, P, P, I, I, I, P],
             "ullm_linear_stream_grouped": [P, P, P, I, I, I, I, I, P, P],
@@ -318,6 +321,12 @@ class Kernels:
         L.ullm_gla_supported.restype = c_int
         L.ullm_gla_state_floats.argtypes = [I, I, I]
         L.ullm_gla_state_floats.restype = c_longlong
+        L.ullm_gla_chunk_supported.argtypes = [I, I, I]
+        L.ullm_gla_chunk_supported.restype = c_int
+        L.ullm_gla_chunk_tiles.argtypes = [I, I]
+        L.ullm_gla_chunk_tiles.restype = c_int
+        L.ullm_gla_chunk_floats.argtypes = [I, I, I]
+        L.ullm_gla_chunk_floats.restype = c_longlong
         L.ullm_ssd_supported.argtypes = [I, I, I, I, I]
         L.ullm_ssd_supported.restype = c_int
         L.ullm_ssd_chunk_supported.argtypes = [I, I, I, I]
@@ -1410,12 +1419,12 @@ class Kernels:
 
     @_timed("gla")
     def gla_recurrence(self, qkv, q_off, k_off, v_off, z, z_bias, inv_tau, q_scale, state, cu_q, req_slots, token_req,
-                       out, requests, heads, dim, vdim, bonus=None):
+                       out, requests, heads, dim, vdim, bonus=None, most_tokens: int = 1 << 30):
         """The recurrence of csrc/gla.cu over the step's tokens, from and into the requests' state rows.
         qkv [T, *]: q, k, v at the given column offsets; z [T, heads * dim] float32 (the decay's projection, a view
         with any row stride; the kernel REPLACES it by the decays; `inv_tau` 0: z holds the decays already), `z_bias` float32
-        [heads * dim] or None; `bonus` float32 [heads, dim] or None: the current token through it alone;
-        out [T, heads * vdim] float32."""
+        [heads * dim] or None; `bonus` float32 [heads, dim] or None: the current token through it alone; requests
+        that bring more than `most_tokens` tokens are left alone; out [T, heads * vdim] float32."""
         _need(qkv, "qkv")
         _need(z, "z", torch.float32, contiguous=False)
         _need(state, "state", torch.float32, contiguous=False)
@@ -1440,8 +1449,48 @@ class Kernels:
         self._check(self.lib.ullm_gla_recurrence(
             _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), q_off, k_off, v_off, _ptr(z), z.stride(0), _ptr(z_bias),
             float(inv_tau), float(q_scale), _ptr(state), state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req),
-            _ptr(out), T, requests, heads, dim, vdim, state.shape[0], _ptr(self.status), _stream(), _ptr(bonus)),
-            f"gla_recurrence (heads {heads}, dim {dim}, vdim {vdim})")
+            _ptr(out), T, requests, heads, dim, vdim, state.shape[0], _ptr(self.status), _stream(), _ptr(bonus),
+            int(most_tokens)), f"gla_recurrence (heads {heads}, dim {dim}, vdim {vdim})")
+
+    def gla_chunk_applies(self, dtype, heads: int, dim: int, vdim: int) -> bool:
+        """True when `gla_chunk` takes these sizes (bfloat16; see csrc/gla_chunk.cu)."""
+        return bool(self.gla_chunk_on and dtype == torch.bfloat16 and self.lib.ullm_gla_chunk_supported(heads, dim, vdim))
+
+    def gla_chunk_scratch(self, workspace, tokens: int, requests: int, heads: int, dim: int, vdim: int):
+        """Scratch rows of `gla_chunk` for a step of this size."""
+        return workspace.get("gla.chunks", self.lib.ullm_gla_chunk_tiles(tokens, requests),
+                             int(self.lib.ullm_gla_chunk_floats(heads, dim, vdim)), torch.float32,
+                             reserve=self.lib.ullm_gla_chunk_tiles(workspace.max_tokens, workspace.max_requests))
+
+    @_timed("gla")
+    def gla_chunk(self, qkv, q_off, k_off, v_off, decay, q_scale, scratch, state, cu_q, req_slots, token_req, out, requests,
+                  heads, dim, vdim, least: int, bonus=None):
+        """`gla_recurrence` in its chunked form on the tensor cores, for the requests that bring MORE than `least` tokens (the
+        others are left alone); `decay` [T, heads * dim] float32: the decays themselves."""
+        _need(qkv, "qkv", torch.bfloat16)
+        _need(decay, "decay", torch.float32, contiguous=False)
+        _need(state, "state", torch.float32, contiguous=False)
+        _need(out, "out", torch.float32)
+        _need(scratch, "scratch", torch.float32)
+        if bonus is not None:
+            _need(bonus, "bonus", torch.float32)
+            if bonus.numel() != heads * dim:
+                raise KernelError("gla_chunk: the bonus has the wrong length")
+        for t_, n_ in ((cu_q, "cu_q"), (req_slots, "req_slots"), (token_req, "token_req")):
+            _need(t_, n_, torch.int32)
+        T = qkv.shape[0]
+        if (decay.shape != (T, heads * dim) or decay.stride(1) != 1 or out.shape != (T, heads * vdim) or state.dim() != 2
+                or state.stride(1) != 1 or state.shape[1] < heads * vdim * dim
+                or scratch.numel() < self.lib.ullm_gla_chunk_tiles(T, requests) * self.lib.ullm_gla_chunk_floats(heads, dim, vdim)):
+            raise KernelError(f"gla_chunk: qkv {tuple(qkv.shape)}, decay {tuple(decay.shape)}, out {tuple(out.shape)}")
+        if max(q_off, k_off) + heads * dim > qkv.shape[1] or v_off + heads * vdim > qkv.shape[1]:
+            raise KernelError("gla_chunk: q, k or v lie outside the rows")
+        self._check(self.lib.ullm_gla_chunk(
+            _ptr(qkv), qkv.stride(0), q_off, k_off, v_off, _ptr(decay), decay.stride(0), _ptr(bonus), float(q_scale),
+            _ptr(scratch), _ptr(state), state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), T, requests,
+            heads, dim, vdim, state.shape[0], int(least), _ptr(self.status), _stream()),
+            f"gla_chunk (heads {heads}, dim {dim}, vdim {vdim})")
+        self.launches += 2
 
     # -- mixes of a row with the row before it; low-rank decays ---------------------------
     @_timed("token_shift")

@@ -10,7 +10,7 @@ With h' the row before h (zeros in front of the first), each of r, k, v, g, w re
 
 The five mixes are one kernel, the five products (r | k | v | g | w1, stacked; an operand each) one launch in decode steps and
 a batched product in prompts, the low-rank decay one kernel (csrc/token_shift.cu); the recurrence is that of csrc/gla.cu
-with its bonus.  Decays, state, read-out and norms are 32-bit in every engine dtype.  The state row of a request holds S of
+and csrc/gla_chunk.cu with their bonus.  Decays, state, read-out and norms are 32-bit in every engine dtype.  The state row of a request holds S of
 every head and the last row h; it is zeroed when a slot is handed out and carried from step to step.
 """
 
@@ -21,6 +21,7 @@ import torch
 from ..csrc import kernels
 from .base import Mixer, ParamDecl, StateNeed
 from .linear import linear
+from .mamba2 import CHUNK_LEAST
 from .registry import register_mixer
 
 _MIXES = ("r", "k", "v", "g", "w")
@@ -103,8 +104,15 @@ class TimeMixing(Mixer):
         w = ws.tokens("wkv.decay", T, S, torch.float32)
         K.low_rank_decay(y[:, 4 * S:4 * S + self.decay_rank], t[n["w2"]], t[n["w0"]], w)
         o = ws.tokens("wkv.o", T, S, torch.float32)
-        K.gla_recurrence(y, 0, S, 2 * S, w, None, 0.0, 1.0, cache.state, ctx.cu_q, ctx.req_slots, ctx.token_req, o,
-                         ctx.num_requests, N, d, d, bonus=t[n["u"]])
+        # prompt portions in chunks on the tensor cores (16-bit, at the sizes that form takes), the rest token by token
+        chunked = ctx.max_q_len > CHUNK_LEAST and K.gla_chunk_applies(x.dtype, N, d, d)
+        if chunked:
+            scratch = K.gla_chunk_scratch(ws, T, ctx.num_requests, N, d, d)
+            K.gla_chunk(y, 0, S, 2 * S, w, 1.0, scratch, cache.state, ctx.cu_q, ctx.req_slots, ctx.token_req, o,
+                        ctx.num_requests, N, d, d, CHUNK_LEAST, bonus=t[n["u"]])
+        if not chunked or ctx.num_requests > 1:
+            K.gla_recurrence(y, 0, S, 2 * S, w, None, 0.0, 1.0, cache.state, ctx.cu_q, ctx.req_slots, ctx.token_req, o,
+                             ctx.num_requests, N, d, d, bonus=t[n["u"]], most_tokens=CHUNK_LEAST if chunked else 1 << 30)
         g = ws.tokens("wkv.gated", T, S, x.dtype)
         K.head_norm_gate(o, y[:, 3 * S:4 * S], t[n["norm"]], self.eps, g, N, d, silu=True)
         if not project_output:
