@@ -215,6 +215,117 @@ __global__ void qkv_rotate_store_kernel(const T* __restrict__ qkv, long long row
   }
 }
 
+// The convolution, the weighted norm per head and the stores alone (no rotation, norm behind it or value mixing), in 16-byte
+// pieces.  One thread: VEC neighbouring channels of TOK tokens in a row; the filter and the rows in front wait in
+// registers, so every projected row is read once (as in csrc/ssd.cu).  The lanes of a head (head_dim / VEC of them, a power
+// of two) sum their squares by shuffles.  `single`: every request of the step has one token; the thread that convolves a
+// channel is then the only reader of its memory and moves it on itself.
+template <typename T, int VEC, int TAPS, int TOK>
+__global__ void __launch_bounds__(128)
+qkv_conv_prepare_kernel(const T* __restrict__ qkv, long long row_stride, int tokens, int num_q, int num_kv, int head_dim,
+                        int v_dim, const T* __restrict__ conv_w, float* __restrict__ conv_state, long long state_stride,
+                        const int* __restrict__ cu_q, const int* __restrict__ token_req, const int* __restrict__ req_slots,
+                        int num_state_slots, const int* __restrict__ positions, const float* __restrict__ q_w,
+                        const float* __restrict__ k_w, float eps, const int* __restrict__ slot_mapping,
+                        T* __restrict__ k_cache, T* __restrict__ v_cache, long long num_slots, T* __restrict__ q_out,
+                        int* status, float temp_coef, int temp_every, int single) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int q_size = num_q * head_dim, k_size = num_kv * head_dim, width = q_size + k_size + num_kv * v_dim;
+  const int raw = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  const bool live = raw < width;  // (every lane takes part in the shuffles)
+  const int c0 = live ? raw : 0;
+  const int kind = c0 < q_size ? 0 : (c0 < q_size + k_size ? 1 : 2);
+  const int lph = head_dim / VEC;
+  const int tok0 = blockIdx.y * TOK, tok1 = min(tokens, tok0 + TOK);
+  float cur[TOK][VEC];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i)
+    if (tok0 + i < tok1) load_vec<T, VEC>(qkv + (long long)(tok0 + i) * row_stride + c0, cur[i]);
+  float w[TAPS][VEC];  // flat: element i * TAPS + j is channel c0 + i's tap j
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load_vec<T, VEC>(conv_w + (long long)c0 * TAPS + j * VEC, w[j]);
+  float nw[VEC];
+  if (kind < 2) load_vec32<VEC>((kind == 0 ? q_w : k_w) + (c0 - (kind == 0 ? 0 : q_size)) % head_dim, nw);
+  float win[TAPS - 1][VEC];
+  int prev = -1, t0 = 0;
+  float* st = nullptr;
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) {
+    const int t = tok0 + i;
+    if (t >= tok1) break;
+    const int r = token_req[t];
+    float y[VEC];
+    if (r < 0) {  // a row that belongs to no request: as projected (nothing reads it)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = cur[i][e];
+      prev = -1;
+    } else {
+      const bool fresh = r != prev;
+      if (fresh) {
+        prev = r;
+        t0 = cu_q[r];
+        const int slot = req_slots[r];
+        st = nullptr;
+        if (slot >= 0 && slot < num_state_slots) st = conv_state + (long long)slot * state_stride + c0;
+        else ullm_report(status, ULLM_STATUS_SLOT, t, slot);
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int back = TAPS - 1 - j;
+          if (t - back >= t0) {
+            load_vec<T, VEC>(qkv + (long long)(t - back) * row_stride + c0, win[j]);
+          } else if (st != nullptr) {
+            load_vec32<VEC>(st + (long long)(TAPS - 1 - (t0 - (t - back))) * width, win[j]);
+          } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) win[j][e] = 0.f;
+          }
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const int f = e * TAPS + j;
+          y[e] = fmaf(w[f / VEC][f % VEC], j < TAPS - 1 ? win[j < TAPS - 1 ? j : 0][e] : cur[i][e], y[e]);
+        }
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) win[j][e] = win[j + 1][e];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) win[TAPS - 2][e] = cur[i][e];
+      if (single && live && st != nullptr) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) store_vec32<VEC>(st + (long long)j * width, win[j]);
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss += y[e] * y[e];
+    for (int d = lph >> 1; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+    if (kind < 2) {
+      float mult = 1.f / sqrtf(ss / (float)head_dim + eps);
+      if (kind == 0 && temp_every > 0) mult *= 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1));
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] *= mult * nw[e];
+    }
+    if (!live) continue;
+    if (kind == 0) {
+      store_vec<T, VEC>(q_out + (long long)t * q_size + c0, y);
+    } else {
+      const int slot = slot_mapping != nullptr ? slot_mapping[t] : -1;
+      if (slot >= num_slots) ullm_report(status, ULLM_STATUS_SLOT, t, slot);
+      if (slot >= 0 && slot < num_slots) {
+        if (kind == 1) store_vec<T, VEC>(k_cache + (long long)slot * k_size + (c0 - q_size), y);
+        else store_vec<T, VEC>(v_cache + (long long)slot * num_kv * v_dim + (c0 - q_size - k_size), y);
+      }
+    }
+  }
+}
+
 // After a step: the state row of every request of the step holds the last taps - 1 projected rows.  One thread
 // per (request, channel); rows are moved in ascending order, so a request that brought fewer than taps - 1 tokens
 // shifts its old rows down before it appends (row s takes old row s + n: always a row not yet written).
@@ -331,5 +442,65 @@ extern "C" int ullm_conv_state_update(int dtype, const void* qkv, long long row_
     return ullm_launch_kernel(conv_state_update_kernel<__half>, grid, block, 0, st, (const __half*)qkv, row_stride,
                               row_width, taps, conv_state, state_stride, cu_q, token_req, req_slots, num_state_slots,
                               requests);
+  return ULLM_ERR_BAD_DTYPE;
+}
+
+template <typename T>
+static int conv_prepare_go(const void* qkv, long long row_stride, int tokens, int num_q, int num_kv, int head_dim, int v_dim,
+                           const void* conv_w, int taps, float* conv_state, long long state_stride, const int* cu_q,
+                           const int* token_req, const int* req_slots, int num_state_slots, const int* positions,
+                           const float* q_w, const float* k_w, float eps, const int* slot_mapping, void* k_cache,
+                           void* v_cache, long long num_slots, void* q_out, int* status, float temp_coef, int temp_every,
+                           int single, cudaStream_t st) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const int lph = head_dim / V;
+  if (head_dim % V || v_dim % V || lph > 32 || (lph & (lph - 1)) || row_stride % V || state_stride % 4 ||
+      (((uintptr_t)qkv | (uintptr_t)conv_w | (uintptr_t)conv_state | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)k_cache |
+        (uintptr_t)v_cache | (uintptr_t)q_out) & 15))
+    return ULLM_ERR_UNSUPPORTED;
+  const int width = num_q * head_dim + num_kv * (head_dim + v_dim);
+  const int tok = tokens >= 512 ? 4 : 1, threads = 128;
+  const dim3 grid((width / V + threads - 1) / threads, (tokens + tok - 1) / tok), block(threads);
+  if (grid.y > 65535) return ULLM_ERR_UNSUPPORTED;
+#define CP_AS(TAPS, TOK)                                                                                              \
+  return ullm_launch_kernel(qkv_conv_prepare_kernel<T, V, TAPS, TOK>, grid, block, 0, st, (const T*)qkv, row_stride,  \
+                            tokens, num_q, num_kv, head_dim, v_dim, (const T*)conv_w, conv_state, state_stride, cu_q, \
+                            token_req, req_slots, num_state_slots, positions, q_w, k_w, eps, slot_mapping,            \
+                            (T*)k_cache, (T*)v_cache, num_slots, (T*)q_out, status, temp_coef, temp_every, single)
+#define CP_GO(TAPS)              \
+  {                              \
+    if (tok == 4) CP_AS(TAPS, 4); \
+    CP_AS(TAPS, 1);              \
+  }
+  if (taps == 2) CP_GO(2);
+  if (taps == 3) CP_GO(3);
+  if (taps == 4) CP_GO(4);
+#undef CP_GO
+#undef CP_AS
+  return ULLM_ERR_UNSUPPORTED;
+}
+
+// `ullm_qkv_prepare` for a convolution of 2 to 4 taps and weighted norms per head without a rotation, in 16-byte pieces;
+// with `single` (every request of the step has one token) the convolution's memory is moved on here and
+// `ullm_conv_state_update` is not needed.  ULLM_ERR_UNSUPPORTED (nothing has run): other sizes or alignments.
+extern "C" int ullm_qkv_conv_prepare(int dtype, const void* qkv, long long row_stride, int tokens, int num_q, int num_kv,
+                                     int head_dim, int v_dim, const void* conv_w, int taps, float* conv_state,
+                                     long long state_stride, const int* cu_q, const int* token_req, const int* req_slots,
+                                     int num_state_slots, const int* positions, const float* q_w, const float* k_w, float eps,
+                                     const int* slot_mapping, void* k_cache, void* v_cache, long long num_slots, void* q_out,
+                                     int* status, float temp_coef, int temp_every, int single, void* stream) {
+  cudaStream_t st = (cudaStream_t)stream;
+  if (tokens < 0 || num_q <= 0 || num_kv <= 0 || head_dim <= 0 || v_dim <= 0) return ULLM_ERR_BAD_SIZE;
+  if (conv_w == nullptr || conv_state == nullptr || q_w == nullptr || k_w == nullptr || (temp_every > 0 && positions == nullptr))
+    return ULLM_ERR_UNSUPPORTED;
+  if (tokens == 0) return ULLM_OK;
+#define CP_ARGS                                                                                                       \
+  qkv, row_stride, tokens, num_q, num_kv, head_dim, v_dim, conv_w, taps, conv_state, state_stride, cu_q, token_req,    \
+      req_slots, num_state_slots, positions, q_w, k_w, eps, slot_mapping, k_cache, v_cache, num_slots, q_out, status, \
+      temp_coef, temp_every, single, st
+  if (dtype == ULLM_DTYPE_F32) return conv_prepare_go<float>(CP_ARGS);
+  if (dtype == ULLM_DTYPE_BF16) return conv_prepare_go<__nv_bfloat16>(CP_ARGS);
+  if (dtype == ULLM_DTYPE_F16) return conv_prepare_go<__half>(CP_ARGS);
+#undef CP_ARGS
   return ULLM_ERR_BAD_DTYPE;
 }

@@ -154,7 +154,8 @@ gla_fold_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int
   }
 }
 
-// fold <- the state in front of every chunk, state <- the state behind the last: four neighbouring key channels per thread
+// fold <- the state in front of every chunk, as pairs of key channels: (two rounded values, two rounded rests), the operands
+// that `gla_out` needs; state <- the state behind the last.  Two neighbouring key channels per thread.
 __global__ void gla_scan_kernel(float* __restrict__ fold, const float* __restrict__ total, float* __restrict__ state,
                                 long long state_stride, const int* __restrict__ cu_q, const int* __restrict__ req_slots,
                                 const int* __restrict__ token_req, int least, int heads, int dim, int vdim,
@@ -174,38 +175,39 @@ __global__ void gla_scan_kernel(float* __restrict__ fold, const float* __restric
     const int m = cu_q[i + 1] - cu_q[i];
     if (m > least) tile += (m + GCH_Q - 1) / GCH_Q;
   }
-  const int e = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  const int e = (blockIdx.x * blockDim.x + threadIdx.x) * 2;
   if (e >= dim * vdim) return;
   const int chunks = (n + GCH_Q - 1) / GCH_Q;
   const long long step = (long long)heads * dim * vdim;
-  float4* f = reinterpret_cast<float4*>(fold + ((long long)tile * heads + head) * dim * vdim + e);
-  const float4* w = reinterpret_cast<const float4*>(total + ((long long)tile * heads + head) * dim + e % dim);
-  float4* st = reinterpret_cast<float4*>(state + (long long)slot * state_stride + (long long)head * dim * vdim + e);
-  float4 s = *st;
+  float* f = fold + ((long long)tile * heads + head) * dim * vdim + e;
+  const float* w = total + ((long long)tile * heads + head) * dim + e % dim;
+  float2* st = reinterpret_cast<float2*>(state + (long long)slot * state_stride + (long long)head * dim * vdim + e);
+  float2 s = *st;
   constexpr int U = 8;
   for (int c0 = 0; c0 < chunks; c0 += U) {
-    float4 d[U], a[U];
+    float2 d[U], a[U];
 #pragma unroll
     for (int j = 0; j < U; ++j)
       if (c0 + j < chunks) {
-        d[j] = f[(c0 + j) * (step / 4)];
-        a[j] = w[(long long)(c0 + j) * heads * (dim / 4)];
+        d[j] = *reinterpret_cast<const float2*>(f + (c0 + j) * step);
+        a[j] = *reinterpret_cast<const float2*>(w + (long long)(c0 + j) * heads * dim);
       }
 #pragma unroll
     for (int j = 0; j < U; ++j)
       if (c0 + j < chunks) {
-        f[(c0 + j) * (step / 4)] = s;
+        uint2 terms;
+        gch_split(s.x, s.y, terms.x, terms.y);
+        *reinterpret_cast<uint2*>(f + (c0 + j) * step) = terms;
         s.x = fmaf(a[j].x, s.x, d[j].x);
         s.y = fmaf(a[j].y, s.y, d[j].y);
-        s.z = fmaf(a[j].z, s.z, d[j].z);
-        s.w = fmaf(a[j].w, s.w, d[j].w);
       }
   }
   *st = s;
 }
 
+// A warp's 16 rows are two stretches, i0 and i0 + 1; its queries are weighted from the start of stretch i0 on.
 template <bool BONUS>
-__global__ void __launch_bounds__(GCH_THREADS)
+__global__ void __launch_bounds__(GCH_THREADS, 3)
 gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int q_off, int k_off, int v_off,
                const float* __restrict__ decay, long long decay_stride, const float* __restrict__ bonus, float q_scale,
                const int* __restrict__ cu_q, const int* __restrict__ token_req, int requests, int least, int heads, int dim,
@@ -217,7 +219,7 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
   const int tile = blockIdx.x, head = blockIdx.y;
   const int cn = gch_find(tile, cu_q, requests, least, t0);
   if (cn == 0 || token_req[t0] < 0) return;
-  const int ks = dim + 4, kb = dim + 2;
+  const int ks = dim + 4, kb = dim + 8;
   float* rp = reinterpret_cast<float*>(gch_smem);                     // [GCH_Q][ks]: q, then weighted q
   float* kq = rp + GCH_Q * ks;                                        // [GCH_Q][ks]: decays, then weighted k
   float* tot = kq + GCH_Q * ks;                                       // [GCH_SUBS][dim]
@@ -227,77 +229,98 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   gch_load_v(v_s, qkv + (long long)t0 * row_stride + v_off + head * vdim, row_stride, vdim, cn);
   {
-    const int pairs = dim >> 1;
-    for (int i = tid; i < GCH_Q * pairs; i += GCH_THREADS) {
-      const int row = i / pairs, ch = (i - row * pairs) << 1;
-      float2 q = make_float2(0.f, 0.f), w = make_float2(1.f, 1.f);
-      __nv_bfloat162 k = __floats2bfloat162_rn(0.f, 0.f);
+    const int pieces = dim >> 3;
+    for (int i = tid; i < GCH_Q * pieces; i += GCH_THREADS) {
+      const int row = i / pieces, ch = (i - row * pieces) << 3;
+      float q[8];
+      float4 w0 = make_float4(1.f, 1.f, 1.f, 1.f), w1 = w0;
+      uint4 k = make_uint4(0, 0, 0, 0);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) q[j] = 0.f;
       if (row < cn) {
         const __nv_bfloat16* src = qkv + (long long)(t0 + row) * row_stride + head * dim + ch;
-        const __nv_bfloat162 qv = *reinterpret_cast<const __nv_bfloat162*>(src + q_off);
-        q = make_float2(__bfloat162float(qv.x) * q_scale, __bfloat162float(qv.y) * q_scale);
-        k = *reinterpret_cast<const __nv_bfloat162*>(src + k_off);
-        w = *reinterpret_cast<const float2*>(decay + (long long)(t0 + row) * decay_stride + head * dim + ch);
+        load_vec<__nv_bfloat16, 8>(src + q_off, q);
+        k = *reinterpret_cast<const uint4*>(src + k_off);
+        const float4* wp = reinterpret_cast<const float4*>(decay + (long long)(t0 + row) * decay_stride + head * dim + ch);
+        w0 = wp[0];
+        w1 = wp[1];
       }
-      *reinterpret_cast<float2*>(rp + row * ks + ch) = q;
-      *reinterpret_cast<float2*>(kq + row * ks + ch) = w;
-      *reinterpret_cast<__nv_bfloat162*>(k_s + row * kb + ch) = k;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) q[j] *= q_scale;
+      store_vec32<8>(rp + row * ks + ch, q);
+      *reinterpret_cast<float4*>(kq + row * ks + ch) = w0;
+      *reinterpret_cast<float4*>(kq + row * ks + ch + 4) = w1;
+      *reinterpret_cast<uint4*>(k_s + row * kb + ch) = k;
     }
   }
   __syncthreads();
-  // ---- scores inside the warp's two stretches: a lane owns key s of one of them and every second channel ----------
+  // ---- scores inside the warp's two stretches: a lane owns key s of one of them and every second pair of channels ----
   {
     const int s = lane & 7, blk = (lane >> 3) & 1, half = lane >> 4, r0 = warp * 16 + blk * 8;
-    float sc[GCH_SUB];
+    float sc[GCH_SUB], own = 0.f;
 #pragma unroll
     for (int t = 0; t < GCH_SUB; ++t) sc[t] = 0.f;
-    const int pairs = dim >> 1;
-    int c = blk * 4;  // (the two stretches' rows lie on the same banks: they take the channels in turn)
-    if (c >= pairs) c -= pairs;
-    for (int i = 0; i < pairs; ++i) {
-      const int ch = 2 * c + half;
-      if (++c == pairs) c = 0;
-      float e = __bfloat162float(k_s[(r0 + s) * kb + ch]);
-      const float eu = BONUS ? e * bonus[head * dim + ch] : 0.f;
+    const int quads = dim >> 2;
+    int c = blk;  // (the two stretches' rows lie on the same banks: they take the channels in turn)
+    for (int i = 0; i < quads; ++i) {
+      const int ch = 4 * c + 2 * half;
+      if (++c == quads) c = 0;
+      const __nv_bfloat162 kv = *reinterpret_cast<const __nv_bfloat162*>(k_s + (r0 + s) * kb + ch);
+      const float2 qs = *reinterpret_cast<const float2*>(rp + (r0 + s) * ks + ch);
+      float ex = __bfloat162float(kv.x), ey = __bfloat162float(kv.y);
+      float2 u = make_float2(1.f, 1.f);
+      if (BONUS) u = *reinterpret_cast<const float2*>(bonus + head * dim + ch);
+      own = fmaf(qs.x * u.x, ex, own);
+      own = fmaf(qs.y * u.y, ey, own);
+      const float* qp = rp + r0 * ks + ch;
+      const float* wp = kq + r0 * ks + ch;
 #pragma unroll
-      for (int t = 0; t < GCH_SUB; ++t) {
-        const float q = rp[(r0 + t) * ks + ch], w = kq[(r0 + t) * ks + ch];
-        if (BONUS) {
-          const float x = t > s ? e : (t == s ? eu : 0.f);
-          sc[t] = fmaf(q, x, sc[t]);
-          e = t > s ? e * w : e;
-        } else {
-          e = t > s ? e * w : e;
-          sc[t] = fmaf(q, t >= s ? e : 0.f, sc[t]);
+      for (int t = 1; t < GCH_SUB; ++t) {  // (what is formed for t <= s is thrown away below)
+        const float2 q = *reinterpret_cast<const float2*>(qp + t * ks), w = *reinterpret_cast<const float2*>(wp + t * ks);
+        if (!BONUS && t > s) {
+          ex *= w.x;
+          ey *= w.y;
+        }
+        sc[t] = fmaf(q.x, ex, sc[t]);
+        sc[t] = fmaf(q.y, ey, sc[t]);
+        if (BONUS && t > s) {
+          ex *= w.x;
+          ey *= w.y;
         }
       }
     }
+    own += __shfl_xor_sync(0xffffffffu, own, 16);
 #pragma unroll
     for (int t = 0; t < GCH_SUB; ++t) {
       sc[t] += __shfl_xor_sync(0xffffffffu, sc[t], 16);
-      if (half == 0) diag[(warp * 2 + blk) * 80 + t * 10 + s] = sc[t];
+      if (half == 0) diag[(warp * 2 + blk) * 80 + t * 10 + s] = t > s ? sc[t] : (t == s ? own : 0.f);
     }
   }
   __syncthreads();
-  // ---- q <- W(start of its stretch, t or t - 1) q,  decays <- W(s, end of its stretch) k ---------------------------
-  for (int i = tid; i < GCH_SUBS * dim; i += GCH_THREADS) {
-    const int sub = i / dim, ch = i - sub * dim, r0 = sub * GCH_SUB;
-    float w[GCH_SUB];
-    float p = 1.f;
+  // ---- q <- W(start of its stretch, t or t - 1) q,  decays <- (rounded, rest) of W(s, end of its stretch) k ----------
+  for (int i = tid; i < GCH_SUBS * (dim >> 1); i += GCH_THREADS) {
+    const int sub = i / (dim >> 1), ch = (i - sub * (dim >> 1)) * 2, r0 = sub * GCH_SUB;
+    float2 w[GCH_SUB];
+    float2 p = make_float2(1.f, 1.f);
 #pragma unroll
     for (int j = 0; j < GCH_SUB; ++j) {
-      w[j] = kq[(r0 + j) * ks + ch];
-      if (!BONUS) p *= w[j];
-      rp[(r0 + j) * ks + ch] *= p;
-      if (BONUS) p *= w[j];
+      w[j] = *reinterpret_cast<const float2*>(kq + (r0 + j) * ks + ch);
+      float2* qp = reinterpret_cast<float2*>(rp + (r0 + j) * ks + ch);
+      float2 q = *qp;
+      if (!BONUS) p.x *= w[j].x, p.y *= w[j].y;
+      q.x *= p.x;
+      q.y *= p.y;
+      *qp = q;
+      if (BONUS) p.x *= w[j].x, p.y *= w[j].y;
     }
-    p = 1.f;
+    p = make_float2(1.f, 1.f);
 #pragma unroll
     for (int j = GCH_SUB - 1; j >= 0; --j) {
-      kq[(r0 + j) * ks + ch] = __bfloat162float(k_s[(r0 + j) * kb + ch]) * p;
-      p *= w[j];
+      const __nv_bfloat162 kv = *reinterpret_cast<const __nv_bfloat162*>(k_s + (r0 + j) * kb + ch);
+      *reinterpret_cast<float2*>(kq + (r0 + j) * ks + ch) = make_float2(__bfloat162float(kv.x) * p.x, __bfloat162float(kv.y) * p.y);
+      p.x *= w[j].x, p.y *= w[j].y;
     }
-    tot[sub * dim + ch] = p;
+    *reinterpret_cast<float2*>(tot + sub * dim + ch) = p;
   }
   __syncthreads();
   if (warp * 16 >= cn) return;
@@ -306,45 +329,56 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
   float acc[GCH_SUBS][4];
 #pragma unroll
   for (int j = 0; j < GCH_SUBS; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  float near[4] = {0.f, 0.f, 0.f, 0.f};  // rows of stretch i0 + 1 against stretch i0
   for (int kk = 0; kk < dim; kk += 16) {
     float* r_lo = rp + (warp * 16 + g) * ks + kk + cp;  // rows of stretch i0
     float* r_hi = r_lo + 8 * ks;                        // rows of stretch i0 + 1
-    float2 q[4] = {*reinterpret_cast<const float2*>(r_lo), *reinterpret_cast<const float2*>(r_hi),
-                   *reinterpret_cast<const float2*>(r_lo + 8), *reinterpret_cast<const float2*>(r_hi + 8)};
+    float2 q0 = *reinterpret_cast<const float2*>(r_lo), q1 = *reinterpret_cast<const float2*>(r_hi),
+           q2 = *reinterpret_cast<const float2*>(r_lo + 8), q3 = *reinterpret_cast<const float2*>(r_hi + 8);
+    unsigned ah[4], al[4], bh[2], bl[2];
+    {
+      ah[0] = ah[2] = al[0] = al[2] = 0u;
+      gch_split(q1.x, q1.y, ah[1], al[1]);
+      gch_split(q3.x, q3.y, ah[3], al[3]);
+      const float2 k0 = *reinterpret_cast<const float2*>(kq + (i0 * 8 + g) * ks + kk + cp);
+      const float2 k1 = *reinterpret_cast<const float2*>(kq + (i0 * 8 + g) * ks + kk + cp + 8);
+      gch_split(k0.x, k0.y, bh[0], bl[0]);
+      gch_split(k1.x, k1.y, bh[1], bl[1]);
+      gch_mma(near, ah, bh[0], bh[1]);
+      gch_mma(near, ah, bl[0], bl[1]);
+      gch_mma(near, al, bh[0], bh[1]);
+    }
+    const float2 d0 = *reinterpret_cast<const float2*>(tot + i0 * dim + kk + cp);
+    const float2 d1 = *reinterpret_cast<const float2*>(tot + i0 * dim + kk + cp + 8);
+    q1.x *= d0.x, q1.y *= d0.y;
+    q3.x *= d1.x, q3.y *= d1.y;
+    gch_split(q0.x, q0.y, ah[0], al[0]);
+    gch_split(q1.x, q1.y, ah[1], al[1]);
+    gch_split(q2.x, q2.y, ah[2], al[2]);
+    gch_split(q3.x, q3.y, ah[3], al[3]);
+    float2 f0 = make_float2(1.f, 1.f), f1 = f0;  // the decays between stretch j's end and stretch i0's start
 #pragma unroll
-    for (int jj = 0; jj < GCH_SUBS - 1; ++jj) {
-      const int j = GCH_SUBS - 2 - jj;
-      if (j <= i0) {
-        unsigned ah[4], al[4];
-        const bool own = j == i0;  // stretch i0 itself: only the rows of the next one see it from here
-        gch_split(own ? 0.f : q[0].x, own ? 0.f : q[0].y, ah[0], al[0]);
-        gch_split(q[1].x, q[1].y, ah[1], al[1]);
-        gch_split(own ? 0.f : q[2].x, own ? 0.f : q[2].y, ah[2], al[2]);
-        gch_split(q[3].x, q[3].y, ah[3], al[3]);
+    for (int jj = 0; jj < GCH_SUBS - 2; ++jj) {
+      const int j = GCH_SUBS - 3 - jj;
+      if (j < i0) {
         const float2 k0 = *reinterpret_cast<const float2*>(kq + (j * 8 + g) * ks + kk + cp);
         const float2 k1 = *reinterpret_cast<const float2*>(kq + (j * 8 + g) * ks + kk + cp + 8);
-        unsigned bh[2], bl[2];
-        gch_split(k0.x, k0.y, bh[0], bl[0]);
-        gch_split(k1.x, k1.y, bh[1], bl[1]);
+        gch_split(k0.x * f0.x, k0.y * f0.y, bh[0], bl[0]);
+        gch_split(k1.x * f1.x, k1.y * f1.y, bh[1], bl[1]);
         gch_mma(acc[j], ah, bh[0], bh[1]);
         gch_mma(acc[j], ah, bl[0], bl[1]);
         gch_mma(acc[j], al, bh[0], bh[1]);
-        // the queries move on to the start of stretch j
-        const float2 d0 = *reinterpret_cast<const float2*>(tot + j * dim + kk + cp);
-        const float2 d1 = *reinterpret_cast<const float2*>(tot + j * dim + kk + cp + 8);
-        if (!own) {
-          q[0].x *= d0.x, q[0].y *= d0.y;
-          q[2].x *= d1.x, q[2].y *= d1.y;
-        }
-        q[1].x *= d0.x, q[1].y *= d0.y;
-        q[3].x *= d1.x, q[3].y *= d1.y;
+        const float2 e0 = *reinterpret_cast<const float2*>(tot + j * dim + kk + cp);
+        const float2 e1 = *reinterpret_cast<const float2*>(tot + j * dim + kk + cp + 8);
+        f0.x *= e0.x, f0.y *= e0.y;
+        f1.x *= e1.x, f1.y *= e1.y;
       }
     }
     // weighted down to the chunk's start: what meets the state
-    *reinterpret_cast<float2*>(r_lo) = q[0];
-    *reinterpret_cast<float2*>(r_hi) = q[1];
-    *reinterpret_cast<float2*>(r_lo + 8) = q[2];
-    *reinterpret_cast<float2*>(r_hi + 8) = q[3];
+    *reinterpret_cast<float2*>(r_lo) = make_float2(q0.x * f0.x, q0.y * f0.y);
+    *reinterpret_cast<float2*>(r_hi) = make_float2(q1.x * f0.x, q1.y * f0.y);
+    *reinterpret_cast<float2*>(r_lo + 8) = make_float2(q2.x * f1.x, q2.y * f1.y);
+    *reinterpret_cast<float2*>(r_hi + 8) = make_float2(q3.x * f1.x, q3.y * f1.y);
   }
   {
     const float2 d0 = *reinterpret_cast<const float2*>(diag + i0 * 80 + g * 10 + cp);
@@ -354,8 +388,8 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
       const float a = j == i0 ? 1.f : 0.f, b = j == i0 + 1 ? 1.f : 0.f;
       acc[j][0] = fmaf(a, d0.x, acc[j][0]);
       acc[j][1] = fmaf(a, d0.y, acc[j][1]);
-      acc[j][2] = fmaf(b, d1.x, acc[j][2]);
-      acc[j][3] = fmaf(b, d1.y, acc[j][3]);
+      acc[j][2] = fmaf(a, near[2], fmaf(b, d1.x, acc[j][2]));
+      acc[j][3] = fmaf(a, near[3], fmaf(b, d1.y, acc[j][3]));
     }
   }
   __syncwarp();
@@ -363,6 +397,7 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
   const float* st = fold + ((long long)tile * heads + head) * vdim * dim;
   const int mat = lane >> 3;
   for (int n0 = 0; n0 < vdim; n0 += 64) {
+    const int nt = min(8, (vdim - n0) >> 3);
     float y[8][4];
 #pragma unroll
     for (int n = 0; n < 8; ++n) y[n][0] = y[n][1] = y[n][2] = y[n][3] = 0.f;
@@ -376,13 +411,14 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
         gch_split(acc[2 * s + 1][2], acc[2 * s + 1][3], ah[3], al[3]);
 #pragma unroll
         for (int n = 0; n < 8; n += 2) {
-          if (n0 + n * 8 >= vdim) continue;
-          unsigned b[4];
-          gch_ldsm4t(b, v_s + (s * 16 + (mat & 1) * 8 + (lane & 7)) * (vdim + 8) + n0 + n * 8 + (mat >> 1) * 8);
-          gch_mma(y[n], ah, b[0], b[1]);
-          gch_mma(y[n + 1], ah, b[2], b[3]);
-          gch_mma(y[n], al, b[0], b[1]);
-          gch_mma(y[n + 1], al, b[2], b[3]);
+          if (n < nt) {
+            unsigned b[4];
+            gch_ldsm4t(b, v_s + (s * 16 + (mat & 1) * 8 + (lane & 7)) * (vdim + 8) + n0 + n * 8 + (mat >> 1) * 8);
+            gch_mma(y[n], ah, b[0], b[1]);
+            gch_mma(y[n + 1], ah, b[2], b[3]);
+            gch_mma(y[n], al, b[0], b[1]);
+            gch_mma(y[n + 1], al, b[2], b[3]);
+          }
         }
       }
     }
@@ -391,28 +427,25 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
       const float2 q0 = *reinterpret_cast<const float2*>(r_lo), q1 = *reinterpret_cast<const float2*>(r_lo + 8 * ks),
                    q2 = *reinterpret_cast<const float2*>(r_lo + 8), q3 = *reinterpret_cast<const float2*>(r_lo + 8 * ks + 8);
       unsigned ah[4], al[4];
+      uint2 x0[8], x1[8];  // (rounded pair, pair of rests)
+      const float* sp = st + (long long)(n0 + g) * dim + kk + cp;
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+        if (n < nt) {
+          x0[n] = *reinterpret_cast<const uint2*>(sp + (long long)n * 8 * dim);
+          x1[n] = *reinterpret_cast<const uint2*>(sp + (long long)n * 8 * dim + 8);
+        }
       gch_split(q0.x, q0.y, ah[0], al[0]);
       gch_split(q1.x, q1.y, ah[1], al[1]);
       gch_split(q2.x, q2.y, ah[2], al[2]);
       gch_split(q3.x, q3.y, ah[3], al[3]);
-      float2 x0[8], x1[8];
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
-        if (n0 + n * 8 >= vdim) continue;
-        const float* sp = st + (long long)(n0 + n * 8 + g) * dim + kk + cp;
-        x0[n] = *reinterpret_cast<const float2*>(sp);
-        x1[n] = *reinterpret_cast<const float2*>(sp + 8);
-      }
-#pragma unroll
-      for (int n = 0; n < 8; ++n) {
-        if (n0 + n * 8 >= vdim) continue;
-        unsigned bh[2], bl[2];
-        gch_split(x0[n].x, x0[n].y, bh[0], bl[0]);
-        gch_split(x1[n].x, x1[n].y, bh[1], bl[1]);
-        gch_mma(y[n], ah, bh[0], bh[1]);
-        gch_mma(y[n], ah, bl[0], bl[1]);
-        gch_mma(y[n], al, bh[0], bh[1]);
-      }
+      for (int n = 0; n < 8; ++n)
+        if (n < nt) {
+          gch_mma(y[n], ah, x0[n].x, x1[n].x);
+          gch_mma(y[n], ah, x0[n].y, x1[n].y);
+          gch_mma(y[n], al, x0[n].x, x1[n].x);
+        }
     }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -421,7 +454,7 @@ gla_out_kernel(const __nv_bfloat16* __restrict__ qkv, long long row_stride, int 
       float* dst = out + ((long long)(t0 + row) * heads + head) * vdim + n0 + cp;
 #pragma unroll
       for (int n = 0; n < 8; ++n)
-        if (n0 + n * 8 < vdim) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(y[n][2 * h], y[n][2 * h + 1]);
+        if (n < nt) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(y[n][2 * h], y[n][2 * h + 1]);
     }
   }
 }
@@ -431,7 +464,7 @@ static size_t gch_fold_smem(int dim, int vdim) {
 }
 static size_t gch_out_smem(int dim, int vdim) {
   return (size_t)(2 * GCH_Q * (dim + 4) + GCH_SUBS * dim + GCH_SUBS * 80) * 4 + (size_t)GCH_Q * (vdim + 8) * 2 +
-         (size_t)GCH_Q * (dim + 2) * 2;
+         (size_t)GCH_Q * (dim + 8) * 2;
 }
 
 // Sizes the chunked form takes (bfloat16): key and value sizes that are multiples of 16, as far as the shared memory reaches.
@@ -468,8 +501,8 @@ extern "C" int ullm_gla_chunk(const void* qkv, long long row_stride, int q_off, 
   if (tokens < 0 || requests < 0 || num_slots <= 0 || scratch == nullptr) return ULLM_ERR_BAD_SIZE;
   if (!ullm_gla_chunk_supported(heads, dim, vdim) || requests > 65535) return ULLM_ERR_UNSUPPORTED;
   if (state_stride < (long long)heads * dim * vdim || state_stride % 4) return ULLM_ERR_BAD_SIZE;
-  if (row_stride % 8 || q_off % 2 || k_off % 2 || v_off % 8 || decay_stride % 2 ||
-      (((uintptr_t)qkv | (uintptr_t)scratch | (uintptr_t)state) & 15) || (((uintptr_t)decay | (uintptr_t)out) & 7))
+  if (row_stride % 8 || q_off % 8 || k_off % 8 || v_off % 8 || decay_stride % 4 ||
+      (((uintptr_t)qkv | (uintptr_t)scratch | (uintptr_t)state | (uintptr_t)decay) & 15) || ((uintptr_t)out & 7))
     return ULLM_ERR_BAD_SIZE;
   if (tokens == 0 || requests == 0) return ULLM_OK;
   const int tiles = ullm_gla_chunk_tiles(tokens, requests);
@@ -485,7 +518,7 @@ extern "C" int ullm_gla_chunk(const void* qkv, long long row_stride, int q_off, 
   rc = ullm_launch_kernel(gla_fold_kernel, grid, block, fs, st, (const __nv_bfloat16*)qkv, row_stride, k_off, v_off, decay,
                           decay_stride, cu_q, token_req, requests, least, heads, dim, vdim, fold, total);
   if (rc != ULLM_OK) return rc;
-  rc = ullm_launch_kernel(gla_scan_kernel, dim3((dim * vdim / 4 + 127) / 128, heads, requests), dim3(128), 0, st, fold,
+  rc = ullm_launch_kernel(gla_scan_kernel, dim3((dim * vdim / 2 + 127) / 128, heads, requests), dim3(128), 0, st, fold,
                           (const float*)total, state, state_stride, cu_q, req_slots, token_req, least, heads, dim, vdim,
                           num_slots, status);
   if (rc != ULLM_OK) return rc;

@@ -316,6 +316,49 @@ __global__ void mlstm_out_gate_kernel(const float* __restrict__ o, const T* __re
   }
 }
 
+// The same in 16-byte pieces: LPH lanes (a power of two) share a head of VEC * LPH columns.
+template <typename T, int VEC>
+__global__ void head_norm_gate_vec_kernel(const float* __restrict__ o, const T* __restrict__ g, long long g_stride,
+                                          const float* __restrict__ w, T* __restrict__ out, long long pieces, int heads,
+                                          int lph, float eps, int w_per_head, int silu) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const bool live = i < pieces;  // (whole heads end together: a head's lanes are all live or all idle)
+  const long long unit = (live ? i : 0) / lph;
+  const int e = (int)((live ? i : 0) - unit * lph) * VEC;
+  const int vdim = lph * VEC;
+  const long long t = unit / heads;
+  const int h = (int)(unit - t * heads);
+  float x[VEC], gv[VEC], wv[VEC];
+  load_vec32<VEC>(o + unit * vdim + e, x);
+  load_vec<T, VEC>(g + t * g_stride + (long long)h * vdim + e, gv);
+  load_vec32<VEC>(w + (w_per_head ? h * vdim : 0) + e, wv);
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) ss += x[j] * x[j];
+  for (int d = lph >> 1; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  const float rstd = 1.f / sqrtf(ss / (float)vdim + eps);
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) x[j] *= rstd * wv[j] * ((silu ? gv[j] : 1.f) / (1.f + expf(-gv[j])));
+  if (live) store_vec<T, VEC>(out + unit * vdim + e, x);
+}
+
+template <typename T>
+static bool head_norm_gate_vec(const float* o, const void* g, long long g_stride, const float* w, void* out, int tokens,
+                               int heads, int vdim, float eps, int w_per_head, int silu, cudaStream_t st, int* rc) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const int lph = vdim / V;
+  if (vdim % V || lph > 32 || (lph & (lph - 1)) || g_stride % V ||
+      (((uintptr_t)o | (uintptr_t)g | (uintptr_t)w | (uintptr_t)out) & 15))
+    return false;
+  const long long pieces = (long long)tokens * heads * lph, blocks = (pieces + 127) / 128;
+  if (blocks > 0x7fffffffLL) return false;
+  *rc = ullm_launch_kernel(head_norm_gate_vec_kernel<T, V>, dim3((int)blocks), dim3(128), 0, st, o, (const T*)g, g_stride, w,
+                           (T*)out, pieces, heads, lph, eps, w_per_head, silu);
+  return true;
+}
+
 // Lanes that share a column: as many as leave a thread about 8 rows (the per-token chain of a thread is what
 // paces the recurrence, and narrower column tiles make more blocks), at most a warp.
 static int mlstm_rs(int dim) {
@@ -424,6 +467,10 @@ extern "C" int ullm_head_norm_gate(int dtype, const float* o, const void* g, lon
   const long long blocks = (units + 3) / 4;
   if (blocks > 0x7fffffffLL) return ULLM_ERR_BAD_SIZE;
   const dim3 grid((int)blocks), block(128);
+  int rc = ULLM_OK;
+  if (dtype == ULLM_DTYPE_F32 && head_norm_gate_vec<float>(o, g, g_stride, w, out, tokens, heads, vdim, eps, w_per_head, silu, st, &rc)) return rc;
+  if (dtype == ULLM_DTYPE_BF16 && head_norm_gate_vec<__nv_bfloat16>(o, g, g_stride, w, out, tokens, heads, vdim, eps, w_per_head, silu, st, &rc)) return rc;
+  if (dtype == ULLM_DTYPE_F16 && head_norm_gate_vec<__half>(o, g, g_stride, w, out, tokens, heads, vdim, eps, w_per_head, silu, st, &rc)) return rc;
   if (dtype == ULLM_DTYPE_F32)
     return ullm_launch_kernel(mlstm_out_gate_kernel<float>, grid, block, 0, st, o, (const float*)g, g_stride, w,
                               (float*)out, units, heads, vdim, eps, w_per_head, silu);

@@ -265,6 +265,7 @@ class Kernels:
             "ullm_softcap_f32": [P, LL, F, P],
             "ullm_qkv_prepare": [I, P, LL, I, I, I, I, I, P, I, P, LL, P, P, P, I, P, P, I, P, P, I, I, F, I, P, P, P, P,
                                  P, LL, P, P, P, F, I],
+            "ullm_qkv_conv_prepare": [I, P, LL, I, I, I, I, I, P, I, P, LL, P, P, P, I, P, P, P, F, P, P, P, LL, P, P, F, I, I, P],
             "ullm_conv_state_update": [I, P, LL, I, I, P, LL, P, P, P, I, I, P],
             "ullm_paged_attention_generic_ex2": [I, P, LL, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, F, LL, P, P, I, I,
                                                  F, P],
@@ -1734,10 +1735,11 @@ class Kernels:
                     conv_w=None, taps: int = 0, conv_state=None, cu_q=None, token_req=None, req_slots=None,
                     inv_freq=None, rotary_dim: int = 0, q_w=None, k_w=None, norm_first: bool = False,
                     norm_last: bool = False, eps: float = 0.0, vmix_mode: int = 0, vmix_lambda=None, v_first=None,
-                    q_temp=None):
+                    q_temp=None, single: bool = False) -> bool:
         """See csrc/attention_prep.cu: short convolution (with the requests' state rows), norm, rotation by computed
         angles, unit norm, value mixing, cache stores; q goes to `q_out` [T, num_q * head_dim].  `q_temp` = (coef, every): every
-        query times 1 + coef ln(floor((p + 1) / every) + 1) at its position p."""
+        query times 1 + coef ln(floor((p + 1) / every) + 1) at its position p.  `single`: every request of the step has one
+        token.  Returns True when the convolution's memory was moved on here (else `conv_state_update` has to follow)."""
         _need(qkv, "qkv", contiguous=False)
         _need(q_out, "q_out", qkv.dtype)
         T, W = qkv.shape
@@ -1774,6 +1776,17 @@ class Kernels:
             if k_pages.shape[-2:] != (num_kv, head_dim) or v_pages.shape[-2:] != (num_kv, v_dim):
                 raise KernelError(f"qkv_prepare: pages {tuple(k_pages.shape)} / {tuple(v_pages.shape)}")
             num_slots = k_pages.numel() // (num_kv * head_dim)
+        if (conv_w is not None and taps > 1 and norm_first and q_w is not None and k_w is not None and not norm_last
+                and rotary_dim == 0 and vmix_mode == 0):
+            code = self.lib.ullm_qkv_conv_prepare(
+                _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), T, num_q, num_kv, head_dim, v_dim, _ptr(conv_w), int(taps),
+                _ptr(conv_state), state_stride, _ptr(cu_q), _ptr(token_req), _ptr(req_slots), state_slots, _ptr(positions),
+                _ptr(q_w), _ptr(k_w), float(eps), _ptr(slot_mapping), _ptr(k_pages), _ptr(v_pages), num_slots, _ptr(q_out),
+                _ptr(self.status), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0, int(bool(single)),
+                _stream())
+            if code != 4:  # (4: sizes or alignments that the general kernel takes)
+                self._check(code, f"qkv_conv_prepare (head_dim {head_dim})")
+                return bool(single)
         self._check(self.lib.ullm_qkv_prepare(
             _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), T, num_q, num_kv, head_dim, v_dim, _ptr(conv_w), int(taps),
             _ptr(conv_state), state_stride, _ptr(cu_q), _ptr(token_req), _ptr(req_slots), state_slots, _ptr(positions),
@@ -1781,6 +1794,7 @@ class Kernels:
             int(vmix_mode), _ptr(vmix_lambda), _ptr(v_first), _ptr(slot_mapping), _ptr(k_pages), _ptr(v_pages), num_slots,
             _ptr(q_out), _ptr(self.status), _stream(), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0),
             f"qkv_prepare (head_dim {head_dim})")
+        return False
 
     @_timed("qk_norm_rope_store")
     def conv_state_update(self, qkv, taps: int, conv_state, cu_q, token_req, req_slots, requests: int):

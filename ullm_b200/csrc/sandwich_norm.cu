@@ -110,10 +110,10 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
     float va[VEC], vb[VEC];
     load_vec<T, VEC>(a + base + c0, va);
     load_vec<T, VEC>(b + base + c0, vb);
+    store_vec32<VEC>(row_a + c0, va);
+    store_vec32<VEC>(row_b + c0, vb);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) {
-      row_a[c0 + i] = va[i];
-      row_b[c0 + i] = vb[i];
       qa += va[i] * va[i];
       qb += vb[i] * vb[i];
     }
@@ -136,15 +136,17 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
   if (wo != nullptr) {  // the weighted sum takes b's place and is normed as one row
     float qo = 0.f;
     for (int c0 = threadIdx.x * VEC; c0 < cols; c0 += blockDim.x * VEC) {
-      float ga[VEC], gb[VEC];
+      float ga[VEC], gb[VEC], va[VEC], vb[VEC];
       load_vec32<VEC>(wa + c0, ga);
       load_vec32<VEC>(wb + c0, gb);
+      load_vec32<VEC>(row_a + c0, va);
+      load_vec32<VEC>(row_b + c0, vb);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) {
-        const float v = row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
-        row_b[c0 + i] = v;
-        qo += v * v;
+        vb[i] = va[i] * ra * ga[i] + vb[i] * rb * gb[i];
+        qo += vb[i] * vb[i];
       }
+      store_vec32<VEC>(row_b + c0, vb);
     }
     qo = warp_sum(qo);
     __syncthreads();  // the two sums have been read
@@ -161,16 +163,18 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
     else
 #pragma unroll
       for (int i = 0; i < VEC; ++i) s[i] = 0.f;
-    float ga[VEC], gb[VEC];
+    float ga[VEC], gb[VEC], va[VEC], vb[VEC];
+    load_vec32<VEC>(row_b + c0, vb);
     if (wo != nullptr) {
       load_vec32<VEC>(wo + c0, ga);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) s[i] += row_b[c0 + i] * ro * ga[i];
+      for (int i = 0; i < VEC; ++i) s[i] += vb[i] * ro * ga[i];
     } else {
+      load_vec32<VEC>(row_a + c0, va);
       load_vec32<VEC>(wa + c0, ga);
       load_vec32<VEC>(wb + c0, gb);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) s[i] += row_a[c0 + i] * ra * ga[i] + row_b[c0 + i] * rb * gb[i];
+      for (int i = 0; i < VEC; ++i) s[i] += va[i] * ra * ga[i] + vb[i] * rb * gb[i];
     }
     if (stream != nullptr) store_vec32<VEC>(stream + base + c0, s);
     if (rows_out != nullptr) store_vec<T, VEC>(rows_out + base + c0, s);
@@ -185,8 +189,7 @@ __global__ void pair_norm_add_norm_kernel(const T* __restrict__ a, const T* __re
       for (int i = 0; i < VEC; ++i) s[i] = tanhf(al * s[i]) * g2[i] + d2[i];
       store_vec<T, VEC>(out + base + c0, s);
     } else {
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) row_a[c0 + i] = s[i];
+      store_vec32<VEC>(row_a + c0, s);
     }
   }
   if (out == nullptr || kind2 >= 2) return;

@@ -37,7 +37,7 @@ struct PairEmbedding {
   const int* cu_q;
 };
 
-template <typename T, typename TAB>
+template <typename T, typename TAB, int VEC>
 __global__ void embed_scaled_kernel(const int* __restrict__ ids, const TAB* __restrict__ table,
                                     float* __restrict__ stream, T* __restrict__ copy, int hidden, int vocab,
                                     float scale, const float* __restrict__ inv_freq,
@@ -78,6 +78,18 @@ __global__ void embed_scaled_kernel(const int* __restrict__ ids, const TAB* __re
     }
     pair = (const TAB*)pe.table + bucket * hidden;
   }
+  if (VEC > 1) {  // (no sinusoid; rows that allow 16-byte pieces)
+    for (int c = threadIdx.x * VEC; c < hidden; c += blockDim.x * VEC) {
+      float v[VEC], x[VEC];
+      load_vec<TAB, VEC>(row + c, v);
+      if (pair != nullptr) load_vec<TAB, VEC>(pair + c, x);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = (bad ? 0.f : v[i] * scale) + (pair != nullptr ? x[i] : 0.f);
+      store_vec32<VEC>(stream + (long long)t * hidden + c, v);
+      if (copy != nullptr) store_vec<T, VEC>(copy + (long long)t * hidden + c, v);
+    }
+    return;
+  }
   const float p = inv_freq != nullptr ? (float)positions[t] : 0.f;
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
     float v = bad ? 0.f : to_f32(row[c]) * scale;
@@ -111,6 +123,68 @@ __global__ void norm_scale_add_kernel(const T* __restrict__ a, float* __restrict
     stream[base + c] = s;
     if (copy != nullptr) copy[base + c] = from_f32<T>(s);
   }
+}
+
+// The same in 16-byte pieces: ITEMS pieces of VEC columns per thread, which wait in registers between the sum and the update.
+template <typename T, int VEC, int ITEMS>
+__global__ void norm_scale_add_vec_kernel(const T* __restrict__ a, float* __restrict__ stream,
+                                          const float* __restrict__ w, T* __restrict__ copy, int cols, float eps,
+                                          float mult) {
+  __shared__ float scratch[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long base = (long long)blockIdx.x * cols;
+  float v[ITEMS][VEC], s[ITEMS][VEC];
+  float acc = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c < cols) {
+      load_vec<T, VEC>(a + base + c, v[i]);
+      load_vec32<VEC>(stream + base + c, s[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c < cols)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc += v[i][j] * v[i][j];
+  }
+  const float rstd = 1.f / sqrtf(block_sum(acc, scratch) / (float)cols + eps);
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c >= cols) continue;
+    float g[VEC];
+    load_vec32<VEC>(w + c, g);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s[i][j] += mult * (v[i][j] * rstd * g[j]);
+    store_vec32<VEC>(stream + base + c, s[i]);
+    if (copy != nullptr) store_vec<T, VEC>(copy + base + c, s[i]);
+  }
+}
+
+template <typename T>
+static bool norm_scale_add_vec(const void* a, float* stream, const float* w, void* copy, int rows, int cols, float eps,
+                               float mult, cudaStream_t st, int* rc) {
+  constexpr int V = 16 / (int)sizeof(T);
+  if (cols % V || (((uintptr_t)a | (uintptr_t)stream | (uintptr_t)w | (uintptr_t)copy) & 15)) return false;
+  const int pieces = cols / V;
+  int threads = 32;
+  while (threads < 256 && threads < pieces) threads <<= 1;
+  const int items = (pieces + threads - 1) / threads;
+#define NSA_GO(I)                                                                                                  \
+  {                                                                                                                \
+    *rc = ullm_launch_kernel(norm_scale_add_vec_kernel<T, V, I>, dim3(rows), dim3(threads), 0, st, (const T*)a,     \
+                             stream, w, (T*)copy, cols, eps, mult);                                                \
+    return true;                                                                                                   \
+  }
+  if (items == 1) NSA_GO(1);
+  if (items == 2) NSA_GO(2);
+  if (items <= 4) NSA_GO(4);
+#undef NSA_GO
+  return false;
 }
 
 // The same, and in the same pass the NEXT norm of the updated stream: out[t] = round(w2 * s / sqrt(mean(s^2) + eps2))
@@ -265,7 +339,15 @@ static int embed_scaled_launch(const int* ids, const void* table, float* stream,
                                int vocab, float scale, const float* inv_freq, const int* positions,
                                const int* last_tokens, const int* token_req, const int* req_slots, int* status,
                                const PairEmbedding& pe, cudaStream_t st) {
-  return ullm_launch_kernel(embed_scaled_kernel<T, TAB>, dim3(tokens), dim3(row_threads(hidden)), 0, st, ids,
+  constexpr int V = 16 / (int)sizeof(TAB);
+  int threads = 32;
+  while (threads < 256 && threads * V < hidden) threads <<= 1;
+  if (inv_freq == nullptr && hidden % V == 0 &&
+      (((uintptr_t)table | (uintptr_t)pe.table | (uintptr_t)stream | (uintptr_t)copy) & 15) == 0)
+    return ullm_launch_kernel(embed_scaled_kernel<T, TAB, V>, dim3(tokens), dim3(threads), 0, st, ids, (const TAB*)table,
+                              stream, (T*)copy, hidden, vocab, scale, inv_freq, positions, last_tokens, token_req,
+                              req_slots, status, pe);
+  return ullm_launch_kernel(embed_scaled_kernel<T, TAB, 1>, dim3(tokens), dim3(row_threads(hidden)), 0, st, ids,
                             (const TAB*)table, stream, (T*)copy, hidden, vocab, scale, inv_freq, positions,
                             last_tokens, token_req, req_slots, status, pe);
 }
@@ -306,6 +388,10 @@ extern "C" int ullm_norm_scale_add(int dtype, const void* a, float* stream, cons
   if (rows < 0 || cols <= 0) return ULLM_ERR_BAD_SIZE;
   if (rows == 0) return ULLM_OK;
   const dim3 grid(rows), block(row_threads(cols));
+  int rc = ULLM_OK;
+  if (dtype == ULLM_DTYPE_F32 && norm_scale_add_vec<float>(a, stream, w, copy, rows, cols, eps, mult, st, &rc)) return rc;
+  if (dtype == ULLM_DTYPE_BF16 && norm_scale_add_vec<__nv_bfloat16>(a, stream, w, copy, rows, cols, eps, mult, st, &rc)) return rc;
+  if (dtype == ULLM_DTYPE_F16 && norm_scale_add_vec<__half>(a, stream, w, copy, rows, cols, eps, mult, st, &rc)) return rc;
   if (dtype == ULLM_DTYPE_F32)
     return ullm_launch_kernel(norm_scale_add_kernel<float>, grid, block, 0, st, (const float*)a, stream, w,
                               (float*)copy, cols, eps, mult);

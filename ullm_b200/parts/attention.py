@@ -359,7 +359,7 @@ class PagedAttention(Mixer, SharesInput):
                 q_head_scale=self.tensors[self.names["temp"]] if self.head_temperature else None,
                 value_unit_norm=self.value_unit_norm)
             return self._attend(q, x, ctx, cache, project_output, out)
-        K.qkv_prepare(
+        moved = K.qkv_prepare(
             qkv, q, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, ctx.positions,
             g.slot_mapping if cache.writes else None, cache.k_pages, cache.v_pages,
             conv_w=self.w_conv, taps=self.conv_taps, conv_state=state, cu_q=ctx.cu_q, token_req=ctx.token_req,
@@ -369,8 +369,9 @@ class PagedAttention(Mixer, SharesInput):
             norm_last=self.unit_norm_after_rotation,
             eps=self.q_norm.eps if self.q_norm is not None else self.norm_eps,
             vmix_mode=mode, vmix_lambda=self.tensors[self.names["vmix"]] if mode == 2 else None, v_first=v_first,
-            **({"q_temp": self.q_temperature} if self.q_temperature else {}))
-        if state is not None:
+            **({"q_temp": self.q_temperature} if self.q_temperature else {}),
+            **({"single": ctx.max_q_len == 1} if self.conv_taps > 1 else {}))
+        if state is not None and not moved:
             K.conv_state_update(qkv, self.conv_taps, state, ctx.cu_q, ctx.token_req, ctx.req_slots, ctx.num_requests)
         return self._attend(q, x, ctx, cache, project_output, out, gate)
 
