@@ -469,6 +469,67 @@ def test_fixed_decays_on_the_state_space_kernels(dtype, heads, dim, vdim):
     close(got, ref.float(), dtype, "gate behind the norm")
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("heads,n,cols,groups", [(2, 64, 64, 2), (4, 128, 64, 1), (3, 20, 13, 3), (2, 512, 24, 1), (1, 4, 1, 1), (6, 48, 80, 2), (2, 200, 40, 2)])
+def test_single_tokens_through_a_state(dtype, heads, n, cols, groups):
+    """Steps of one token per request, with a row that belongs to no request: state-space and per-channel decays, bonus and
+    scale, silu on the way in, one row of decays for all tokens; other slots stay as they are."""
+    from ullm_b200.csrc import kernels
+
+    K, td = kernels(), getattr(torch, dtype)
+    g = torch.Generator().manual_seed(n + cols)
+    B, slots = 5, [3, 0, 5, 1, 2]
+    T = B + 1
+    sizes = heads * cols * n
+    state0 = torch.randn(7, (sizes + 11) // 4 * 4, generator=g) * 0.5
+    args = (i32(list(range(T + 1))), i32(slots + [0]), i32(list(range(B)) + [-1]))
+
+    def check(name, out, state, ref, new):
+        K.raise_on_status()
+        assert not out[B].any()
+        close(out[:B], ref.reshape(B, -1).float(), "float32", f"{name}: outputs")
+        want = state0.clone().double()
+        for b, s in enumerate(slots):
+            want[s, :sizes] = new[b].reshape(-1)
+        close(state, want.float(), "float32", f"{name}: states")
+
+    # state-space form
+    gs = groups * n
+    xbc = torch.randn(T, heads * cols + 2 * gs + 3, generator=g).to(td)
+    for one_row, silu in ((False, False), (True, True)):
+        rows = 1 if one_row else T
+        dt, logd, D = torch.rand(rows, heads, generator=g), -torch.rand(rows, heads, generator=g) * 3, torch.randn(heads, generator=g)
+        x = pn.silu(xbc.double()) if silu else xbc.double()
+        v = x[:B, :heads * cols].view(B, heads, cols)
+        k, q = (x[:B, o:o + gs].view(B, groups, n).repeat_interleave(heads // groups, 1) for o in (heads * cols, heads * cols + gs))
+        S = torch.stack([state0[s, :sizes].double().view(heads, cols, n) for s in slots])
+        d = dt.double().expand(T, -1)[:B]
+        new = logd.double().exp().expand(T, -1)[:B, :, None, None] * S + v[..., None] * (d[..., None] * k)[:, :, None, :]
+        ref = torch.einsum("bhcn,bhn->bhc", new, q) + D.double()[None, :, None] * v
+        state, out = state0.to(device()), torch.full((T, heads * cols), 5.0, device=device())
+        K.ssd_recurrence(xbc.to(device()), heads * cols, heads * cols + gs, dt.to(device()), logd.to(device()), D.to(device()), state,
+                         *args, out, T, heads, n, cols, groups, silu_in=silu, single=True)
+        check(f"state space, one row {one_row}", out, state, ref, new)
+    # a decay per key channel
+    qkv = torch.randn(T, heads * (2 * n + cols) + 5, generator=g).to(td)
+    q, k = (qkv[:B, o * heads * n:(o + 1) * heads * n].double().view(B, heads, n) for o in range(2))
+    v = qkv[:B, 2 * heads * n:2 * heads * n + heads * cols].double().view(B, heads, cols)
+    z, zb, u = torch.randn(T, heads * n, generator=g), torch.randn(heads * n, generator=g), torch.randn(heads, n, generator=g)
+    for bonus in (False, True):
+        w = torch.sigmoid(z.double()) if bonus else torch.sigmoid(z.double() + zb.double()) ** 0.25
+        zin = w.float() if bonus else z
+        w = w[:B].view(B, heads, 1, n)
+        kv = v[..., None] * k[:, :, None, :]
+        new = w * S + kv
+        seen = S + u.double()[None, :, None, :] * kv if bonus else new
+        ref = torch.einsum("bhcn,bhn->bhc", seen, q) * 0.6
+        state, out = state0.to(device()), torch.full((T, heads * cols), 5.0, device=device())
+        K.gla_recurrence(qkv.to(device()), 0, heads * n, 2 * heads * n, zin.to(device()), None if bonus else zb.to(device()),
+                         0.0 if bonus else 0.25, 0.6, state, *args, out, T, heads, n, cols, bonus=u.to(device()) if bonus else None,
+                         single=True)
+        check(f"per-channel decays, bonus {bonus}", out, state, ref, new)
+
+
 ATTENTION = [  # heads, kv heads, dim, vdim, pages of
     (4, 2, 64, 64, 16), (6, 1, 64, 80, 8), (2, 2, 128, 128, 16), (8, 1, 32, 48, 4), (16, 1, 128, 128, 16), (3, 3, 16, 96, 8),
     (4, 4, 20, 12, 8), (64, 1, 64, 64, 16)]

@@ -134,7 +134,8 @@ class Kernels:
                 "ULLM_B200_DECODE_BALANCED", "ULLM_B200_SMALL_M_LINEAR", "ULLM_B200_STREAM_WEIGHT_MB",
                 "ULLM_B200_FUSED_MLP_ROWS", "ULLM_B200_LT_ROWS", "ULLM_B200_FUSED_TAIL_ROWS",
                 "ULLM_B200_STREAM_ALL_ROWS", "ULLM_B200_CHAIN_NORMS", "ULLM_B200_GENERAL_ATTN_TC", "ULLM_B200_SSD_CHUNK",
-                "ULLM_B200_PAIR_BIASED_ROWS", "ULLM_B200_GLA_CHUNK")
+                "ULLM_B200_PAIR_BIASED_ROWS", "ULLM_B200_GLA_CHUNK",
+                "ULLM_B200_STATE_STEP")
 
     def apply_switches(self, env) -> None:
         """Sets every kernel choice from `env` (a mapping; the process environment at start-up): a switch that is
@@ -164,6 +165,8 @@ class Kernels:
         self.ssd_chunk_on = get("ULLM_B200_SSD_CHUNK", "1") != "0"
         # the same for the recurrence with a decay per key channel
         self.gla_chunk_on = get("ULLM_B200_GLA_CHUNK", "1") != "0"
+        # steps of single tokens through a state: the kernel built around the state's stream; 0: the general recurrences
+        self.state_step_on = get("ULLM_B200_STATE_STEP", "1") != "0"
         # rows from which a step with distance biases (heads of 128) takes the tcgen05 prompt kernel
         self.pair_biased_rows = int(get("ULLM_B200_PAIR_BIASED_ROWS", "128"))
         self.window_attention_tc = get("ULLM_B200_WINDOW_ATTN_TC", "1") != "0"
@@ -293,6 +296,8 @@ class Kernels:
             "ullm_sigmoid_gate": [I, P, P, LL, I, I, P],
             "ullm_mingru": [I, P, LL, I, I, I, P, P, P, LL, P, P, P, P, LL, F, I, I, I, P, P],
             "ullm_gla_recurrence": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, P, I],
+            "ullm_ssd_step": [I, P, LL, I, I, P, P, P, P, LL, P, P, P, I, I, I, I, I, I, P, P, LL, I],
+            "ullm_gla_step": [I, P, LL, I, I, I, P, LL, P, F, F, P, LL, P, P, P, I, I, I, I, I, P, P, P],
             "ullm_gla_chunk": [P, LL, I, I, I, P, LL, P, F, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, P, P],
             "ullm_token_shift_mix": [I, P, LL, P, I, I, P, P, LL, I, P, P, P, I, I, P, P],
             "ullm_low_rank_decay": [I, P, LL, I, I, P, P, P, I, I, I, P],
@@ -1420,12 +1425,14 @@ class Kernels:
 
     @_timed("gla")
     def gla_recurrence(self, qkv, q_off, k_off, v_off, z, z_bias, inv_tau, q_scale, state, cu_q, req_slots, token_req,
-                       out, requests, heads, dim, vdim, bonus=None, most_tokens: int = 1 << 30):
+                       out, requests, heads, dim, vdim, bonus=None, most_tokens: int = 1 << 30,
+                       single: bool = False):
         """The recurrence of csrc/gla.cu over the step's tokens, from and into the requests' state rows.
         qkv [T, *]: q, k, v at the given column offsets; z [T, heads * dim] float32 (the decay's projection, a view
         with any row stride; the kernel REPLACES it by the decays; `inv_tau` 0: z holds the decays already), `z_bias` float32
         [heads * dim] or None; `bonus` float32 [heads, dim] or None: the current token through it alone; requests
-        that bring more than `most_tokens` tokens are left alone; out [T, heads * vdim] float32."""
+        that bring more than `most_tokens` tokens are left alone; `single`: every request of the step has one token (a
+        kernel of its own where sizes and alignments allow; z then stays as it is); out [T, heads * vdim] float32."""
         _need(qkv, "qkv")
         _need(z, "z", torch.float32, contiguous=False)
         _need(state, "state", torch.float32, contiguous=False)
@@ -1447,6 +1454,13 @@ class Kernels:
             raise KernelError("gla_recurrence: q, k or v lie outside the rows")
         if z_bias is not None and z_bias.numel() != heads * dim:
             raise KernelError("gla_recurrence: the decay bias has the wrong length")
+        if single and self.state_step_on and T == requests:
+            code = self.lib.ullm_gla_step(
+                _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), q_off, k_off, v_off, _ptr(z), z.stride(0), _ptr(z_bias),
+                float(inv_tau), float(q_scale), _ptr(state), state.stride(0), _ptr(req_slots), _ptr(token_req), _ptr(out),
+                requests, heads, dim, vdim, state.shape[0], _ptr(self.status), _stream(), _ptr(bonus))
+            if code != 4:
+                return self._check(code, f"gla_step (heads {heads}, dim {dim}, vdim {vdim})")
         self._check(self.lib.ullm_gla_recurrence(
             _DT[qkv.dtype], _ptr(qkv), qkv.stride(0), q_off, k_off, v_off, _ptr(z), z.stride(0), _ptr(z_bias),
             float(inv_tau), float(q_scale), _ptr(state), state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req),
@@ -1654,11 +1668,12 @@ class Kernels:
     @_timed("ssd")
     def ssd_recurrence(self, xbc, b_off: int, c_off: int, dt, log_decay, d_skip, state, cu_q, req_slots, token_req, out,
                        requests: int, heads: int, n_state: int, pdim: int, groups: int, most_tokens: int = 1 << 30,
-                       silu_in: bool = False):
+                       silu_in: bool = False, single: bool = False):
         """The recurrence over the step's tokens, from and into the requests' state rows (float32
         [slots, >= heads * pdim * n_state]); out [T, heads * pdim] float32.  Requests that bring more than
         `most_tokens` tokens are left alone.  dt and log_decay may have ONE row that serves all tokens; `silu_in`: x, B
-        and C pass a silu as they are read."""
+        and C pass a silu as they are read.  `single`: every request of the step has one token (a kernel of its own where
+        sizes and alignments allow)."""
         _need(xbc, "xbc")
         _need(state, "state", torch.float32, contiguous=False)
         for t_, n_ in ((dt, "dt"), (log_decay, "log_decay"), (d_skip, "d_skip"), (out, "out")):
@@ -1672,6 +1687,13 @@ class Kernels:
             raise KernelError(f"ssd_recurrence: xbc {tuple(xbc.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
         if max(b_off, c_off) + groups * n_state > xbc.shape[1] or heads * pdim > xbc.shape[1]:
             raise KernelError("ssd_recurrence: x, B or C lie outside the rows")
+        if single and self.state_step_on and T == requests:
+            code = self.lib.ullm_ssd_step(
+                _DT[xbc.dtype], _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(state),
+                state.stride(0), _ptr(req_slots), _ptr(token_req), _ptr(out), requests, heads, n_state, pdim, groups,
+                state.shape[0], _ptr(self.status), _stream(), heads if dt.shape[0] == T else 0, int(bool(silu_in)))
+            if code != 4:
+                return self._check(code, f"ssd_step (heads {heads}, state {n_state}, columns {pdim})")
         self._check(self.lib.ullm_ssd_recurrence(
             _DT[xbc.dtype], _ptr(xbc), xbc.stride(0), b_off, c_off, _ptr(dt), _ptr(log_decay), _ptr(d_skip), _ptr(state),
             state.stride(0), _ptr(cu_q), _ptr(req_slots), _ptr(token_req), _ptr(out), requests, heads, n_state, pdim,

@@ -99,63 +99,73 @@ low_rank_decay_kernel(const T* __restrict__ a, long long a_stride, int tokens, i
   }
 }
 
-// The same for prompts: a block of 64 channels x 64 tokens, a thread four of each, so that two 16-byte reads of shared memory
-// serve sixteen multiply-adds.
+// The same for prompts: a block of 128 channels x 64 tokens, a thread eight by four, so that three 16-byte reads of shared
+// memory serve 32 multiply-adds and every tanh is formed once per 128 channels.
 #define LRP_TILE 64
+#define LRP_C 128
 template <typename T>
 __global__ void __launch_bounds__(256)
 low_rank_decay_tiled_kernel(const T* __restrict__ a, long long a_stride, int tokens, int rank, const T* __restrict__ w2,
                             const float* __restrict__ w0, float* __restrict__ out, int out_stride, int channels, int log_out) {
-  __shared__ __align__(16) float w_s[LRD_R][LRP_TILE + 4];
+  __shared__ __align__(16) float w_s[LRD_R][LRP_C + 4];
   __shared__ __align__(16) float a_s[LRD_R][LRP_TILE + 4];
   pdl_launch_dependents();
   pdl_wait();
-  const int c0 = blockIdx.x * LRP_TILE, t0 = blockIdx.y * LRP_TILE;
-  const int c = (threadIdx.x & 15) * 4, t = (threadIdx.x >> 4) * 4;
-  float acc[4][4];  // [token][channel]
+  const int c0 = blockIdx.x * LRP_C, t0 = blockIdx.y * LRP_TILE;
+  const int c = (threadIdx.x & 15) * 4, t = (threadIdx.x >> 4) * 4;  // channels c .. c + 3 and c + 64 .. c + 67
+  float acc[4][8];  // [token][channel]
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
   for (int r0 = 0; r0 < rank; r0 += LRD_R) {
     const int n = min(LRD_R, rank - r0);
-    for (int i = threadIdx.x; i < LRP_TILE * LRD_R; i += 256) {
+    for (int i = threadIdx.x; i < LRP_C * LRD_R; i += 256) {
       const int row = i / LRD_R, r = i - row * LRD_R;
       w_s[r][row] = (c0 + row < channels && r < n) ? to_f32(w2[(long long)(c0 + row) * rank + r0 + r]) : 0.f;
+    }
+    for (int i = threadIdx.x; i < LRP_TILE * LRD_R; i += 256) {
+      const int row = i / LRD_R, r = i - row * LRD_R;
       a_s[r][row] = (t0 + row < tokens && r < n) ? tanhf(to_f32(a[(long long)(t0 + row) * a_stride + r0 + r])) : 0.f;
     }
     __syncthreads();
 #pragma unroll 8
     for (int r = 0; r < LRD_R; ++r) {
-      const float4 w = *reinterpret_cast<const float4*>(&w_s[r][c]), x = *reinterpret_cast<const float4*>(&a_s[r][t]);
-      const float wv[4] = {w.x, w.y, w.z, w.w}, xv[4] = {x.x, x.y, x.z, x.w};
+      const float4 w = *reinterpret_cast<const float4*>(&w_s[r][c]), w4 = *reinterpret_cast<const float4*>(&w_s[r][c + 64]),
+                   x = *reinterpret_cast<const float4*>(&a_s[r][t]);
+      const float wv[8] = {w.x, w.y, w.z, w.w, w4.x, w4.y, w4.z, w4.w}, xv[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(wv[j], xv[i], acc[i][j]);
+        for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(wv[j], xv[i], acc[i][j]);
     }
     __syncthreads();
   }
-  float b[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) b[j] = c0 + c + j < channels ? w0[c0 + c + j] : 0.f;
-  const bool wide = (out_stride & 3) == 0 && c0 + c + 4 <= channels && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
+  for (int h = 0; h < 2; ++h) {
+    const int ch = c0 + c + 64 * h;
+    if (ch >= channels) return;
+    float b[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    if (t0 + t + i >= tokens) return;
-    float v[4];
+    for (int j = 0; j < 4; ++j) b[j] = ch + j < channels ? w0[ch + j] : 0.f;
+    const bool wide = (out_stride & 3) == 0 && ch + 4 <= channels && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float l = -expf(acc[i][j] + b[j]);
-      v[j] = log_out ? l : expf(l);
-    }
-    float* dst = out + (long long)(t0 + t + i) * out_stride + c0 + c;
-    if (wide) {
-      *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
-    } else {
+    for (int i = 0; i < 4; ++i) {
+      if (t0 + t + i >= tokens) break;
+      float v[4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (c0 + c + j < channels) dst[j] = v[j];
+      for (int j = 0; j < 4; ++j) {
+        const float l = -expf(acc[i][4 * h + j] + b[j]);
+        v[j] = log_out ? l : expf(l);
+      }
+      float* dst = out + (long long)(t0 + t + i) * out_stride + ch;
+      if (wide) {
+        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (ch + j < channels) dst[j] = v[j];
+      }
     }
   }
 }
@@ -205,7 +215,8 @@ extern "C" int ullm_low_rank_decay(int dtype, const void* a, long long a_stride,
   if (tokens < 0 || rank <= 0 || channels <= 0 || a_stride < rank || out_stride < channels) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
   const int tok = tokens <= 16 ? 4 : LRP_TILE;
-  const dim3 grid((channels + LRD_C - 1) / LRD_C, (tokens + tok - 1) / tok), block(LRD_C * LRD_TG);
+  const int cb = tok == 4 ? LRD_C : LRP_C;
+  const dim3 grid((channels + cb - 1) / cb, (tokens + tok - 1) / tok), block(LRD_C * LRD_TG);
   if (grid.y > 65535) return ULLM_ERR_UNSUPPORTED;
 #define LR_GO(T)                                                                                                       \
   {                                                                                                                    \

@@ -96,7 +96,8 @@ class GatedLinearAttention(Mixer):
         K.linear_f32_out(y[:, 2 * qk + 2 * vs:], self.tensors[n["a2"]], z)
         o = ws.tokens("gla.o", T, vs, torch.float32)
         K.gla_recurrence(y, 0, qk, 2 * qk, z, self.tensors[n["a2_bias"]], 1.0 / self.tau, d ** -0.5, cache.state,
-                         ctx.cu_q, ctx.req_slots, ctx.token_req, o, ctx.num_requests, N, d, dv)
+                         ctx.cu_q, ctx.req_slots, ctx.token_req, o, ctx.num_requests, N, d, dv,
+                         single=ctx.max_q_len == 1)
         gated = ws.tokens("gla.gated", T, vs, x.dtype)
         K.head_norm_gate(o, y[:, 2 * qk + vs:2 * qk + 2 * vs], self.tensors[n["norm"]], self.eps, gated, N, dv, silu=True)
         out = ws.tokens("mixer.out", T, self.hidden_size, x.dtype)

@@ -99,7 +99,7 @@ class FixedDecayAttention(Mixer):
         if not chunked or ctx.num_requests > 1:
             K.ssd_recurrence(u, vs, vs + qk, self.steps, self.log_decay, self.skip, cache.state, ctx.cu_q, ctx.req_slots,
                              ctx.token_req, o, ctx.num_requests, N, d, dv, N, CHUNK_LEAST if chunked else 1 << 30,
-                             silu_in=not chunked)
+                             silu_in=not chunked, single=ctx.max_q_len == 1)
         g = ws.tokens("lin.gated", T, vs, x.dtype)
         K.ssd_gate_norm(o, u[:, vs + 2 * qk:], t[n["norm"]], 1, self.eps, g, gate_behind=True)
         if not project_output:

@@ -111,7 +111,8 @@ class Mamba2(Mixer, SharesInput):
                         ctx.token_req, y, ctx.num_requests, N, S, P, G, CHUNK_LEAST)
         if not chunked or ctx.num_requests > 1:
             K.ssd_recurrence(xbc, inner, inner + G * S, dt, log_decay, t[n["d"]], cache.state, ctx.cu_q, ctx.req_slots,
-                             ctx.token_req, y, ctx.num_requests, N, S, P, G, CHUNK_LEAST if chunked else 1 << 30)
+                             ctx.token_req, y, ctx.num_requests, N, S, P, G, CHUNK_LEAST if chunked else 1 << 30,
+                             single=ctx.max_q_len == 1)
         g = ws.tokens("ssd.gated", T, inner, x.dtype)
         K.ssd_gate_norm(y, u[:, :inner], t[n["norm"]], self.norm_groups, self.eps, g)
         if not project_output:

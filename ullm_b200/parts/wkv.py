@@ -112,7 +112,8 @@ class TimeMixing(Mixer):
                         ctx.num_requests, N, d, d, CHUNK_LEAST, bonus=t[n["u"]])
         if not chunked or ctx.num_requests > 1:
             K.gla_recurrence(y, 0, S, 2 * S, w, None, 0.0, 1.0, cache.state, ctx.cu_q, ctx.req_slots, ctx.token_req, o,
-                             ctx.num_requests, N, d, d, bonus=t[n["u"]], most_tokens=CHUNK_LEAST if chunked else 1 << 30)
+                             ctx.num_requests, N, d, d, bonus=t[n["u"]], most_tokens=CHUNK_LEAST if chunked else 1 << 30,
+                             single=ctx.max_q_len == 1)
         g = ws.tokens("wkv.gated", T, S, x.dtype)
         K.head_norm_gate(o, y[:, 3 * S:4 * S], t[n["norm"]], self.eps, g, N, d, silu=True)
         if not project_output:
