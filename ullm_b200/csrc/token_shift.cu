@@ -55,7 +55,7 @@ __global__ void token_shift_mix_kernel(const T* __restrict__ h, long long h_stri
 #define LRD_TG 4
 #define LRD_R 32
 
-template <typename T, int TOK>  // TOK tokens per block, TOK / LRD_TG per thread (steps of few tokens)
+template <typename T, int TOK>  // TOK tokens per block, TOK / LRD_TG per thread
 __global__ void __launch_bounds__(LRD_C * LRD_TG)
 low_rank_decay_kernel(const T* __restrict__ a, long long a_stride, int tokens, int rank, const T* __restrict__ w2,
                       const float* __restrict__ w0, float* __restrict__ out, int out_stride, int channels, int log_out) {
@@ -99,73 +99,66 @@ low_rank_decay_kernel(const T* __restrict__ a, long long a_stride, int tokens, i
   }
 }
 
-// The same for prompts: a block of 128 channels x 64 tokens, a thread eight by four, so that three 16-byte reads of shared
-// memory serve 32 multiply-adds and every tanh is formed once per 128 channels.
-#define LRP_TILE 64
-#define LRP_C 128
-template <typename T>
-__global__ void __launch_bounds__(256)
-low_rank_decay_tiled_kernel(const T* __restrict__ a, long long a_stride, int tokens, int rank, const T* __restrict__ w2,
-                            const float* __restrict__ w0, float* __restrict__ out, int out_stride, int channels, int log_out) {
-  __shared__ __align__(16) float w_s[LRD_R][LRP_C + 4];
-  __shared__ __align__(16) float a_s[LRD_R][LRP_TILE + 4];
+// The same for bfloat16 prompts on the tensor cores (mma.sync m16n8k16): w2 is an exact operand, tanh(a) enters as two
+// bfloat16 terms, rounded value and rounded rest, so the sums keep 16 bits of it or more.  A block: 64 tokens x 64 channels, a
+// warp 16 of the tokens.
+__device__ __forceinline__ void lrm_mma(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__global__ void __launch_bounds__(128)
+low_rank_decay_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_stride, int tokens, int rank,
+                          const __nv_bfloat16* __restrict__ w2, const float* __restrict__ w0, float* __restrict__ out,
+                          int out_stride, int channels, int log_out) {
   pdl_launch_dependents();
   pdl_wait();
-  const int c0 = blockIdx.x * LRP_C, t0 = blockIdx.y * LRP_TILE;
-  const int c = (threadIdx.x & 15) * 4, t = (threadIdx.x >> 4) * 4;  // channels c .. c + 3 and c + 64 .. c + 67
-  float acc[4][8];  // [token][channel]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, cp = (lane & 3) * 2;
+  const int t0 = blockIdx.y * 64 + warp * 16, c0 = blockIdx.x * 64;
+  float acc[8][4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+  for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+  for (int k0 = 0; k0 < rank; k0 += 16) {
+    unsigned ah[4], al[4];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
-  for (int r0 = 0; r0 < rank; r0 += LRD_R) {
-    const int n = min(LRD_R, rank - r0);
-    for (int i = threadIdx.x; i < LRP_C * LRD_R; i += 256) {
-      const int row = i / LRD_R, r = i - row * LRD_R;
-      w_s[r][row] = (c0 + row < channels && r < n) ? to_f32(w2[(long long)(c0 + row) * rank + r0 + r]) : 0.f;
+    for (int q = 0; q < 4; ++q) {  // rows + 8 (q & 1), columns + 8 (q >> 1)
+      const int t = t0 + g + 8 * (q & 1), k = k0 + cp + 8 * (q >> 1);
+      float2 v = make_float2(0.f, 0.f);
+      if (t < tokens && k < rank) {
+        const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(a + (long long)t * a_stride + k);
+        v = make_float2(tanhf(__bfloat162float(x.x)), tanhf(__bfloat162float(x.y)));
+      }
+      const __nv_bfloat162 h = __floats2bfloat162_rn(v.x, v.y);
+      const __nv_bfloat162 l = __floats2bfloat162_rn(v.x - __bfloat162float(h.x), v.y - __bfloat162float(h.y));
+      ah[q] = *reinterpret_cast<const unsigned*>(&h);
+      al[q] = *reinterpret_cast<const unsigned*>(&l);
     }
-    for (int i = threadIdx.x; i < LRP_TILE * LRD_R; i += 256) {
-      const int row = i / LRD_R, r = i - row * LRD_R;
-      a_s[r][row] = (t0 + row < tokens && r < n) ? tanhf(to_f32(a[(long long)(t0 + row) * a_stride + r0 + r])) : 0.f;
-    }
-    __syncthreads();
-#pragma unroll 8
-    for (int r = 0; r < LRD_R; ++r) {
-      const float4 w = *reinterpret_cast<const float4*>(&w_s[r][c]), w4 = *reinterpret_cast<const float4*>(&w_s[r][c + 64]),
-                   x = *reinterpret_cast<const float4*>(&a_s[r][t]);
-      const float wv[8] = {w.x, w.y, w.z, w.w, w4.x, w4.y, w4.z, w4.w}, xv[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(wv[j], xv[i], acc[i][j]);
+    for (int n = 0; n < 8; ++n) {
+      const int c = c0 + n * 8 + g;
+      const __nv_bfloat16* wp = w2 + (long long)c * rank + k0 + cp;
+      const unsigned b0 = c < channels && k0 + cp < rank ? *reinterpret_cast<const unsigned*>(wp) : 0u;
+      const unsigned b1 = c < channels && k0 + cp + 8 < rank ? *reinterpret_cast<const unsigned*>(wp + 8) : 0u;
+      lrm_mma(acc[n], ah, b0, b1);
+      lrm_mma(acc[n], al, b0, b1);
     }
-    __syncthreads();
   }
 #pragma unroll
-  for (int h = 0; h < 2; ++h) {
-    const int ch = c0 + c + 64 * h;
-    if (ch >= channels) return;
-    float b[4];
+  for (int n = 0; n < 8; ++n) {
+    const int c = c0 + n * 8 + cp;
+    if (c >= channels) continue;  // (channels are even here)
+    const float2 b = *reinterpret_cast<const float2*>(w0 + c);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) b[j] = ch + j < channels ? w0[ch + j] : 0.f;
-    const bool wide = (out_stride & 3) == 0 && ch + 4 <= channels && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      if (t0 + t + i >= tokens) break;
-      float v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float l = -expf(acc[i][4 * h + j] + b[j]);
-        v[j] = log_out ? l : expf(l);
+    for (int h = 0; h < 2; ++h) {
+      const int t = t0 + g + 8 * h;
+      if (t >= tokens) continue;
+      float x = -expf(acc[n][2 * h] + b.x), y = -expf(acc[n][2 * h + 1] + b.y);
+      if (!log_out) {
+        x = expf(x);
+        y = expf(y);
       }
-      float* dst = out + (long long)(t0 + t + i) * out_stride + ch;
-      if (wide) {
-        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (ch + j < channels) dst[j] = v[j];
-      }
+      *reinterpret_cast<float2*>(out + (long long)t * out_stride + c) = make_float2(x, y);
     }
   }
 }
@@ -214,16 +207,20 @@ extern "C" int ullm_low_rank_decay(int dtype, const void* a, long long a_stride,
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens < 0 || rank <= 0 || channels <= 0 || a_stride < rank || out_stride < channels) return ULLM_ERR_BAD_SIZE;
   if (tokens == 0) return ULLM_OK;
-  const int tok = tokens <= 16 ? 4 : LRP_TILE;
-  const int cb = tok == 4 ? LRD_C : LRP_C;
-  const dim3 grid((channels + cb - 1) / cb, (tokens + tok - 1) / tok), block(LRD_C * LRD_TG);
+  if (dtype == ULLM_DTYPE_BF16 && tokens > 16 && rank % 2 == 0 && a_stride % 2 == 0 && channels % 2 == 0 && out_stride % 2 == 0 &&
+      (((uintptr_t)a | (uintptr_t)w2) & 3) == 0 && (((uintptr_t)w0 | (uintptr_t)out) & 7) == 0 && (tokens + 63) / 64 <= 65535)
+    return ullm_launch_kernel(low_rank_decay_mma_kernel, dim3((channels + 63) / 64, (tokens + 63) / 64), dim3(128), 0, st,
+                              (const __nv_bfloat16*)a, a_stride, tokens, rank, (const __nv_bfloat16*)w2, w0, out, out_stride,
+                              channels, log_out);
+  const int tok = tokens <= 16 ? 4 : 32;
+  const dim3 grid((channels + LRD_C - 1) / LRD_C, (tokens + tok - 1) / tok), block(LRD_C * LRD_TG);
   if (grid.y > 65535) return ULLM_ERR_UNSUPPORTED;
 #define LR_GO(T)                                                                                                       \
   {                                                                                                                    \
     if (tok == 4)                                                                                                      \
       return ullm_launch_kernel(low_rank_decay_kernel<T, 4>, grid, block, 0, st, (const T*)a, a_stride, tokens, rank,   \
                                 (const T*)w2, w0, out, out_stride, channels, log_out);                                 \
-    return ullm_launch_kernel(low_rank_decay_tiled_kernel<T>, grid, block, 0, st, (const T*)a, a_stride, tokens, rank,  \
+    return ullm_launch_kernel(low_rank_decay_kernel<T, 32>, grid, block, 0, st, (const T*)a, a_stride, tokens, rank,    \
                               (const T*)w2, w0, out, out_stride, channels, log_out);                                   \
   }
   if (dtype == ULLM_DTYPE_F32) LR_GO(float);
